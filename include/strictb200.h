@@ -224,6 +224,9 @@ int strictb200_gemm_int8(strictb200_ctx* ctx, int64_t M, int64_t N, int64_t K, c
 /* bf16 activations in (split inside, using context scratch); bf16 out. */
 int strictb200_gemm_int8w(strictb200_ctx* ctx, int64_t M, int64_t N, int64_t K, const uint16_t* d_x_bf16, const int8_t* d_wq, const float* d_sw,
                           uint16_t* d_y_bf16);
+/* Y[M,N] = X[M,K] . W[N,K]^T, bf16 operands, fp32 accumulation on the tensor cores. out_dtype: 0 bf16, 1 fp32. K % 8 == 0. */
+int strictb200_gemm_bf16(strictb200_ctx* ctx, int64_t M, int64_t N, int64_t K, const uint16_t* d_x, const uint16_t* d_w, void* d_y,
+                         int out_dtype);
 /* fp32 Y[M,N] = X[M,K] . W[N,K]^T + bias[N] (bias may be NULL). */
 int strictb200_gemm_f32(strictb200_ctx* ctx, int64_t M, int64_t N, int64_t K, const float* d_x, const float* d_w,
                         const float* d_bias, float* d_y);
@@ -281,7 +284,7 @@ int strictb200_embedding_bf16(strictb200_ctx* ctx, const uint16_t* d_table, cons
 int strictb200_argmax(strictb200_ctx* ctx, const float* d_x, int64_t M, int64_t N, int32_t* d_out);
 
 /* ---- model / KV-cache objects (new API in the style of the existing surface) ---- */
-enum strictb200_arch { STRICTB200_GPT2 = 0, STRICTB200_QWEN3 = 1 };
+enum strictb200_arch { STRICTB200_GPT2 = 0, STRICTB200_QWEN3 = 1, STRICTB200_STACK = 2 /* strictb200_stack_create */ };
 typedef struct strictb200_model_config {
   int32_t arch;       /* strictb200_arch */
   int32_t n_layers, d_model, n_q_heads, n_kv_heads, head_dim, d_ff, vocab;
@@ -293,6 +296,34 @@ typedef struct strictb200_model_config {
 
 int strictb200_model_create(strictb200_ctx* ctx, const strictb200_model_config* cfg, strictb200_model** out);
 int strictb200_model_destroy(strictb200_model* m);
+/* ---- models described layer by layer (single GPU) ----
+ * Every layer: x <- x + mixer(norm1(x)) + ff(norm2(x)), both norms of the same x, each an RMS norm over norm_groups equal
+ * consecutive parts of the row. The model is strictb200_model like any other: the cache, prefill, decode, generate and
+ * tensor calls below take it.
+ * Mixer "latent attention": per head `dim` unrotated and `rot_dim` rotated query/key dimensions and `vdim` value
+ * dimensions; a position leaves one RMS-normed latent of kv_rank values and one rotated key part that all heads share
+ * (what the cache holds); keys and values of a head are linear in the latent. Rotation pairs (2i, 2i+1), angle
+ * pos * rot_base^(-2i/rot_dim). Scores are multiplied by `scale`; a position sees `window` keys, itself included
+ * (0: every earlier one). kv_from >= 0: no latents of its own, it reads those of that earlier layer.
+ * Feed-forward: down(xIELU(up(h))), or none.
+ * dtype BF16: bf16 weights, cache and matrix operands; fp32 residual, norms, scores and softmax. FP32: all fp32. */
+enum strictb200_mixer { STRICTB200_MIXER_LATENT = 1 };
+enum strictb200_mlp { STRICTB200_MLP_NONE = 0, STRICTB200_MLP_XIELU = 1 };
+enum strictb200_dtype { STRICTB200_BF16 = 0, STRICTB200_FP32 = 1 };
+typedef struct strictb200_layer_config {
+  int32_t mixer; /* strictb200_mixer */
+  int32_t heads, dim, rot_dim, vdim, kv_rank;
+  int32_t window, kv_from; /* 0: no window; -1: latents of its own */
+  int32_t mlp, d_ff;       /* strictb200_mlp */
+  double scale, rot_base;
+} strictb200_layer_config;
+typedef struct strictb200_stack_config {
+  int32_t n_layers, d_model, vocab, max_pos;
+  int32_t norm_groups;
+  int32_t dtype; /* strictb200_dtype */
+  double eps;
+} strictb200_stack_config;
+int strictb200_stack_create(strictb200_ctx* ctx, const strictb200_stack_config* cfg, const strictb200_layer_config* layers, strictb200_model** out);
 /* Fill every tensor from the seeded generator (std 0.02, norm gains 1, biases 0). Under
  * tensor parallelism each rank generates only its own shard. */
 int strictb200_model_init_random(strictb200_model* m, uint64_t seed);
@@ -301,7 +332,8 @@ int strictb200_model_init_random(strictb200_model* m, uint64_t seed);
  * "layers.<i>.{norm1.g,norm1.b,norm2.g,norm2.b,qnorm.g,knorm.g}", Qwen3:
  * "layers.<i>.{wqkv,wo,wgu,wdown}.{q,s}", GPT-2: "layers.<i>.{wqkv,wo,wfc,wproj}.{w,b}".
  * fp32 host data except ".q" (E4M3 bytes); "embed" of a Qwen3 model is given as fp32 and
- * rounded to bf16. */
+ * rounded to bf16. Models described layer by layer: "embed", "head", "final.norm", "l<i>.norm1", "l<i>.norm2",
+ * "l<i>.mix.{q,dkv,dkv.norm,uk,uv,o}", "l<i>.mlp.{up,down,act}", host data bf16 or fp32 by its size. */
 int strictb200_model_set_tensor(strictb200_model* m, const char* name, const void* h_data, size_t bytes);
 int strictb200_model_get_tensor(strictb200_model* m, const char* name, void* h_data, size_t bytes);
 int strictb200_model_weight_bytes(strictb200_model* m, uint64_t* out);
@@ -319,6 +351,11 @@ int strictb200_kv_fill_synthetic(strictb200_kv* kv, uint64_t seed, int len);
  * fp32 logits [B,vocab] to h_logits. */
 int strictb200_prefill(strictb200_model* m, strictb200_kv* kv, const int32_t* h_tokens, const int32_t* h_lens, int B, int S,
                        int32_t* h_next, float* h_logits);
+/* The same with the logits of chosen rows: of sequence b the h_n_want[b] places h_want[..] (0 .. h_lens[b]-1 among the new
+ * tokens, the sequences' lists one after the other); h_logits receives one row of `vocab` values per place, in that order.
+ * h_want and h_logits may be NULL when no row is wanted. */
+int strictb200_prefill_rows(strictb200_model* m, strictb200_kv* kv, const int32_t* h_tokens, const int32_t* h_lens, int B, int S,
+                            const int32_t* h_want, const int32_t* h_n_want, int32_t* h_next, float* h_logits);
 /* One decode step for every sequence of the cache: h_ids[B] in, greedy next ids out. */
 int strictb200_decode_step(strictb200_model* m, strictb200_kv* kv, const int32_t* h_ids, int32_t* h_next, float* h_logits);
 /* n_steps greedy steps entirely on the device starting from h_ids; h_out [n_steps,B]. */
@@ -329,7 +366,9 @@ int strictb200_decode_steps_device(strictb200_model* m, strictb200_kv* kv, int32
 int strictb200_kv_device_ids(strictb200_kv* kv, int32_t** d_ids_out);
 /* 1 = capture the decode step in a CUDA graph and replay it (default), 0 = plain launches. */
 int strictb200_model_set_graph(strictb200_model* m, int enabled);
-/* Kernel classes of the Qwen3 decode step, for strictb200_profile_decode. */
+/* Kernel classes of the decode step, for strictb200_profile_decode. A step of a model described layer by layer reports
+ * under the nearest class: GEMM_QKV the layer's input product (feed-forward included), ROPE the kernel between it and the
+ * attention, GEMM_O the output product, ATTN_MERGE the merge with the value projection. */
 enum strictb200_kernel_class {
   STRICTB200_K_EMBED = 0,     /* embedding gather, length update */
   STRICTB200_K_GEMM_QKV = 1,

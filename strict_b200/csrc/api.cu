@@ -128,8 +128,9 @@ int sb_trace_set_gemm_split(const SbTraceDev&);  // one per instrumented transla
 int sb_trace_set_norm(const SbTraceDev&);
 int sb_trace_set_rope(const SbTraceDev&);
 int sb_trace_set_attention(const SbTraceDev&);
+int sb_trace_set_latent(const SbTraceDev&);
 static int trace_set_all(const SbTraceDev& t) {
-  return sb_trace_set_gemm_split(t) | sb_trace_set_norm(t) | sb_trace_set_rope(t) | sb_trace_set_attention(t);
+  return sb_trace_set_gemm_split(t) | sb_trace_set_norm(t) | sb_trace_set_rope(t) | sb_trace_set_attention(t) | sb_trace_set_latent(t);
 }
 
 extern "C" {

@@ -65,6 +65,11 @@ __device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map
                "l"(map), "r"(x), "r"(y), "r"(bar)
                : "memory");
 }
+__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
+  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];" ::"r"(dst),
+               "l"(map), "r"(x), "r"(y), "r"(z), "r"(bar)
+               : "memory");
+}
 __device__ __forceinline__ void set_status(int* status, int code) {
   *(volatile int*)status = code;
   __threadfence_system();
@@ -148,6 +153,13 @@ struct TcAttnArgs {
   float scale_log2;
   bf16* out;
   int* status;
+  // keys of a layer with per-head keys rebuilt from latents (LatentPrefillArgs); unused by the GQA form
+  const int32_t* koff;   // [B] row of the sequence's first key in the key and value arrays
+  const int32_t* kpos0;  // [B] position of that key
+  int window;            // keys a row sees, itself included
+  int nks_q, nks_r;      // 16-wide reduction steps of the unrotated and of the rotated part
+  int dv;                // value width
+  int64_t ldo;           // row stride of out
 };
 
 __global__ void __launch_bounds__(128) attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
@@ -384,13 +396,26 @@ __global__ void __launch_bounds__(128) attn_prefill_tc_kernel(const __grid_const
 //                while the A threads run their softmax the tensor pipe works on tile B, and so on
 //   warp 17      one lane issues the TMA copies into two-stage K and V rings
 // The whole tensor memory (512 columns) and 193 KB of shared memory: one block per SM.
+//
+// The tile shapes are parameters: a query/key row is QA 64-dim atoms of its own head followed by RA
+// atoms that all heads share on the key side (the rotated part of latent attention; its own array
+// and copy), a value row VA atoms. Head widths that do not fill their last atom are cut by the
+// tensor maps (dims x heads x rows), which fill with zeros; reduction steps beyond the width are not
+// issued. KST = stages of the K ring. WIN adds a sliding window: the walk over the key tiles begins
+// at the first tile any row of the block sees, and rows drop keys below their own window.
 constexpr int TC2_THREADS = 576;  // 16 softmax warps + MMA warp + TMA warp
 
-__global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+template <int QA, int RA, int VA, int KST>
+constexpr int tc2_tile_bytes() { return (2 * (QA + RA) + KST * (QA + RA) + 2 * VA) * HALF_BYTES; }
+
+template <int QA, int RA, int VA, int KST, bool WIN>
+__global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_qr,
+                                                                      const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_kr,
                                                                       const __grid_constant__ CUtensorMap map_v, TcAttnArgs a) {
+  constexpr int QK_BYTES = (QA + RA) * HALF_BYTES, V_BYTES = VA * HALF_BYTES;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
-  __shared__ __align__(8) uint64_t bar_q, k_full[2], k_empty[2], v_full[2], v_empty[2], bar_s[2], bar_p[2], bar_o[2];
+  __shared__ __align__(8) uint64_t bar_q, k_full[KST], k_empty[KST], v_full[2], v_empty[2], bar_s[2], bar_p[2], bar_o[2];
   __shared__ uint32_t tmem_base_slot;
   __shared__ float x_max[2][2][BQ], x_sum[2][BQ];  // [tile][column half][row]: exchange between the two threads of a row
 
@@ -399,20 +424,28 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
   const int n_new = len - pst;
   if (q0 >= n_new) return;  // whole block, before anything is allocated
   const int64_t row0 = a.qstart ? a.qstart[b] : (int64_t)b * a.S;
-  const int hk = h / (a.Hq / a.Hkv);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int kv_row0 = (b * a.Hkv + hk) * a.maxlen;
+  // position and row of the first key of the walk, and the head coordinate of the keys
+  int kp0 = 0, kv_row0, kh = 0;
+  if (RA) {
+    kh = h;
+    kp0 = a.kpos0[b];
+    if (WIN) kp0 += max(0, pst + q0 - a.window + 1 - kp0) / BKV * BKV;
+    kv_row0 = a.koff[b] + kp0 - a.kpos0[b];
+  } else {
+    kv_row0 = (b * a.Hkv + h / (a.Hq / a.Hkv)) * a.maxlen;
+  }
   // K/V tiles each query tile needs (tile B is empty when the sequence ends inside tile A)
   int nt[2];
-  nt[0] = (min(len, pst + q0 + BQ) + BKV - 1) / BKV;
-  nt[1] = q0 + BQ < n_new ? (min(len, pst + q0 + 2 * BQ) + BKV - 1) / BKV : 0;
+  nt[0] = (min(len, pst + q0 + BQ) - kp0 + BKV - 1) / BKV;
+  nt[1] = q0 + BQ < n_new ? (min(len, pst + q0 + 2 * BQ) - kp0 + BKV - 1) / BKV : 0;
   const int ntiles = max(nt[0], nt[1]);
 
-  const uint32_t sQ = smem_u32(smem), sK = sQ + 2 * TILE_BYTES, sV = sK + 2 * TILE_BYTES;
+  const uint32_t sQ = smem_u32(smem), sK = sQ + 2 * QK_BYTES, sV = sK + KST * QK_BYTES;
   if (threadIdx.x == 0) {
     mbar_init(smem_u32(&bar_q), 1);
     for (int i = 0; i < 2; i++) {
-      mbar_init(smem_u32(&k_full[i]), 1); mbar_init(smem_u32(&k_empty[i]), 1);
+      if (i < KST) { mbar_init(smem_u32(&k_full[i]), 1); mbar_init(smem_u32(&k_empty[i]), 1); }
       mbar_init(smem_u32(&v_full[i]), 1); mbar_init(smem_u32(&v_empty[i]), 1);
       mbar_init(smem_u32(&bar_s[i]), 1); mbar_init(smem_u32(&bar_p[i]), 2 * BQ); mbar_init(smem_u32(&bar_o[i]), 1);
     }
@@ -427,27 +460,26 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
   tc_fence_after();
   const uint32_t tmem = tmem_base_slot;
   constexpr uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(128 >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-  constexpr uint32_t idesc_pv = idesc_s | (1u << 16);
+  constexpr uint32_t idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(VA * 64 >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
 
   if (warp == 17) {
     // ---- TMA producer
     if (lane == 0) {
-      mbar_expect_tx(smem_u32(&bar_q), (nt[1] ? 2 : 1) * TILE_BYTES);
+      mbar_expect_tx(smem_u32(&bar_q), (nt[1] ? 2 : 1) * QK_BYTES);
       for (int w = 0; w < (nt[1] ? 2 : 1); w++) {
-        tma_load_2d(sQ + w * TILE_BYTES, &map_q, h * D, (int)(row0 + q0 + w * BQ), smem_u32(&bar_q));
-        tma_load_2d(sQ + w * TILE_BYTES + HALF_BYTES, &map_q, h * D + 64, (int)(row0 + q0 + w * BQ), smem_u32(&bar_q));
+        for (int i = 0; i < QA; i++) tma_load_3d(sQ + w * QK_BYTES + i * HALF_BYTES, &map_q, i * 64, h, (int)(row0 + q0 + w * BQ), smem_u32(&bar_q));
+        for (int i = 0; i < RA; i++) tma_load_3d(sQ + w * QK_BYTES + (QA + i) * HALF_BYTES, &map_qr, i * 64, h, (int)(row0 + q0 + w * BQ), smem_u32(&bar_q));
       }
       for (int t = 0; t < ntiles; t++) {
-        const int st = t & 1;
-        const uint32_t ph = (uint32_t)((t >> 1) & 1);
-        if (t >= 2 && !mbar_wait(smem_u32(&k_empty[st]), ph ^ 1)) { set_status(a.status, 11); break; }
-        mbar_expect_tx(smem_u32(&k_full[st]), TILE_BYTES);
-        tma_load_2d(sK + st * TILE_BYTES, &map_k, 0, kv_row0 + t * BKV, smem_u32(&k_full[st]));
-        tma_load_2d(sK + st * TILE_BYTES + HALF_BYTES, &map_k, 64, kv_row0 + t * BKV, smem_u32(&k_full[st]));
-        if (t >= 2 && !mbar_wait(smem_u32(&v_empty[st]), ph ^ 1)) { set_status(a.status, 12); break; }
-        mbar_expect_tx(smem_u32(&v_full[st]), TILE_BYTES);
-        tma_load_2d(sV + st * TILE_BYTES, &map_v, 0, kv_row0 + t * BKV, smem_u32(&v_full[st]));
-        tma_load_2d(sV + st * TILE_BYTES + HALF_BYTES, &map_v, 64, kv_row0 + t * BKV, smem_u32(&v_full[st]));
+        const int kst = t % KST, vst = t & 1;
+        const int row = kv_row0 + t * BKV;
+        if (t >= KST && !mbar_wait(smem_u32(&k_empty[kst]), (uint32_t)((t / KST) & 1) ^ 1)) { set_status(a.status, 11); break; }
+        mbar_expect_tx(smem_u32(&k_full[kst]), QK_BYTES);
+        for (int i = 0; i < QA; i++) tma_load_3d(sK + kst * QK_BYTES + i * HALF_BYTES, &map_k, i * 64, kh, row, smem_u32(&k_full[kst]));
+        for (int i = 0; i < RA; i++) tma_load_3d(sK + kst * QK_BYTES + (QA + i) * HALF_BYTES, &map_kr, i * 64, 0, row, smem_u32(&k_full[kst]));
+        if (t >= 2 && !mbar_wait(smem_u32(&v_empty[vst]), (uint32_t)((t >> 1) & 1) ^ 1)) { set_status(a.status, 12); break; }
+        mbar_expect_tx(smem_u32(&v_full[vst]), V_BYTES);
+        for (int i = 0; i < VA; i++) tma_load_3d(sV + vst * V_BYTES + i * HALF_BYTES, &map_v, i * 64, kh, row, smem_u32(&v_full[vst]));
       }
     }
   } else if (warp == 16) {
@@ -456,12 +488,13 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
     // the A threads are in the softmax of step t+1 the pipe works on tile B, and vice versa.
     if (lane == 0) {
       auto issue_s = [&](int w, int t) {
-        const int st = t & 1;
+        const int st = t % KST;
         const uint32_t tS = tmem + (uint32_t)(w * 256);
 #pragma unroll
-        for (int s = 0; s < 8; s++) {
+        for (int s = 0; s < 4 * (QA + RA); s++) {
+          if (RA && (s < 4 * QA ? s >= a.nks_q : s - 4 * QA >= a.nks_r)) continue;  // beyond the head's width
           const uint32_t off = (uint32_t)((s >> 2) * HALF_BYTES + (s & 3) * 32);
-          tc_mma_ss(tS, desc_kmajor(sQ + w * TILE_BYTES + off), desc_kmajor(sK + st * TILE_BYTES + off), idesc_s, s ? 1u : 0u);
+          tc_mma_ss(tS, desc_kmajor(sQ + w * QK_BYTES + off), desc_kmajor(sK + st * QK_BYTES + off), idesc_s, s ? 1u : 0u);
         }
         tc_commit(smem_u32(&bar_s[w]));
       };
@@ -485,7 +518,7 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
             const uint32_t tS = tmem + (uint32_t)(w * 256), tO = tS + 128;
 #pragma unroll
             for (int s = 0; s < 8; s++) {
-              const uint64_t dv = desc_mnmajor(sV + st * TILE_BYTES + (uint32_t)(s * 2048));
+              const uint64_t dv = desc_mnmajor(sV + st * V_BYTES + (uint32_t)(s * 2048));
               const uint32_t pcol = (uint32_t)((s >> 1) * 32 + (s & 1) * 8);
               tc_mma_ts(tO, tS + pcol, dv, idesc_pv, (t | s) ? 1u : 0u);
               tc_mma_ts(tO, tS + pcol + 16, dv, idesc_pv, 1u);
@@ -494,7 +527,7 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
           }
           if (t + 1 < nt[w]) {
             if (!k_next_ready) {
-              good = mbar_wait(smem_u32(&k_full[(t + 1) & 1]), (uint32_t)(((t + 1) >> 1) & 1));
+              good = mbar_wait(smem_u32(&k_full[(t + 1) % KST]), (uint32_t)(((t + 1) / KST) & 1));
               if (!good) break;
               tc_fence_after();
               k_next_ready = true;
@@ -504,7 +537,7 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
         }
         if (!good) break;
         tc_commit(smem_u32(&v_empty[st]));                               // both PV products have read the V tile
-        if (t + 1 < ntiles) tc_commit(smem_u32(&k_empty[(t + 1) & 1]));  // both S products of the next step have read its K tile
+        if (t + 1 < ntiles) tc_commit(smem_u32(&k_empty[(t + 1) % KST]));  // both S products of the next step have read its K tile
       }
       if (!good) set_status(a.status, 13);
     }
@@ -522,9 +555,10 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
       const uint32_t ph = (uint32_t)(t & 1);
       if (!mbar_wait(smem_u32(&bar_s[w]), ph)) { if (row == 0) set_status(a.status, 14); ok = false; break; }
       tc_fence_after();
-      const int k0 = t * BKV;
+      const int k0 = kp0 + t * BKV;
       const int k_lim = min(len, qpos + 1) - k0;
-      const bool full = k0 + BKV <= min(len, pst + qw + 1);
+      const int k_low = WIN ? qpos - a.window + 1 - k0 : 0;  // keys [k_low, k_lim) of the tile are visible to this row
+      const bool full = k0 + BKV <= min(len, pst + qw + 1) && (!WIN || pst + qw + BQ - a.window <= k0);
       float m_tile = -INFINITY;
 #pragma unroll 1
       for (int c = 2 * half; c < 2 * half + 2; c++) {
@@ -537,7 +571,7 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
         } else {
 #pragma unroll
           for (int j = 0; j < 32; j++)
-            if (c * 32 + j < k_lim) m_tile = fmaxf(m_tile, __uint_as_float(r[j]));
+            if (c * 32 + j < k_lim && (!WIN || c * 32 + j >= k_low)) m_tile = fmaxf(m_tile, __uint_as_float(r[j]));
         }
       }
       x_max[w][half][row] = m_tile;
@@ -552,7 +586,7 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
         if (!mbar_wait(smem_u32(&bar_o[w]), ph ^ 1)) { if (row == 0) set_status(a.status, 15); ok = false; break; }
         tc_fence_after();
 #pragma unroll 1
-        for (int c = 2 * half; c < 2 * half + 2; c++) {
+        for (int c = VA * half; c < VA * half + VA; c++) {
           uint32_t r[32];
           tc_ld32(tO + lane_base + (uint32_t)(c * 32), r);
           tc_wait_ld();
@@ -574,8 +608,8 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
           float p0 = ex2_approx(fmaf(__uint_as_float(r[2 * j]), a.scale_log2, -m_use));
           float p1 = ex2_approx(fmaf(__uint_as_float(r[2 * j + 1]), a.scale_log2, -m_use));
           if (!full) {
-            if (kk >= k_lim) p0 = 0.f;
-            if (kk + 1 >= k_lim) p1 = 0.f;
+            if (kk >= k_lim || (WIN && kk < k_low)) p0 = 0.f;
+            if (kk + 1 >= k_lim || (WIN && kk + 1 < k_low)) p1 = 0.f;
           }
           row_sum += p0 + p1;
           const uint32_t b0 = __float_as_uint(p0), b1 = __float_as_uint(p1);
@@ -603,15 +637,21 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
     if (ok && nt[w] > 0) {
       const bool live = qw + row < n_new;
       const float inv = 1.0f / x_sum[w][row];
-      bf16* dst = a.out + ((row0 + qw + row) * a.Hq + h) * D;
+      bf16* dst = RA ? a.out + (row0 + qw + row) * a.ldo + (int64_t)h * a.dv : a.out + ((row0 + qw + row) * a.Hq + h) * D;
+      const bool whole = !RA || (((a.dv & 7) == 0) && ((a.ldo & 7) == 0));
 #pragma unroll 1
-      for (int c = 2 * half; c < 2 * half + 2; c++) {
+      for (int c = VA * half; c < VA * half + VA; c++) {
         uint32_t r[32];
         tc_ld32(tO + lane_base + (uint32_t)(c * 32), r);
         tc_wait_ld();
-        if (live) {
+        if (live && !whole) {
+#pragma unroll
+          for (int i = 0; i < 32; i++)
+            if (c * 32 + i < a.dv) dst[c * 32 + i] = __float2bfloat16_rn(__uint_as_float(r[i]) * inv);
+        } else if (live) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
+            if (RA && c * 32 + i >= a.dv) break;
             uint4 wv;
             wv.x = f32_to_bf16_bits(__uint_as_float(r[i]) * inv) | (f32_to_bf16_bits(__uint_as_float(r[i + 1]) * inv) << 16);
             wv.y = f32_to_bf16_bits(__uint_as_float(r[i + 2]) * inv) | (f32_to_bf16_bits(__uint_as_float(r[i + 3]) * inv) << 16);
@@ -657,6 +697,29 @@ int make_map(CUtensorMap* map, const void* base, int64_t rows, int64_t cols, int
   return STRICTB200_OK;
 }
 
+// 3D map of bf16 rows of `heads` heads (width x heads x rows, strides in elements), box = 64 x 1 x 128, 128-byte swizzle.
+int make_map3(CUtensorMap* map, const void* base, int64_t width, int64_t heads, int64_t rows, int64_t head_stride, int64_t row_stride) {
+  cuuint64_t dims[3] = {(cuuint64_t)width, (cuuint64_t)heads, (cuuint64_t)rows};
+  cuuint64_t strides[2] = {(cuuint64_t)head_stride * 2, (cuuint64_t)row_stride * 2};
+  cuuint32_t box[3] = {64u, 1u, 128u};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = g_encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                        CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return sb_fail(STRICTB200_ERR_CUDA, "cuTensorMapEncodeTiled failed with code " + std::to_string((int)r));
+  return STRICTB200_OK;
+}
+
+template <int QA, int RA, int VA, int KST, bool WIN>
+int launch_tc2(strictb200_ctx* ctx, const CUtensorMap* m, const TcAttnArgs& a, int B, int S) {
+  const size_t smem = tc2_tile_bytes<QA, RA, VA, KST>() + 1024;
+  static SbDeviceOnce once;  // one per instantiation
+  SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(attn_prefill_tc2_kernel<QA, RA, VA, KST, WIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
+  dim3 grid((unsigned)((S + 2 * BQ - 1) / (2 * BQ)), (unsigned)a.Hq, (unsigned)B);
+  attn_prefill_tc2_kernel<QA, RA, VA, KST, WIN><<<grid, TC2_THREADS, smem, ctx->stream>>>(m[0], m[1], m[2], m[3], m[4], a);
+  SB_LAUNCHED(ctx);
+  return STRICTB200_OK;
+}
+
 }  // namespace
 
 // q, out: [q_rows, Hq, 128]; caches [B, Hkv, maxlen, 128]. ERR_UNSUPPORTED for shapes this kernel does not take.
@@ -666,6 +729,17 @@ int k_attn_prefill_tc(strictb200_ctx* ctx, const bf16* q, const bf16* kc, const 
   if ((int64_t)B * Hkv * maxlen > INT32_MAX || q_rows > INT32_MAX) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "attention: cache too large for 32-bit tile coordinates");
   if (((uintptr_t)q | (uintptr_t)kc | (uintptr_t)vc) & 15) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "attention: operands must be 16-byte aligned");
   SB_TRY(get_encode());
+  TcAttnArgs a{lens, past, qstart, S, Hq, Hkv, maxlen, scale * LOG2E, out, ctx->d_status, nullptr, nullptr, 0, 0, 0, D, (int64_t)Hq * D};
+  // two query tiles per block (ping-pong) from 256 new tokens per sequence on; the attn_tc option (1 / 2) forces a kernel
+  const int forced = ctx->opt.attn_tc;
+  if (forced == 2 || (forced != 1 && S >= 2 * BQ)) {
+    CUtensorMap m[5];
+    SB_TRY(make_map3(&m[0], q, D, Hq, q_rows, D, (int64_t)Hq * D));
+    SB_TRY(make_map3(&m[2], kc, D, 1, (int64_t)B * Hkv * maxlen, D, D));
+    SB_TRY(make_map3(&m[4], vc, D, 1, (int64_t)B * Hkv * maxlen, D, D));
+    m[1] = m[0]; m[3] = m[2];
+    return launch_tc2<2, 0, 2, 2, false>(ctx, m, a, B, S);
+  }
   CUtensorMap mq, mk, mv;
   SB_TRY(make_map(&mq, q, q_rows, (int64_t)Hq * D, (int64_t)Hq * D));
   SB_TRY(make_map(&mk, kc, (int64_t)B * Hkv * maxlen, D, D));
@@ -673,20 +747,36 @@ int k_attn_prefill_tc(strictb200_ctx* ctx, const bf16* q, const bf16* kc, const 
   const size_t smem = 3 * TILE_BYTES + 1024;
   static SbDeviceOnce once;
   SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
-  TcAttnArgs a{lens, past, qstart, S, Hq, Hkv, maxlen, scale * LOG2E, out, ctx->d_status};
-  // two query tiles per block (ping-pong) from 256 new tokens per sequence on; the attn_tc option (1 / 2) forces a kernel
-  const int forced = ctx->opt.attn_tc;
-  if (forced == 2 || (forced != 1 && S >= 2 * BQ)) {
-    const size_t smem2 = 6 * TILE_BYTES + 1024;
-    static SbDeviceOnce once2;
-    SB_CUDA(once2.run(ctx->device, [&] { return cudaFuncSetAttribute(attn_prefill_tc2_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2); }));
-    dim3 grid2((unsigned)((S + 2 * BQ - 1) / (2 * BQ)), (unsigned)Hq, (unsigned)B);
-    attn_prefill_tc2_kernel<<<grid2, TC2_THREADS, smem2, ctx->stream>>>(mq, mk, mv, a);
-    SB_LAUNCHED(ctx);
-    return STRICTB200_OK;
-  }
   dim3 grid((unsigned)((S + BQ - 1) / BQ), (unsigned)Hq, (unsigned)B);
   attn_prefill_tc_kernel<<<grid, 128, smem, ctx->stream>>>(mq, mk, mv, a);
   SB_LAUNCHED(ctx);
   return STRICTB200_OK;
+}
+
+bool sb_latent_prefill_fits(int dim, int rot, int vdim) { return dim <= 128 && rot <= 64 && vdim <= 128; }
+
+int k_attn_prefill_latent(strictb200_ctx* ctx, const LatentPrefillArgs& p) {
+  if (!sb_latent_prefill_fits(p.dim, p.rot, p.vdim)) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "latent prefill attention: head too wide for the tensor-core kernel");
+  if (p.H > 65535 || p.B > 65535 || p.q_rows > INT32_MAX || p.k_rows > INT32_MAX)
+    return sb_fail(STRICTB200_ERR_UNSUPPORTED, "latent prefill attention: too many heads, sequences or rows");
+  SB_TRY(get_encode());
+  TcAttnArgs a{};
+  a.lens = p.lens; a.past = p.past; a.qstart = p.qstart; a.S = p.S; a.Hq = p.H; a.Hkv = p.H;
+  a.scale_log2 = p.scale * LOG2E; a.out = p.out; a.status = ctx->d_status;
+  a.koff = p.koff; a.kpos0 = p.kpos0; a.window = p.window; a.nks_q = (p.dim + 15) / 16; a.nks_r = (p.rot + 15) / 16; a.dv = p.vdim; a.ldo = p.ldo;
+  CUtensorMap m[5];
+  SB_TRY(make_map3(&m[0], p.q, p.dim, p.H, p.q_rows, p.q_head, p.q_head * p.H));
+  SB_TRY(make_map3(&m[1], p.q + p.q_rot, p.rot, p.H, p.q_rows, p.q_head, p.q_head * p.H));
+  SB_TRY(make_map3(&m[2], p.k, p.dim, p.H, p.k_rows, p.k_head, p.ldk));
+  SB_TRY(make_map3(&m[3], p.k_rot, p.rot, 1, p.k_rows, p.ld_rot, p.ld_rot));
+  SB_TRY(make_map3(&m[4], p.v, p.vdim, p.H, p.k_rows, p.v_head, p.ldk));
+  const int S = p.S, B = p.B;
+#define LATENT_TC2(QA, VA, KST) return p.window > 0 ? launch_tc2<QA, 1, VA, KST, true>(ctx, m, a, B, S) : launch_tc2<QA, 1, VA, KST, false>(ctx, m, a, B, S)
+  if (p.dim <= 64) {
+    if (p.vdim <= 64) LATENT_TC2(1, 1, 2);
+    LATENT_TC2(1, 2, 2);
+  }
+  if (p.vdim <= 64) LATENT_TC2(2, 1, 1);
+  LATENT_TC2(2, 2, 1);  // three 64-dim atoms per query and key row: one stage of keys is what shared memory leaves
+#undef LATENT_TC2
 }

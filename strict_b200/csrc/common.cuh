@@ -204,6 +204,23 @@ struct RowNormArgs {
 int k_rownorm(strictb200_ctx*, const RowNormArgs& a, int64_t M, int64_t d);
 int k_reduce_scale(strictb200_ctx*, const float* part, int splits, const float* sx, const float* sw, int64_t M, int64_t N, float* out,
                    bf16* out_bf16 = nullptr);
+// Grouped RMS norm of the residual stream, one or two gains over one normalisation:
+//   x += sum over splits of part (when given); every group of d / groups consecutive columns is divided by its own root mean
+//   square; y1 = x_n * g1 and, with g2, y2 = x_n * g2, as bf16 or fp32 rows
+struct GroupNormArgs {
+  float* x = nullptr;            // [M, ldx] fp32 residual stream, in/out
+  int64_t ldx = 0;
+  const float* part = nullptr;   // [splits][M, ldp] raw sums of the projections that feed the residual, may be null
+  int64_t ldp = 0;
+  int splits = 1;
+  const float *g1 = nullptr, *g2 = nullptr;  // [d]; g1 null: only the residual update
+  float eps = 1e-5f;
+  int groups = 1;
+  void *y1 = nullptr, *y2 = nullptr;
+  int64_t ldy = 0;
+  bool f32 = false;              // y in fp32
+};
+int k_group_norm(strictb200_ctx*, const GroupNormArgs& a, int64_t M, int64_t d);
 int k_layernorm(strictb200_ctx*, const float* x, const float* g, const float* b, float eps, int64_t M, int64_t d, float* y);
 int k_add_f32(strictb200_ctx*, float* x, const float* y, int64_t n);
 int k_swiglu(strictb200_ctx*, const bf16* gate_up, const float* gate_up_f32, int64_t M, int64_t I, bf16* y, uint8_t* q, float* qscale);
@@ -216,6 +233,10 @@ int k_gelu_tanh(strictb200_ctx*, const float* x, int64_t n, float* y);
 __device__ __forceinline__ float sb_gelu_tanh(float v) {
   const float u = __fmul_rn(0.797884583f, __fadd_rn(v, __fmul_rn(0.044715f, __fmul_rn(__fmul_rn(v, v), v))));
   return __fmul_rn(__fmul_rn(0.5f, v), __fadd_rn(1.0f, tanhf(u)));
+}
+// xIELU: pos * z^2 + z/2 above zero, neg * (exp(z) - 1 - z) + z/2 below; pos = softplus(p), neg = 1/2 + softplus(q)
+__device__ __forceinline__ float sb_xielu(float z, float pos, float neg) {
+  return z > 0.f ? fmaf(pos * z, z, 0.5f * z) : fmaf(neg, expm1f(z) - z, 0.5f * z);
 }
 #endif
 // rope.cu
@@ -240,7 +261,7 @@ struct RopeArgs {
   bf16* vcache = nullptr;
 };
 int k_rope_qknorm_kvappend(strictb200_ctx*, const RopeArgs& a, int64_t T);
-int sb_rope_table(strictb200_ctx*, int max_pos, int D, float theta, float** d_cos, float** d_sin);
+int sb_rope_table(strictb200_ctx*, int max_pos, int D, double theta, float** d_cos, float** d_sin);
 // gemm_fp8.cu
 struct GemmArgs {
   int64_t M = 0, N = 0, K = 0;
@@ -260,12 +281,130 @@ struct GemmArgs {
 };
 int k_gemm_fp8(strictb200_ctx*, const GemmArgs& a);
 int sb_gemm_pick_splits(strictb200_ctx*, int64_t M, int64_t N, int64_t K);
+int sb_pick_splits_kb(strictb200_ctx*, int64_t M, int64_t N, int64_t nkb);  // the same rule for nkb K blocks of 128 bytes
+// gemm_bf16.cu: Y[M,N] = X[M,K] . W[N,K]^T, bf16 operands on the kernels of the E4M3 path (tcgen05 kind::f16), fp32 accumulation.
+// Where a finished value goes. Columns from n_switch on (0 = none) belong to a second product of the same launch: its
+// operand rows are x_row_off + m, and with act_out set the value leaves through the activation.
+struct Bf16Epilogue {
+  float* out_f32 = nullptr;   // [M, ldo]
+  bf16* out_bf16 = nullptr;   // [M, ldo] (used when out_f32 is null)
+  int64_t ldo = 0;
+  int accumulate = 0;         // out_f32 += value (the residual stream)
+  int n_switch = 0, x_row_off = 0;
+  bf16* act_out = nullptr;    // [M, ld_act], column n - n_switch
+  int64_t ld_act = 0;
+  float act_pos = 0.f, act_neg = 0.f;  // xIELU coefficients (sb_xielu)
+};
+struct GemmBf16Args {
+  int64_t M = 0, N = 0, K = 0;  // K in elements; rows may end inside a 64-element block (the copies fill with zeros)
+  const bf16* x = nullptr;
+  int64_t ldx = 0, x_rows = 0;  // rows of x that exist (0 = M)
+  const bf16* w = nullptr;
+  int64_t ldw = 0;
+  float* part = nullptr;        // [splits][M,N] raw sums instead of an epilogue
+  int splits = 1;
+  Bf16Epilogue e;
+};
+int k_gemm_bf16(strictb200_ctx*, const GemmBf16Args& g);
+int sb_gemm_bf16_splits(strictb200_ctx*, int64_t M, int64_t N, int64_t K);
 // gemm_f32.cu
 int k_gemm_f32(strictb200_ctx*, int64_t M, int64_t N, int64_t K, const float* x, const float* w, const float* bias, float* y,
                int accumulate);
+struct GemmF32Args {
+  int64_t M = 0, N = 0, K = 0;
+  const float* x = nullptr;
+  int64_t ldx = 0;
+  const float* w = nullptr;
+  int64_t ldw = 0;
+  const float* bias = nullptr;
+  float* y = nullptr;
+  int64_t ldy = 0;
+  int mode = 0;  // 0 store, 1 add to y, 2 GELU, 3 xIELU
+  float act_pos = 0.f, act_neg = 0.f;
+};
+int k_gemm_f32(strictb200_ctx*, const GemmF32Args& g);
 // attention.cu
 int k_attn_prefill(strictb200_ctx*, const bf16* q, const bf16* kc, const bf16* vc, const int32_t* lens, const int32_t* past,
                    const int32_t* qstart, int B, int S, int64_t q_rows, int Hq, int Hkv, int D, int maxlen, float scale, bf16* out);
+// attention_tc.cu: prompt rows of a latent-attention layer over keys and values rebuilt per head (kv_expand) and the shared rotated key part
+struct LatentPrefillArgs {
+  const bf16* q = nullptr;      // [q_rows, H, q_head]: the unrotated dims first, the rotated ones from q_rot on
+  int64_t q_rows = 0, q_head = 0, q_rot = 0;
+  const bf16* k = nullptr;      // row r, head h: k + r * ldk + h * k_head
+  const bf16* v = nullptr;      // row r, head h: v + r * ldk + h * v_head
+  int64_t k_rows = 0, ldk = 0, k_head = 0, v_head = 0;
+  const bf16* k_rot = nullptr;  // row r: k_rot + r * ld_rot
+  int64_t ld_rot = 0;
+  const int32_t *lens = nullptr, *past = nullptr, *qstart = nullptr;  // [B]
+  const int32_t *koff = nullptr, *kpos0 = nullptr;                    // [B] row and position of the first key of a sequence
+  int B = 0, S = 0, H = 0, dim = 0, rot = 0, vdim = 0;
+  int window = 0;               // 0: every earlier key
+  float scale = 1.f;
+  bf16* out = nullptr;          // row t, head h: out + t * ldo + h * vdim
+  int64_t ldo = 0;
+};
+bool sb_latent_prefill_fits(int dim, int rot, int vdim);
+int k_attn_prefill_latent(strictb200_ctx*, const LatentPrefillArgs& a);
+// latent.cu: latent attention (one low-rank vector and one rotated key part per position instead of keys and values per head)
+#ifdef __CUDACC__
+#define SB_HD __host__ __device__
+#else
+#define SB_HD
+#endif
+struct LatentShape {
+  int H = 0, dim = 0, rot = 0, vdim = 0, rank = 0;
+  int window = 0;                  // keys a position sees, itself included; 0 = every earlier one
+  float scale = 1.f;
+  SB_HD int dim_p() const { return (dim + 7) & ~7; }
+  SB_HD int kv_head() const { return ((dim > vdim ? dim : vdim) + 7) & ~7; }  // head stride of the rebuilt keys and values, one for both
+  SB_HD int rot8() const { return (rot + 7) & ~7; }
+  SB_HD int q_head() const { return dim_p() + rot8(); }   // head stride of the query buffer; the rotated part begins at dim_p
+  SB_HD int rank_p() const { return (rank + 15) & ~15; }  // a cache row: latent, rotated key part, each padded with zeros
+  SB_HD int row() const { return rank_p() + ((rot + 15) & ~15); }
+  SB_HD int n_q() const { return H * (dim + rot); }
+  SB_HD int n_kv() const { return 2 * H * kv_head(); }    // rows of the [uk | uv] matrix, ld = rank_p
+};
+// The projection's output becomes queries (rotated) and, for a layer with latents of its own, a cache row.
+struct LatentSplitArgs {
+  LatentShape s;
+  const float* in = nullptr;       // [splits][T, ld_in]: queries head by head, then latent and rotated key part
+  int64_t ld_in = 0;
+  int splits = 1;
+  const int32_t *seq = nullptr, *pos = nullptr, *lens = nullptr;  // row t: sequence seq[t] (null: t) at pos[t] (null: lens[seq])
+  const float *cos_t = nullptr, *sin_t = nullptr;                 // [max_pos, rot/2]
+  int max_pos = 0, maxlen = 0;
+  const float* norm_w = nullptr;   // [rank]
+  float eps = 1e-5f;
+  void* q_out = nullptr;           // [T, H, q_head]
+  void* cache = nullptr;           // [B, maxlen, row]; null: the layer reads another layer's latents
+  bool f32 = false;
+};
+int k_latent_split(strictb200_ctx*, const LatentSplitArgs& a, int64_t T);
+// The decode step's form: the same, with the queries carried into latent space (q . W_uk per head), and the feed-forward
+// half of the projection through its activation.
+struct LatentDecodeInArgs {
+  LatentSplitArgs a;
+  const bf16* wkv = nullptr;       // [n_kv, rank_p]
+  bf16* q_abs = nullptr;           // [B, H, row]
+  int act_col = 0, n_act = 0;      // columns [act_col, act_col + n_act) of `in` through xIELU to act[b * ld_act + i]
+  float act_pos = 0.f, act_neg = 0.f;
+  bf16* act = nullptr;
+  int64_t ld_act = 0;
+};
+bool sb_latent_decode_fits(const LatentShape& s);
+int k_latent_decode_in(strictb200_ctx*, const LatentDecodeInArgs& a, int64_t B);
+// Split-key attention of one new token per sequence over the latents of its window, then the merge of the key chunks and the
+// value projection of every head. len_plan: lengths the chunks are planned for.
+int sb_latent_decode_chunk(strictb200_ctx*, const LatentShape& s, int B, int len_plan);
+size_t sb_latent_decode_scratch(const LatentShape& s, int B);
+int k_latent_attn_decode(strictb200_ctx*, const LatentShape& s, const bf16* q_abs, const bf16* cache, const int32_t* lens, int B, int maxlen, int chunk,
+                         int nsplit, float* scratch, const bf16* wkv, bf16* out, int64_t ldo);
+// Any widths, bf16 or fp32, prompt rows and decode rows: one block per row and head, straight from the cache.
+int k_latent_attn_any(strictb200_ctx*, const LatentShape& s, bool f32, const void* q, const void* cache, const void* wkv, const int32_t* seq,
+                      const int32_t* pos, const int32_t* lens, int64_t T, int maxlen, void* out, int64_t ldo);
+// rows of the cache of several sequences one after the other: dst row koff[j] + i = cache row kpos0[j] + i of sequence j, i < n[j]
+int k_latent_gather(strictb200_ctx*, const bf16* cache, int64_t maxlen, int row, const int32_t* koff, const int32_t* kpos0, const int32_t* lens, int nb,
+                    int max_n, bf16* dst);
 size_t sb_attn_decode_scratch(int B, int Hq, int D, int nsplit);
 int sb_attn_decode_splits(strictb200_ctx*, int B, int Hkv, int maxlen);
 int sb_attn_decode_chunk(strictb200_ctx*, int B, int Hkv, int maxlen, int len_plan);  // keys per block for sequences of about len_plan keys (at most 8 chunks cover maxlen)
@@ -301,6 +440,17 @@ void sb_tp_abort(strictb200_ctx*);       // ncclCommAbort: stops the communicato
 
 // ------------------------------------------------------------------ device helpers
 #ifdef __CUDACC__
+// One finished value of a bf16 GEMM (Bf16Epilogue).
+__device__ __forceinline__ void sb_bf16_store(const Bf16Epilogue& e, int64_t m, int n, float v) {
+  if (e.act_out && n >= e.n_switch) {
+    e.act_out[m * e.ld_act + (n - e.n_switch)] = __float2bfloat16_rn(sb_xielu(v, e.act_pos, e.act_neg));
+  } else if (e.out_f32) {
+    float* o = e.out_f32 + m * e.ldo + n;
+    *o = e.accumulate ? *o + v : v;
+  } else {
+    e.out_bf16[m * e.ldo + n] = __float2bfloat16_rn(v);
+  }
+}
 // Programmatic dependent launch. A kernel launched through sb_launch may begin while its
 // predecessor in the stream is still running: pdl_trigger() lets the successor start launching,
 // pdl_wait() blocks until the predecessor has completed and its writes are visible. Every such

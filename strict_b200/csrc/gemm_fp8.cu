@@ -263,7 +263,10 @@ int launch_skinny(strictb200_ctx* ctx, const GemmDev& d) {
 // Number of K splits for a skinny GEMM so that the grid covers the SMs about twice.
 int sb_gemm_pick_splits(strictb200_ctx* ctx, int64_t M, int64_t N, int64_t K) {
   if (M > 128 || K % 128) return 1;
-  const int64_t tiles = (N + SK_ROWS - 1) / SK_ROWS, nkb = K / 128;
+  return sb_pick_splits_kb(ctx, M, N, K / 128);
+}
+int sb_pick_splits_kb(strictb200_ctx* ctx, int64_t M, int64_t N, int64_t nkb) {
+  const int64_t tiles = (N + SK_ROWS - 1) / SK_ROWS;
   if (M > 32) {
     // 33..128 tokens: one block per SM fits (its ring fills the shared memory); split K until the grid covers the GPU
     int64_t s = ctx->sm_count / tiles;

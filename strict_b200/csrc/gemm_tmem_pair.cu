@@ -127,6 +127,17 @@ __device__ __forceinline__ uint64_t smem_desc(uint32_t addr) {
   return (uint64_t)((addr >> 4) & 0x3FFF) | (1ull << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
 }
 
+// The same with bf16 operands (K = 16 elements = the same 32 bytes per instruction).
+__device__ __forceinline__ void tc_mma_bf16_pair(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::2.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5, %5, %5, %5, %5}, p;\n\t}"
+      :
+      : "r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(0u)
+      : "memory");
+}
+
 struct PairArgs {
   int M, Mq, N, K;
   const float* sx;
@@ -136,8 +147,12 @@ struct PairArgs {
   int* status;   // host-visible error word
   int tiles_n;   // 256-channel tiles; tile = tt * tiles_n + tn
   int tiles;
+  Bf16Epilogue e;  // BF16 only
 };
 
+// BF16: plain bf16 operands, one operand row (accumulator column) per token, so a tile is 256 channels x 256 tokens; K
+// counts bytes, and a row that ends inside a 128-byte block is filled with zeros by the copy.
+template <bool BF16>
 __global__ void __launch_bounds__(192) gemm_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                                                         PairArgs a) {
   extern __shared__ __align__(1024) uint8_t smem_raw[];
@@ -150,7 +165,7 @@ __global__ void __launch_bounds__(192) gemm_pair_kernel(const __grid_constant__ 
   uint32_t rank;
   asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(rank));
   const bool leader = rank == 0;
-  const int nkb = a.K / BK;
+  const int nkb = (a.K + BK - 1) / BK;
   const int pairs = gridDim.x / 2, c = blockIdx.x / 2;
   const int tile_begin = (int)((int64_t)c * a.tiles / pairs), tile_end = (int)((int64_t)(c + 1) * a.tiles / pairs);
   const int n_my = (tile_end - tile_begin) * nkb;  // K blocks this pair walks through
@@ -181,7 +196,8 @@ __global__ void __launch_bounds__(192) gemm_pair_kernel(const __grid_constant__ 
         if (it >= STAGES && !mbar_wait(smem_u32(&bar_empty[s]), ((it / STAGES) & 1) ^ 1)) { set_status(a.status, 1); abort_flag = 1; break; }
         if (*(volatile int*)&abort_flag) break;
         const int tile = tile_begin + it / nkb, kb = it % nkb;
-        const int wy = (tile % a.tiles_n) * 2 * BN + (int)rank * BN, xy = (tile / a.tiles_n) * 2 * BTH + (int)rank * BTH;
+        const int wy = (tile % a.tiles_n) * 2 * BN + (int)rank * BN, xy0 = (tile / a.tiles_n) * 2 * BTH + (int)rank * BTH;
+        const int xy = BF16 && a.e.n_switch > 0 && (tile % a.tiles_n) * 2 * BN >= a.e.n_switch ? a.e.x_row_off + xy0 : xy0;
         const uint32_t full_leader = map_to_rank(smem_u32(&bar_full[s]), 0);
         if (leader) mbar_expect_tx(smem_u32(&bar_full[s]), 2 * STAGE_BYTES);  // the bytes of both blocks
         const uint32_t dst = smem_u32(smem + (size_t)s * STAGE_BYTES);
@@ -191,8 +207,8 @@ __global__ void __launch_bounds__(192) gemm_pair_kernel(const __grid_constant__ 
     }
   } else if (warp == 1) {
     if (leader && lane == 0) {
-      // instruction descriptor: D = F32, A = B = E4M3, both K-major, N = 256 (>> 3 at bit 17), M = 256 (>> 4 at bit 24)
-      constexpr uint32_t idesc = (1u << 4) | ((uint32_t)(256 >> 3) << 17) | ((uint32_t)(256 >> 4) << 24);
+      // instruction descriptor: D = F32, A = B = E4M3 (or bf16), both K-major, N = 256 (>> 3 at bit 17), M = 256 (>> 4 at bit 24)
+      constexpr uint32_t idesc = (1u << 4) | (BF16 ? (1u << 7) | (1u << 10) : 0u) | ((uint32_t)(256 >> 3) << 17) | ((uint32_t)(256 >> 4) << 24);
       // The operand tiles cannot arrive before the producer's dependency wait has returned; waiting for the same
       // dependency here keeps the bounded waits below for progress inside this kernel (a predecessor that itself
       // waits for another rank may take longer than any of them).
@@ -212,7 +228,8 @@ __global__ void __launch_bounds__(192) gemm_pair_kernel(const __grid_constant__ 
         const uint32_t acc = tmem + (uint32_t)((seg & 1) * ACC_COLS);
 #pragma unroll
         for (int k = 0; k < BK / UMMA_K; k++)
-          tc_mma_f8_pair(acc, da + (uint64_t)(k * (UMMA_K >> 4)), db + (uint64_t)(k * (UMMA_K >> 4)), idesc, (kb | k) ? 1u : 0u);
+          if (BF16) tc_mma_bf16_pair(acc, da + (uint64_t)(k * (UMMA_K >> 4)), db + (uint64_t)(k * (UMMA_K >> 4)), idesc, (kb | k) ? 1u : 0u);
+          else tc_mma_f8_pair(acc, da + (uint64_t)(k * (UMMA_K >> 4)), db + (uint64_t)(k * (UMMA_K >> 4)), idesc, (kb | k) ? 1u : 0u);
         tc_commit_pair(smem_u32(&bar_empty[s]));                             // the stage is free in both blocks
         if (kb == nkb - 1) tc_commit_pair(smem_u32(&bar_acc_full[seg & 1]));  // accumulator complete, both blocks
       }
@@ -231,12 +248,19 @@ __global__ void __launch_bounds__(192) gemm_pair_kernel(const __grid_constant__ 
       const uint32_t acc = tmem + (uint32_t)((seg & 1) * ACC_COLS) + ((uint32_t)(lg * 32) << 16);
       const int n = (tile % a.tiles_n) * 2 * BN + (int)rank * BN + ch;
       const int tok_base = (tile / a.tiles_n) * BTH;  // 256 operand rows = 128 tokens per tile
-      const float swn = n < a.N ? a.sw[n] : 0.f;
+      const float swn = !BF16 && n < a.N ? a.sw[n] : 0.f;
 #pragma unroll 1
       for (int grp = 0; grp < ACC_COLS / 16; grp++) {
         uint32_t r[16];
         tc_ld16(acc + (uint32_t)(grp * 16), r);
         tc_wait_ld();
+        if constexpr (BF16) {
+#pragma unroll
+          for (int j = 0; j < 16; j++) {
+            const int tok = 2 * tok_base + grp * 16 + j;  // 256 tokens per tile
+            if (tok < a.M && n < a.N) sb_bf16_store(a.e, tok, n, __uint_as_float(r[j]));
+          }
+        } else {
 #pragma unroll
         for (int j = 0; j < 8; j++) {
           const int tok = tok_base + grp * 8 + j;  // operand rows 16g.. hold tokens 8g..
@@ -246,6 +270,7 @@ __global__ void __launch_bounds__(192) gemm_pair_kernel(const __grid_constant__ 
             if (a.out_f32) ((float*)a.out)[(int64_t)tok * a.N + n] = y;
             else ((bf16*)a.out)[(int64_t)tok * a.N + n] = __float2bfloat16_rn(y);
           }
+        }
         }
       }
       // the accumulator is drained in this block: tell the leader's MMA warp
@@ -301,14 +326,33 @@ int k_gemm_fp8_tmem_pair(strictb200_ctx* ctx, const GemmArgs& g) {
   if (tiles > INT32_MAX / 2) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_fp8: too many output tiles");
   const size_t smem = (size_t)STAGES * STAGE_BYTES + 1024;  // + slack for the 1024-byte round-up
   static SbDeviceOnce once;
-  SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(gemm_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
+  SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(gemm_pair_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
   CUtensorMap mw, mx;
   SB_TRY(make_map(&mw, g.wq, g.N, g.K, g.ldw));
   SB_TRY(make_map(&mx, g.xq, Mq, g.K, g.ldx));
-  PairArgs pa{(int)g.M, (int)Mq, (int)g.N, (int)g.K, g.sx, g.sw, g.out, g.out_f32, ctx->d_status, (int)tiles_n, (int)tiles};
+  PairArgs pa{(int)g.M, (int)Mq, (int)g.N, (int)g.K, g.sx, g.sw, g.out, g.out_f32, ctx->d_status, (int)tiles_n, (int)tiles, {}};
   int64_t pairs = ctx->sm_count / 2;
   if (pairs > tiles) pairs = tiles;
-  SB_CUDA(sb_launch_cluster(ctx, gemm_pair_kernel, dim3((unsigned)(2 * pairs)), dim3(192), smem, dim3(2, 1, 1), mw, mx, pa));
+  SB_CUDA(sb_launch_cluster(ctx, gemm_pair_kernel<false>, dim3((unsigned)(2 * pairs)), dim3(192), smem, dim3(2, 1, 1), mw, mx, pa));
+  ctx->launches++;
+  return STRICTB200_OK;
+}
+
+// The same for bf16 operands, finished values through b.e.
+int k_gemm_bf16_tmem_pair(strictb200_ctx* ctx, const GemmBf16Args& b) {
+  SB_TRY(get_encode());
+  const int64_t kbytes = 2 * b.K, tiles_n = (b.N + 2 * BN - 1) / (2 * BN), tiles_t = (b.M + 2 * BTH - 1) / (2 * BTH), tiles = tiles_n * tiles_t;
+  if (tiles > INT32_MAX / 2) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_bf16: too many output tiles");
+  const size_t smem = (size_t)STAGES * STAGE_BYTES + 1024;
+  static SbDeviceOnce once;
+  SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(gemm_pair_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
+  CUtensorMap mw, mx;
+  SB_TRY(make_map(&mw, b.w, b.N, kbytes, 2 * b.ldw));
+  SB_TRY(make_map(&mx, b.x, b.x_rows ? b.x_rows : b.M, kbytes, 2 * b.ldx));
+  PairArgs pa{(int)b.M, (int)b.M, (int)b.N, (int)kbytes, nullptr, nullptr, nullptr, 1, ctx->d_status, (int)tiles_n, (int)tiles, b.e};
+  int64_t pairs = ctx->sm_count / 2;
+  if (pairs > tiles) pairs = tiles;
+  SB_CUDA(sb_launch_cluster(ctx, gemm_pair_kernel<true>, dim3((unsigned)(2 * pairs)), dim3(192), smem, dim3(2, 1, 1), mw, mx, pa));
   ctx->launches++;
   return STRICTB200_OK;
 }

@@ -74,6 +74,16 @@ __device__ __forceinline__ void tc_mma_f8(uint32_t tmem_d, uint64_t desc_a, uint
       : "r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(0u)
       : "memory");
 }
+// bf16 operands (K = 16 elements = the same 32 bytes per instruction).
+__device__ __forceinline__ void tc_mma_bf16(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
+      :
+      : "r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(0u)
+      : "memory");
+}
 // Signed 8-bit integer operands, 32-bit integer accumulator (same operand layout and K = 32 per instruction).
 __device__ __forceinline__ void tc_mma_i8(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
   asm volatile(
@@ -112,14 +122,19 @@ struct TmemArgs {
   int raw;
   int* status;  // host-visible error word
   int prefetch;  // issue the first ring of weight loads before the dependency wait
+  Bf16Epilogue e;  // BF16 only
 };
+enum { KIND_F8 = 0, KIND_I8 = 1, KIND_BF16 = 2 };
 
 // I8: both operands are signed 8-bit integers (weights int8, activations as two int8 terms
 // x = s * (128 * hi + lo), gemm_int8.cu) and the accumulators 32-bit integers; the epilogue joins
 // the two terms in 64-bit integers, so the result does not depend on the K split or on any order.
-template <int BT, int STAGES, bool I8>
+// BF16: plain bf16 operands, one operand row (accumulator column) per token; K counts bytes all the
+// same, and a row that ends inside a 128-byte block is filled with zeros by the copy.
+template <int BT, int STAGES, int KIND>
 __global__ void __launch_bounds__(192) gemm_tmem_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                                                         TmemArgs a) {
+  constexpr bool I8 = KIND == KIND_I8;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   // dynamic shared memory is only guaranteed 16-byte aligned: round up to the 1024 the swizzle needs
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -133,7 +148,8 @@ __global__ void __launch_bounds__(192) gemm_tmem_kernel(const __grid_constant__ 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n0 = blockIdx.x * BN, t0 = blockIdx.y * BT;
   // split z owns the k-blocks [z * nkb_all / splits, (z + 1) * nkb_all / splits): sizes differ by at most one
-  const int nkb_all = a.K / BK;
+  const int nkb_all = (a.K + BK - 1) / BK;
+  const int x0 = KIND == KIND_BF16 && a.e.n_switch > 0 && n0 >= a.e.n_switch ? a.e.x_row_off + t0 : t0;  // first operand row
   const int kb_first = (int)((int64_t)blockIdx.z * nkb_all / a.splits), kb_last = (int)((int64_t)(blockIdx.z + 1) * nkb_all / a.splits);
   const int k_begin = kb_first * BK, nkb = kb_last - kb_first;
 
@@ -169,7 +185,7 @@ __global__ void __launch_bounds__(192) gemm_tmem_kernel(const __grid_constant__ 
       pdl_wait();
       SB_TRACE_WAITED();
       for (int kb = 0; kb < npre; kb++)
-        tma_load_2d(smem_u32(smem + (size_t)kb * STAGE_BYTES) + BN * BK, &map_x, k_begin + kb * BK, t0, smem_u32(&bar_full[kb]));
+        tma_load_2d(smem_u32(smem + (size_t)kb * STAGE_BYTES) + BN * BK, &map_x, k_begin + kb * BK, x0, smem_u32(&bar_full[kb]));
       for (int kb = npre; kb < nkb; kb++) {
         int s = kb % STAGES;
         if (!mbar_wait(smem_u32(&bar_empty[s]), ((kb / STAGES) & 1) ^ 1)) { set_status(a.status, 1); abort_flag = 1; break; }
@@ -178,14 +194,14 @@ __global__ void __launch_bounds__(192) gemm_tmem_kernel(const __grid_constant__ 
         uint32_t dst = smem_u32(smem + (size_t)s * STAGE_BYTES);
         mbar_expect_tx(full, STAGE_BYTES);
         tma_load_2d_hint(dst, &map_w, k_begin + kb * BK, n0, full, w_policy);
-        tma_load_2d(dst + BN * BK, &map_x, k_begin + kb * BK, t0, full);
+        tma_load_2d(dst + BN * BK, &map_x, k_begin + kb * BK, x0, full);
       }
     }
   } else if (warp == 1) {
     if (lane == 0) {
       // instruction descriptor: D = F32 (bits 4-5 = 1), A = B = E4M3 (0), both K-major, N >> 3 at bit 17, M >> 4 at bit 24;
-      // integers: D = S32 (bits 4-5 = 2), A (bits 7-9) = B (bits 10-12) = signed 8 bit (1)
-      constexpr uint32_t idesc = (I8 ? (2u << 4) | (1u << 7) | (1u << 10) : (1u << 4)) | ((uint32_t)(BT >> 3) << 17) | ((uint32_t)(BN >> 4) << 24);
+      // integers: D = S32 (bits 4-5 = 2), A (bits 7-9) = B (bits 10-12) = signed 8 bit (1); bf16: D = F32, A = B = bf16 (1)
+      constexpr uint32_t idesc = (I8 ? (2u << 4) | (1u << 7) | (1u << 10) : KIND == KIND_BF16 ? (1u << 4) | (1u << 7) | (1u << 10) : (1u << 4)) | ((uint32_t)(BT >> 3) << 17) | ((uint32_t)(BN >> 4) << 24);
       // The operand tiles cannot arrive before the producer's dependency wait has returned; waiting for the same
       // dependency here keeps the bounded waits below for progress inside this kernel (a predecessor that itself
       // waits for another rank may take longer than any of them).
@@ -201,6 +217,7 @@ __global__ void __launch_bounds__(192) gemm_tmem_kernel(const __grid_constant__ 
         for (int k = 0; k < BK / UMMA_K; k++) {
           // +32 bytes of K inside the swizzle atom = +2 in the (address >> 4) field
           if (I8) tc_mma_i8(tmem, da + (uint64_t)(k * (UMMA_K >> 4)), db + (uint64_t)(k * (UMMA_K >> 4)), idesc, (kb | k) ? 1u : 0u);
+          else if (KIND == KIND_BF16) tc_mma_bf16(tmem, da + (uint64_t)(k * (UMMA_K >> 4)), db + (uint64_t)(k * (UMMA_K >> 4)), idesc, (kb | k) ? 1u : 0u);
           else tc_mma_f8(tmem, da + (uint64_t)(k * (UMMA_K >> 4)), db + (uint64_t)(k * (UMMA_K >> 4)), idesc, (kb | k) ? 1u : 0u);
         }
         tc_commit(smem_u32(&bar_empty[s]));  // stage is free once these MMAs have read it
@@ -218,12 +235,23 @@ __global__ void __launch_bounds__(192) gemm_tmem_kernel(const __grid_constant__ 
     tc_fence_after();
     if (ok) {
       const bool raw = a.raw || a.splits > 1;
-      const float swn = (!raw && n < a.N) ? a.sw[n] : 0.f;
+      const float swn = (KIND != KIND_BF16 && !raw && n < a.N) ? a.sw[n] : 0.f;
 #pragma unroll 1
       for (int grp = 0; grp < BT / 16; grp++) {
         uint32_t r[16];
         tc_ld16(tmem + ((uint32_t)(lg * 32) << 16) + (uint32_t)(grp * 16), r);
         tc_wait_ld();
+        if (KIND == KIND_BF16) {
+#pragma unroll
+          for (int j = 0; j < 16; j++) {
+            const int tok = t0 + grp * 16 + j;
+            if (tok < a.M && n < a.N) {
+              if (raw) a.part[((int64_t)blockIdx.z * a.M + tok) * a.N + n] = __uint_as_float(r[j]);
+              else sb_bf16_store(a.e, tok, n, __uint_as_float(r[j]));
+            }
+          }
+          continue;
+        }
         const int tok0 = ((t0 + grp * 16) >> 1);  // operand rows 16g.. hold tokens 8g..
 #pragma unroll
         for (int j = 0; j < 8; j++) {
@@ -261,7 +289,7 @@ __global__ void __launch_bounds__(192) gemm_tmem_kernel(const __grid_constant__ 
     tc_fence_after();
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"((uint32_t)TMEM_COLS) : "memory");
   }
-  SB_TRACE_END(SB_K_GEMM, (uint32_t)a.N ^ ((uint32_t)a.K << 12));
+  SB_TRACE_END(SB_K_GEMM, (uint32_t)a.N ^ ((uint32_t)(KIND == KIND_BF16 ? a.K / 2 : a.K) << 12));
 }
 
 typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
@@ -290,18 +318,18 @@ int make_map(CUtensorMap* map, const void* base, int64_t rows, int64_t K, int64_
   return STRICTB200_OK;
 }
 
-template <int BT, int STAGES, bool I8 = false>
-int launch(strictb200_ctx* ctx, const GemmArgs& g, const TmemArgs& ta) {
+template <int BT, int STAGES, int KIND = KIND_F8>
+int launch(strictb200_ctx* ctx, const GemmArgs& g, const TmemArgs& ta, int64_t x_rows = 0) {
   constexpr int STAGE_BYTES = BN * BK + BT * BK;
   size_t smem = (size_t)STAGES * STAGE_BYTES + 1024;  // + slack for the 1024-byte round-up
   static SbDeviceOnce once;  // one per instantiation
-  SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(gemm_tmem_kernel<BT, STAGES, I8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
+  SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(gemm_tmem_kernel<BT, STAGES, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
   CUtensorMap mw, mx;
   SB_TRY(make_map(&mw, g.wq, g.N, g.K, g.ldw, BN));
-  SB_TRY(make_map(&mx, g.xq, ta.Mq, g.K, g.ldx, BT));
+  SB_TRY(make_map(&mx, g.xq, x_rows ? x_rows : ta.Mq, g.K, g.ldx, BT));
   dim3 grid((unsigned)((g.N + BN - 1) / BN), (unsigned)((ta.Mq + BT - 1) / BT), (unsigned)g.splits);
   if (grid.y > 65535) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_fp8: M too large for one launch");
-  SB_CUDA(sb_launch(ctx, gemm_tmem_kernel<BT, STAGES, I8>, grid, dim3(192), smem, mw, mx, ta));
+  SB_CUDA(sb_launch(ctx, gemm_tmem_kernel<BT, STAGES, KIND>, grid, dim3(192), smem, mw, mx, ta));
   ctx->launches++;
   return STRICTB200_OK;
 }
@@ -325,14 +353,33 @@ int k_gemm_fp8_tmem_split(strictb200_ctx* ctx, const GemmArgs& g) {
   const int64_t blocks = ((g.N + BN - 1) / BN) * g.splits;
   const int deep = ctx->opt.deep_ring;
   if (g.i8) {  // integer operands: the same tiles; token tiles beyond the first go to grid.y
-    if (ta.Mq <= 32) return launch<32, 5, true>(ctx, g, ta);
-    if (ta.Mq <= 64) return launch<64, 4, true>(ctx, g, ta);
-    if (ta.Mq <= 128) return launch<128, 4, true>(ctx, g, ta);
-    return launch<256, 4, true>(ctx, g, ta);
+    if (ta.Mq <= 32) return launch<32, 5, KIND_I8>(ctx, g, ta);
+    if (ta.Mq <= 64) return launch<64, 4, KIND_I8>(ctx, g, ta);
+    if (ta.Mq <= 128) return launch<128, 4, KIND_I8>(ctx, g, ta);
+    return launch<256, 4, KIND_I8>(ctx, g, ta);
   }
   if (ta.Mq <= 32) return deep && blocks <= ctx->sm_count ? launch<32, 10>(ctx, g, ta) : launch<32, 5>(ctx, g, ta);
   if (ta.Mq <= 64) return deep && blocks <= ctx->sm_count ? launch<64, 9>(ctx, g, ta) : launch<64, 4>(ctx, g, ta);
   if (ta.Mq <= 128) return launch<128, 4>(ctx, g, ta);
   if (ta.Mq <= 256) return launch<256, 4>(ctx, g, ta);
   return sb_fail(STRICTB200_ERR_UNSUPPORTED, "the split tensor-memory GEMM takes at most 128 tokens");
+}
+
+// bf16 operands: at most 256 tokens (one operand row each). Raw partials per K split, or finished values through g.e.
+int k_gemm_bf16_tmem_split(strictb200_ctx* ctx, const GemmBf16Args& b) {
+  const int64_t kbytes = 2 * b.K, nkb = (kbytes + BK - 1) / BK;
+  if (b.splits < 1 || b.splits > nkb) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_bf16: more K splits than K blocks");
+  if (b.splits > 1 && !b.part) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_bf16: split-K needs a partial buffer");
+  if (b.M > 256) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "the split bf16 GEMM takes at most 256 tokens");
+  SB_TRY(get_encode());
+  TmemArgs ta{(int)b.M, (int)b.M, (int)b.N, (int)kbytes, nullptr, nullptr, nullptr, 1, b.part, b.splits, b.part ? 1 : 0, ctx->d_status, ctx->opt.prefetch, b.e};
+  GemmArgs g;
+  g.M = b.M; g.N = b.N; g.K = kbytes;
+  g.xq = (const uint8_t*)b.x; g.ldx = 2 * b.ldx; g.wq = (const uint8_t*)b.w; g.ldw = 2 * b.ldw; g.splits = b.splits;
+  const int64_t blocks = ((b.N + BN - 1) / BN) * b.splits, x_rows = b.x_rows ? b.x_rows : b.M;
+  const bool deep = ctx->opt.deep_ring && blocks <= ctx->sm_count;
+  if (b.M <= 32) return deep ? launch<32, 10, KIND_BF16>(ctx, g, ta, x_rows) : launch<32, 5, KIND_BF16>(ctx, g, ta, x_rows);
+  if (b.M <= 64) return deep ? launch<64, 9, KIND_BF16>(ctx, g, ta, x_rows) : launch<64, 4, KIND_BF16>(ctx, g, ta, x_rows);
+  if (b.M <= 128) return launch<128, 4, KIND_BF16>(ctx, g, ta, x_rows);
+  return launch<256, 4, KIND_BF16>(ctx, g, ta, x_rows);
 }

@@ -11,110 +11,9 @@
 //     head  = this rank's slice of the vocabulary rows
 //   embedding bf16 [V, d] (replicated); norm gains fp32; RoPE cos/sin fp32 [max_pos, D/2]
 //   KV cache bf16 [L][B][Hkv_local][maxlen][D] for K and for V (fp32 for GPT-2)
-#include <algorithm>
-#include <cstring>
-#include <string>
-#include <vector>
-
-#include "common.cuh"
+#include "model.cuh"
 
 namespace {
-
-enum { T_NORM1 = 0, T_Q = 1, T_K = 2, T_V = 3, T_QN = 4, T_KN = 5, T_O = 6, T_NORM2 = 7, T_GATE = 8, T_UP = 9, T_DOWN = 10 };
-enum { G_EMBED = 1, G_WPE = 2, G_HEAD = 3, G_NORMF = 4 };
-inline uint64_t layer_tensor(int l, int kind) { return 16ull * (uint64_t)(l + 1) + (uint64_t)kind; }
-
-struct QW {
-  uint8_t* q = nullptr;
-  float* s = nullptr;
-  int64_t N = 0, K = 0;
-};
-struct FW {
-  float* w = nullptr;
-  float* b = nullptr;
-  int64_t N = 0, K = 0;
-};
-struct LayerW {
-  float *norm1_g = nullptr, *norm1_b = nullptr, *norm2_g = nullptr, *norm2_b = nullptr, *qn_g = nullptr, *kn_g = nullptr;
-  QW wqkv, wo, wgu, wdown;
-  FW fqkv, fo, ffc, fproj;
-};
-
-}  // namespace
-
-struct strictb200_model {
-  strictb200_ctx* ctx = nullptr;
-  strictb200_model_config c;
-  int world = 1, rank = 0;
-  int Hq_l = 0, Hkv_l = 0;
-  int64_t I_l = 0, V_l = 0;
-  std::vector<LayerW> L;
-  bf16* embed = nullptr;   // Qwen3
-  float* wte = nullptr;    // GPT-2
-  float* wpe = nullptr;
-  float *normf_g = nullptr, *normf_b = nullptr;
-  QW head;
-  float *rope_cos = nullptr, *rope_sin = nullptr;
-  std::vector<void*> allocs;
-  uint64_t weight_bytes = 0;  // bytes of the tensors a decode step streams (linears + head)
-  int use_graph = 1;
-};
-
-struct strictb200_kv {
-  strictb200_model* m = nullptr;
-  int B = 0, maxlen = 0;
-  void *k = nullptr, *v = nullptr;
-  size_t layer_stride = 0;  // elements per layer
-  int32_t* d_lens = nullptr;
-  std::vector<int32_t> h_lens;
-  // decode state
-  int32_t *d_ids = nullptr, *d_next = nullptr, *d_hist = nullptr;
-  int hist_cap = 0;
-  void* dec = nullptr;  // one allocation carved into the decode buffers
-  size_t dec_bytes = 0;
-  cudaGraphExec_t graph = nullptr;
-  uint64_t graph_kernels = 0;
-  bool warmed = false;
-  int nsplit = 1;        // key chunks per sequence of the decode attention, and
-  int chunk = 0;         // keys per chunk: planned for the lengths the cache holds now (plan_attention), 0 = not planned yet
-  int plan_until = 0;    // the plan is kept until a sequence grows beyond this length
-  std::vector<void*> allocs;
-};
-
-namespace {
-
-template <typename T>
-int dalloc(strictb200_model* m, T** p, size_t count) {
-  *p = nullptr;
-  if (!count) return STRICTB200_OK;
-  void* v;
-  SB_CUDA(cudaMalloc(&v, count * sizeof(T)));
-  m->allocs.push_back(v);
-  *p = (T*)v;
-  return STRICTB200_OK;
-}
-int fill_f32(strictb200_ctx* ctx, float* p, size_t n, float v) {
-  std::vector<float> h(n, v);
-  SB_CUDA(cudaMemcpyAsync(p, h.data(), n * 4, cudaMemcpyHostToDevice, ctx->stream));
-  SB_CUDA(cudaStreamSynchronize(ctx->stream));
-  return STRICTB200_OK;
-}
-int alloc_qw(strictb200_model* m, QW& w, int64_t N, int64_t K) {
-  w.N = N; w.K = K;
-  SB_TRY(dalloc(m, &w.q, (size_t)N * K));
-  SB_TRY(dalloc(m, &w.s, (size_t)N));
-  m->weight_bytes += (uint64_t)N * K + (uint64_t)N * 4;
-  return STRICTB200_OK;
-}
-int alloc_fw(strictb200_model* m, FW& w, int64_t N, int64_t K) {
-  w.N = N; w.K = K;
-  SB_TRY(dalloc(m, &w.w, (size_t)N * K));
-  SB_TRY(dalloc(m, &w.b, (size_t)N));
-  SB_TRY(fill_f32(m->ctx, w.b, N, 0.f));
-  m->weight_bytes += (uint64_t)N * K * 4 + (uint64_t)N * 4;
-  return STRICTB200_OK;
-}
-
 // ------------------------------------------------------------------ decode buffers
 struct DecBuf {
   float* x;        // [B,d] fp32 residual stream
@@ -135,21 +34,6 @@ struct DecBuf {
   int32_t* best_idx;
   void* am_ws;     // chunk winners of the two-stage argmax
 };
-
-size_t align256(size_t x) { return (x + 255) & ~(size_t)255; }
-
-struct Carver {
-  char* base;
-  size_t off = 0;
-  template <typename T>
-  T* take(size_t count) {
-    T* p = base ? (T*)(base + off) : nullptr;
-    off += align256(count * sizeof(T));
-    return p;
-  }
-};
-
-struct GemmPlan { int splits; };
 
 int plan_splits(strictb200_model* m, int64_t M, int64_t N, int64_t K) { return sb_gemm_pick_splits(m->ctx, M, N, K); }
 // K splits of the decode gate/up projection: 1 (the GEMM writes the scaled fp32 result) unless the
@@ -272,18 +156,7 @@ float* kv_vf(strictb200_kv* kv, int l) { return (float*)kv->v + (size_t)l * kv->
 // ------------------------------------------------------------------ per-class device timing
 // When ctx->prof is set, every call of the decode body is bracketed by a pair of CUDA events
 // tagged with its kernel class; strictb200_profile_decode sums them up afterwards.
-struct ProfSpan { int cls; cudaEvent_t a, b; };
 }  // namespace
-struct SbProfiler {
-  std::vector<ProfSpan> spans;
-  std::vector<cudaEvent_t> pool;
-  size_t used = 0;
-  ProfSpan* open = nullptr;  // the span of the call that is being made
-  cudaEvent_t get() {
-    if (used == pool.size()) { cudaEvent_t e; cudaEventCreate(&e); pool.push_back(e); }
-    return pool[used++];
-  }
-};
 // Inside a bracketed call: what is launched from here on belongs to class `cls` (a call that
 // launches kernels of two classes, e.g. the attention kernel and the merge of its key chunks).
 void sb_prof_split(strictb200_ctx* ctx, int cls) {
@@ -296,21 +169,6 @@ void sb_prof_split(strictb200_ctx* ctx, int cls) {
   p->open->a = e;
 }
 namespace {
-template <typename F>
-int prof(strictb200_ctx* ctx, int cls, F&& f) {
-  SbProfiler* p = ctx->prof;
-  if (!p) return f();
-  ProfSpan sp{cls, p->get(), p->get()};
-  cudaEventRecord(sp.a, ctx->stream);
-  p->open = &sp;
-  int st = f();
-  p->open = nullptr;
-  cudaEventRecord(sp.b, ctx->stream);
-  p->spans.push_back(sp);
-  return st;
-}
-#define PROF(cls, expr) SB_TRY(prof(ctx, cls, [&]() -> int { return (expr); }))
-
 // ------------------------------------------------------------------ Qwen3 decode step body
 // Everything below is enqueued on the stream with device-resident state only, so the whole
 // body can be captured into a CUDA graph.
@@ -435,6 +293,7 @@ int gpt2_decode_body(strictb200_model* m, strictb200_kv* kv, DecBuf& b) {
 }
 
 int decode_body(strictb200_model* m, strictb200_kv* kv) {
+  if (m->stack) return sb_stack_decode_body(m, kv);
   DecBuf b;
   size_t total;
   carve_decode(kv, (char*)kv->dec, &b, &total);
@@ -461,6 +320,11 @@ int decode_enqueue(strictb200_model* m, strictb200_kv* kv) {
       }
       kv->plan_until = std::min(kv->maxlen, longest + 256);
     }
+  }
+  if (m->stack) {
+    int longest = 0;
+    for (int b = 0; b < kv->B; b++) longest = std::max(longest, kv->h_lens[b] + 1);
+    if (sb_stack_plan(m, kv, longest) && kv->graph) { cudaGraphExecDestroy(kv->graph); kv->graph = nullptr; }
   }
   if (!m->use_graph || !kv->warmed) {
     // the first step runs as plain launches: it also performs the one-time kernel attribute set-up
@@ -491,32 +355,14 @@ int decode_enqueue(strictb200_model* m, strictb200_kv* kv) {
 // ------------------------------------------------------------------ prefill
 // Activations and index arrays of a prefill chunk are carved out of one grow-only scratch
 // buffer of the context: after the first prompt of a given size no prefill allocates.
-int prefill_scratch(strictb200_ctx* ctx, size_t bytes, char** out) {
-  if (bytes > ctx->prefill_ws_bytes) {
-    SB_CUDA(cudaStreamSynchronize(ctx->stream));
-    if (ctx->prefill_ws) SB_CUDA(cudaFree(ctx->prefill_ws));
-    ctx->prefill_ws = nullptr;
-    ctx->prefill_ws_bytes = 0;
-    SB_CUDA(cudaMalloc(&ctx->prefill_ws, bytes));
-    ctx->prefill_ws_bytes = bytes;
-  }
-  *out = (char*)ctx->prefill_ws;
-  return STRICTB200_OK;
-}
-struct ChunkIdx {
-  int32_t *tok, *seq, *pos, *la, *past, *qs, *last;
-};
-void carve_idx(Carver& cv, int64_t T, int nb, ChunkIdx* o) {
-  o->tok = cv.take<int32_t>(T); o->seq = cv.take<int32_t>(T); o->pos = cv.take<int32_t>(T);
-  o->la = cv.take<int32_t>(nb); o->past = cv.take<int32_t>(nb); o->qs = cv.take<int32_t>(nb); o->last = cv.take<int32_t>(nb);
-}
 struct QwenChunk {
   float *x, *qkv, *gu, *y, *sa, *last;
   bf16 *qb, *att;
   uint8_t* aq;
+  int32_t* pick;
   DecBuf hb;
 };
-void carve_qwen_chunk(strictb200_model* m, Carver& cv, int64_t T, int nb, QwenChunk* o) {
+void carve_qwen_chunk(strictb200_model* m, Carver& cv, int64_t T, int nb /* output rows */, QwenChunk* o) {
   const int64_t d = m->c.d_model, D = m->c.head_dim;
   const int64_t nq = (int64_t)m->Hq_l * D, nqkv = nq + 2 * (int64_t)m->Hkv_l * D;
   const int64_t amax = std::max<int64_t>(d, std::max<int64_t>(nq, m->I_l));
@@ -526,8 +372,9 @@ void carve_qwen_chunk(strictb200_model* m, Carver& cv, int64_t T, int nb, QwenCh
   o->att = cv.take<bf16>(T * nq);
   o->gu = cv.take<float>(T * 2 * m->I_l);
   o->y = cv.take<float>(T * d);
-  o->aq = cv.take<uint8_t>(sb_qrows(T) * amax);
-  o->sa = cv.take<float>(T);
+  o->aq = cv.take<uint8_t>(sb_qrows(std::max<int64_t>(T, nb)) * amax);
+  o->sa = cv.take<float>(std::max<int64_t>(T, nb));
+  o->pick = cv.take<int32_t>(nb);
   o->last = cv.take<float>((size_t)nb * d);
   o->hb = DecBuf{};
   o->hb.logits = cv.take<float>((size_t)nb * m->V_l);
@@ -538,9 +385,10 @@ void carve_qwen_chunk(strictb200_model* m, Carver& cv, int64_t T, int nb, QwenCh
 }
 struct Gpt2Chunk {
   float *xf, *af, *bf_, *last, *lastn, *logits;
+  int32_t* pick;
   void* am_ws;
 };
-void carve_gpt2_chunk(strictb200_model* m, Carver& cv, int64_t T, int nb, Gpt2Chunk* o) {
+void carve_gpt2_chunk(strictb200_model* m, Carver& cv, int64_t T, int nb /* output rows */, Gpt2Chunk* o) {
   const int64_t d = m->c.d_model, wd = std::max<int64_t>(3 * d, m->c.d_ff);
   o->xf = cv.take<float>(T * d);
   o->af = cv.take<float>(T * wd);
@@ -548,12 +396,13 @@ void carve_gpt2_chunk(strictb200_model* m, Carver& cv, int64_t T, int nb, Gpt2Ch
   o->last = cv.take<float>((size_t)nb * d);
   o->lastn = cv.take<float>((size_t)nb * d);
   o->logits = cv.take<float>((size_t)nb * m->c.vocab);
+  o->pick = cv.take<int32_t>(nb);
   o->am_ws = cv.take<uint8_t>(sb_argmax_scratch(nb, m->c.vocab));
 }
 
-int qwen_prefill_chunk(strictb200_model* m, strictb200_kv* kv, int64_t T, int nb, const int32_t* d_tok, const int32_t* d_seq,
-                       const int32_t* d_pos, const int32_t* d_lens_after, const int32_t* d_past, const int32_t* d_qstart,
-                       const int32_t* d_last_rows, int b0, int32_t* d_next, float* h_logits, int max_new, QwenChunk& cb) {
+int qwen_prefill_chunk(strictb200_model* m, strictb200_kv* kv, const PrefillChunk& pc, QwenChunk& cb) {
+  const int64_t T = pc.T;
+  const int nb = pc.nb, b0 = pc.b0, n_rows = pc.n_rows;
   strictb200_ctx* ctx = m->ctx;
   const auto& c = m->c;
   const int64_t d = c.d_model, D = c.head_dim;
@@ -563,7 +412,7 @@ int qwen_prefill_chunk(strictb200_model* m, strictb200_kv* kv, int64_t T, int nb
   bf16 *qb = cb.qb, *att = cb.att;
   uint8_t* aq = cb.aq;
   float *x = cb.x, *y = cb.y, *sa = cb.sa, *qkv = cb.qkv, *gu = cb.gu;
-  SB_TRY(k_embedding_bf16_f32(ctx, m->embed, d_tok, T, d, c.vocab, x));
+  SB_TRY(k_embedding_bf16_f32(ctx, m->embed, pc.ix.tok, T, d, c.vocab, x));
   {
     RowNormArgs a;
     a.x_f32 = x; a.gain = m->L[0].norm1_g; a.eps = c.eps; a.q = aq; a.qscale = sa;
@@ -578,13 +427,13 @@ int qwen_prefill_chunk(strictb200_model* m, strictb200_kv* kv, int64_t T, int nb
     SB_TRY(run_gemm(m, T, w.wqkv, aq, sa, qkv, 1, nullptr, 1, 0));
     {
       RopeArgs r;
-      r.qkv_f32 = qkv; r.seq = d_seq; r.pos = d_pos;
+      r.qkv_f32 = qkv; r.seq = pc.ix.seq; r.pos = pc.ix.pos;
       r.cos_t = m->rope_cos; r.sin_t = m->rope_sin; r.qgain = w.qn_g; r.kgain = w.kn_g; r.eps = c.eps;
       r.Hq = m->Hq_l; r.Hkv = m->Hkv_l; r.D = (int)D; r.maxlen = kv->maxlen; r.max_pos = c.max_pos;
       r.q_out = qb; r.kcache = kc; r.vcache = vc;
       SB_TRY(k_rope_qknorm_kvappend(ctx, r, T));
     }
-    SB_TRY(k_attn_prefill(ctx, qb, kc, vc, d_lens_after, d_past, d_qstart, nb, max_new, T, m->Hq_l, m->Hkv_l, (int)D, kv->maxlen, scale, att));
+    SB_TRY(k_attn_prefill(ctx, qb, kc, vc, pc.ix.la, pc.ix.past, pc.ix.qs, nb, pc.max_new, T, m->Hq_l, m->Hkv_l, (int)D, kv->maxlen, scale, att));
     SB_TRY(k_quantize_rows(ctx, att, T, nq, nq, aq, sa));
     {
       RowNormArgs a;
@@ -605,34 +454,144 @@ int qwen_prefill_chunk(strictb200_model* m, strictb200_kv* kv, int64_t T, int nb
       SB_TRY(k_rownorm(ctx, a, T, d));
     }
   }
-  // last real row of every sequence -> final norm -> head -> greedy pick
+  // the rows asked for and the last real row of every sequence -> final norm -> head -> greedy pick
   float* last = cb.last;
-  SB_TRY(k_gather_rows(ctx, x, d_last_rows, nb, d * 4, last));
+  SB_TRY(k_gather_rows(ctx, x, pc.ix.last, n_rows, d * 4, last));
   {
     RowNormArgs a;
     a.x_f32 = last; a.gain = m->normf_g; a.eps = c.eps; a.q = aq; a.qscale = sa;
-    SB_TRY(k_rownorm(ctx, a, nb, d));
+    SB_TRY(k_rownorm(ctx, a, n_rows, d));
   }
-  SB_TRY(head_and_pick(m, nb, aq, sa, cb.hb, d_next, h_logits, nb));
+  if (n_rows == nb) {
+    SB_TRY(head_and_pick(m, nb, aq, sa, cb.hb, pc.d_next, pc.h_logits, nb));
+  } else {
+    // wanted rows: their logits come with those of the last rows; the picks are the last rows'
+    SB_TRY(head_and_pick(m, n_rows, aq, sa, cb.hb, cb.pick, nullptr, n_rows));
+    SB_CUDA(cudaMemcpyAsync(pc.d_next, cb.pick + (n_rows - nb), (size_t)nb * 4, cudaMemcpyDeviceToDevice, ctx->stream));
+    if (pc.h_logits) {
+      const float* src = cb.hb.logits;
+      if (m->world > 1) {
+        SB_TRY(sb_tp_allgather(ctx, cb.hb.logits, cb.hb.logits_all, (int64_t)n_rows * m->V_l * 4));
+        void* tmp;
+        SB_TRY(sb_ws2(ctx, (size_t)m->world * n_rows * m->V_l * 4, &tmp));
+        interleave_logits_kernel<<<ctx->sm_count * 4, 256, 0, ctx->stream>>>(cb.hb.logits_all, m->world, n_rows, m->V_l, (float*)tmp);
+        SB_LAUNCHED(ctx);
+        src = (const float*)tmp;
+      }
+      SB_CUDA(cudaMemcpyAsync(pc.h_logits, src, (size_t)pc.n_logits * c.vocab * 4, cudaMemcpyDeviceToHost, ctx->stream));
+    }
+  }
   SB_CUDA(cudaStreamSynchronize(ctx->stream));
   return STRICTB200_OK;
 }
 
-int gpt2_prefill_chunk(strictb200_model* m, strictb200_kv* kv, int64_t T, int nb, const int32_t* d_tok, const int32_t* d_seq,
-                       const int32_t* d_pos, const int32_t* d_last_rows, int32_t* d_next, float* h_logits, Gpt2Chunk& cb) {
+int gpt2_prefill_chunk(strictb200_model* m, strictb200_kv* kv, const PrefillChunk& pc, Gpt2Chunk& cb) {
+  const int64_t T = pc.T;
+  const int n_rows = pc.n_rows;
   strictb200_ctx* ctx = m->ctx;
   const auto& c = m->c;
   const int64_t d = c.d_model;
   float *xf = cb.xf, *af = cb.af, *bf_ = cb.bf_, *last = cb.last, *lastn = cb.lastn, *logits = cb.logits;
-  SB_TRY(k_embedding_f32(ctx, m->wte, m->wpe, d_tok, d_pos, nullptr, T, d, c.vocab, c.max_pos, xf));
-  SB_TRY(gpt2_layers(m, kv, T, xf, af, bf_, d_seq, d_pos));
-  SB_TRY(k_gather_rows(ctx, xf, d_last_rows, nb, d * 4, last));
-  SB_TRY(k_layernorm(ctx, last, m->normf_g, m->normf_b, c.eps, nb, d, lastn));
-  SB_TRY(k_gemm_f32(ctx, nb, c.vocab, d, lastn, m->wte, nullptr, logits, 0));
-  SB_TRY(k_argmax(ctx, logits, nb, c.vocab, c.vocab, d_next, nullptr, cb.am_ws));
-  if (h_logits) SB_CUDA(cudaMemcpyAsync(h_logits, logits, (size_t)nb * c.vocab * 4, cudaMemcpyDeviceToHost, ctx->stream));
+  SB_TRY(k_embedding_f32(ctx, m->wte, m->wpe, pc.ix.tok, pc.ix.pos, nullptr, T, d, c.vocab, c.max_pos, xf));
+  SB_TRY(gpt2_layers(m, kv, T, xf, af, bf_, pc.ix.seq, pc.ix.pos));
+  SB_TRY(k_gather_rows(ctx, xf, pc.ix.last, n_rows, d * 4, last));
+  SB_TRY(k_layernorm(ctx, last, m->normf_g, m->normf_b, c.eps, n_rows, d, lastn));
+  SB_TRY(k_gemm_f32(ctx, n_rows, c.vocab, d, lastn, m->wte, nullptr, logits, 0));
+  SB_TRY(k_argmax(ctx, logits, n_rows, c.vocab, c.vocab, cb.pick, nullptr, cb.am_ws));
+  SB_CUDA(cudaMemcpyAsync(pc.d_next, cb.pick + (n_rows - pc.nb), (size_t)pc.nb * 4, cudaMemcpyDeviceToDevice, ctx->stream));
+  if (pc.h_logits) SB_CUDA(cudaMemcpyAsync(pc.h_logits, logits, (size_t)pc.n_logits * c.vocab * 4, cudaMemcpyDeviceToHost, ctx->stream));
   SB_CUDA(cudaStreamSynchronize(ctx->stream));
   return STRICTB200_OK;
+}
+
+// h_n_want null: the logits of every sequence's last new token; else those of the wanted places (strictb200_prefill_rows).
+int prefill_impl(strictb200_model* m, strictb200_kv* kv, const int32_t* h_tokens, const int32_t* h_lens, int B, int S, const int32_t* h_want,
+                 const int32_t* h_n_want, int32_t* h_next, float* h_logits) {
+  if (!m || !kv || !h_tokens || !h_lens || !h_next) return sb_fail(STRICTB200_ERR_INVALID_ARG, "null argument");
+  strictb200_ctx* ctx = m->ctx;
+  SB_ENTER(ctx);
+  SB_REQUIRE(kv->m == m, "cache belongs to another model");
+  SB_REQUIRE(B == kv->B && S > 0, "batch must match the cache and S must be positive");
+  const auto& c = m->c;
+  const int32_t* want = h_want;
+  for (int b = 0; b < B; b++) {
+    SB_REQUIRE(h_lens[b] > 0 && h_lens[b] <= S, "every sequence needs between 1 and S tokens");
+    SB_REQUIRE(kv->h_lens[b] + h_lens[b] <= kv->maxlen && kv->h_lens[b] + h_lens[b] <= c.max_pos, "prompt does not fit the cache");
+    for (int i = 0; i < h_lens[b]; i++)
+      SB_REQUIRE(h_tokens[(size_t)b * S + i] >= 0 && h_tokens[(size_t)b * S + i] < c.vocab, "token id outside the vocabulary");
+    if (h_n_want && h_n_want[b]) {
+      SB_REQUIRE(h_n_want[b] > 0 && h_want && h_logits, "wanted rows need their places and a buffer");
+      for (int i = 0; i < h_n_want[b]; i++, want++) SB_REQUIRE(*want >= 0 && *want < h_lens[b], "wanted row outside the new tokens");
+    }
+  }
+  want = h_want;
+  size_t logits_done = 0;  // rows of h_logits written by earlier chunks
+  const int64_t MAX_T = ctx->opt.prefill_chunk > 0 ? ctx->opt.prefill_chunk : 16384;  // token rows per chunk (bounds the activation scratch)
+  int b0 = 0;
+  int32_t* d_next = kv->d_next;  // the decode step's own buffer: nothing else uses it during a prefill
+  while (b0 < B) {
+    int nb = 0;
+    int64_t T = 0;
+    while (b0 + nb < B && (nb == 0 || T + h_lens[b0 + nb] <= MAX_T)) { T += h_lens[b0 + nb]; nb++; }
+    std::vector<int32_t> tok(T), seq(T), pos(T), la(nb), past(nb), qstart(nb), last;
+    int64_t t = 0;
+    int max_new = 0;
+    for (int j = 0; j < nb; j++) {
+      int b = b0 + j;
+      qstart[j] = (int32_t)t;
+      past[j] = kv->h_lens[b];
+      la[j] = kv->h_lens[b] + h_lens[b];
+      max_new = std::max(max_new, h_lens[b]);
+      for (int i = 0; h_n_want && i < h_n_want[b]; i++) last.push_back((int32_t)t + *want++);
+      for (int i = 0; i < h_lens[b]; i++, t++) {
+        tok[t] = h_tokens[(size_t)b * S + i];
+        seq[t] = c.arch == STRICTB200_GPT2 ? b : j;  // the GPT-2 path addresses the cache by absolute sequence index
+        pos[t] = kv->h_lens[b] + i;
+      }
+    }
+    // rows that leave the stack: the wanted ones, then every sequence's last (its greedy pick)
+    const int n_want = (int)last.size();
+    for (int j = 0; j < nb; j++) last.push_back(qstart[j] + h_lens[b0 + j] - 1);
+    const int n_rows = n_want + nb;
+    const int n_logits = h_n_want ? n_want : nb;
+    float* hl = h_logits && n_logits ? h_logits + logits_done * c.vocab : nullptr;
+    logits_done += n_logits;
+    // one carve pass to size the scratch, one to place the buffers
+    PrefillChunk pc;
+    pc.T = T; pc.nb = nb; pc.b0 = b0; pc.max_new = max_new; pc.h_past = past.data(); pc.h_after = la.data();
+    pc.n_rows = n_rows; pc.d_next = d_next + b0; pc.h_logits = hl; pc.n_logits = n_logits;
+    ChunkIdx& ix = pc.ix;
+    QwenChunk qc;
+    Gpt2Chunk gc;
+    char *base = nullptr, *rest = nullptr;
+    for (int pass = 0; pass < 2; pass++) {
+      Carver cv{base};
+      carve_idx(cv, T, nb, n_rows, &ix);
+      if (m->stack) rest = cv.take<char>(sb_stack_prefill_bytes(m, pc));
+      else if (c.arch == STRICTB200_QWEN3) carve_qwen_chunk(m, cv, T, n_rows, &qc);
+      else carve_gpt2_chunk(m, cv, T, n_rows, &gc);
+      if (pass == 0) SB_TRY(prefill_scratch(ctx, cv.off, &base));
+    }
+    SB_CUDA(cudaMemcpyAsync(ix.tok, tok.data(), T * 4, cudaMemcpyHostToDevice, ctx->stream));
+    SB_CUDA(cudaMemcpyAsync(ix.seq, seq.data(), T * 4, cudaMemcpyHostToDevice, ctx->stream));
+    SB_CUDA(cudaMemcpyAsync(ix.pos, pos.data(), T * 4, cudaMemcpyHostToDevice, ctx->stream));
+    SB_CUDA(cudaMemcpyAsync(ix.la, la.data(), nb * 4, cudaMemcpyHostToDevice, ctx->stream));
+    SB_CUDA(cudaMemcpyAsync(ix.past, past.data(), nb * 4, cudaMemcpyHostToDevice, ctx->stream));
+    SB_CUDA(cudaMemcpyAsync(ix.qs, qstart.data(), nb * 4, cudaMemcpyHostToDevice, ctx->stream));
+    SB_CUDA(cudaMemcpyAsync(ix.last, last.data(), (size_t)n_rows * 4, cudaMemcpyHostToDevice, ctx->stream));
+    // the chunk functions end with a stream synchronise, so the host vectors above outlive their copies
+    if (m->stack) SB_TRY(sb_stack_prefill_chunk(m, kv, pc, rest));
+    else if (c.arch == STRICTB200_QWEN3) SB_TRY(qwen_prefill_chunk(m, kv, pc, qc));
+    else SB_TRY(gpt2_prefill_chunk(m, kv, pc, gc));
+    SB_TRY(sb_check_status(ctx, "prefill"));
+    for (int j = 0; j < nb; j++) kv->h_lens[b0 + j] += h_lens[b0 + j];
+    b0 += nb;
+  }
+  kv->plan_until = 0;  // the lengths jumped: the next decode step plans the attention's key chunks for them
+  SB_CUDA(cudaMemcpyAsync(kv->d_lens, kv->h_lens.data(), (size_t)B * 4, cudaMemcpyHostToDevice, ctx->stream));
+  SB_CUDA(cudaMemcpyAsync(h_next, d_next, (size_t)B * 4, cudaMemcpyDeviceToHost, ctx->stream));
+  SB_TRY(sb_sync(ctx, "prefill"));
+  return sb_check_status(ctx, "prefill");
 }
 
 // ------------------------------------------------------------------ named tensors
@@ -808,6 +767,7 @@ int strictb200_model_destroy(strictb200_model* m) {
   cudaSetDevice(m->ctx->device);
   cudaStreamSynchronize(m->ctx->stream);
   for (void* p : m->allocs) cudaFree(p);
+  sb_stack_destroy(m);
   delete m;
   return STRICTB200_OK;
 }
@@ -816,6 +776,7 @@ int strictb200_model_init_random(strictb200_model* m, uint64_t seed) {
   if (!m) return sb_fail(STRICTB200_ERR_INVALID_ARG, "null model");
   strictb200_ctx* ctx = m->ctx;
   SB_ENTER(ctx);
+  if (m->stack) return sb_stack_init_random(m, seed);
   const auto& c = m->c;
   const float SD = 0.02f;
   const int64_t d = c.d_model, D = c.head_dim, I = c.d_ff;
@@ -862,6 +823,7 @@ int strictb200_model_set_tensor(strictb200_model* m, const char* name, const voi
   if (!m || !name || !h_data) return sb_fail(STRICTB200_ERR_INVALID_ARG, "null argument");
   strictb200_ctx* ctx = m->ctx;
   SB_ENTER(ctx);
+  if (m->stack) return sb_stack_tensor(m, name, h_data, nullptr, bytes);
   Slice s;
   if (!find_slice(m, name, &s)) return sb_fail(STRICTB200_ERR_INVALID_ARG, std::string("unknown tensor ") + name);
   size_t helem = s.host_f32 ? 4 : s.elem;
@@ -898,6 +860,7 @@ int strictb200_model_get_tensor(strictb200_model* m, const char* name, void* h_d
   if (!m || !name || !h_data) return sb_fail(STRICTB200_ERR_INVALID_ARG, "null argument");
   strictb200_ctx* ctx = m->ctx;
   SB_ENTER(ctx);
+  if (m->stack) return sb_stack_tensor(m, name, nullptr, h_data, bytes);
   if (m->world != 1) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "get_tensor reads whole tensors and needs a single-rank model");
   Slice s;
   if (!find_slice(m, name, &s)) return sb_fail(STRICTB200_ERR_INVALID_ARG, std::string("unknown tensor ") + name);
@@ -946,6 +909,10 @@ int strictb200_kv_create(strictb200_model* m, int batch, int maxlen, strictb200_
   const size_t esz = qwen ? 2 : 4;
   kv->layer_stride = (size_t)batch * (qwen ? m->Hkv_l : m->c.n_kv_heads) * kv->maxlen * m->c.head_dim;
   size_t bytes = kv->layer_stride * m->c.n_layers * esz;
+  if (m->stack) {  // one array of latent rows; nothing in v
+    SB_TRY(sb_stack_kv_layout(m, kv, &kv->layer_stride));
+    bytes = kv->layer_stride * (m->c.n_layers ? sb_stack_esz(m) : 0);
+  }
   auto fail = [&](int s) { strictb200_kv_destroy(kv); return s; };
   auto alloc = [&](void** p, size_t n) -> int {
     SB_CUDA(cudaMalloc(p, n ? n : 1));
@@ -955,9 +922,10 @@ int strictb200_kv_create(strictb200_model* m, int batch, int maxlen, strictb200_
   int st;
 #define K_TRY(e) do { st = (e); if (st != STRICTB200_OK) return fail(st); } while (0)
   K_TRY(alloc(&kv->k, bytes));
-  K_TRY(alloc(&kv->v, bytes));
+  if (!m->stack) K_TRY(alloc(&kv->v, bytes));
   // zero so that the padding rows of a partly filled 64-key tile are finite
-  if (cudaMemsetAsync(kv->k, 0, bytes, ctx->stream) != cudaSuccess || cudaMemsetAsync(kv->v, 0, bytes, ctx->stream) != cudaSuccess)
+  if (cudaMemsetAsync(kv->k, 0, bytes, ctx->stream) != cudaSuccess ||
+      (kv->v && cudaMemsetAsync(kv->v, 0, bytes, ctx->stream) != cudaSuccess))
     return fail(sb_fail(STRICTB200_ERR_CUDA, "memset of the cache failed"));
   K_TRY(alloc((void**)&kv->d_lens, (size_t)batch * 4));
   K_TRY(alloc((void**)&kv->d_ids, (size_t)batch * 4));
@@ -967,8 +935,10 @@ int strictb200_kv_create(strictb200_model* m, int batch, int maxlen, strictb200_
   kv->h_lens.assign(batch, 0);
   kv->nsplit = qwen ? sb_attn_decode_splits(ctx, batch, m->Hkv_l, kv->maxlen) : 1;
   DecBuf tmp;
-  carve_decode(kv, nullptr, &tmp, &kv->dec_bytes);
+  if (m->stack) kv->dec_bytes = sb_stack_decode_bytes(m, kv);
+  else carve_decode(kv, nullptr, &tmp, &kv->dec_bytes);
   K_TRY(alloc(&kv->dec, kv->dec_bytes));
+  if (m->stack) cudaMemsetAsync(kv->dec, 0, kv->dec_bytes, ctx->stream);  // padding columns of the buffers stay zero
 #undef K_TRY
   if (cudaStreamSynchronize(ctx->stream) != cudaSuccess) return fail(sb_fail(STRICTB200_ERR_CUDA, "cache set-up failed"));
   *out = kv;
@@ -1012,7 +982,10 @@ int strictb200_kv_fill_synthetic(strictb200_kv* kv, uint64_t seed, int len) {
   SB_ENTER(ctx);
   SB_REQUIRE(len >= 0 && len <= kv->maxlen && len < m->c.max_pos, "len outside the cache");
   size_t n = kv->layer_stride * m->c.n_layers;
-  if (m->c.arch == STRICTB200_QWEN3) {
+  if (m->stack) {
+    if (sb_stack_esz(m) == 2) SB_TRY(k_gen_normal_bf16(ctx, sb_stream_key(seed, 0x4B00), 0, (int64_t)kv->layer_stride, 1.0f, (bf16*)kv->k));
+    else SB_TRY(k_gen_normal_f32(ctx, sb_stream_key(seed, 0x4B00), 0, (int64_t)kv->layer_stride, 1.0f, (float*)kv->k));
+  } else if (m->c.arch == STRICTB200_QWEN3) {
     SB_TRY(k_gen_normal_bf16(ctx, sb_stream_key(seed, 0x4B00 + m->rank), 0, (int64_t)n, 1.0f, (bf16*)kv->k));
     SB_TRY(k_gen_normal_bf16(ctx, sb_stream_key(seed, 0x5600 + m->rank), 0, (int64_t)n, 1.0f, (bf16*)kv->v));
   } else {
@@ -1030,76 +1003,12 @@ int strictb200_kv_fill_synthetic(strictb200_kv* kv, uint64_t seed, int len) {
 // ---------------------------------------------------------------- prefill / decode
 int strictb200_prefill(strictb200_model* m, strictb200_kv* kv, const int32_t* h_tokens, const int32_t* h_lens, int B, int S,
                        int32_t* h_next, float* h_logits) {
-  if (!m || !kv || !h_tokens || !h_lens || !h_next) return sb_fail(STRICTB200_ERR_INVALID_ARG, "null argument");
-  strictb200_ctx* ctx = m->ctx;
-  SB_ENTER(ctx);
-  SB_REQUIRE(kv->m == m, "cache belongs to another model");
-  SB_REQUIRE(B == kv->B && S > 0, "batch must match the cache and S must be positive");
-  const auto& c = m->c;
-  for (int b = 0; b < B; b++) {
-    SB_REQUIRE(h_lens[b] > 0 && h_lens[b] <= S, "every sequence needs between 1 and S tokens");
-    SB_REQUIRE(kv->h_lens[b] + h_lens[b] <= kv->maxlen && kv->h_lens[b] + h_lens[b] <= c.max_pos, "prompt does not fit the cache");
-    for (int i = 0; i < h_lens[b]; i++)
-      SB_REQUIRE(h_tokens[(size_t)b * S + i] >= 0 && h_tokens[(size_t)b * S + i] < c.vocab, "token id outside the vocabulary");
-  }
-  const int64_t MAX_T = ctx->opt.prefill_chunk > 0 ? ctx->opt.prefill_chunk : 16384;  // token rows per chunk (bounds the activation scratch)
-  int b0 = 0;
-  int32_t* d_next = kv->d_next;  // the decode step's own buffer: nothing else uses it during a prefill
-  while (b0 < B) {
-    int nb = 0;
-    int64_t T = 0;
-    while (b0 + nb < B && (nb == 0 || T + h_lens[b0 + nb] <= MAX_T)) { T += h_lens[b0 + nb]; nb++; }
-    std::vector<int32_t> tok(T), seq(T), pos(T), la(nb), past(nb), qstart(nb), last(nb);
-    int64_t t = 0;
-    int max_new = 0;
-    for (int j = 0; j < nb; j++) {
-      int b = b0 + j;
-      qstart[j] = (int32_t)t;
-      past[j] = kv->h_lens[b];
-      la[j] = kv->h_lens[b] + h_lens[b];
-      max_new = std::max(max_new, h_lens[b]);
-      for (int i = 0; i < h_lens[b]; i++, t++) {
-        tok[t] = h_tokens[(size_t)b * S + i];
-        seq[t] = c.arch == STRICTB200_QWEN3 ? j : b;  // the fp32 path addresses the cache by absolute sequence index
-        pos[t] = kv->h_lens[b] + i;
-      }
-      last[j] = (int32_t)t - 1;
-    }
-    // one carve pass to size the scratch, one to place the buffers
-    ChunkIdx ix;
-    QwenChunk qc;
-    Gpt2Chunk gc;
-    char* base = nullptr;
-    for (int pass = 0; pass < 2; pass++) {
-      Carver cv{base};
-      carve_idx(cv, T, nb, &ix);
-      if (c.arch == STRICTB200_QWEN3) carve_qwen_chunk(m, cv, T, nb, &qc);
-      else carve_gpt2_chunk(m, cv, T, nb, &gc);
-      if (pass == 0) SB_TRY(prefill_scratch(ctx, cv.off, &base));
-    }
-    SB_CUDA(cudaMemcpyAsync(ix.tok, tok.data(), T * 4, cudaMemcpyHostToDevice, ctx->stream));
-    SB_CUDA(cudaMemcpyAsync(ix.seq, seq.data(), T * 4, cudaMemcpyHostToDevice, ctx->stream));
-    SB_CUDA(cudaMemcpyAsync(ix.pos, pos.data(), T * 4, cudaMemcpyHostToDevice, ctx->stream));
-    SB_CUDA(cudaMemcpyAsync(ix.la, la.data(), nb * 4, cudaMemcpyHostToDevice, ctx->stream));
-    SB_CUDA(cudaMemcpyAsync(ix.past, past.data(), nb * 4, cudaMemcpyHostToDevice, ctx->stream));
-    SB_CUDA(cudaMemcpyAsync(ix.qs, qstart.data(), nb * 4, cudaMemcpyHostToDevice, ctx->stream));
-    SB_CUDA(cudaMemcpyAsync(ix.last, last.data(), nb * 4, cudaMemcpyHostToDevice, ctx->stream));
-    float* hl = h_logits ? h_logits + (size_t)b0 * c.vocab : nullptr;
-    // both chunk functions end with a stream synchronise, so the host vectors above outlive their copies
-    if (c.arch == STRICTB200_QWEN3) {
-      SB_TRY(qwen_prefill_chunk(m, kv, T, nb, ix.tok, ix.seq, ix.pos, ix.la, ix.past, ix.qs, ix.last, b0, d_next + b0, hl, max_new, qc));
-    } else {
-      SB_TRY(gpt2_prefill_chunk(m, kv, T, nb, ix.tok, ix.seq, ix.pos, ix.last, d_next + b0, hl, gc));
-    }
-    SB_TRY(sb_check_status(ctx, "prefill"));
-    for (int j = 0; j < nb; j++) kv->h_lens[b0 + j] += h_lens[b0 + j];
-    b0 += nb;
-  }
-  kv->plan_until = 0;  // the lengths jumped: the next decode step plans the attention's key chunks for them
-  SB_CUDA(cudaMemcpyAsync(kv->d_lens, kv->h_lens.data(), (size_t)B * 4, cudaMemcpyHostToDevice, ctx->stream));
-  SB_CUDA(cudaMemcpyAsync(h_next, d_next, (size_t)B * 4, cudaMemcpyDeviceToHost, ctx->stream));
-  SB_TRY(sb_sync(ctx, "prefill"));
-  return sb_check_status(ctx, "prefill");
+  return prefill_impl(m, kv, h_tokens, h_lens, B, S, nullptr, nullptr, h_next, h_logits);
+}
+int strictb200_prefill_rows(strictb200_model* m, strictb200_kv* kv, const int32_t* h_tokens, const int32_t* h_lens, int B, int S,
+                            const int32_t* h_want, const int32_t* h_n_want, int32_t* h_next, float* h_logits) {
+  if (!h_n_want) return sb_fail(STRICTB200_ERR_INVALID_ARG, "null argument");
+  return prefill_impl(m, kv, h_tokens, h_lens, B, S, h_want, h_n_want, h_next, h_logits);
 }
 
 int strictb200_decode_step(strictb200_model* m, strictb200_kv* kv, const int32_t* h_ids, int32_t* h_next, float* h_logits) {
@@ -1111,7 +1020,9 @@ int strictb200_decode_step(strictb200_model* m, strictb200_kv* kv, const int32_t
   SB_CUDA(cudaMemcpyAsync(kv->d_ids, h_ids, (size_t)kv->B * 4, cudaMemcpyHostToDevice, ctx->stream));
   SB_TRY(decode_enqueue(m, kv));
   SB_CUDA(cudaMemcpyAsync(h_next, kv->d_next, (size_t)kv->B * 4, cudaMemcpyDeviceToHost, ctx->stream));
-  if (h_logits) {
+  if (h_logits && m->stack) {
+    SB_CUDA(cudaMemcpyAsync(h_logits, sb_stack_decode_logits(m, kv), (size_t)kv->B * m->V_l * 4, cudaMemcpyDeviceToHost, ctx->stream));
+  } else if (h_logits) {
     DecBuf b;
     size_t total;
     carve_decode(kv, (char*)kv->dec, &b, &total);
@@ -1178,7 +1089,7 @@ int strictb200_profile_decode(strictb200_model* m, strictb200_kv* kv, int n_step
   strictb200_ctx* ctx = m->ctx;
   SB_ENTER(ctx);
   SB_REQUIRE(kv->m == m && n_steps > 0 && n_classes >= STRICTB200_K_COUNT, "bad arguments");
-  if (m->c.arch != STRICTB200_QWEN3) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "per-class timing covers the Qwen3 decode step");
+  if (m->c.arch == STRICTB200_GPT2) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "per-class timing does not cover the GPT-2 decode step");
   for (int i = 0; i < n_classes; i++) { ms_out[i] = 0.f; calls_out[i] = 0; }
   SbProfiler prof;
   int saved = m->use_graph;
@@ -1209,6 +1120,11 @@ int strictb200_decode_bytes(strictb200_model* m, strictb200_kv* kv, uint64_t* ou
   if (!m || !kv || !out) return sb_fail(STRICTB200_ERR_INVALID_ARG, "null argument");
   const auto& c = m->c;
   uint64_t kvb = 0;
+  if (m->stack) {
+    for (int b = 0; b < kv->B; b++) kvb += sb_stack_cache_read_bytes(m, kv->h_lens[b] + 1);
+    *out = m->weight_bytes + kvb;
+    return STRICTB200_OK;
+  }
   const uint64_t esz = c.arch == STRICTB200_QWEN3 ? 2 : 4;
   const uint64_t heads = c.arch == STRICTB200_QWEN3 ? m->Hkv_l : c.n_kv_heads;
   for (int b = 0; b < kv->B; b++) kvb += (uint64_t)(kv->h_lens[b] + 1) * heads * c.head_dim * 2 * esz * c.n_layers;

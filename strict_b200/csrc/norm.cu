@@ -782,3 +782,157 @@ int k_reduce_scale(strictb200_ctx* ctx, const float* part, int splits, const flo
   ctx->launches++;
   return STRICTB200_OK;
 }
+
+// ------------------------------------------------------------------ grouped RMS norm of the residual stream
+namespace {
+struct GroupNormDev {
+  float* x;
+  int64_t ldx;
+  const float* part;
+  int64_t ldp;
+  int splits;
+  const float *g1, *g2;
+  float eps;
+  void *y1, *y2;
+  int64_t ldy;
+  int gw;  // columns per group
+  int cb;  // blocks (one cluster) per group
+  int* status;
+};
+template <typename T>
+__device__ __forceinline__ void store4(T* p, float a, float b, float c, float d);
+template <>
+__device__ __forceinline__ void store4<float>(float* p, float a, float b, float c, float d) { *(float4*)p = make_float4(a, b, c, d); }
+template <>
+__device__ __forceinline__ void store4<bf16>(bf16* p, float a, float b, float c, float d) {
+  *(uint2*)p = make_uint2(f32_to_bf16_bits(a) | (f32_to_bf16_bits(b) << 16), f32_to_bf16_bits(c) | (f32_to_bf16_bits(d) << 16));
+}
+template <typename T>
+__device__ __forceinline__ T from_f32(float v);
+template <>
+__device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
+
+// grid (M, groups * cb): a block owns one group of a row, or one of the cb slices a cluster shares (the sum of squares is
+// then exchanged). The sums, the new residual and both outputs pass through registers once; the gains are constants and are
+// fetched before the dependency wait. A thread owns NI float4s: one in the decode step's blocks, up to four in a prompt's.
+template <typename T, int NI>
+__global__ void __launch_bounds__(NI == 1 ? 1024 : 512) group_norm_kernel(GroupNormDev a, int64_t M) {
+  __shared__ float red[32];
+  __shared__ __align__(8) ClusterExchange xch;
+  SB_TRACE_BEGIN();
+  if (a.cb > 1) cluster_exchange_init(&xch);
+  const int64_t row = blockIdx.x;
+  const int n = a.gw / a.cb, c0 = (int)blockIdx.y / a.cb * a.gw + (int)blockIdx.y % a.cb * n;
+  pdl_trigger();
+  float4 g1[NI], g2[NI], v[NI];
+#pragma unroll
+  for (int i = 0; i < NI; i++) {
+    const int k = (i * (int)blockDim.x + (int)threadIdx.x) * 4;
+    if (k < n && a.g1) {
+      g1[i] = *(const float4*)(a.g1 + c0 + k);
+      if (a.g2) g2[i] = *(const float4*)(a.g2 + c0 + k);
+    }
+  }
+  pdl_wait();
+  SB_TRACE_WAITED();
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NI; i++) {
+    const int k = (i * (int)blockDim.x + (int)threadIdx.x) * 4;
+    if (k < n) {
+      float* xp = a.x + row * a.ldx + c0 + k;
+      float4 x = *(const float4*)xp;
+      if (a.part) {
+        float4 p[8], t = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int s = 0; s < 8; s++)
+          if (s < a.splits) p[s] = *(const float4*)(a.part + ((int64_t)s * M + row) * a.ldp + c0 + k);
+#pragma unroll
+        for (int s = 0; s < 8; s++)
+          if (s < a.splits) { t.x += p[s].x; t.y += p[s].y; t.z += p[s].z; t.w += p[s].w; }
+        x.x += t.x; x.y += t.y; x.z += t.z; x.w += t.w;
+        *(float4*)xp = x;
+      }
+      v[i] = x;
+      ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+    }
+  }
+  if (!a.g1) return;
+  ss = block_sum(ss, red);
+  if (a.cb > 1) {
+    const uint32_t rank = blockIdx.y % a.cb;
+    if (!cluster_exchange(&xch, ss, a.cb, rank) && threadIdx.x == 0) { *(volatile int*)a.status = 6; __threadfence_system(); }
+    ss = 0.f;
+    for (int r = 0; r < a.cb; r++) ss += ((volatile float*)xch.slot[0])[r];
+  }
+  const float r = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.gw), a.eps)));
+#pragma unroll
+  for (int i = 0; i < NI; i++) {
+    const int k = (i * (int)blockDim.x + (int)threadIdx.x) * 4;
+    if (k < n) {
+      const float4 t = make_float4(v[i].x * r, v[i].y * r, v[i].z * r, v[i].w * r);
+      store4<T>((T*)a.y1 + row * a.ldy + c0 + k, t.x * g1[i].x, t.y * g1[i].y, t.z * g1[i].z, t.w * g1[i].w);
+      if (a.g2) store4<T>((T*)a.y2 + row * a.ldy + c0 + k, t.x * g2[i].x, t.y * g2[i].y, t.z * g2[i].z, t.w * g2[i].w);
+    }
+  }
+  SB_TRACE_END(SB_K_ROWNORM, 0);
+}
+
+// Group widths that are no multiple of four, or too wide for the kernel above: one column at a time, two passes.
+template <typename T>
+__global__ void __launch_bounds__(256) group_norm_any_kernel(GroupNormDev a, int64_t M) {
+  __shared__ float red[32];
+  pdl_trigger();
+  pdl_wait();
+  const int64_t row = blockIdx.x;
+  const int c0 = (int)blockIdx.y * a.gw;
+  float ss = 0.f;
+  for (int k = threadIdx.x; k < a.gw; k += blockDim.x) {
+    float* xp = a.x + row * a.ldx + c0 + k;
+    float x = *xp;
+    if (a.part) {
+      float t = 0.f;
+      for (int s = 0; s < a.splits; s++) t += a.part[((int64_t)s * M + row) * a.ldp + c0 + k];
+      x += t;
+      *xp = x;
+    }
+    ss += x * x;
+  }
+  if (!a.g1) return;
+  ss = block_sum(ss, red);
+  const float r = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.gw), a.eps)));
+  for (int k = threadIdx.x; k < a.gw; k += blockDim.x) {
+    const float t = a.x[row * a.ldx + c0 + k] * r;  // this thread's own column
+    ((T*)a.y1)[row * a.ldy + c0 + k] = from_f32<T>(t * a.g1[c0 + k]);
+    if (a.g2) ((T*)a.y2)[row * a.ldy + c0 + k] = from_f32<T>(t * a.g2[c0 + k]);
+  }
+}
+}  // namespace
+
+int k_group_norm(strictb200_ctx* ctx, const GroupNormArgs& a, int64_t M, int64_t d) {
+  if (a.groups < 1 || d % a.groups) return sb_fail(STRICTB200_ERR_INVALID_ARG, "group_norm: the width must be a multiple of the groups");
+  if (a.groups > 16383 || a.splits < 1 || a.splits > 8) return sb_fail(STRICTB200_ERR_INVALID_ARG, "group_norm: at most 16383 groups and 8 partial sums");
+  GroupNormDev v{a.x, a.ldx, a.part, a.ldp, a.splits, a.g1, a.g2, a.eps, a.y1, a.y2, a.ldy, (int)(d / a.groups), 1, ctx->d_status};
+  const bool vec = v.gw % 4 == 0 && a.ldx % 4 == 0 && a.ldp % 4 == 0 && a.ldy % 4 == 0 && v.gw <= 8192;
+  if (!vec) {
+    dim3 grid((unsigned)M, (unsigned)a.groups);
+    if (a.f32) SB_CUDA(sb_launch(ctx, group_norm_any_kernel<float>, grid, dim3(256), 0, v, M));
+    else SB_CUDA(sb_launch(ctx, group_norm_any_kernel<bf16>, grid, dim3(256), 0, v, M));
+    ctx->launches++;
+    return STRICTB200_OK;
+  }
+  // few rows (decode): a wide group is shared by a cluster, so that its partial sums come through several SMs' paths to L2
+  const int want = ctx->opt.row_cluster > 8 ? 8 : ctx->opt.row_cluster;
+  if (want > 1 && M <= 256 && v.gw >= 1024 && v.gw % (4 * want) == 0) v.cb = want;
+  const int n4 = v.gw / v.cb / 4;
+  const int ni = n4 <= 1024 && (M <= 256 || n4 <= 256) ? 1 : 4;
+  const int threads = ((n4 + ni - 1) / ni + 31) / 32 * 32;
+  dim3 grid((unsigned)M, (unsigned)(a.groups * v.cb));
+  auto go = [&](auto kernel) { return v.cb > 1 ? sb_launch_cluster(ctx, kernel, grid, dim3(threads), 0, dim3(1, v.cb, 1), v, M) : sb_launch(ctx, kernel, grid, dim3(threads), 0, v, M); };
+  if (a.f32) SB_CUDA(ni == 1 ? go(group_norm_kernel<float, 1>) : go(group_norm_kernel<float, 4>));
+  else SB_CUDA(ni == 1 ? go(group_norm_kernel<bf16, 1>) : go(group_norm_kernel<bf16, 4>));
+  ctx->launches++;
+  return STRICTB200_OK;
+}

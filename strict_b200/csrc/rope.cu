@@ -203,11 +203,11 @@ int k_rope_qknorm_kvappend(strictb200_ctx* ctx, const RopeArgs& a, int64_t T) {
 
 // cos/sin of pos * theta^(-2i/D), evaluated in double on the host and rounded to fp32: part of
 // the model constants (like the weights), not of the per-token path.
-int sb_rope_table(strictb200_ctx* ctx, int max_pos, int D, float theta, float** d_cos, float** d_sin) {
+int sb_rope_table(strictb200_ctx* ctx, int max_pos, int D, double theta, float** d_cos, float** d_sin) {
   int h = D / 2;
   std::vector<float> c((size_t)max_pos * h), s((size_t)max_pos * h);
   std::vector<double> inv(h);
-  for (int i = 0; i < h; i++) inv[i] = std::pow((double)theta, -2.0 * (double)i / (double)D);
+  for (int i = 0; i < h; i++) inv[i] = std::pow(theta, -2.0 * (double)i / (double)D);
   for (int p = 0; p < max_pos; p++)
     for (int i = 0; i < h; i++) {
       double ang = (double)p * inv[i];

@@ -37,6 +37,10 @@ __global__ void embedding_f32_kernel(const float* __restrict__ wte, const float*
   int64_t t = blockIdx.x;
   int64_t id = ids[t];
   if (id < 0 || id >= vocab) id = 0;
+  if (!wpe) {  // no learned positions
+    for (int64_t i = threadIdx.x; i < d; i += blockDim.x) out[t * d + i] = wte[id * d + i];
+    return;
+  }
   int p = pos ? pos[t] : lens[t];
   if (p < 0 || p >= max_pos) p = 0;
   for (int64_t i = threadIdx.x; i < d; i += blockDim.x) out[t * d + i] = __fadd_rn(wte[id * d + i], wpe[(int64_t)p * d + i]);

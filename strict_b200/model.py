@@ -2,7 +2,9 @@
 
 Model configs of the benchmark are in CONFIGS; `Model(ctx, cfg)` allocates the weights on the
 context's device (this rank's shard under tensor parallelism), `init_random(seed)` fills them
-from the seeded generator, `new_cache(batch, maxlen)` creates the KV cache object.
+from the seeded generator, `new_cache(batch, maxlen)` creates the KV cache object. A configuration
+with arch STACK describes its layers one by one (stack_config); checkpoints in a folder are read by
+checkpoint.py, which picks the configuration by the architecture that config.json names.
 """
 import ctypes as C
 
@@ -10,7 +12,10 @@ import numpy as np
 
 from . import native as N
 
-GPT2, QWEN3 = 0, 1
+GPT2, QWEN3, STACK = 0, 1, 2
+BF16, FP32 = 0, 1            # strictb200_dtype
+MIXER_LATENT = 1             # strictb200_mixer
+MLP_NONE, MLP_XIELU = 0, 1   # strictb200_mlp
 
 CONFIGS = {
     # GPT-2 small: 12 layers, d 768, 12 heads x 64, MLP 3072, LN eps 1e-5, 1024 positions, tied
@@ -34,10 +39,38 @@ def make_config(cfg):
     return c
 
 
+def latent_layer(heads, dim, rot_dim, vdim, kv_rank, scale, rot_base, window=0, kv_from=-1, d_ff=0):
+    """One layer of a STACK configuration: latent attention, and an xIELU feed-forward when d_ff > 0."""
+    return dict(mixer=MIXER_LATENT, heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, window=window, kv_from=kv_from,
+                mlp=MLP_XIELU if d_ff else MLP_NONE, d_ff=d_ff, scale=scale, rot_base=rot_base)
+
+
+def stack_config(layers, d_model, vocab, max_pos, norm_groups, eps, dtype=BF16):
+    """Configuration of a model described layer by layer (strictb200_stack_create)."""
+    return dict(arch=STACK, n_layers=len(layers), d_model=d_model, vocab=vocab, max_pos=max_pos, norm_groups=norm_groups, eps=eps, dtype=dtype,
+                layers=list(layers))
+
+
+def make_stack_config(cfg):
+    c = N.StackConfig()
+    for k in ("n_layers", "d_model", "vocab", "max_pos", "norm_groups", "dtype"):
+        setattr(c, k, int(cfg[k]))
+    c.eps = float(cfg["eps"])
+    layers = (N.LayerConfig * len(cfg["layers"]))()
+    for dst, src in zip(layers, cfg["layers"]):
+        for k, t in N.LayerConfig._fields_:
+            setattr(dst, k, float(src[k]) if t is C.c_double else int(src[k]))
+    return c, layers
+
+
 class Model:
     def __init__(self, ctx, cfg):
         self.ctx, self.cfg = ctx, dict(cfg)
         self.h = C.c_void_p()
+        if cfg["arch"] == STACK:
+            c, layers = make_stack_config(cfg)
+            N.check(N.lib().strictb200_stack_create(ctx.h, C.byref(c), layers, C.byref(self.h)))
+            return
         c = make_config(cfg)
         N.check(N.lib().strictb200_model_create(ctx.h, C.byref(c), C.byref(self.h)))
 
@@ -98,6 +131,19 @@ class KvCache:
         nxt = np.empty(B, np.int32)
         logits = np.empty((B, self.model.cfg["vocab"]), np.float32) if want_logits else None
         N.check(N.lib().strictb200_prefill(self.model.h, self.h, N.ptr(tokens), N.ptr(lens), B, S, N.ptr(nxt), N.ptr(logits)))
+        return nxt, logits
+
+    def prefill_rows(self, tokens, want, lens=None):
+        """tokens [B,S] int32 and, per sequence, the places among its new tokens whose logits are asked for;
+        returns (next_ids[B], logits[places, V]), the sequences' places one after the other."""
+        tokens = np.ascontiguousarray(tokens, dtype=np.int32)
+        B, S = tokens.shape
+        lens = np.full(B, S, np.int32) if lens is None else np.ascontiguousarray(lens, dtype=np.int32)
+        n_want = np.array([len(w) for w in want], np.int32)
+        places = np.array([p for w in want for p in w], np.int32)
+        nxt = np.empty(B, np.int32)
+        logits = np.empty((len(places), self.model.cfg["vocab"]), np.float32)
+        N.check(N.lib().strictb200_prefill_rows(self.model.h, self.h, N.ptr(tokens), N.ptr(lens), B, S, N.ptr(places), N.ptr(n_want), N.ptr(nxt), N.ptr(logits)))
         return nxt, logits
 
     def decode_step(self, ids, want_logits=False, out=None):

@@ -28,6 +28,17 @@ class ModelConfig(C.Structure):
                 ("max_pos", C.c_int32), ("tied", C.c_int32), ("eps", C.c_float), ("rope_theta", C.c_float)]
 
 
+class LayerConfig(C.Structure):
+    """strictb200_layer_config"""
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "rot_dim", "vdim", "kv_rank", "window", "kv_from", "mlp", "d_ff")] + \
+               [("scale", C.c_double), ("rot_base", C.c_double)]
+
+
+class StackConfig(C.Structure):
+    """strictb200_stack_config"""
+    _fields_ = [(n, C.c_int32) for n in ("n_layers", "d_model", "vocab", "max_pos", "norm_groups", "dtype")] + [("eps", C.c_double)]
+
+
 _lib = None
 
 vp, i32, i64, u64, f32, u32, sz = C.c_void_p, C.c_int, C.c_int64, C.c_uint64, C.c_float, C.c_uint32, C.c_size_t
@@ -76,6 +87,7 @@ SIGNATURES = {
     "strictb200_quantize_rows_int8": [vp, vp, i64, i64, vp, vp],
     "strictb200_gemm_int8": [vp, i64, i64, i64, vp, vp, vp, vp, vp],
     "strictb200_gemm_int8w": [vp, i64, i64, i64, vp, vp, vp, vp],
+    "strictb200_gemm_bf16": [vp, i64, i64, i64, vp, vp, vp, i32],
     "strictb200_gemm_f32": [vp, i64, i64, i64, vp, vp, vp, vp],
     "strictb200_rmsnorm": [vp, vp, vp, vp, f32, i64, i64, vp],
     "strictb200_layernorm": [vp, vp, vp, vp, f32, i64, i64, vp],
@@ -88,6 +100,7 @@ SIGNATURES = {
     "strictb200_embedding_bf16": [vp, vp, vp, i64, i64, i64, vp],
     "strictb200_argmax": [vp, vp, i64, i64, vp],
     "strictb200_model_create": [vp, C.POINTER(ModelConfig), C.POINTER(vp)],
+    "strictb200_stack_create": [vp, C.POINTER(StackConfig), C.POINTER(LayerConfig), C.POINTER(vp)],
     "strictb200_model_destroy": [vp],
     "strictb200_model_init_random": [vp, u64],
     "strictb200_model_set_tensor": [vp, C.c_char_p, vp, sz],
@@ -100,6 +113,7 @@ SIGNATURES = {
     "strictb200_kv_lens": [vp, vp],
     "strictb200_kv_fill_synthetic": [vp, u64, i32],
     "strictb200_prefill": [vp, vp, vp, vp, i32, i32, vp, vp],
+    "strictb200_prefill_rows": [vp, vp, vp, vp, i32, i32, vp, vp, vp, vp],
     "strictb200_decode_step": [vp, vp, vp, vp, vp],
     "strictb200_generate": [vp, vp, vp, i32, vp],
     "strictb200_decode_steps_device": [vp, vp, vp, i32],
