@@ -240,6 +240,13 @@ int strictb200_gemm_f32(strictb200_ctx* ctx, int64_t M, int64_t N, int64_t K, co
  * reachable through strictb200_tp_allreduce_rownorm under tensor parallelism). */
 int strictb200_rmsnorm(strictb200_ctx* ctx, const uint16_t* d_x, uint16_t* d_residual, const float* d_gain, float eps, int64_t M,
                        int64_t d, uint16_t* d_y);
+/* Grouped RMS norm with one or two gains: the d columns in `groups` equal consecutive parts, each divided by its own
+ * sqrt(mean(x^2) + eps); y1 = x_n * gain1 and, if not NULL, y2 = x_n * gain2. Rows of d columns; fp32 in, out_dtype 0 bf16,
+ * 1 fp32. Partial sums d_part [splits][M,d] (may be NULL, at most 8) are first added to d_x in place. */
+int strictb200_group_rmsnorm(strictb200_ctx* ctx, float* d_x, const float* d_part, int splits, const float* d_gain1, const float* d_gain2,
+                             float eps, int groups, int64_t M, int64_t d, void* d_y1, void* d_y2, int out_dtype);
+/* y = softplus(p) x^2 + x/2 above zero, (1/2 + softplus(q)) (exp(x) - 1 - x) + x/2 otherwise. */
+int strictb200_xielu(strictb200_ctx* ctx, const float* d_x, int64_t count, float p, float q, float* d_y);
 int strictb200_layernorm(strictb200_ctx* ctx, const float* d_x, const float* d_gain, const float* d_bias, float eps, int64_t M,
                          int64_t d, float* d_y);
 /* y = bf16(silu(gate) * up); gate_up is [M, 2*I] with gate in columns [0,I). */

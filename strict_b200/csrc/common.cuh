@@ -221,6 +221,7 @@ struct GroupNormArgs {
   bool f32 = false;              // y in fp32
 };
 int k_group_norm(strictb200_ctx*, const GroupNormArgs& a, int64_t M, int64_t d);
+void sb_xielu_coefficients(float p, float q, float* pos, float* neg);
 int k_layernorm(strictb200_ctx*, const float* x, const float* g, const float* b, float eps, int64_t M, int64_t d, float* y);
 int k_add_f32(strictb200_ctx*, float* x, const float* y, int64_t n);
 int k_swiglu(strictb200_ctx*, const bf16* gate_up, const float* gate_up_f32, int64_t M, int64_t I, bf16* y, uint8_t* q, float* qscale);

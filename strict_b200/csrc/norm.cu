@@ -1,6 +1,8 @@
 // Row-wise kernels of the residual stream: two-term E4M3 split of bf16 rows, fused
 // (split-K reduce + dequant) + residual add + RMSNorm + quantise, LayerNorm, SwiGLU, GELU.
 // All are HBM/L2 streams: one block per token row, 128-bit loads, warp-shuffle reductions.
+#include <cmath>
+
 #include "common.cuh"
 
 namespace {
@@ -935,4 +937,43 @@ int k_group_norm(strictb200_ctx* ctx, const GroupNormArgs& a, int64_t M, int64_t
   else SB_CUDA(ni == 1 ? go(group_norm_kernel<bf16, 1>) : go(group_norm_kernel<bf16, 4>));
   ctx->launches++;
   return STRICTB200_OK;
+}
+
+namespace {
+__global__ void xielu_kernel(const float* __restrict__ x, int64_t n, float pos, float neg, float* __restrict__ y) {
+  const int64_t step = (int64_t)gridDim.x * blockDim.x;
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += step) y[i] = sb_xielu(x[i], pos, neg);
+}
+}  // namespace
+
+// Coefficients of xIELU from its two numbers, in double.
+void sb_xielu_coefficients(float p, float q, float* pos, float* neg) {
+  auto softplus = [](double z) { return std::log1p(std::exp(-std::fabs(z))) + (z > 0 ? z : 0.0); };
+  *pos = (float)softplus(p);
+  *neg = (float)(0.5 + softplus(q));
+}
+
+extern "C" int strictb200_xielu(strictb200_ctx* ctx, const float* d_x, int64_t count, float p, float q, float* d_y) {
+  SB_ENTER(ctx);
+  SB_REQUIRE(count >= 0, "negative size");
+  if (!count) return STRICTB200_OK;
+  SB_REQUIRE(d_x && d_y, "null pointer");
+  float pos, neg;
+  sb_xielu_coefficients(p, q, &pos, &neg);
+  xielu_kernel<<<stream_grid(ctx, count, 256), 256, 0, ctx->stream>>>(d_x, count, pos, neg, d_y);
+  SB_LAUNCHED(ctx);
+  return STRICTB200_OK;
+}
+
+extern "C" int strictb200_group_rmsnorm(strictb200_ctx* ctx, float* d_x, const float* d_part, int splits, const float* d_gain1, const float* d_gain2,
+                                        float eps, int groups, int64_t M, int64_t d, void* d_y1, void* d_y2, int out_dtype) {
+  SB_ENTER(ctx);
+  SB_REQUIRE(M >= 0 && M <= INT32_MAX && d > 0 && d <= INT32_MAX, "bad shape");
+  if (!M) return STRICTB200_OK;
+  SB_REQUIRE(d_x && d_gain1 && d_y1 && (!d_gain2 || d_y2), "null pointer");
+  SB_REQUIRE(out_dtype == 0 || out_dtype == 1, "out_dtype: 0 bf16, 1 fp32");
+  GroupNormArgs a;
+  a.x = d_x; a.ldx = d; a.part = d_part; a.ldp = d; a.splits = splits; a.g1 = d_gain1; a.g2 = d_gain2; a.eps = eps; a.groups = groups;
+  a.y1 = d_y1; a.y2 = d_y2; a.ldy = d; a.f32 = out_dtype == 1;
+  return k_group_norm(ctx, a, M, d);
 }

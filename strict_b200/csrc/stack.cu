@@ -36,7 +36,6 @@ struct StackLayer {
 };
 
 int64_t pad8(int64_t n) { return (n + 7) / 8 * 8; }
-float softplus(double z) { return (float)(std::log1p(std::exp(-std::fabs(z))) + std::max(z, 0.0)); }
 
 }  // namespace
 
@@ -152,10 +151,7 @@ bool find_slot(strictb200_model* m, const std::string& name, Slot* o) {
   return false;
 }
 
-void set_act(StackLayer& w) {
-  w.act_pos = softplus(w.act[0]);
-  w.act_neg = (float)(0.5 + (double)softplus(w.act[1]));
-}
+void set_act(StackLayer& w) { sb_xielu_coefficients(w.act[0], w.act[1], &w.act_pos, &w.act_neg); }
 
 // ------------------------------------------------------------------ pieces both schedules use
 // y = x . w^T of one matrix that is no part of a combined launch (the LM head)

@@ -90,6 +90,8 @@ SIGNATURES = {
     "strictb200_gemm_bf16": [vp, i64, i64, i64, vp, vp, vp, i32],
     "strictb200_gemm_f32": [vp, i64, i64, i64, vp, vp, vp, vp],
     "strictb200_rmsnorm": [vp, vp, vp, vp, f32, i64, i64, vp],
+    "strictb200_group_rmsnorm": [vp, vp, vp, i32, vp, vp, f32, i32, i64, i64, vp, vp, i32],
+    "strictb200_xielu": [vp, vp, i64, f32, f32, vp],
     "strictb200_layernorm": [vp, vp, vp, vp, f32, i64, i64, vp],
     "strictb200_swiglu": [vp, vp, i64, i64, vp],
     "strictb200_gelu_tanh": [vp, vp, i64, vp],
