@@ -1,0 +1,158 @@
+"""Prefill and decode throughput of the Kipatar design at sizes that resemble a real model's layers (random
+weights), beside the framework's closest existing model (Qwen3: grouped-query attention, sequential SwiGLU
+layers, E4M3 weights) at equal width, depth, heads, feed-forward and vocabulary.
+
+    python bench.py --design kipatar [--steps K] [--warmup W] [--sizes 8b,0.6b] [--layers N]
+
+Prints one JSON line. Times are CUDA events on the library's stream (prefill: the public prefill call,
+host ids in, greedy ids out; decode: graph-replayed steps with ids resident on the device). A step streams
+more than L2 holds in every configuration but the few-layer ones of --layers. `kernels` are plain launches
+of the decode step, one pair of events per call, with the bytes a call must move and their share of the
+copy bandwidth; `flops_frac` is a prefill's useful matrix work over the measured bf16 throughput.
+"""
+import json
+import os
+
+import numpy as np
+
+from . import clocks, native as N
+from .kernel import Context, DeviceVariable
+from .model import CONFIGS, STACK, Model, latent_layer, stack_config
+
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+
+# name -> (Qwen3 configuration, latent rank, rotated dims, window, [(batch, prompt)] for decode, for prefill)
+SIZES = {
+    "8b": ("qwen3-8b", 512, 64, 2048, [(32, 2048), (1, 2048)], [(8, 2048), (1, 2048), (1, 8192)]),
+    "0.6b": ("qwen3-0.6b", 256, 64, 1024, [(32, 2048), (1, 2048)], [(8, 2048), (1, 2048)]),
+}
+
+
+def kipatar_like(qwen, rank, rot, window, max_pos):
+    """The design at the sizes of a Qwen3 configuration: as many heads, heads as wide, the same feed-forward width. Every
+    fourth layer reads the latents of the one before it."""
+    layers = [latent_layer(heads=qwen["n_q_heads"], dim=qwen["head_dim"], rot_dim=rot, vdim=qwen["head_dim"], kv_rank=rank,
+                           scale=(qwen["head_dim"] + rot) ** -0.5, rot_base=1e6, window=window, kv_from=i - 1 if i % 4 == 3 else -1, d_ff=qwen["d_ff"])
+              for i in range(qwen["n_layers"])]
+    return stack_config(layers, d_model=qwen["d_model"], vocab=qwen["vocab"], max_pos=max_pos, norm_groups=8, eps=1e-6)
+
+
+def peaks():
+    path = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    if os.path.exists(path):
+        p = json.load(open(path))
+        return float(p["hbm_gbs"]), float(p["bf16_tflops"]), float(p.get("bf16_tflops_sustained", p["bf16_tflops"])), "measured"
+    return 6650.0, 1590.0, 1400.0, "fallback"
+
+
+def seen(n, window):
+    """Sum over the positions 0..n-1 of the keys each sees."""
+    w = window or n
+    return sum(min(i + 1, w) for i in range(n)) if n < w else w * (w + 1) // 2 + (n - w) * w
+
+
+def prefill_flops(cfg, B, S):
+    """Useful matrix work of a prompt: linear layers (the head on the last row only) and attention over the keys each position sees."""
+    d, T, f = cfg["d_model"], B * S, 0
+    if cfg["arch"] == STACK:
+        for y in cfg["layers"]:
+            H, q, own = y["heads"], y["dim"] + y["rot_dim"], y["kv_from"] < 0
+            f += 2 * T * (d * (H * q + (y["kv_rank"] + y["rot_dim"] if own else 0) + H * y["vdim"] + 2 * y["d_ff"]) + y["kv_rank"] * H * (y["dim"] + y["vdim"]))
+            f += 2 * B * seen(S, y["window"]) * H * (q + y["vdim"])
+        return f
+    D, H, Hkv = cfg["head_dim"], cfg["n_q_heads"], cfg["n_kv_heads"]
+    return cfg["n_layers"] * (2 * T * d * ((2 * H + 2 * Hkv) * D + 3 * cfg["d_ff"]) + 4 * B * seen(S, 0) * H * D)
+
+
+def call_bytes(cfg, B, length):
+    """Bytes a call of each kernel class of the decode step must move (weights or cache once), averaged over the layers."""
+    d = cfg["d_model"]
+    if cfg["arch"] == STACK:
+        L = cfg["layers"]
+        mean = lambda f: sum(f(y) for y in L) / len(L)  # noqa: E731
+        return {"gemm_qkv": 2 * d * mean(lambda y: y["heads"] * (y["dim"] + y["rot_dim"]) + (y["kv_rank"] + y["rot_dim"] if y["kv_from"] < 0 else 0) + y["d_ff"]),
+                "rope_kvappend": 2 * mean(lambda y: y["heads"] * y["dim"] * y["kv_rank"]),
+                "attn_decode": 2 * B * mean(lambda y: min(length, y["window"] or length) * (y["kv_rank"] + y["rot_dim"])),
+                "attn_merge": 2 * mean(lambda y: y["heads"] * y["vdim"] * y["kv_rank"]),
+                "gemm_o": 2 * d * mean(lambda y: y["heads"] * y["vdim"] + y["d_ff"]), "head": 2 * cfg["vocab"] * d}
+    D, H, Hkv, I = cfg["head_dim"], cfg["n_q_heads"], cfg["n_kv_heads"], cfg["d_ff"]
+    return {"gemm_qkv": (H + 2 * Hkv) * D * d, "gemm_o": H * D * d, "gemm_gate_up": 2 * I * d, "gemm_down": d * I, "head": cfg["vocab"] * d,
+            "attn_decode": B * length * Hkv * D * 4}
+
+
+def ids(ctx, n, vocab, seed):
+    v = DeviceVariable(ctx, n, np.int32)
+    N.check(N.lib().strictb200_gen_tokens(ctx.h, seed, 1, n, vocab, v.p))
+    out = v.to_host()
+    v.free()
+    return out
+
+
+def run_model(ctx, cfg, decode, prefill, steps, warmup):
+    hbm, burst, sustained, _ = peaks()
+    model = Model(ctx, cfg).init_random(5)
+    out = {"weights_gb": model.weight_bytes() / 1e9, "prefill": [], "decode": []}
+    for B, S in prefill:
+        toks = ids(ctx, B * S, cfg["vocab"], 6).reshape(B, S)
+        kv = model.new_cache(B, S)
+        for _ in range(3):
+            kv.reset()
+            kv.prefill(toks)
+        times = []
+        sampler = clocks.ClockSampler(0)
+        sampler.start()
+        for _ in range(max(3, min(steps, 5))):
+            kv.reset()
+            ctx.synchronize()
+            ctx.timer_begin()
+            kv.prefill(toks)
+            times.append(ctx.timer_end())
+        ms, flops = float(np.median(times)), prefill_flops(cfg, B, S)
+        out["prefill"].append({"batch": B, "prompt": S, "ms": ms, "tokens_per_s": B * S / ms * 1e3, "tflops": flops / ms / 1e9,
+                               "flops_frac": flops / ms / 1e9 / sustained, "clocks": sampler.stop()})
+        kv.dispose()
+    for B, S in decode:
+        kv = model.new_cache(B, S + 2 * (steps + warmup) + 16)
+        kv.fill_synthetic(7, S)
+        kv.decode_step(ids(ctx, B, cfg["vocab"], 8))
+        kv.decode_steps_device(max(3, warmup))
+        ctx.synchronize()
+        sampler = clocks.ClockSampler(0)
+        sampler.start()
+        nbytes = kv.decode_bytes()
+        ctx.timer_begin()
+        kv.decode_steps_device(steps)
+        ms = ctx.timer_end() / steps
+        clk = sampler.stop()
+        kernels, per_call = {}, call_bytes(cfg, B, int(kv.lens().mean()))
+        for k, (tot, calls) in kv.profile_decode(3).items():
+            if calls:
+                us = tot / calls * 1e3
+                kernels[k] = {"us": us, "calls_per_step": calls / 3}
+                if k in per_call:
+                    calls_of_bytes = calls / 3 if k != "head" else 1  # the head's product and its pick are two calls
+                    kernels[k]["hbm_frac"] = per_call[k] / (tot * 1e3 / (3 * calls_of_bytes) * 1e-6) / 1e9 / hbm
+        out["decode"].append({"batch": B, "context": S, "ms": ms, "tokens_per_s": B / ms * 1e3, "step_gb": nbytes / 1e9,
+                              "hbm_frac": nbytes / (ms * 1e-3) / 1e9 / hbm, "kernels": kernels, "clocks": clk})
+        kv.dispose()
+    ctx.device_status()
+    model.dispose()
+    return out
+
+
+def run(sizes, steps, warmup, layers=0):
+    ctx = Context(0)
+    hbm, burst, sustained, kind = peaks()
+    result = {"design": "kipatar", "data": "synthetic (random weights)", "peaks": {"hbm_gbs": hbm, "bf16_tflops": burst, "bf16_tflops_sustained": sustained, "kind": kind},
+              "steps": steps, "warmup": warmup, "sizes": {}}
+    for name in sizes:
+        base, rank, rot, window, decode, prefill = SIZES[name]
+        qwen = dict(CONFIGS[base], max_pos=16384)
+        if layers:
+            qwen["n_layers"] = layers
+        ours = kipatar_like(qwen, rank, rot, window, 16384)
+        result["sizes"][name] = {"config": {"width": qwen["d_model"], "layers": qwen["n_layers"], "heads": qwen["n_q_heads"], "dim": qwen["head_dim"], "rot_dim": rot,
+                                            "kv_rank": rank, "window": window, "ff": qwen["d_ff"], "vocab": qwen["vocab"], "norm_groups": 8, "kv_from": "every fourth layer"},
+                                 "kipatar": run_model(ctx, ours, decode, prefill, steps, warmup), "qwen3": run_model(ctx, qwen, decode, prefill, steps, warmup)}
+    ctx.dispose()
+    print(json.dumps(result), flush=True)
