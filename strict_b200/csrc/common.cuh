@@ -230,6 +230,15 @@ int k_swiglu_part(strictb200_ctx*, const float* part, int splits, const float* s
                   float* qscale);
 int k_gelu_tanh(strictb200_ctx*, const float* x, int64_t n, float* y);
 #ifdef __CUDACC__
+// xIELU for results that are rounded to bf16: exp through ex2, and the series of exp(z) - 1 - z where that would cancel
+__device__ __forceinline__ float sb_xielu_bf16(float z, float pos, float neg) {
+  const float zz = z * z;
+  const float series = zz * fmaf(z, fmaf(z, 0.041666667f, 0.16666667f), 0.5f);
+  float e;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(z * 1.4426950408889634f));
+  const float t = z > -0.0625f ? series : e - 1.0f - z;
+  return fmaf(z > 0.f ? pos : neg, z > 0.f ? zz : t, 0.5f * z);
+}
 // tanh-approximated GELU in fp32 with the operation order of the element-wise kernel
 __device__ __forceinline__ float sb_gelu_tanh(float v) {
   const float u = __fmul_rn(0.797884583f, __fadd_rn(v, __fmul_rn(0.044715f, __fmul_rn(__fmul_rn(v, v), v))));
@@ -441,15 +450,38 @@ void sb_tp_abort(strictb200_ctx*);       // ncclCommAbort: stops the communicato
 
 // ------------------------------------------------------------------ device helpers
 #ifdef __CUDACC__
-// One finished value of a bf16 GEMM (Bf16Epilogue).
-__device__ __forceinline__ void sb_bf16_store(const Bf16Epilogue& e, int64_t m, int n, float v) {
-  if (e.act_out && n >= e.n_switch) {
-    e.act_out[m * e.ld_act + (n - e.n_switch)] = __float2bfloat16_rn(sb_xielu(v, e.act_pos, e.act_neg));
-  } else if (e.out_f32) {
-    float* o = e.out_f32 + m * e.ldo + n;
-    *o = e.accumulate ? *o + v : v;
-  } else {
-    e.out_bf16[m * e.ldo + n] = __float2bfloat16_rn(v);
+__device__ __forceinline__ uint32_t f32_to_bf16_bits(float f);
+// Sixteen tokens m0.. of one output channel n per lane (channels of a warp are consecutive, the first one even, all on the
+// same side of n_switch). bf16 rows: neighbouring lanes trade tokens so that each stores two channels at a time.
+__device__ __forceinline__ void sb_bf16_store16(const Bf16Epilogue& e, int M, int N, int m0, int n, const uint32_t* r) {
+  const bool act = e.act_out && n >= e.n_switch;
+  if (!act && e.out_f32) {
+    if (n >= N) return;
+    float* o = e.out_f32 + (int64_t)m0 * e.ldo + n;
+#pragma unroll
+    for (int j = 0; j < 16; j++, o += e.ldo)
+      if (m0 + j < M) *o = e.accumulate ? *o + __uint_as_float(r[j]) : __uint_as_float(r[j]);
+    return;
+  }
+  const int64_t ld = act ? e.ld_act : e.ldo;
+  bf16* o = act ? e.act_out + (n - e.n_switch) : e.out_bf16 + n;
+  float v[16];
+#pragma unroll
+  for (int j = 0; j < 16; j++) v[j] = act ? sb_xielu_bf16(__uint_as_float(r[j]), e.act_pos, e.act_neg) : __uint_as_float(r[j]);
+  if ((ld & 1) == 0 && (N & 1) == 0 && ((uintptr_t)(act ? e.act_out : e.out_bf16) & 3) == 0) {  // the same for every lane
+    const bool odd = n & 1;
+    o += (int64_t)(m0 + (odd ? 8 : 0)) * ld - (odd ? 1 : 0);
+#pragma unroll
+    for (int j = 0; j < 8; j++, o += ld) {
+      const float got = __shfl_xor_sync(0xffffffffu, odd ? v[j] : v[8 + j], 1);
+      const float lo = odd ? got : v[j], hi = odd ? v[8 + j] : got;
+      if (m0 + j + (odd ? 8 : 0) < M && n < N) *(uint32_t*)o = f32_to_bf16_bits(lo) | (f32_to_bf16_bits(hi) << 16);
+    }
+  } else if (n < N) {
+    o += (int64_t)m0 * ld;
+#pragma unroll
+    for (int j = 0; j < 16; j++, o += ld)
+      if (m0 + j < M) *o = __float2bfloat16_rn(v[j]);
   }
 }
 // Programmatic dependent launch. A kernel launched through sb_launch may begin while its

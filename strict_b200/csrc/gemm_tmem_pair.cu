@@ -255,11 +255,7 @@ __global__ void __launch_bounds__(192) gemm_pair_kernel(const __grid_constant__ 
         tc_ld16(acc + (uint32_t)(grp * 16), r);
         tc_wait_ld();
         if constexpr (BF16) {
-#pragma unroll
-          for (int j = 0; j < 16; j++) {
-            const int tok = 2 * tok_base + grp * 16 + j;  // 256 tokens per tile
-            if (tok < a.M && n < a.N) sb_bf16_store(a.e, tok, n, __uint_as_float(r[j]));
-          }
+          sb_bf16_store16(a.e, a.M, a.N, 2 * tok_base + grp * 16, n, r);  // 256 tokens per tile
         } else {
 #pragma unroll
         for (int j = 0; j < 8; j++) {

@@ -242,13 +242,14 @@ __global__ void __launch_bounds__(192) gemm_tmem_kernel(const __grid_constant__ 
         tc_ld16(tmem + ((uint32_t)(lg * 32) << 16) + (uint32_t)(grp * 16), r);
         tc_wait_ld();
         if (KIND == KIND_BF16) {
+          if (raw) {
 #pragma unroll
-          for (int j = 0; j < 16; j++) {
-            const int tok = t0 + grp * 16 + j;
-            if (tok < a.M && n < a.N) {
-              if (raw) a.part[((int64_t)blockIdx.z * a.M + tok) * a.N + n] = __uint_as_float(r[j]);
-              else sb_bf16_store(a.e, tok, n, __uint_as_float(r[j]));
+            for (int j = 0; j < 16; j++) {
+              const int tok = t0 + grp * 16 + j;
+              if (tok < a.M && n < a.N) a.part[((int64_t)blockIdx.z * a.M + tok) * a.N + n] = __uint_as_float(r[j]);
             }
+          } else {
+            sb_bf16_store16(a.e, a.M, a.N, t0 + grp * 16, n, r);
           }
           continue;
         }

@@ -41,8 +41,9 @@ __device__ __forceinline__ void ldsm_x2(uint32_t addr, uint32_t* r) {
 __device__ __forceinline__ void ldsm_x2_t(uint32_t addr, uint32_t* r) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
 }
+// not volatile: the compiler may move fragment loads ahead of products that do not need them
 __device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
-  asm volatile(
+  asm(
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
@@ -81,6 +82,17 @@ __device__ __forceinline__ float proj(const SplitDev& a, int64_t T, int64_t t, i
   for (int s = 0; s < a.splits; s++) v += a.in[((int64_t)s * T + t) * a.ld_in + col];
   return v;
 }
+// four columns at a time (col and the row stride multiples of 4; at most 8 splits), every split's load in flight at once
+__device__ __forceinline__ float4 proj4(const SplitDev& a, int64_t T, int64_t t, int64_t col) {
+  float4 p[8], v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int s = 0; s < 8; s++)
+    if (s < a.splits) p[s] = *(const float4*)(a.in + ((int64_t)s * T + t) * a.ld_in + col);
+#pragma unroll
+  for (int s = 0; s < 8; s++)
+    if (s < a.splits) { v.x += p[s].x; v.y += p[s].y; v.z += p[s].z; v.w += p[s].w; }
+  return v;
+}
 // pair i of a rotated vector (dimension 2i with 2i + 1)
 __device__ __forceinline__ void rotate(const SplitDev& a, int p, int i, float& u, float& v) {
   const float c = a.cos_t[(int64_t)p * (a.rot / 2) + i], s = a.sin_t[(int64_t)p * (a.rot / 2) + i];
@@ -92,23 +104,46 @@ __device__ __forceinline__ void rotate(const SplitDev& a, int p, int i, float& u
 template <typename T>
 __device__ __forceinline__ void append_latent(const SplitDev& a, int64_t rows, int64_t t, int b, int p, float* red) {
   const int64_t c0 = (int64_t)a.H * (a.dim + a.rot);
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < a.rank; i += blockDim.x) {
-    const float v = proj(a, rows, t, c0 + i);
-    ss += v * v;
+  T* dst = (T*)a.cache + ((int64_t)b * a.maxlen + p) * a.row;
+  // the rotated part is requested first, by threads from the end of the block, so that its loads run beside the latent's
+  const int ri = (int)blockDim.x - 1 - (int)threadIdx.x;
+  float u = 0.f, v = 0.f;
+  if (ri < a.rot / 2) { u = proj(a, rows, t, c0 + a.rank + 2 * ri); v = proj(a, rows, t, c0 + a.rank + 2 * ri + 1); }
+  float x[4], ss = 0.f;  // the first 4 * blockDim columns stay in registers
+#pragma unroll
+  for (int j = 0; j < 4; j++) {
+    const int i = j * (int)blockDim.x + (int)threadIdx.x;
+    x[j] = i < a.rank ? proj(a, rows, t, c0 + i) : 0.f;
+  }
+#pragma unroll
+  for (int j = 0; j < 4; j++) ss += x[j] * x[j];
+  for (int i = 4 * (int)blockDim.x + (int)threadIdx.x; i < a.rank; i += blockDim.x) {
+    const float w = proj(a, rows, t, c0 + i);
+    ss += w * w;
   }
   ss = block_sum(ss, red);
   const float r = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.rank), a.eps)));
-  T* dst = (T*)a.cache + ((int64_t)b * a.maxlen + p) * a.row;
-  for (int i = threadIdx.x; i < a.rank; i += blockDim.x) dst[i] = to_t<T>(proj(a, rows, t, c0 + i) * r * a.norm_w[i]);
-  for (int i = threadIdx.x; i < a.rot / 2; i += blockDim.x) {
-    float u = proj(a, rows, t, c0 + a.rank + 2 * i), v = proj(a, rows, t, c0 + a.rank + 2 * i + 1);
+#pragma unroll
+  for (int j = 0; j < 4; j++) {
+    const int i = j * (int)blockDim.x + (int)threadIdx.x;
+    if (i < a.rank) dst[i] = to_t<T>(x[j] * r * a.norm_w[i]);
+  }
+  for (int i = 4 * (int)blockDim.x + (int)threadIdx.x; i < a.rank; i += blockDim.x) dst[i] = to_t<T>(proj(a, rows, t, c0 + i) * r * a.norm_w[i]);
+  if (ri < a.rot / 2) {
+    rotate(a, p, ri, u, v);
+    dst[a.rank_p + 2 * ri] = to_t<T>(u);
+    dst[a.rank_p + 2 * ri + 1] = to_t<T>(v);
+  }
+  for (int i = (int)blockDim.x + ri; i < a.rot / 2; i += blockDim.x) {
+    u = proj(a, rows, t, c0 + a.rank + 2 * i);
+    v = proj(a, rows, t, c0 + a.rank + 2 * i + 1);
     rotate(a, p, i, u, v);
     dst[a.rank_p + 2 * i] = to_t<T>(u);
     dst[a.rank_p + 2 * i + 1] = to_t<T>(v);
   }
 }
 
+// grid (T, 2 with latents of its own, else 1)
 template <typename T>
 __global__ void __launch_bounds__(256) latent_split_kernel(SplitDev a, int64_t rows) {
   __shared__ float red[32];
@@ -117,18 +152,34 @@ __global__ void __launch_bounds__(256) latent_split_kernel(SplitDev a, int64_t r
   const int64_t t = blockIdx.x;
   const int b = a.seq ? a.seq[t] : (int)t, p = a.pos ? a.pos[t] : a.lens[b];
   if (p < 0 || p >= a.maxlen || p >= a.max_pos) return;  // host validates; never index outside the cache
+  if (blockIdx.y == 1) {  // the latent's half of the row
+    append_latent<T>(a, rows, t, b, p, red);
+    return;
+  }
   T* q = (T*)a.q_out + t * a.H * a.q_head;
-  const int half = (a.dim + a.rot) / 2;
-  if (((a.dim | a.rot) & 1) == 0 && a.splits == 1 && a.ld_in % 2 == 0) {
-    // two columns at a time
-    for (int i = threadIdx.x; i < a.H * half; i += blockDim.x) {
-      const int h = i / half, j = i - h * half;
-      const float2 w = *(const float2*)(a.in + t * a.ld_in + 2 * i);
-      float u = w.x, v = w.y;
-      if (2 * j >= a.dim) rotate(a, p, j - a.dim / 2, u, v);
-      T* dst = q + h * a.q_head + (2 * j < a.dim ? 2 * j : a.q_rot + 2 * j - a.dim);
-      if (sizeof(T) == 2) *(uint32_t*)dst = pack_bf16(u, v);
-      else *(float2*)dst = make_float2(u, v);
+  if (((a.dim | a.rot) & 3) == 0 && a.splits == 1 && a.ld_in % 4 == 0) {
+    // four columns at a time, four requests in flight per thread
+    const int quarter = (a.dim + a.rot) / 4, n = a.H * quarter;
+    const float4* in = (const float4*)(a.in + t * a.ld_in);
+    for (int i0 = threadIdx.x; i0 < n; i0 += 4 * (int)blockDim.x) {
+      float4 w[4];
+#pragma unroll
+      for (int u = 0; u < 4; u++)
+        if (i0 + u * (int)blockDim.x < n) w[u] = __ldcs(in + i0 + u * (int)blockDim.x);
+#pragma unroll
+      for (int u = 0; u < 4; u++) {
+        const int i = i0 + u * (int)blockDim.x;
+        if (i < n) {
+          const int h = i / quarter, j = (i - h * quarter) * 4;
+          if (j >= a.dim) {
+            rotate(a, p, (j - a.dim) / 2, w[u].x, w[u].y);
+            rotate(a, p, (j - a.dim) / 2 + 1, w[u].z, w[u].w);
+          }
+          T* dst = q + h * a.q_head + (j < a.dim ? j : a.q_rot + j - a.dim);
+          if (sizeof(T) == 2) *(uint2*)dst = make_uint2(pack_bf16(w[u].x, w[u].y), pack_bf16(w[u].z, w[u].w));
+          else *(float4*)dst = w[u];
+        }
+      }
     }
   } else {
     for (int i = threadIdx.x; i < a.H * a.dim; i += blockDim.x) {
@@ -144,7 +195,6 @@ __global__ void __launch_bounds__(256) latent_split_kernel(SplitDev a, int64_t r
       q[h * a.q_head + a.q_rot + 2 * j + 1] = to_t<T>(v);
     }
   }
-  if (a.cache) append_latent<T>(a, rows, t, b, p, red);
 }
 
 __global__ void __launch_bounds__(128) latent_gather_kernel(const bf16* __restrict__ cache, int64_t maxlen, int row, const int32_t* __restrict__ koff,
@@ -167,7 +217,8 @@ struct DecodeInDev {
   bf16* act;
   int64_t ld_act;
   int n_rt, n_grp;      // latent tiles of 64 and token groups of 16: blocks of the first role
-  int act_blocks;       // blocks per token of the activation
+  int rot_blocks;       // blocks per token of the rotation (256 pairs each)
+  int act_blocks;       // ... and of the activation
 };
 constexpr int QA_COLS = 64, QA_LD = QA_COLS + 8;
 __host__ __device__ inline int decode_in_smem(int dim) {
@@ -175,7 +226,8 @@ __host__ __device__ inline int decode_in_smem(int dim) {
   return d16 * QA_LD * 2 + 16 * (d16 + 8) * 2;
 }
 // One launch, four roles by block index: H * n_rt * n_grp blocks multiply queries with W_uk (64 latents of one head, 16
-// tokens), then B blocks rotate the queries' second part, B append the cache row, B * act_blocks run the activation.
+// tokens), then B * rot_blocks rotate the queries' second part, B append the cache row (a layer with latents of its own),
+// B * act_blocks run the activation.
 __global__ void __launch_bounds__(256) latent_decode_in_kernel(DecodeInDev d, int B) {
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ float red[32];
@@ -197,7 +249,14 @@ __global__ void __launch_bounds__(256) latent_decode_in_kernel(DecodeInDev d, in
     cp_async_commit();
     pdl_wait();
     SB_TRACE_WAITED();
-    for (int i = threadIdx.x; i < 16 * d16; i += blockDim.x) {
+    if (((a.dim | a.rot) & 3) == 0 && a.ld_in % 4 == 0) {
+      for (int i = threadIdx.x; i < 4 * d16; i += blockDim.x) {
+        const int m = i / (d16 / 4), k = (i - m * (d16 / 4)) * 4;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (b0 + m < B && k < a.dim) v = proj4(a, B, b0 + m, (int64_t)h * (a.dim + a.rot) + k);
+        *(uint2*)(qt + m * (d16 + 8) + k) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+      }
+    } else for (int i = threadIdx.x; i < 16 * d16; i += blockDim.x) {
       const int m = i / d16, k = i - m * d16;
       qt[m * (d16 + 8) + k] = b0 + m < B && k < a.dim ? __float2bfloat16_rn(proj(a, B, b0 + m, (int64_t)h * (a.dim + a.rot) + k)) : __float2bfloat16_rn(0.f);
     }
@@ -222,11 +281,11 @@ __global__ void __launch_bounds__(256) latent_decode_in_kernel(DecodeInDev d, in
   pdl_wait();
   SB_TRACE_WAITED();
   blk -= n_mul;
-  if (blk < B) {
-    const int b = blk, p = a.lens[b], rp = a.row - a.rank_p;
+  if (blk < B * d.rot_blocks) {
+    const int b = blk / d.rot_blocks, p = a.lens[b], rp = a.row - a.rank_p;
     if (p < 0 || p >= a.maxlen || p >= a.max_pos) return;
-    for (int i = threadIdx.x; i < a.H * (rp / 2); i += blockDim.x) {
-      const int h = i / (rp / 2), j = i - h * (rp / 2);
+    const int i = (blk % d.rot_blocks) * 256 + (int)threadIdx.x, h = i / (rp / 2), j = i - h * (rp / 2);
+    if (h < a.H) {
       float u = 0.f, v = 0.f;
       if (2 * j < a.rot) {
         const int64_t col = (int64_t)h * (a.dim + a.rot) + a.dim + 2 * j;
@@ -236,27 +295,42 @@ __global__ void __launch_bounds__(256) latent_decode_in_kernel(DecodeInDev d, in
       }
       *(uint32_t*)(d.q_abs + ((int64_t)b * a.H + h) * a.row + a.rank_p + 2 * j) = pack_bf16(u, v);
     }
-  } else if (blk < 2 * B) {
-    if (!a.cache) return;
-    const int b = blk - B, p = a.lens[b];
+    SB_TRACE_END(SB_K_ROPE, 0);
+    return;
+  }
+  blk -= B * d.rot_blocks;
+  if (a.cache && blk < B) {
+    const int p = a.lens[blk];
     if (p < 0 || p >= a.maxlen || p >= a.max_pos) return;
-    append_latent<bf16>(a, B, b, b, p, red);
+    append_latent<bf16>(a, B, blk, blk, p, red);
+    SB_TRACE_END(SB_K_ROPE, 0);
+    return;
+  }
+  if (a.cache) blk -= B;
+  const int b = blk / d.act_blocks, c0 = (blk % d.act_blocks) * 1024;
+  bf16* act = d.act + (int64_t)b * d.ld_act;
+  if (((d.act_col | d.n_act) & 3) == 0 && a.ld_in % 4 == 0 && ((uintptr_t)act & 7) == 0) {
+    const int i = c0 + (int)threadIdx.x * 4;
+    if (i < d.n_act) {
+      const float4 v = proj4(a, B, b, d.act_col + i);
+      *(uint2*)(act + i) = make_uint2(pack_bf16(sb_xielu_bf16(v.x, d.act_pos, d.act_neg), sb_xielu_bf16(v.y, d.act_pos, d.act_neg)),
+                                      pack_bf16(sb_xielu_bf16(v.z, d.act_pos, d.act_neg), sb_xielu_bf16(v.w, d.act_pos, d.act_neg)));
+    }
   } else {
-    blk -= 2 * B;
-    const int b = blk / d.act_blocks, c0 = (blk % d.act_blocks) * 1024;
-    for (int i = c0 + (int)threadIdx.x; i < min(c0 + 1024, d.n_act); i += blockDim.x)
-      d.act[(int64_t)b * d.ld_act + i] = __float2bfloat16_rn(sb_xielu(proj(a, B, b, d.act_col + i), d.act_pos, d.act_neg));
+    for (int i = c0 + (int)threadIdx.x; i < min(c0 + 1024, d.n_act); i += blockDim.x) act[i] = __float2bfloat16_rn(sb_xielu_bf16(proj(a, B, b, d.act_col + i), d.act_pos, d.act_neg));
   }
   SB_TRACE_END(SB_K_ROPE, 0);
 }
 
 // ------------------------------------------------------------------ decode: split-key attention over the latents
-// grid (nsplit, ceil(H / (16 MT)), B), 256 threads. Rows of the MMA tiles = up to 16 MT heads, 64 keys per step.
-//   S partials  warp (ks, kh): reduction steps ks, ks + 4, .. of the cache row for the 32 keys of half kh; its share of the
-//               queries stays in registers for the whole block, so a step reads the key tile from shared memory once
-//   softmax     the four partial scores of a (head, key) are added in slice order; running maximum and sum per head
-//   O += P c    every warp owns 8 NV latent columns of all heads; the key tile is its operand again
-constexpr int LKT = 64;
+// grid (nsplit, ceil(H / (16 MT)), B), 256 threads. Rows of the MMA tiles = up to 16 MT heads, 32 keys per step. Three
+// products of three different steps share an iteration, so one barrier per step is enough:
+//   S(t+1) partials  warp (ks, kh): reduction steps ks, ks + 4, .. of the cache row for the 16 keys of half kh; its share of
+//                    the queries stays in registers for the whole block, so a step reads the key tile from shared memory once
+//   softmax(t)       the four partial scores of a (head, key) are added in slice order; running maximum and sum per head
+//   O += P(t-1) c    every warp owns 8 NV latent columns of all heads; the key tile is its operand again
+// Key tiles pass through a ring of NS stages (t-1, t, t+1 in use, the rest in flight).
+constexpr int LKT = 32;
 struct AttnDecodeDev {
   const bf16* q;
   const bf16* cache;
@@ -267,27 +341,35 @@ struct AttnDecodeDev {
   float* ml_part;
   int prefetch;
 };
-template <int MT>
-__host__ __device__ constexpr int attn_decode_fixed_smem() { return 4 * MT * 16 * 68 * 4 + 2 * MT * 16 * 72 * 2 + MT * 16 * 4; }
+constexpr int SP_LD = 36, PP_LD = 40;  // row strides of the score (fp32) and weight (bf16) tiles
+constexpr int decode_stages(int ksm) { return ksm > 5 ? 4 : 6; }
+constexpr size_t attn_decode_smem(int mt, int ksm, int row) {
+  return (size_t)decode_stages(ksm) * LKT * (row * 2 + 16) + (size_t)2 * 4 * mt * 16 * SP_LD * 4 + (size_t)2 * 2 * mt * 16 * PP_LD * 2 + 2 * mt * 16 * 4;
+}
 
 template <int MT, int KSM, int NV>
 __global__ void __launch_bounds__(256) latent_attn_decode_kernel(AttnDecodeDev a) {
+  constexpr int NS = decode_stages(KSM), R = MT * 16;
   extern __shared__ __align__(128) uint8_t smem[];
   SB_TRACE_BEGIN();
   pdl_trigger();
-  const int split = blockIdx.x, h0 = blockIdx.y * MT * 16, b = blockIdx.z;
+  const int split = blockIdx.x, h0 = blockIdx.y * R, b = blockIdx.z;
   const int RS = a.row * 2 + 16;  // shared-memory row stride: an odd number of 16-byte chunks
-  uint8_t* tiles = smem;
-  float* sp = (float*)(smem + 2 * LKT * RS);           // [4][MT*16][68]
-  bf16* pp = (bf16*)(sp + 4 * MT * 16 * 68);           // [2][MT*16][72]
-  float* corr_s = (float*)(pp + 2 * MT * 16 * 72);     // [MT*16]
+  uint8_t* tiles = smem;                               // [NS][LKT][RS]
+  float* sp = (float*)(smem + NS * LKT * RS);          // [2][4][R][SP_LD]
+  bf16* pp = (bf16*)(sp + 2 * 4 * R * SP_LD);          // [2][hi, lo][R][PP_LD]
+  float* corr_s = (float*)(pp + 2 * 2 * R * PP_LD);    // [2][R]
   const bf16* base = a.cache + (int64_t)b * a.maxlen * a.row;
   const int cpr = a.row / 8;  // 16-byte chunks per row
+  const int ld_r = (int)threadIdx.x / cpr, ld_c = (int)threadIdx.x % cpr, st_r = 256 / cpr, st_c = 256 % cpr;
   auto load_tile = [&](int stage, int key0, int n) {
-    for (int c = threadIdx.x; c < LKT * cpr; c += 256) {
-      const int r = c / cpr, cc = c - r * cpr;
+    const uint32_t dst = smem_u32(tiles + stage * LKT * RS);
+    for (int r = ld_r, c = ld_c; r < LKT;) {
       const bool ok = r < n;
-      cp_async16(smem_u32(tiles + (stage * LKT + r) * RS + cc * 16), base + (int64_t)(key0 + (ok ? r : 0)) * a.row + cc * 8, ok);
+      cp_async16(dst + r * RS + c * 16, base + (int64_t)(key0 + (ok ? r : 0)) * a.row + c * 8, ok);
+      r += st_r;
+      c += st_c;
+      if (c >= cpr) { c -= cpr; r++; }
     }
   };
   auto range = [&](int len, int& kb, int& ke) {
@@ -295,28 +377,32 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(AttnDecodeDev a
     kb = lo + split * a.chunk;
     ke = min(len, kb + a.chunk);
   };
-  // The first tile is requested before the dependency wait when it holds rows of earlier steps only; the length is read
-  // again after the wait.
+  // Tiles that hold rows of earlier steps only are requested before the dependency wait; the length they are derived from is
+  // read again after it.
   int kb, ke;
   const int len_early = min(ld_volatile_i32(a.lens + b) + 1, a.maxlen);
   range(len_early, kb, ke);
-  const bool early = a.prefetch && kb + LKT <= min(ke, len_early - 1);
-  if (early) { load_tile(0, kb, LKT); cp_async_commit(); }
+  int n_early = 0;
+  if (a.prefetch)
+    for (; n_early < NS - 2 && kb + (n_early + 1) * LKT <= min(ke, len_early - 1); n_early++) { load_tile(n_early, kb + n_early * LKT, LKT); cp_async_commit(); }
   pdl_wait();
   SB_TRACE_WAITED();
   const int len = min(ld_volatile_i32(a.lens + b) + 1, a.maxlen);
-  bool have = early;
-  if (len != len_early && early) {  // not expected: the length belongs to the previous step
+  if (len != len_early && n_early) {  // not expected: the length belongs to the previous step
     cp_async_wait<0>();
     __syncthreads();
-    have = false;
+    n_early = 0;
   }
   range(len, kb, ke);
   if (kb >= ke) return;
-  if (!have) { load_tile(0, kb, min(LKT, ke - kb)); cp_async_commit(); }
+  const int ntiles = (ke - kb + LKT - 1) / LKT;
+  for (int t = n_early; t < NS - 2; t++) {  // one group per tile, empty beyond the last
+    if (t < ntiles) load_tile(t, kb + t * LKT, min(LKT, ke - kb - t * LKT));
+    cp_async_commit();
+  }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tig = lane & 3, mi = lane >> 3, r8 = lane & 7;
   const int ks = warp & 3, kh = warp >> 2;
-  const int nks = a.row / 16, ntiles = (ke - kb + LKT - 1) / LKT;
+  const int nks = a.row / 16;
 
   uint32_t qf[MT][KSM][4];
 #pragma unroll
@@ -339,126 +425,132 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(AttnDecodeDev a
     for (int j = 0; j < NV; j++)
 #pragma unroll
       for (int i = 0; i < 4; i++) o[m][j][i] = 0.f;
-  constexpr int TPR = 256 / (MT * 16), KPT = LKT / TPR;  // softmax: threads per head row, keys per thread
+  constexpr int TPR = 256 / R, KPT = LKT / TPR;  // softmax: threads per head row, keys per thread (2 or 4)
   const int srow = threadIdx.x / TPR, skey = (threadIdx.x % TPR) * KPT;
   float m_run = -INFINITY, l_run = 0.f;
   const int dim0 = warp * NV * 8;
 
-  for (int t = 0; t < ntiles; t++) {
-    cp_async_wait<0>();
-    __syncthreads();  // tile t has landed, and everyone has left tile t - 1
-    if (t + 1 < ntiles) { load_tile((t + 1) & 1, kb + (t + 1) * LKT, min(LKT, ke - kb - (t + 1) * LKT)); cp_async_commit(); }
-    const uint32_t tile = smem_u32(tiles + (t & 1) * LKT * RS);
-    {
-      float s[MT][4][4];
+  auto scores = [&](int t) {
+    const uint32_t tile = smem_u32(tiles + (t % NS) * LKT * RS) + (uint32_t)((kh * 16 + (mi >> 1) * 8 + r8) * RS + (mi & 1) * 16);
+    float s[MT][2][4];
 #pragma unroll
-      for (int m = 0; m < MT; m++)
+    for (int m = 0; m < MT; m++)
 #pragma unroll
-        for (int j = 0; j < 4; j++)
+      for (int j = 0; j < 2; j++)
 #pragma unroll
-          for (int i = 0; i < 4; i++) s[m][j][i] = 0.f;
+        for (int i = 0; i < 4; i++) s[m][j][i] = 0.f;
 #pragma unroll
-      for (int k = 0; k < KSM; k++) {
-        const int step = ks + 4 * k;
-        if (step < nks) {
+    for (int k = 0; k < KSM; k++) {
+      const int step = ks + 4 * k;
+      if (step < nks) {
+        uint32_t kf[4];
+        ldsm_x4(tile + (uint32_t)(step * 32), kf);
 #pragma unroll
-          for (int jp = 0; jp < 2; jp++) {
-            uint32_t kf[4];
-            ldsm_x4(tile + (uint32_t)((kh * 32 + jp * 16 + (mi >> 1) * 8 + r8) * RS + step * 32 + (mi & 1) * 16), kf);
-#pragma unroll
-            for (int m = 0; m < MT; m++) {
-              mma_bf16(s[m][2 * jp], qf[m][k], kf[0], kf[1]);
-              mma_bf16(s[m][2 * jp + 1], qf[m][k], kf[2], kf[3]);
-            }
-          }
+        for (int m = 0; m < MT; m++) {
+          mma_bf16(s[m][0], qf[m][k], kf[0], kf[1]);
+          mma_bf16(s[m][1], qf[m][k], kf[2], kf[3]);
         }
       }
-#pragma unroll
-      for (int m = 0; m < MT; m++)
-#pragma unroll
-        for (int j = 0; j < 4; j++) {
-          float* w = sp + (ks * MT * 16 + m * 16 + g) * 68 + kh * 32 + j * 8 + 2 * tig;
-          *(float2*)w = make_float2(s[m][j][0], s[m][j][1]);
-          *(float2*)(w + 8 * 68) = make_float2(s[m][j][2], s[m][j][3]);
-        }
     }
-    __syncthreads();
-    {
-      float v[KPT];
-      float mx = -INFINITY;
-      const int lim = ke - kb - t * LKT;
+    float* w0 = sp + (((t & 1) * 4 + ks) * R + g) * SP_LD + kh * 16 + 2 * tig;
 #pragma unroll
-      for (int i = 0; i < KPT; i += 4) {
-        float4 x[4];
+    for (int m = 0; m < MT; m++)
 #pragma unroll
-        for (int p = 0; p < 4; p++) x[p] = *(const float4*)(sp + (p * MT * 16 + srow) * 68 + skey + i);
-        v[i] = ((x[0].x + x[1].x) + x[2].x) + x[3].x;
-        v[i + 1] = ((x[0].y + x[1].y) + x[2].y) + x[3].y;
-        v[i + 2] = ((x[0].z + x[1].z) + x[2].z) + x[3].z;
-        v[i + 3] = ((x[0].w + x[1].w) + x[2].w) + x[3].w;
+      for (int j = 0; j < 2; j++) {
+        float* w = w0 + m * 16 * SP_LD + j * 8;
+        *(float2*)w = make_float2(s[m][j][0], s[m][j][1]);
+        *(float2*)(w + 8 * SP_LD) = make_float2(s[m][j][2], s[m][j][3]);
       }
+  };
+  auto softmax = [&](int t) {
+    float v[KPT];
+    const float* sr = sp + ((t & 1) * 4 * R + srow) * SP_LD + skey;
 #pragma unroll
-      for (int i = 0; i < KPT; i++) {
-        v[i] = skey + i < lim ? v[i] * a.scale_log2 : -INFINITY;
-        mx = fmaxf(mx, v[i]);
-      }
+    for (int i = 0; i < KPT; i += 2) {
+      float2 x[4];
 #pragma unroll
-      for (int off = 1; off < TPR; off <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-      const float m_new = fmaxf(m_run, mx);  // finite: every tile holds a visible key
-      const float corr = exp2f(m_run - m_new);
-      m_run = m_new;
-      float ls = 0.f;
-      uint32_t hi[KPT / 2], lo[KPT / 2];
-#pragma unroll
-      for (int i = 0; i < KPT; i += 2) {
-        const float p0 = exp2f(v[i] - m_new), p1 = exp2f(v[i + 1] - m_new);
-        ls += p0 + p1;
-        const float a0 = round_bf16(p0), a1 = round_bf16(p1);
-        hi[i / 2] = pack_bf16(a0, a1);
-        lo[i / 2] = pack_bf16(p0 - a0, p1 - a1);
-      }
-      l_run = l_run * corr + ls;
-      if (KPT == 8) {
-        *(uint4*)(pp + srow * 72 + skey) = make_uint4(hi[0], hi[1], hi[KPT / 2 - 2], hi[KPT / 2 - 1]);
-        *(uint4*)(pp + (MT * 16 + srow) * 72 + skey) = make_uint4(lo[0], lo[1], lo[KPT / 2 - 2], lo[KPT / 2 - 1]);
-      } else {
-        *(uint2*)(pp + srow * 72 + skey) = make_uint2(hi[0], hi[1]);
-        *(uint2*)(pp + (MT * 16 + srow) * 72 + skey) = make_uint2(lo[0], lo[1]);
-      }
-      if (skey == 0) corr_s[srow] = corr;
+      for (int p = 0; p < 4; p++) x[p] = *(const float2*)(sr + p * R * SP_LD + i);
+      v[i] = ((x[0].x + x[1].x) + x[2].x) + x[3].x;
+      v[i + 1] = ((x[0].y + x[1].y) + x[2].y) + x[3].y;
     }
-    __syncthreads();
-    if (dim0 < a.rank_p) {
+    const int lim = ke - kb - t * LKT;
+    float mx = -INFINITY;
 #pragma unroll
-      for (int m = 0; m < MT; m++) {
-        const float c0 = corr_s[m * 16 + g], c1 = corr_s[m * 16 + g + 8];
+    for (int i = 0; i < KPT; i++) {
+      v[i] = skey + i < lim ? v[i] * a.scale_log2 : -INFINITY;
+      mx = fmaxf(mx, v[i]);
+    }
+#pragma unroll
+    for (int off = 1; off < TPR; off <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+    const float m_new = fmaxf(m_run, mx);  // finite: every tile holds a visible key
+    const float corr = exp2f(m_run - m_new);
+    m_run = m_new;
+    float ls = 0.f;
+    bf16* ph = pp + ((t & 1) * 2 * R + srow) * PP_LD + skey;
+#pragma unroll
+    for (int i = 0; i < KPT; i += 2) {
+      const float p0 = exp2f(v[i] - m_new), p1 = exp2f(v[i + 1] - m_new);
+      ls += p0 + p1;
+      const float a0 = round_bf16(p0), a1 = round_bf16(p1);
+      *(uint32_t*)(ph + i) = pack_bf16(a0, a1);
+      *(uint32_t*)(ph + R * PP_LD + i) = pack_bf16(p0 - a0, p1 - a1);
+    }
+    l_run = l_run * corr + ls;
+    if (skey == 0) corr_s[(t & 1) * R + srow] = corr;
+  };
+  auto accumulate = [&](int t) {
+    if (dim0 >= a.rank_p) return;
+    const float* cs = corr_s + (t & 1) * R;
+#pragma unroll
+    for (int m = 0; m < MT; m++) {
+      const float c0 = cs[m * 16 + g], c1 = cs[m * 16 + g + 8];
+      if (!__all_sync(0xffffffffu, c0 == 1.0f && c1 == 1.0f)) {
 #pragma unroll
         for (int j = 0; j < NV; j++) { o[m][j][0] *= c0; o[m][j][1] *= c0; o[m][j][2] *= c1; o[m][j][3] *= c1; }
       }
+    }
+    const uint32_t tile = smem_u32(tiles + (t % NS) * LKT * RS) + (uint32_t)(((mi & 1) * 8 + r8) * RS + (dim0 + (mi >> 1) * 8) * 2);
+    const uint32_t ps = smem_u32(pp + (t & 1) * 2 * R * PP_LD + ((mi & 1) * 8 + r8) * PP_LD + (mi >> 1) * 8);
 #pragma unroll
-      for (int kk = 0; kk < 4; kk++) {
-        uint32_t ph[MT][4], pl[MT][4];
+    for (int kk = 0; kk < LKT / 16; kk++) {
+      uint32_t ph[MT][4], pl[MT][4];
 #pragma unroll
-        for (int m = 0; m < MT; m++) {
-          ldsm_x4(smem_u32(pp + (m * 16 + (mi & 1) * 8 + r8) * 72 + kk * 16 + (mi >> 1) * 8), ph[m]);
-          ldsm_x4(smem_u32(pp + ((MT + m) * 16 + (mi & 1) * 8 + r8) * 72 + kk * 16 + (mi >> 1) * 8), pl[m]);
-        }
+      for (int m = 0; m < MT; m++) {
+        ldsm_x4(ps + (uint32_t)((m * 16 * PP_LD + kk * 16) * 2), ph[m]);
+        ldsm_x4(ps + (uint32_t)(((R + m * 16) * PP_LD + kk * 16) * 2), pl[m]);
+      }
 #pragma unroll
-        for (int jp = 0; jp < NV / 2; jp++) {
-          if (dim0 + jp * 16 < a.rank_p) {
-            uint32_t vf[4];
-            ldsm_x4_t(tile + (uint32_t)((kk * 16 + (mi & 1) * 8 + r8) * RS + (dim0 + jp * 16 + (mi >> 1) * 8) * 2), vf);
+      for (int jp = 0; jp < NV / 2; jp++) {
+        if (dim0 + jp * 16 < a.rank_p) {
+          uint32_t vf[4];
+          ldsm_x4_t(tile + (uint32_t)(kk * 16 * RS + jp * 32), vf);
 #pragma unroll
-            for (int m = 0; m < MT; m++) {
-              mma_bf16(o[m][2 * jp], ph[m], vf[0], vf[1]);
-              mma_bf16(o[m][2 * jp + 1], ph[m], vf[2], vf[3]);
-              mma_bf16(o[m][2 * jp], pl[m], vf[0], vf[1]);
-              mma_bf16(o[m][2 * jp + 1], pl[m], vf[2], vf[3]);
-            }
+          for (int m = 0; m < MT; m++) {
+            mma_bf16(o[m][2 * jp], ph[m], vf[0], vf[1]);
+            mma_bf16(o[m][2 * jp + 1], ph[m], vf[2], vf[3]);
+          }
+#pragma unroll
+          for (int m = 0; m < MT; m++) {
+            mma_bf16(o[m][2 * jp], pl[m], vf[0], vf[1]);
+            mma_bf16(o[m][2 * jp + 1], pl[m], vf[2], vf[3]);
           }
         }
       }
     }
+  };
+
+  cp_async_wait<NS - 3>();
+  __syncthreads();
+  scores(0);
+  for (int t = 0; t <= ntiles; t++) {
+    cp_async_wait<NS - 4>();  // tile t + 1 has landed
+    __syncthreads();          // S(t), P(t-1) and tile t + 1 of every thread; everyone has left tile t - 2
+    const int next = t + NS - 2;
+    if (next < ntiles) load_tile(next % NS, kb + next * LKT, min(LKT, ke - kb - next * LKT));
+    cp_async_commit();
+    if (t + 1 < ntiles) scores(t + 1);
+    if (t < ntiles) softmax(t);
+    if (t > 0) accumulate(t - 1);
   }
 #pragma unroll
   for (int off = 1; off < TPR; off <<= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, off);
@@ -518,18 +610,31 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(MergeDev a) {
     float f = l16 < ns ? exp2f(ml.x - M) : 0.f, L = f * ml.y;
 #pragma unroll
     for (int off = 1; off < 16; off <<= 1) L += __shfl_xor_sync(0xffffffffu, L, off);
-    fs[m][l16] = ns > 0 ? f / L : 0.f;
-    __syncwarp();
-    for (int c = l16 * 4; c < a.rank_p; c += 64) {
-      float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 4
-      for (int s = 0; s < ns; s++) {
-        const float4 x = *(const float4*)(a.o_part + (base + s) * a.rank_p + c);
-        const float w = fs[m][s];
-        acc.x += w * x.x; acc.y += w * x.y; acc.z += w * x.z; acc.w += w * x.w;
+    fs[m][l16] = l16 < ns ? f / L : 0.f;
+  }
+  __syncthreads();
+  // every thread of the block takes groups of four columns of any of the tokens; all chunks' loads of a group in flight at once
+  const int c4n = a.rank_p / 4;
+#pragma unroll 2
+  for (int i = threadIdx.x; i < 16 * c4n; i += 256) {
+    const int m = i / c4n, c = (i - m * c4n) * 4, b = b0 + m;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (b < a.B) {
+      const float* src = a.o_part + (((int64_t)b * a.H + h) * a.nsplit) * a.rank_p + c;
+      for (int s0 = 0; s0 < a.nsplit; s0 += 8) {
+        float4 x[8];
+#pragma unroll
+        for (int s = 0; s < 8; s++)
+          if (s0 + s < a.nsplit && fs[m][s0 + s] != 0.f) x[s] = *(const float4*)(src + (int64_t)(s0 + s) * a.rank_p);
+#pragma unroll
+        for (int s = 0; s < 8; s++)
+          if (s0 + s < a.nsplit && fs[m][s0 + s] != 0.f) {
+            const float w = fs[m][s0 + s];
+            acc.x += w * x[s].x; acc.y += w * x[s].y; acc.z += w * x[s].z; acc.w += w * x[s].w;
+          }
       }
-      *(uint2*)(ot + m * ld + c) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
     }
+    *(uint2*)(ot + m * ld + c) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
   }
   cp_async_wait<0>();
   __syncthreads();
@@ -644,7 +749,7 @@ constexpr size_t SMEM_MAX = 227 * 1024 - 1024;  // what a block may take, less t
 template <int MT, int KSM, int NV>
 int launch_attn_decode(strictb200_ctx* ctx, const AttnDecodeDev& a, int B) {
   static size_t have[64] = {};
-  const size_t smem = (size_t)2 * LKT * (a.row * 2 + 16) + attn_decode_fixed_smem<MT>();
+  const size_t smem = attn_decode_smem(MT, KSM, a.row);
   SB_TRY(allow_smem(ctx, latent_attn_decode_kernel<MT, KSM, NV>, smem, have));
   SB_CUDA(sb_launch(ctx, latent_attn_decode_kernel<MT, KSM, NV>, dim3(a.nsplit, (a.H + MT * 16 - 1) / (MT * 16), B), dim3(256), smem, a));
   ctx->launches++;
@@ -657,8 +762,9 @@ SB_TRACE_TU(latent)
 
 int k_latent_split(strictb200_ctx* ctx, const LatentSplitArgs& a, int64_t T) {
   const SplitDev d = split_dev(a);
-  if (a.f32) SB_CUDA(sb_launch(ctx, latent_split_kernel<float>, dim3((unsigned)T), dim3(256), 0, d, T));
-  else SB_CUDA(sb_launch(ctx, latent_split_kernel<bf16>, dim3((unsigned)T), dim3(256), 0, d, T));
+  const dim3 grid((unsigned)T, a.cache ? 2u : 1u);
+  if (a.f32) SB_CUDA(sb_launch(ctx, latent_split_kernel<float>, grid, dim3(256), 0, d, T));
+  else SB_CUDA(sb_launch(ctx, latent_split_kernel<bf16>, grid, dim3(256), 0, d, T));
   ctx->launches++;
   return STRICTB200_OK;
 }
@@ -680,13 +786,20 @@ int k_latent_decode_in(strictb200_ctx* ctx, const LatentDecodeInArgs& x, int64_t
   static size_t have[64] = {};
   const LatentShape& s = x.a.s;
   DecodeInDev d{split_dev(x.a), x.wkv, s.kv_head(), x.q_abs, x.act_col, x.n_act, x.act_pos, x.act_neg, x.act, x.ld_act,
-                (s.rank_p() + QA_COLS - 1) / QA_COLS, (int)((B + 15) / 16), (x.n_act + 1023) / 1024};
+                (s.rank_p() + QA_COLS - 1) / QA_COLS, (int)((B + 15) / 16), (s.H * (s.row() - s.rank_p()) / 2 + 255) / 256, (x.n_act + 1023) / 1024};
   const size_t smem = decode_in_smem(s.dim);
   SB_TRY(allow_smem(ctx, latent_decode_in_kernel, smem, have));
-  const int64_t blocks = (int64_t)s.H * d.n_rt * d.n_grp + 2 * B + B * d.act_blocks;
+  const int64_t blocks = (int64_t)s.H * d.n_rt * d.n_grp + B * (d.rot_blocks + (x.a.cache ? 1 : 0) + d.act_blocks);
+  if (x.a.splits > 8) return sb_fail(STRICTB200_ERR_INVALID_ARG, "latent decode: at most 8 partial sums");
   SB_CUDA(sb_launch(ctx, latent_decode_in_kernel, dim3((unsigned)blocks), dim3(256), smem, d, (int)B));
   ctx->launches++;
   return STRICTB200_OK;
+}
+
+// Reduction steps per slice the kernel is built for: rows of up to 192, 320 and 576 elements.
+int decode_ksm(const LatentShape& s) {
+  const int nks = (s.row() / 16 + 3) / 4;
+  return s.rank_p() <= 128 && nks <= 3 ? 3 : s.rank_p() <= 256 && nks <= 5 ? 5 : 9;
 }
 
 // Keys per block: waves of blocks x (key tiles per block + what a block costs besides), over the multiples of the tile that
@@ -694,14 +807,13 @@ int k_latent_decode_in(strictb200_ctx* ctx, const LatentDecodeInArgs& x, int64_t
 int sb_latent_decode_chunk(strictb200_ctx* ctx, const LatentShape& s, int B, int len_plan) {
   const int n = s.window > 0 ? std::min(s.window, len_plan) : len_plan, tiles = std::max(1, (n + LKT - 1) / LKT);
   const int mt = s.H <= 16 ? 1 : 2;
-  const size_t smem = (size_t)2 * LKT * (s.row() * 2 + 16) + (mt == 1 ? attn_decode_fixed_smem<1>() : attn_decode_fixed_smem<2>());
-  const int per_sm = std::max<int>(1, std::min<int>(4, (int)(227 * 1024 / (smem + 1024))));
+  const int per_sm = std::max<int>(1, std::min<int>(2, (int)(227 * 1024 / (attn_decode_smem(mt, decode_ksm(s), s.row()) + 1024))));
   const int64_t slots = (int64_t)ctx->sm_count * per_sm, pairs = (int64_t)B * ((s.H + mt * 16 - 1) / (mt * 16));
   int best = tiles;
   double best_cost = 1e30;
   for (int c = (tiles + MAX_SPLITS - 1) / MAX_SPLITS; c <= tiles; c++) {
     const int64_t blocks = pairs * ((tiles + c - 1) / c), waves = (blocks + slots - 1) / slots;
-    const double cost = (double)waves * (c + 1.5) + 0.05 * ((tiles + c - 1) / c);  // every chunk adds to the merge
+    const double cost = (double)waves * (c + 3) + 0.05 * ((tiles + c - 1) / c);  // every chunk adds to the merge
     if (cost < best_cost - 1e-9) { best_cost = cost; best = c; }
   }
   return best * LKT;
@@ -714,10 +826,10 @@ int k_latent_attn_decode(strictb200_ctx* ctx, const LatentShape& s, const bf16* 
   if (nsplit < 1 || nsplit > MAX_SPLITS || chunk < LKT || chunk % LKT || B > 65535) return sb_fail(STRICTB200_ERR_INVALID_ARG, "latent decode attention: bad key chunks");
   float* ml = scratch + (size_t)B * s.H * nsplit * s.rank_p();
   AttnDecodeDev a{q_abs, cache, lens, s.H, s.row(), s.rank_p(), maxlen, s.window, chunk, nsplit, s.scale * LOG2E, scratch, ml, ctx->opt.attn_prefetch};
-  const int rp = s.rank_p(), nks = (s.row() / 16 + 3) / 4;
+  const int rp = s.rank_p(), ksm = decode_ksm(s);
 #define LATENT_DECODE(KSM, NV) SB_TRY((s.H <= 16 ? launch_attn_decode<1, KSM, NV>(ctx, a, B) : launch_attn_decode<2, KSM, NV>(ctx, a, B)))
-  if (rp <= 128 && nks <= 3) LATENT_DECODE(3, 2);
-  else if (rp <= 256 && nks <= 5) LATENT_DECODE(5, 4);
+  if (ksm == 3) LATENT_DECODE(3, 2);
+  else if (ksm == 5) LATENT_DECODE(5, 4);
   else LATENT_DECODE(9, 8);
 #undef LATENT_DECODE
   sb_prof_split(ctx, STRICTB200_K_ATTN_MERGE);

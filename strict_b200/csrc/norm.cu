@@ -882,6 +882,48 @@ __global__ void __launch_bounds__(NI == 1 ? 1024 : 512) group_norm_kernel(GroupN
   SB_TRACE_END(SB_K_ROWNORM, 0);
 }
 
+// Many rows (prompts): one block per row whatever the number of groups. A warp's 128 columns lie in one group (group widths
+// are multiples of 128 here); their sums of squares meet in shared memory.
+template <typename T, int NI>
+__global__ void __launch_bounds__(256) group_norm_rows_kernel(GroupNormDev a, int64_t M, int d) {
+  __shared__ float sums[NI * 8];
+  pdl_trigger();
+  pdl_wait();
+  const int64_t row = blockIdx.x;
+  float4 v[NI];
+#pragma unroll
+  for (int i = 0; i < NI; i++) {
+    const int k = (i * 256 + (int)threadIdx.x) * 4;
+    if (k < d) v[i] = *(const float4*)(a.x + row * a.ldx + k);
+  }
+#pragma unroll
+  for (int i = 0; i < NI; i++) {
+    const int k = (i * 256 + (int)threadIdx.x) * 4;
+    float ss = 0.f;
+    if (k < d) ss = v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) sums[i * 8 + (threadIdx.x >> 5)] = ss;
+  }
+  __syncthreads();
+  const int per = a.gw / 128;  // warps' shares per group
+#pragma unroll
+  for (int i = 0; i < NI; i++) {
+    const int k = (i * 256 + (int)threadIdx.x) * 4;
+    if (k < d) {
+      const int first = k / a.gw * per;
+      float ss = 0.f;
+      for (int j = 0; j < per; j++) ss += sums[first + j];
+      const float r = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.gw), a.eps)));
+      const float4 g = *(const float4*)(a.g1 + k), t = make_float4(v[i].x * r, v[i].y * r, v[i].z * r, v[i].w * r);
+      store4<T>((T*)a.y1 + row * a.ldy + k, t.x * g.x, t.y * g.y, t.z * g.z, t.w * g.w);
+      if (a.g2) {
+        const float4 h = *(const float4*)(a.g2 + k);
+        store4<T>((T*)a.y2 + row * a.ldy + k, t.x * h.x, t.y * h.y, t.z * h.z, t.w * h.w);
+      }
+    }
+  }
+}
+
 // Group widths that are no multiple of four, or too wide for the kernel above: one column at a time, two passes.
 template <typename T>
 __global__ void __launch_bounds__(256) group_norm_any_kernel(GroupNormDev a, int64_t M) {
@@ -922,6 +964,13 @@ int k_group_norm(strictb200_ctx* ctx, const GroupNormArgs& a, int64_t M, int64_t
     dim3 grid((unsigned)M, (unsigned)a.groups);
     if (a.f32) SB_CUDA(sb_launch(ctx, group_norm_any_kernel<float>, grid, dim3(256), 0, v, M));
     else SB_CUDA(sb_launch(ctx, group_norm_any_kernel<bf16>, grid, dim3(256), 0, v, M));
+    ctx->launches++;
+    return STRICTB200_OK;
+  }
+  if (M > 256 && !a.part && a.g1 && v.gw % 128 == 0 && d <= 8192) {
+    auto rows = [&](auto kernel) { return sb_launch(ctx, kernel, dim3((unsigned)M), dim3(256), 0, v, M, (int)d); };
+    if (a.f32) SB_CUDA(d <= 4096 ? rows(group_norm_rows_kernel<float, 4>) : rows(group_norm_rows_kernel<float, 8>));
+    else SB_CUDA(d <= 1024 ? rows(group_norm_rows_kernel<bf16, 1>) : d <= 4096 ? rows(group_norm_rows_kernel<bf16, 4>) : rows(group_norm_rows_kernel<bf16, 8>));
     ctx->launches++;
     return STRICTB200_OK;
   }
