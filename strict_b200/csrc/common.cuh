@@ -403,12 +403,12 @@ struct LatentDecodeInArgs {
 };
 bool sb_latent_decode_fits(const LatentShape& s);
 int k_latent_decode_in(strictb200_ctx*, const LatentDecodeInArgs& a, int64_t B);
-// Split-key attention of one new token per sequence over the latents of its window, then the merge of the key chunks and the
-// value projection of every head. len_plan: lengths the chunks are planned for.
+// Split-key attention of one new token per sequence over the latents of its window (the key chunks of a sequence are merged
+// inside a cluster), then the value projection of every head. len_plan: lengths the chunks are planned for.
 int sb_latent_decode_chunk(strictb200_ctx*, const LatentShape& s, int B, int len_plan);
 size_t sb_latent_decode_scratch(const LatentShape& s, int B);
 int k_latent_attn_decode(strictb200_ctx*, const LatentShape& s, const bf16* q_abs, const bf16* cache, const int32_t* lens, int B, int maxlen, int chunk,
-                         int nsplit, float* scratch, const bf16* wkv, bf16* out, int64_t ldo);
+                         int nsplit, bf16* scratch, const bf16* wkv, bf16* out, int64_t ldo);
 // Any widths, bf16 or fp32, prompt rows and decode rows: one block per row and head, straight from the cache.
 int k_latent_attn_any(strictb200_ctx*, const LatentShape& s, bool f32, const void* q, const void* cache, const void* wkv, const int32_t* seq,
                       const int32_t* pos, const int32_t* lens, int64_t T, int maxlen, void* out, int64_t ldo);

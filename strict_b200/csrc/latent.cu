@@ -7,11 +7,13 @@
 //  * decode: nothing is rebuilt. A head's query is carried into latent space (q' = q W_uk), so that q' . c replaces
 //    q . W_uk c, all heads read the same cache row (the heads are the rows of the MMA tile) and the weighted sum of latents
 //    goes through W_uv once per head. Three launches: queries into latent space beside everything else the projection
-//    feeds (rotation, cache append, activation); split-key attention; merge of the key chunks + W_uv.
+//    feeds (rotation, cache append, activation); split-key attention, merged inside a cluster; W_uv.
 //  * any other width, and fp32: one block per row and head, straight from the cache.
 //
 // Scores, softmax weights, norms and rotations are fp32; the weights enter the product with the latents as two bf16 terms
 // (hi + lo), whose sum carries 16 mantissa bits.
+#include <cuda.h>
+
 #include <algorithm>
 #include <mutex>
 
@@ -38,8 +40,48 @@ __device__ __forceinline__ void ldsm_x4_t(uint32_t addr, uint32_t* r) {
 __device__ __forceinline__ void ldsm_x2(uint32_t addr, uint32_t* r) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
 }
-__device__ __forceinline__ void ldsm_x2_t(uint32_t addr, uint32_t* r) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
+__device__ __forceinline__ void mbar_init(uint32_t bar, uint32_t count) { asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count)); }
+__device__ __forceinline__ void mbar_expect_tx(uint32_t bar, uint32_t bytes) {
+  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory");
+}
+// Bounded wait for the phase with the given parity. Returns false when the limit expired.
+__device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity) {
+  for (uint32_t i = 0; i < (1u << 22); i++) {
+    uint32_t done;
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+        "selp.u32 %0, 1, 0, p;\n\t}"
+        : "=r"(done)
+        : "r"(bar), "r"(parity)
+        : "memory");
+    if (done) return true;
+  }
+  return false;
+}
+__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar, uint64_t policy) {
+  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes.L2::cache_hint [%0], [%1, {%2, %3}], [%4], %5;" ::"r"(dst),
+               "l"(map), "r"(x), "r"(y), "r"(bar), "l"(policy)
+               : "memory");
+}
+// the address of this block's shared-memory location in block `rank` of the cluster
+__device__ __forceinline__ uint32_t map_to_rank(uint32_t local, uint32_t rank) {
+  uint32_t r;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(local), "r"(rank));
+  return r;
+}
+__device__ __forceinline__ float2 ld_cluster2(uint32_t addr) {
+  float2 v;
+  asm volatile("ld.shared::cluster.v2.f32 {%0,%1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(addr) : "memory");
+  return v;
+}
+__device__ __forceinline__ float4 ld_cluster4(uint32_t addr) {
+  float4 v;
+  asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr) : "memory");
+  return v;
+}
+__device__ __forceinline__ void cluster_sync() {
+  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 // not volatile: the compiler may move fragment loads ahead of products that do not need them
 __device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
@@ -47,6 +89,24 @@ __device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// the same with a zero accumulator
+__device__ __forceinline__ void mma_bf16_zero(float* d, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%10,%10,%10,%10};\n"
+      : "=f"(d[0]), "=f"(d[1]), "=f"(d[2]), "=f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1), "f"(0.f));
+}
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// two fp32 values as two bf16 terms, p = hi + lo to 2^-17
+__device__ __forceinline__ void split_bf16x2(float p0, float p1, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(p0 - __uint_as_float(hi << 16), p1 - __uint_as_float(hi & 0xFFFF0000u));
+  lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) { return f32_to_bf16_bits(lo) | (f32_to_bf16_bits(hi) << 16); }
 __device__ __forceinline__ int ld_volatile_i32(const int32_t* p) {
@@ -84,6 +144,7 @@ __device__ __forceinline__ float proj(const SplitDev& a, int64_t T, int64_t t, i
 }
 // four columns at a time (col and the row stride multiples of 4; at most 8 splits), every split's load in flight at once
 __device__ __forceinline__ float4 proj4(const SplitDev& a, int64_t T, int64_t t, int64_t col) {
+  if (a.splits == 1) return *(const float4*)(a.in + t * a.ld_in + col);
   float4 p[8], v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
   for (int s = 0; s < 8; s++)
@@ -216,17 +277,17 @@ struct DecodeInDev {
   float act_pos, act_neg;
   bf16* act;
   int64_t ld_act;
-  int n_rt, n_grp;      // latent tiles of 64 and token groups of 16: blocks of the first role
+  int n_rt, n_grp;      // latent tiles of 128 and token groups of 16: blocks of the first role
   int rot_blocks;       // blocks per token of the rotation (256 pairs each)
   int act_blocks;       // ... and of the activation
 };
-constexpr int QA_COLS = 64, QA_LD = QA_COLS + 8;
+constexpr int QA_COLS = 128, QA_LD = QA_COLS + 8;
 __host__ __device__ inline int decode_in_smem(int dim) {
   const int d16 = (dim + 15) & ~15;
   return d16 * QA_LD * 2 + 16 * (d16 + 8) * 2;
 }
-// One launch, four roles by block index: H * n_rt * n_grp blocks multiply queries with W_uk (64 latents of one head, 16
-// tokens), then B * rot_blocks rotate the queries' second part, B append the cache row (a layer with latents of its own),
+// One launch, four roles by block index: H * n_rt * n_grp blocks multiply queries with W_uk (128 latents of one head,
+// 16 tokens), then B * rot_blocks rotate the queries' second part, B append the cache row (a layer with latents of its own),
 // B * act_blocks run the activation.
 __global__ void __launch_bounds__(256) latent_decode_in_kernel(DecodeInDev d, int B) {
   extern __shared__ __align__(128) uint8_t smem[];
@@ -263,17 +324,22 @@ __global__ void __launch_bounds__(256) latent_decode_in_kernel(DecodeInDev d, in
     cp_async_wait<0>();
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mi = lane >> 3, r8 = lane & 7;
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
     for (int k = 0; k < d16; k += 16) {
-      uint32_t qa[4], wb[2];
+      uint32_t qa[4], wb[4];
       ldsm_x4(smem_u32(qt + ((mi & 1) * 8 + r8) * (d16 + 8) + k + (mi >> 1) * 8), qa);
-      ldsm_x2_t(smem_u32(wt + (k + (mi & 1) * 8 + r8) * QA_LD + warp * 8), wb);
-      mma_bf16(acc, qa, wb[0], wb[1]);
+      ldsm_x4_t(smem_u32(wt + (k + (mi & 1) * 8 + r8) * QA_LD + warp * 16 + (mi >> 1) * 8), wb);
+      mma_bf16(acc[0], qa, wb[0], wb[1]);
+      mma_bf16(acc[1], qa, wb[2], wb[3]);
     }
-    const int g = lane >> 2, col = r0 + warp * 8 + 2 * (lane & 3);
-    if (col < a.rank_p) {
-      if (b0 + g < B) *(uint32_t*)(d.q_abs + ((int64_t)(b0 + g) * a.H + h) * a.row + col) = pack_bf16(acc[0], acc[1]);
-      if (b0 + g + 8 < B) *(uint32_t*)(d.q_abs + ((int64_t)(b0 + g + 8) * a.H + h) * a.row + col) = pack_bf16(acc[2], acc[3]);
+    const int g = lane >> 2;
+#pragma unroll
+    for (int j = 0; j < 2; j++) {
+      const int col = r0 + warp * 16 + j * 8 + 2 * (lane & 3);
+      if (col < a.rank_p) {
+        if (b0 + g < B) *(uint32_t*)(d.q_abs + ((int64_t)(b0 + g) * a.H + h) * a.row + col) = pack_bf16(acc[j][0], acc[j][1]);
+        if (b0 + g + 8 < B) *(uint32_t*)(d.q_abs + ((int64_t)(b0 + g + 8) * a.H + h) * a.row + col) = pack_bf16(acc[j][2], acc[j][3]);
+      }
     }
     SB_TRACE_END(SB_K_ROPE, 0);
     return;
@@ -323,54 +389,59 @@ __global__ void __launch_bounds__(256) latent_decode_in_kernel(DecodeInDev d, in
 }
 
 // ------------------------------------------------------------------ decode: split-key attention over the latents
-// grid (nsplit, ceil(H / (16 MT)), B), 256 threads. Rows of the MMA tiles = up to 16 MT heads, 32 keys per step. Three
-// products of three different steps share an iteration, so one barrier per step is enough:
-//   S(t+1) partials  warp (ks, kh): reduction steps ks, ks + 4, .. of the cache row for the 16 keys of half kh; its share of
+// grid (nsplit, ceil(H / (16 MT)), B), 32 NW threads; the nsplit blocks of a (sequence, head group) are one cluster. Rows of
+// the MMA tiles = up to 16 MT heads, 32 keys per step. Three products of three different steps share an iteration:
+//   S(t+1) partials  warp (ks, kh): reduction steps ks, ks + SL, .. of the cache row for the 16 keys of half kh; its share of
 //                    the queries stays in registers for the whole block, so a step reads the key tile from shared memory once
-//   softmax(t)       the four partial scores of a (head, key) are added in slice order; running maximum and sum per head
+//   softmax(t)       the SL partial scores of a (head, key) are added in slice order; running maximum and sum per head
 //   O += P(t-1) c    every warp owns 8 NV latent columns of all heads; the key tile is its operand again
-// Key tiles pass through a ring of NS stages (t-1, t, t+1 in use, the rest in flight).
-constexpr int LKT = 32;
+// A key tile is copied by TMA in atoms of 32 rows x 64 columns (128-byte swizzle: 16-byte chunk c of row r lies at c ^ (r & 7));
+// tiles pass through a ring of four stages (t-1, t, t+1 in use, t+2 in flight). At the end the cluster's blocks weigh each other's sums through distributed shared memory, so what leaves
+// is one bf16 row of latents per head.
+constexpr int LKT = 32, NS = 4;
+constexpr int MAX_SPLITS = 8;  // blocks of a cluster
 struct AttnDecodeDev {
   const bf16* q;
-  const bf16* cache;
   const int32_t* lens;
   int H, row, rank_p, maxlen, window, chunk, nsplit;
   float scale_log2;
-  float* o_part;
-  float* ml_part;
+  bf16* out;   // [B, H, rank_p] weighted sum of latents
   int prefetch;
+  int* status;
 };
 constexpr int SP_LD = 36, PP_LD = 40;  // row strides of the score (fp32) and weight (bf16) tiles
-constexpr int decode_stages(int ksm) { return ksm > 5 ? 4 : 6; }
-constexpr size_t attn_decode_smem(int mt, int ksm, int row) {
-  return (size_t)decode_stages(ksm) * LKT * (row * 2 + 16) + (size_t)2 * 4 * mt * 16 * SP_LD * 4 + (size_t)2 * 2 * mt * 16 * PP_LD * 2 + 2 * mt * 16 * 4;
+constexpr int ATOM = LKT * 128;        // bytes of a tile's 64-column atom
+constexpr size_t attn_decode_smem(int mt, int nw, int row) {
+  return 1024 /* round-up to the swizzle's alignment */ + (size_t)NS * ((row + 63) / 64) * ATOM + (size_t)(nw / 2) * mt * 16 * SP_LD * 4 + (size_t)2 * 2 * mt * 16 * PP_LD * 2 + 2 * mt * 16 * 4;
 }
 
-template <int MT, int KSM, int NV>
-__global__ void __launch_bounds__(256) latent_attn_decode_kernel(AttnDecodeDev a) {
-  constexpr int NS = decode_stages(KSM), R = MT * 16;
-  extern __shared__ __align__(128) uint8_t smem[];
+template <int MT, int NW, int KSM, int NV>
+__global__ void __launch_bounds__(NW * 32) latent_attn_decode_kernel(const __grid_constant__ CUtensorMap map, AttnDecodeDev a) {
+  constexpr int R = MT * 16, SL = NW / 2, NT = NW * 32;
+  extern __shared__ __align__(1024) uint8_t smem_raw[];
+  uint8_t* smem = smem_raw + ((1024 - (smem_u32(smem_raw) & 1023)) & 1023);
+  __shared__ __align__(8) uint64_t full[NS];
+  __shared__ float2 ml_s[R];
+  __shared__ float fs[R][MAX_SPLITS];
   SB_TRACE_BEGIN();
   pdl_trigger();
   const int split = blockIdx.x, h0 = blockIdx.y * R, b = blockIdx.z;
-  const int RS = a.row * 2 + 16;  // shared-memory row stride: an odd number of 16-byte chunks
-  uint8_t* tiles = smem;                               // [NS][LKT][RS]
-  float* sp = (float*)(smem + NS * LKT * RS);          // [2][4][R][SP_LD]
-  bf16* pp = (bf16*)(sp + 2 * 4 * R * SP_LD);          // [2][hi, lo][R][PP_LD]
+  const int n_atoms = (a.row + 63) / 64, stage_bytes = n_atoms * ATOM;
+  float* sp = (float*)(smem + NS * stage_bytes);       // [SL][R][SP_LD], behind the ring of key tiles
+  bf16* pp = (bf16*)(sp + SL * R * SP_LD);             // [2][hi, lo][R][PP_LD]
   float* corr_s = (float*)(pp + 2 * 2 * R * PP_LD);    // [2][R]
-  const bf16* base = a.cache + (int64_t)b * a.maxlen * a.row;
-  const int cpr = a.row / 8;  // 16-byte chunks per row
-  const int ld_r = (int)threadIdx.x / cpr, ld_c = (int)threadIdx.x % cpr, st_r = 256 / cpr, st_c = 256 % cpr;
-  auto load_tile = [&](int stage, int key0, int n) {
-    const uint32_t dst = smem_u32(tiles + stage * LKT * RS);
-    for (int r = ld_r, c = ld_c; r < LKT;) {
-      const bool ok = r < n;
-      cp_async16(dst + r * RS + c * 16, base + (int64_t)(key0 + (ok ? r : 0)) * a.row + c * 8, ok);
-      r += st_r;
-      c += st_c;
-      if (c >= cpr) { c -= cpr; r++; }
-    }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tig = lane & 3, mi = lane >> 3, r8 = lane & 7;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < NS; i++) mbar_init(smem_u32(&full[i]), 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  __syncthreads();
+  const uint64_t policy = l2_evict_first_policy();
+  // One thread. Rows beyond the chunk are whatever the cache holds there (finite, or zeros beyond its end); their weights are zero.
+  auto load_tile = [&](int t, int kb) {
+    const uint32_t bar = smem_u32(&full[t & (NS - 1)]), dst = smem_u32(smem) + (uint32_t)((t & (NS - 1)) * stage_bytes);
+    mbar_expect_tx(bar, (uint32_t)stage_bytes);
+    for (int i = 0; i < n_atoms; i++) tma_load_2d(dst + i * ATOM, &map, i * 64, b * a.maxlen + kb + t * LKT, bar, policy);
   };
   auto range = [&](int len, int& kb, int& ke) {
     const int lo = a.window > 0 ? max(0, len - a.window) : 0;
@@ -378,30 +449,23 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(AttnDecodeDev a
     ke = min(len, kb + a.chunk);
   };
   // Tiles that hold rows of earlier steps only are requested before the dependency wait; the length they are derived from is
-  // read again after it.
+  // read again after it. (It belongs to the previous step and has not changed; if it had, the sequence would be refused below.)
   int kb, ke;
   const int len_early = min(ld_volatile_i32(a.lens + b) + 1, a.maxlen);
   range(len_early, kb, ke);
   int n_early = 0;
   if (a.prefetch)
-    for (; n_early < NS - 2 && kb + (n_early + 1) * LKT <= min(ke, len_early - 1); n_early++) { load_tile(n_early, kb + n_early * LKT, LKT); cp_async_commit(); }
+    for (; n_early < NS - 2 && kb + (n_early + 1) * LKT <= min(ke, len_early - 1); n_early++)
+      if (threadIdx.x == 0) load_tile(n_early, kb);
   pdl_wait();
   SB_TRACE_WAITED();
   const int len = min(ld_volatile_i32(a.lens + b) + 1, a.maxlen);
-  if (len != len_early && n_early) {  // not expected: the length belongs to the previous step
-    cp_async_wait<0>();
-    __syncthreads();
-    n_early = 0;
-  }
-  range(len, kb, ke);
-  if (kb >= ke) return;
-  const int ntiles = (ke - kb + LKT - 1) / LKT;
-  for (int t = n_early; t < NS - 2; t++) {  // one group per tile, empty beyond the last
-    if (t < ntiles) load_tile(t, kb + t * LKT, min(LKT, ke - kb - t * LKT));
-    cp_async_commit();
-  }
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tig = lane & 3, mi = lane >> 3, r8 = lane & 7;
-  const int ks = warp & 3, kh = warp >> 2;
+  bool bad = len != len_early && n_early;
+  if (!bad) range(len, kb, ke);
+  const int ntiles = kb < ke ? (ke - kb + LKT - 1) / LKT : 0;
+  if (threadIdx.x == 0)
+    for (int t = n_early; t < min(NS - 2, ntiles); t++) load_tile(t, kb);
+  const int ks = warp % SL, kh = warp / SL;
   const int nks = a.row / 16;
 
   uint32_t qf[MT][KSM][4];
@@ -409,7 +473,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(AttnDecodeDev a
   for (int m = 0; m < MT; m++)
 #pragma unroll
     for (int k = 0; k < KSM; k++) {
-      const int step = ks + 4 * k, ha = h0 + m * 16 + g, hb = ha + 8;
+      const int step = ks + SL * k, ha = h0 + m * 16 + g, hb = ha + 8;
       const bf16* q0 = a.q + ((int64_t)b * a.H + ha) * a.row + step * 16 + 2 * tig;
       const bf16* q1 = q0 + 8 * (int64_t)a.row;
       const bool v = step < nks;
@@ -425,54 +489,62 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(AttnDecodeDev a
     for (int j = 0; j < NV; j++)
 #pragma unroll
       for (int i = 0; i < 4; i++) o[m][j][i] = 0.f;
-  constexpr int TPR = 256 / R, KPT = LKT / TPR;  // softmax: threads per head row, keys per thread (2 or 4)
+  constexpr int TPR = NT / R, KPT = LKT / TPR;  // softmax: threads per head row (16 or 32: never across warps), keys per thread
   const int srow = threadIdx.x / TPR, skey = (threadIdx.x % TPR) * KPT;
   float m_run = -INFINITY, l_run = 0.f;
   const int dim0 = warp * NV * 8;
+  const bool has_cols = dim0 < a.rank_p;
 
-  auto scores = [&](int t) {
-    const uint32_t tile = smem_u32(tiles + (t % NS) * LKT * RS) + (uint32_t)((kh * 16 + (mi >> 1) * 8 + r8) * RS + (mi & 1) * 16);
-    float s[MT][2][4];
-#pragma unroll
-    for (int m = 0; m < MT; m++)
-#pragma unroll
-      for (int j = 0; j < 2; j++)
-#pragma unroll
-        for (int i = 0; i < 4; i++) s[m][j][i] = 0.f;
+  float s[MT][2][4];
+  // this lane's place in an atom of the key tile: reduction steps ks, ks + SL, .. all lie in the same two 16-byte chunks
+  const uint32_t k_lane = smem_u32(smem) + (uint32_t)((ks >> 2) * ATOM + (kh * 16 + (mi >> 1) * 8 + r8) * 128 + ((((ks & 3) * 2 + (mi & 1)) ^ r8) << 4));
+  auto scores = [&](int t) {  // into registers
+    const uint32_t tile = k_lane + (uint32_t)((t & (NS - 1)) * stage_bytes);
 #pragma unroll
     for (int k = 0; k < KSM; k++) {
-      const int step = ks + 4 * k;
-      if (step < nks) {
+      if (ks + SL * k < nks) {
         uint32_t kf[4];
-        ldsm_x4(tile + (uint32_t)(step * 32), kf);
+        ldsm_x4(tile + (uint32_t)(SL / 4 * k * ATOM), kf);
 #pragma unroll
         for (int m = 0; m < MT; m++) {
-          mma_bf16(s[m][0], qf[m][k], kf[0], kf[1]);
-          mma_bf16(s[m][1], qf[m][k], kf[2], kf[3]);
+          if (k == 0) {
+            mma_bf16_zero(s[m][0], qf[m][k], kf[0], kf[1]);
+            mma_bf16_zero(s[m][1], qf[m][k], kf[2], kf[3]);
+          } else {
+            mma_bf16(s[m][0], qf[m][k], kf[0], kf[1]);
+            mma_bf16(s[m][1], qf[m][k], kf[2], kf[3]);
+          }
         }
+      } else if (k == 0) {
+#pragma unroll
+        for (int m = 0; m < MT; m++)
+#pragma unroll
+          for (int i = 0; i < 4; i++) s[m][0][i] = s[m][1][i] = 0.f;
       }
     }
-    float* w0 = sp + (((t & 1) * 4 + ks) * R + g) * SP_LD + kh * 16 + 2 * tig;
+  };
+  float* const sp_w = sp + (ks * R + g) * SP_LD + kh * 16 + 2 * tig;
+  auto store_scores = [&]() {
 #pragma unroll
     for (int m = 0; m < MT; m++)
 #pragma unroll
       for (int j = 0; j < 2; j++) {
-        float* w = w0 + m * 16 * SP_LD + j * 8;
+        float* w = sp_w + m * 16 * SP_LD + j * 8;
         *(float2*)w = make_float2(s[m][j][0], s[m][j][1]);
         *(float2*)(w + 8 * SP_LD) = make_float2(s[m][j][2], s[m][j][3]);
       }
   };
+  const float* const sp_r = sp + srow * SP_LD + skey;
+  float v[KPT];
+  auto fetch_scores = [&]() {  // the slices' sums, in slice order
+#pragma unroll
+    for (int i = 0; i < KPT; i++) v[i] = sp_r[i];
+#pragma unroll
+    for (int p = 1; p < SL; p++)
+#pragma unroll
+      for (int i = 0; i < KPT; i++) v[i] += sp_r[p * R * SP_LD + i];
+  };
   auto softmax = [&](int t) {
-    float v[KPT];
-    const float* sr = sp + ((t & 1) * 4 * R + srow) * SP_LD + skey;
-#pragma unroll
-    for (int i = 0; i < KPT; i += 2) {
-      float2 x[4];
-#pragma unroll
-      for (int p = 0; p < 4; p++) x[p] = *(const float2*)(sr + p * R * SP_LD + i);
-      v[i] = ((x[0].x + x[1].x) + x[2].x) + x[3].x;
-      v[i + 1] = ((x[0].y + x[1].y) + x[2].y) + x[3].y;
-    }
     const int lim = ke - kb - t * LKT;
     float mx = -INFINITY;
 #pragma unroll
@@ -483,23 +555,34 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(AttnDecodeDev a
 #pragma unroll
     for (int off = 1; off < TPR; off <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
     const float m_new = fmaxf(m_run, mx);  // finite: every tile holds a visible key
-    const float corr = exp2f(m_run - m_new);
+    const float corr = ex2_approx(m_run - m_new);
     m_run = m_new;
     float ls = 0.f;
     bf16* ph = pp + ((t & 1) * 2 * R + srow) * PP_LD + skey;
+    if (KPT == 1) {
+      const float p0 = ex2_approx(v[0] - m_new), a0 = round_bf16(p0);
+      ls = p0;
+      ph[0] = __float2bfloat16_rn(a0);
+      ph[R * PP_LD] = __float2bfloat16_rn(p0 - a0);
+    } else {
 #pragma unroll
-    for (int i = 0; i < KPT; i += 2) {
-      const float p0 = exp2f(v[i] - m_new), p1 = exp2f(v[i + 1] - m_new);
-      ls += p0 + p1;
-      const float a0 = round_bf16(p0), a1 = round_bf16(p1);
-      *(uint32_t*)(ph + i) = pack_bf16(a0, a1);
-      *(uint32_t*)(ph + R * PP_LD + i) = pack_bf16(p0 - a0, p1 - a1);
+      for (int i = 0; i + 1 < KPT; i += 2) {
+        const float p0 = ex2_approx(v[i] - m_new), p1 = ex2_approx(v[i + 1] - m_new);
+        ls += p0 + p1;
+        uint32_t hi, lo;
+        split_bf16x2(p0, p1, hi, lo);
+        *(uint32_t*)(ph + i) = hi;
+        *(uint32_t*)(ph + R * PP_LD + i) = lo;
+      }
     }
     l_run = l_run * corr + ls;
     if (skey == 0) corr_s[(t & 1) * R + srow] = corr;
   };
+  uint32_t v_chunk[NV / 2];  // swizzled place of this lane's 16-byte chunk of the warp's latent columns (all in one atom)
+#pragma unroll
+  for (int jp = 0; jp < NV / 2; jp++) v_chunk[jp] = (uint32_t)(((((dim0 >> 3) & 7) + jp * 2 + (mi >> 1)) ^ r8) << 4);
   auto accumulate = [&](int t) {
-    if (dim0 >= a.rank_p) return;
+    if (!has_cols) return;
     const float* cs = corr_s + (t & 1) * R;
 #pragma unroll
     for (int m = 0; m < MT; m++) {
@@ -509,7 +592,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(AttnDecodeDev a
         for (int j = 0; j < NV; j++) { o[m][j][0] *= c0; o[m][j][1] *= c0; o[m][j][2] *= c1; o[m][j][3] *= c1; }
       }
     }
-    const uint32_t tile = smem_u32(tiles + (t % NS) * LKT * RS) + (uint32_t)(((mi & 1) * 8 + r8) * RS + (dim0 + (mi >> 1) * 8) * 2);
+    const uint32_t tile = smem_u32(smem) + (uint32_t)((t & (NS - 1)) * stage_bytes + (dim0 >> 6) * ATOM + ((mi & 1) * 8 + r8) * 128);
     const uint32_t ps = smem_u32(pp + (t & 1) * 2 * R * PP_LD + ((mi & 1) * 8 + r8) * PP_LD + (mi >> 1) * 8);
 #pragma unroll
     for (int kk = 0; kk < LKT / 16; kk++) {
@@ -523,7 +606,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(AttnDecodeDev a
       for (int jp = 0; jp < NV / 2; jp++) {
         if (dim0 + jp * 16 < a.rank_p) {
           uint32_t vf[4];
-          ldsm_x4_t(tile + (uint32_t)(kk * 16 * RS + jp * 32), vf);
+          ldsm_x4_t(tile + (uint32_t)(kk * 16 * 128) + v_chunk[jp], vf);
 #pragma unroll
           for (int m = 0; m < MT; m++) {
             mma_bf16(o[m][2 * jp], ph[m], vf[0], vf[1]);
@@ -538,52 +621,91 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(AttnDecodeDev a
       }
     }
   };
+  auto arrived = [&](int t) {  // tile t has landed (bounded)
+    if (!mbar_wait(smem_u32(&full[t & (NS - 1)]), (uint32_t)(t / NS) & 1)) bad = true;
+  };
 
-  cp_async_wait<NS - 3>();
-  __syncthreads();
-  scores(0);
-  for (int t = 0; t <= ntiles; t++) {
-    cp_async_wait<NS - 4>();  // tile t + 1 has landed
-    __syncthreads();          // S(t), P(t-1) and tile t + 1 of every thread; everyone has left tile t - 2
-    const int next = t + NS - 2;
-    if (next < ntiles) load_tile(next % NS, kb + next * LKT, min(LKT, ke - kb - next * LKT));
-    cp_async_commit();
-    if (t + 1 < ntiles) scores(t + 1);
-    if (t < ntiles) softmax(t);
-    if (t > 0) accumulate(t - 1);
+  if (ntiles > 0) {
+    arrived(0);
+    scores(0);
+    store_scores();
+    for (int t = 0; t <= ntiles; t++) {
+      if (t + 1 < ntiles) arrived(t + 1);
+      __syncthreads();  // S(t) and P(t-1) of every thread; everyone has left tile t - 2
+      if (threadIdx.x == 0 && t + 2 < ntiles) load_tile(t + 2, kb);
+      if (t < ntiles) fetch_scores();
+      if (t + 1 < ntiles) scores(t + 1);
+      __syncthreads();  // everyone has fetched S(t)
+      if (t + 1 < ntiles) store_scores();
+      if (t < ntiles) softmax(t);
+      if (t > 0) accumulate(t - 1);
+    }
   }
 #pragma unroll
   for (int off = 1; off < TPR; off <<= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, off);
-  if (skey == 0 && h0 + srow < a.H) *(float2*)(a.ml_part + (((int64_t)b * a.H + h0 + srow) * a.nsplit + split) * 2) = make_float2(m_run, l_run);
+  __syncthreads();  // the ring is free: it holds this block's sums now
+  float* so = (float*)smem;  // [R][rank_p + 4]
+  const int so_ld = a.rank_p + 4;
+  if (skey == 0) ml_s[srow] = make_float2(m_run, l_run);
 #pragma unroll
   for (int m = 0; m < MT; m++)
 #pragma unroll
     for (int j = 0; j < NV; j++) {
-      const int col = dim0 + j * 8 + 2 * tig, ha = h0 + m * 16 + g;
+      const int col = dim0 + j * 8 + 2 * tig;
       if (col < a.rank_p) {
-        if (ha < a.H) *(float2*)(a.o_part + (((int64_t)b * a.H + ha) * a.nsplit + split) * a.rank_p + col) = make_float2(o[m][j][0], o[m][j][1]);
-        if (ha + 8 < a.H) *(float2*)(a.o_part + (((int64_t)b * a.H + ha + 8) * a.nsplit + split) * a.rank_p + col) = make_float2(o[m][j][2], o[m][j][3]);
+        *(float2*)(so + (m * 16 + g) * so_ld + col) = make_float2(o[m][j][0], o[m][j][1]);
+        *(float2*)(so + (m * 16 + g + 8) * so_ld + col) = make_float2(o[m][j][2], o[m][j][3]);
       }
     }
+  cluster_sync();
+  if (threadIdx.x < R) {
+    float2 ml[MAX_SPLITS];
+    float M = -INFINITY, L = 0.f;
+#pragma unroll
+    for (int i = 0; i < MAX_SPLITS; i++)
+      if (i < a.nsplit) { ml[i] = ld_cluster2(map_to_rank(smem_u32(&ml_s[threadIdx.x]), i)); M = fmaxf(M, ml[i].x); }
+#pragma unroll
+    for (int i = 0; i < MAX_SPLITS; i++)
+      if (i < a.nsplit) { ml[i].x = ml[i].y > 0.f ? exp2f(ml[i].x - M) : 0.f; L += ml[i].x * ml[i].y; }
+    const float inv = 1.0f / L;
+#pragma unroll
+    for (int i = 0; i < MAX_SPLITS; i++)
+      if (i < a.nsplit) fs[threadIdx.x][i] = ml[i].x * inv;
+  }
+  __syncthreads();
+  const int c4n = a.rank_p / 4, heads = min(R, a.H - h0);
+  const uint32_t so_a = smem_u32(so);
+  for (int i = split * NT + (int)threadIdx.x; i < heads * c4n; i += a.nsplit * NT) {
+    const int h = i / c4n, c = (i - h * c4n) * 4;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f), x[MAX_SPLITS];
+#pragma unroll
+    for (int p = 0; p < MAX_SPLITS; p++)
+      if (p < a.nsplit) x[p] = ld_cluster4(map_to_rank(so_a + (uint32_t)((h * so_ld + c) * 4), p));
+#pragma unroll
+    for (int p = 0; p < MAX_SPLITS; p++)
+      if (p < a.nsplit && fs[h][p] != 0.f) {  // a block without keys holds zeros; its weight is zero
+        const float w = fs[h][p];
+        acc.x += w * x[p].x; acc.y += w * x[p].y; acc.z += w * x[p].z; acc.w += w * x[p].w;
+      }
+    *(uint2*)(a.out + ((int64_t)b * a.H + h0 + h) * a.rank_p + c) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
+  }
+  if (bad && lane == 0) { *(volatile int*)a.status = 17; __threadfence_system(); }
+  cluster_sync();  // nobody leaves while another block may still read its shared memory
   SB_TRACE_END(SB_K_ATTN, 0);
 }
 
-// grid (H, ceil(vdim / 64), ceil(B / 16)), 256 threads: merges the key chunks of one head for 16 tokens, then its 64 value
-// columns from W_uv (a constant, requested before the dependency wait).
-constexpr int MAX_SPLITS = 16;
-struct MergeDev {
-  const float* o_part;
-  const float* ml_part;
-  const int32_t* lens;
-  int B, H, rank_p, vdim, window, maxlen, chunk, nsplit;
+// grid (H, ceil(vdim / 64), ceil(B / 16)), 256 threads: 64 value columns of one head for 16 tokens, W_uv times the weighted
+// latents (W_uv is a constant, requested before the dependency wait).
+struct ValueDev {
+  const bf16* lat;  // [B, H, rank_p]
+  int B, H, rank_p, vdim;
   const bf16* wv;   // value rows: head h, value v at (h * kv_head + v) * rank_p
   int kv_head;
   bf16* out;
   int64_t ldo;
 };
-__global__ void __launch_bounds__(256) latent_merge_kernel(MergeDev a) {
+__global__ void __launch_bounds__(256) latent_value_kernel(ValueDev a) {
   extern __shared__ __align__(128) uint8_t smem[];
-  __shared__ float fs[16][MAX_SPLITS];
   SB_TRACE_BEGIN();
   pdl_trigger();
   const int h = blockIdx.x, v0 = blockIdx.y * 64, b0 = blockIdx.z * 16, ld = a.rank_p + 8;
@@ -595,62 +717,40 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(MergeDev a) {
     const bool ok = v0 + r < a.vdim;
     cp_async16(smem_u32(wt + r * ld + cc * 8), a.wv + ((int64_t)h * a.kv_head + (ok ? v0 + r : 0)) * a.rank_p + cc * 8, ok);
   }
-  cp_async_commit();
   pdl_wait();
   SB_TRACE_WAITED();
-  {
-    const int m = threadIdx.x >> 4, l16 = threadIdx.x & 15, b = b0 + m;
-    const int len = b < a.B ? min(a.lens[b] + 1, a.maxlen) : 0;
-    const int n = a.window > 0 ? min(len, a.window) : len, ns = (n + a.chunk - 1) / a.chunk;
-    const int64_t base = ((int64_t)(b < a.B ? b : 0) * a.H + h) * a.nsplit;
-    float2 ml = l16 < ns ? *(const float2*)(a.ml_part + (base + l16) * 2) : make_float2(-INFINITY, 0.f);
-    float M = ml.x;
-#pragma unroll
-    for (int off = 1; off < 16; off <<= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, off));
-    float f = l16 < ns ? exp2f(ml.x - M) : 0.f, L = f * ml.y;
-#pragma unroll
-    for (int off = 1; off < 16; off <<= 1) L += __shfl_xor_sync(0xffffffffu, L, off);
-    fs[m][l16] = l16 < ns ? f / L : 0.f;
+  for (int c = threadIdx.x; c < 16 * cpr; c += 256) {
+    const int m = c / cpr, cc = c - m * cpr;
+    const bool ok = b0 + m < a.B;
+    cp_async16(smem_u32(ot + m * ld + cc * 8), a.lat + ((int64_t)(ok ? b0 + m : 0) * a.H + h) * a.rank_p + cc * 8, ok);
   }
-  __syncthreads();
-  // every thread of the block takes groups of four columns of any of the tokens; all chunks' loads of a group in flight at once
-  const int c4n = a.rank_p / 4;
-#pragma unroll 2
-  for (int i = threadIdx.x; i < 16 * c4n; i += 256) {
-    const int m = i / c4n, c = (i - m * c4n) * 4, b = b0 + m;
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (b < a.B) {
-      const float* src = a.o_part + (((int64_t)b * a.H + h) * a.nsplit) * a.rank_p + c;
-      for (int s0 = 0; s0 < a.nsplit; s0 += 8) {
-        float4 x[8];
-#pragma unroll
-        for (int s = 0; s < 8; s++)
-          if (s0 + s < a.nsplit && fs[m][s0 + s] != 0.f) x[s] = *(const float4*)(src + (int64_t)(s0 + s) * a.rank_p);
-#pragma unroll
-        for (int s = 0; s < 8; s++)
-          if (s0 + s < a.nsplit && fs[m][s0 + s] != 0.f) {
-            const float w = fs[m][s0 + s];
-            acc.x += w * x[s].x; acc.y += w * x[s].y; acc.z += w * x[s].z; acc.w += w * x[s].w;
-          }
-      }
-    }
-    *(uint2*)(ot + m * ld + c) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
-  }
+  cp_async_commit();
   cp_async_wait<0>();
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mi = lane >> 3, r8 = lane & 7;
-  float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-  for (int k = 0; k < a.rank_p; k += 16) {
-    uint32_t oa[4], wb[2];
-    ldsm_x4(smem_u32(ot + ((mi & 1) * 8 + r8) * ld + k + (mi >> 1) * 8), oa);
-    ldsm_x2(smem_u32(wt + (warp * 8 + r8) * ld + k + (mi & 1) * 8), wb);
-    mma_bf16(acc[(k >> 4) & 1], oa, wb[0], wb[1]);
+  float acc[4][4];
+#pragma unroll
+  for (int i = 0; i < 4; i++)
+#pragma unroll
+    for (int j = 0; j < 4; j++) acc[i][j] = 0.f;
+  for (int k0 = 0; k0 < a.rank_p; k0 += 64) {
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      const int k = k0 + 16 * i;
+      if (k < a.rank_p) {
+        uint32_t oa[4], wb[2];
+        ldsm_x4(smem_u32(ot + ((mi & 1) * 8 + r8) * ld + k + (mi >> 1) * 8), oa);
+        ldsm_x2(smem_u32(wt + (warp * 8 + r8) * ld + k + (mi & 1) * 8), wb);
+        mma_bf16(acc[i], oa, wb[0], wb[1]);
+      }
+    }
   }
   const int g = lane >> 2, v = v0 + warp * 8 + 2 * (lane & 3);
 #pragma unroll
   for (int i = 0; i < 4; i++) {
     const int b = b0 + g + (i >> 1) * 8, vc = v + (i & 1);
-    if (b < a.B && vc < a.vdim) a.out[(int64_t)b * a.ldo + (int64_t)h * a.vdim + vc] = __float2bfloat16_rn(acc[0][i] + acc[1][i]);
+    if (b < a.B && vc < a.vdim)
+      a.out[(int64_t)b * a.ldo + (int64_t)h * a.vdim + vc] = __float2bfloat16_rn((acc[0][i] + acc[1][i]) + (acc[2][i] + acc[3][i]));
   }
   SB_TRACE_END(SB_K_COMBINE, 0);
 }
@@ -738,7 +838,7 @@ int allow_smem(strictb200_ctx* ctx, F kernel, size_t bytes, size_t* have /* [64]
   static std::mutex mu;
   std::lock_guard<std::mutex> lock(mu);
   size_t& h = have[ctx->device & 63];
-  if (bytes > 48 * 1024 && bytes > h) {
+  if (bytes > 32 * 1024 && bytes > h) {  // the default limit of 48 KB counts the static share too
     SB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes));
     h = bytes;
   }
@@ -746,12 +846,43 @@ int allow_smem(strictb200_ctx* ctx, F kernel, size_t bytes, size_t* have /* [64]
 }
 constexpr size_t SMEM_MAX = 227 * 1024 - 1024;  // what a block may take, less the kernels' static share
 
-template <int MT, int KSM, int NV>
-int launch_attn_decode(strictb200_ctx* ctx, const AttnDecodeDev& a, int B) {
+typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                             const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+// 2D map of a layer's cache rows [rows, row], box = 32 rows x 64 columns (128 bytes), 128-byte swizzle.
+int cache_map(CUtensorMap* map, const bf16* base, int64_t rows, int row) {
+  static EncodeFn encode = nullptr;
+  if (!encode) {
+    void* fn = nullptr;
+    cudaDriverEntryPointQueryResult q;
+    SB_CUDA(cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &q));
+    if (!fn || q != cudaDriverEntryPointSuccess) return sb_fail(STRICTB200_ERR_CUDA, "cuTensorMapEncodeTiled is not available from this driver");
+    encode = (EncodeFn)fn;
+  }
+  cuuint64_t dims[2] = {(cuuint64_t)row, (cuuint64_t)rows};
+  cuuint64_t strides[1] = {(cuuint64_t)row * 2};
+  cuuint32_t box[2] = {64u, (cuuint32_t)LKT};
+  cuuint32_t estr[2] = {1, 1};
+  CUresult r = encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<bf16*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                      CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return sb_fail(STRICTB200_ERR_CUDA, "cuTensorMapEncodeTiled failed with code " + std::to_string((int)r));
+  return STRICTB200_OK;
+}
+
+// The kernel's shapes: warps, reduction steps per slice, latent columns per warp. Rows of up to 192 (rank 128), 384 (rank 256)
+// and 640 (rank 512) elements.
+int decode_shape(const LatentShape& s) {
+  const int rp = s.rank_p(), row = s.row();
+  return rp <= 128 && row <= 192 ? 0 : rp <= 256 && row <= 384 ? 1 : 2;
+}
+int decode_warps(const LatentShape& s) { return decode_shape(s) == 0 ? 8 : 16; }
+
+template <int MT, int NW, int KSM, int NV>
+int launch_attn_decode(strictb200_ctx* ctx, const CUtensorMap& map, const AttnDecodeDev& a, int B) {
   static size_t have[64] = {};
-  const size_t smem = attn_decode_smem(MT, KSM, a.row);
-  SB_TRY(allow_smem(ctx, latent_attn_decode_kernel<MT, KSM, NV>, smem, have));
-  SB_CUDA(sb_launch(ctx, latent_attn_decode_kernel<MT, KSM, NV>, dim3(a.nsplit, (a.H + MT * 16 - 1) / (MT * 16), B), dim3(256), smem, a));
+  const size_t smem = attn_decode_smem(MT, NW, a.row);
+  SB_TRY(allow_smem(ctx, latent_attn_decode_kernel<MT, NW, KSM, NV>, smem, have));
+  SB_CUDA(sb_launch_cluster(ctx, latent_attn_decode_kernel<MT, NW, KSM, NV>, dim3(a.nsplit, (a.H + MT * 16 - 1) / (MT * 16), B), dim3(NW * 32), smem,
+                            dim3(a.nsplit, 1, 1), map, a));
   ctx->launches++;
   return STRICTB200_OK;
 }
@@ -779,7 +910,7 @@ int k_latent_gather(strictb200_ctx* ctx, const bf16* cache, int64_t maxlen, int 
 }
 
 bool sb_latent_decode_fits(const LatentShape& s) {
-  return s.rank_p() <= 512 && s.row() <= 576 && decode_in_smem(s.dim) <= (int)SMEM_MAX && s.dim <= 512;
+  return s.rank_p() <= 512 && s.row() <= 640 && s.dim <= 512 && decode_in_smem(s.dim) <= (int)SMEM_MAX;
 }
 
 int k_latent_decode_in(strictb200_ctx* ctx, const LatentDecodeInArgs& x, int64_t B) {
@@ -796,48 +927,46 @@ int k_latent_decode_in(strictb200_ctx* ctx, const LatentDecodeInArgs& x, int64_t
   return STRICTB200_OK;
 }
 
-// Reduction steps per slice the kernel is built for: rows of up to 192, 320 and 576 elements.
-int decode_ksm(const LatentShape& s) {
-  const int nks = (s.row() / 16 + 3) / 4;
-  return s.rank_p() <= 128 && nks <= 3 ? 3 : s.rank_p() <= 256 && nks <= 5 ? 5 : 9;
-}
-
 // Keys per block: waves of blocks x (key tiles per block + what a block costs besides), over the multiples of the tile that
-// leave at most MAX_SPLITS chunks of the window (or of the planned length, where that is shorter).
+// leave at most MAX_SPLITS chunks of the window (or of the planned length, where that is shorter). The chunks of a (sequence,
+// head group) are one cluster, and clusters of 3, 5, 6 or 7 blocks pack the SMs of a GPC badly: 1, 2, 4 or 8 chunks.
 int sb_latent_decode_chunk(strictb200_ctx* ctx, const LatentShape& s, int B, int len_plan) {
   const int n = s.window > 0 ? std::min(s.window, len_plan) : len_plan, tiles = std::max(1, (n + LKT - 1) / LKT);
   const int mt = s.H <= 16 ? 1 : 2;
-  const int per_sm = std::max<int>(1, std::min<int>(2, (int)(227 * 1024 / (attn_decode_smem(mt, decode_ksm(s), s.row()) + 1024))));
+  const int per_sm = std::max<int>(1, std::min<int>(2, (int)(227 * 1024 / (attn_decode_smem(mt, decode_warps(s), s.row()) + 2048))));
   const int64_t slots = (int64_t)ctx->sm_count * per_sm, pairs = (int64_t)B * ((s.H + mt * 16 - 1) / (mt * 16));
   int best = tiles;
   double best_cost = 1e30;
-  for (int c = (tiles + MAX_SPLITS - 1) / MAX_SPLITS; c <= tiles; c++) {
-    const int64_t blocks = pairs * ((tiles + c - 1) / c), waves = (blocks + slots - 1) / slots;
-    const double cost = (double)waves * (c + 3) + 0.05 * ((tiles + c - 1) / c);  // every chunk adds to the merge
+  for (int k = 1; k <= MAX_SPLITS && k <= tiles; k *= 2) {
+    const int c = (tiles + k - 1) / k;
+    const int64_t blocks = pairs * k, waves = (blocks + slots - 1) / slots;
+    const double cost = (double)waves * (c + 4);
     if (cost < best_cost - 1e-9) { best_cost = cost; best = c; }
   }
   return best * LKT;
 }
-size_t sb_latent_decode_scratch(const LatentShape& s, int B) { return (size_t)B * s.H * MAX_SPLITS * (s.rank_p() + 2) * sizeof(float); }
+size_t sb_latent_decode_scratch(const LatentShape& s, int B) { return (size_t)B * s.H * s.rank_p() * sizeof(bf16); }
 
 int k_latent_attn_decode(strictb200_ctx* ctx, const LatentShape& s, const bf16* q_abs, const bf16* cache, const int32_t* lens, int B, int maxlen, int chunk,
-                         int nsplit, float* scratch, const bf16* wkv, bf16* out, int64_t ldo) {
+                         int nsplit, bf16* scratch, const bf16* wkv, bf16* out, int64_t ldo) {
   if (!sb_latent_decode_fits(s)) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "latent decode attention: rows too wide for the tensor-core kernel");
   if (nsplit < 1 || nsplit > MAX_SPLITS || chunk < LKT || chunk % LKT || B > 65535) return sb_fail(STRICTB200_ERR_INVALID_ARG, "latent decode attention: bad key chunks");
-  float* ml = scratch + (size_t)B * s.H * nsplit * s.rank_p();
-  AttnDecodeDev a{q_abs, cache, lens, s.H, s.row(), s.rank_p(), maxlen, s.window, chunk, nsplit, s.scale * LOG2E, scratch, ml, ctx->opt.attn_prefetch};
-  const int rp = s.rank_p(), ksm = decode_ksm(s);
-#define LATENT_DECODE(KSM, NV) SB_TRY((s.H <= 16 ? launch_attn_decode<1, KSM, NV>(ctx, a, B) : launch_attn_decode<2, KSM, NV>(ctx, a, B)))
-  if (ksm == 3) LATENT_DECODE(3, 2);
-  else if (ksm == 5) LATENT_DECODE(5, 4);
-  else LATENT_DECODE(9, 8);
+  if ((int64_t)B * maxlen > INT32_MAX) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "latent decode attention: cache too large for 32-bit tile coordinates");
+  CUtensorMap map;
+  SB_TRY(cache_map(&map, cache, (int64_t)B * maxlen, s.row()));
+  AttnDecodeDev a{q_abs, lens, s.H, s.row(), s.rank_p(), maxlen, s.window, chunk, nsplit, s.scale * LOG2E, scratch, ctx->opt.attn_prefetch, ctx->d_status};
+  const int rp = s.rank_p(), shape = decode_shape(s);
+#define LATENT_DECODE(NW, KSM, NV) SB_TRY((s.H <= 16 ? launch_attn_decode<1, NW, KSM, NV>(ctx, map, a, B) : launch_attn_decode<2, NW, KSM, NV>(ctx, map, a, B)))
+  if (shape == 0) LATENT_DECODE(8, 3, 2);
+  else if (shape == 1) LATENT_DECODE(16, 3, 2);
+  else LATENT_DECODE(16, 5, 4);
 #undef LATENT_DECODE
   sb_prof_split(ctx, STRICTB200_K_ATTN_MERGE);
   static size_t have[64] = {};
   const size_t smem = (size_t)(64 + 16) * (rp + 8) * 2;
-  SB_TRY(allow_smem(ctx, latent_merge_kernel, smem, have));
-  MergeDev m{scratch, ml, lens, B, s.H, rp, s.vdim, s.window, maxlen, chunk, nsplit, wkv + (int64_t)s.H * s.kv_head() * rp, s.kv_head(), out, ldo};
-  SB_CUDA(sb_launch(ctx, latent_merge_kernel, dim3(s.H, (s.vdim + 63) / 64, (B + 15) / 16), dim3(256), smem, m));
+  SB_TRY(allow_smem(ctx, latent_value_kernel, smem, have));
+  ValueDev m{scratch, B, s.H, rp, s.vdim, wkv + (int64_t)s.H * s.kv_head() * rp, s.kv_head(), out, ldo};
+  SB_CUDA(sb_launch(ctx, latent_value_kernel, dim3(s.H, (s.vdim + 63) / 64, (B + 15) / 16), dim3(256), smem, m));
   ctx->launches++;
   return STRICTB200_OK;
 }

@@ -407,7 +407,7 @@ int sb_stack_decode_body(strictb200_model* m, strictb200_kv* kv) {
     in.act = (bf16*)b.oa + w.ko_p; in.ld_act = w.ldo;
     PROF(STRICTB200_K_ROPE, k_latent_decode_in(ctx, in, B));
     PROF(STRICTB200_K_ATTN, k_latent_attn_decode(ctx, w.s, (const bf16*)b.q, (const bf16*)latents(m, kv, l, 0), kv->d_lens, (int)B, kv->maxlen,
-                                                 kv->layer_chunk[l] / 32, kv->layer_chunk[l] % 32, b.attn_ws, (const bf16*)w.w_kv, (bf16*)b.oa, w.ldo));
+                                                 kv->layer_chunk[l] / 32, kv->layer_chunk[l] % 32, (bf16*)b.attn_ws, (const bf16*)w.w_kv, (bf16*)b.oa, w.ldo));
     GemmBf16Args o;
     o.M = B; o.N = d; o.K = w.ldo; o.x = (const bf16*)b.oa; o.ldx = w.ldo; o.w = (const bf16*)w.w_out; o.ldw = w.ldo;
     o.part = b.part2; o.splits = sb_gemm_bf16_splits(ctx, B, d, w.ldo);
