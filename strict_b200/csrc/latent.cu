@@ -90,12 +90,6 @@ __device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-// the same with a zero accumulator
-__device__ __forceinline__ void mma_bf16_zero(float* d, const uint32_t* a, uint32_t b0, uint32_t b1) {
-  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%10,%10,%10,%10};\n"
-      : "=f"(d[0]), "=f"(d[1]), "=f"(d[2]), "=f"(d[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1), "f"(0.f));
-}
 __device__ __forceinline__ float ex2_approx(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -389,276 +383,362 @@ __global__ void __launch_bounds__(256) latent_decode_in_kernel(DecodeInDev d, in
 }
 
 // ------------------------------------------------------------------ decode: split-key attention over the latents
-// grid (nsplit, ceil(H / (16 MT)), B), 32 NW threads; the nsplit blocks of a (sequence, head group) are one cluster. Rows of
-// the MMA tiles = up to 16 MT heads, 32 keys per step. Three products of three different steps share an iteration:
-//   S(t+1) partials  warp (ks, kh): reduction steps ks, ks + SL, .. of the cache row for the 16 keys of half kh; its share of
-//                    the queries stays in registers for the whole block, so a step reads the key tile from shared memory once
-//   softmax(t)       the SL partial scores of a (head, key) are added in slice order; running maximum and sum per head
-//   O += P(t-1) c    every warp owns 8 NV latent columns of all heads; the key tile is its operand again
-// A key tile is copied by TMA in atoms of 32 rows x 64 columns (128-byte swizzle: 16-byte chunk c of row r lies at c ^ (r & 7));
-// tiles pass through a ring of four stages (t-1, t, t+1 in use, t+2 in flight). At the end the cluster's blocks weigh each other's sums through distributed shared memory, so what leaves
-// is one bf16 row of latents per head.
-constexpr int LKT = 32, NS = 4;
-constexpr int MAX_SPLITS = 8;  // blocks of a cluster
+// grid (nsplit, ceil(H / 32), B), 256 threads; the nsplit blocks of a (sequence, head group) are one cluster. The work is two
+// products per tile of 64 keys on the tcgen05 tensor cores, with the long dimension of each as the tensor-memory lanes:
+//   S^T = K Q^T      A = the key tile [64 keys x row] (K-major), B = the queries [32 heads x row] (K-major, staged once);
+//                    lane = key, column = head. M is 128: lanes 64.. read past the tile and are ignored.
+//   O^T += c^T P     A = the same tile read MN-major, [128 latents x 64 keys] per block of 128 latents, B = the weights
+//                    [64 keys x 64], MN-major: columns 0..31 the heads' hi terms, 32..63 their lo terms (P = hi + lo);
+//                    lane = latent, column = head; the two halves are added at the end
+// Roles by warp: 0, 1, 4, 5 softmax (warp & 1 = which 32 keys, warp >> 2 = which 16 heads), 2 MMA issue, 3 TMA producer,
+// 6, 7 help to rescale O^T (their lanes are out of the softmax warps' reach). S^T is double-buffered, so S^T(t+1) runs under
+// the softmax of tile t. A head's running maximum is followed lazily (only when it grew by more than 2^8, as in the prompt's
+// kernel), so O^T is hardly ever rescaled.
+// Key tiles are TMA atoms of 64 rows x 64 columns (128-byte swizzle) in a ring of NS stages. At the end the cluster's blocks
+// weigh each other's sums through distributed shared memory; what leaves is one bf16 row of latents per head.
+// Every mbarrier wait is bounded: on expiry the error word is set and the block runs to its end.
+constexpr int LKT = 64, LHEADS = 32;
+constexpr int MAX_SPLITS = 8;               // blocks of a cluster
+constexpr int ATOM = LKT * 128;             // bytes of a key tile's 64-column atom
+constexpr int Q_ATOM = LHEADS * 128;        // ... and of the queries'
+constexpr int P_BYTES = LKT * 128;
 struct AttnDecodeDev {
-  const bf16* q;
   const int32_t* lens;
-  int H, row, rank_p, maxlen, window, chunk, nsplit;
+  int H, row, rank_p, maxlen, window, chunk, nsplit, stages;
   float scale_log2;
   bf16* out;   // [B, H, rank_p] weighted sum of latents
   int prefetch;
   int* status;
 };
-constexpr int SP_LD = 36, PP_LD = 40;  // row strides of the score (fp32) and weight (bf16) tiles
-constexpr int ATOM = LKT * 128;        // bytes of a tile's 64-column atom
-constexpr size_t attn_decode_smem(int mt, int nw, int row) {
-  return 1024 /* round-up to the swizzle's alignment */ + (size_t)NS * ((row + 63) / 64) * ATOM + (size_t)(nw / 2) * mt * 16 * SP_LD * 4 + (size_t)2 * 2 * mt * 16 * PP_LD * 2 + 2 * mt * 16 * 4;
+constexpr int MAX_STAGES = 4;
+inline int decode_atoms(int row) { return (row + 63) / 64; }
+inline size_t attn_decode_smem(int row, int stages) {
+  return 1024 /* round-up to the swizzle's alignment */ + (size_t)stages * decode_atoms(row) * ATOM + (size_t)decode_atoms(row) * Q_ATOM + 2 * P_BYTES;
+}
+// stages of the ring: as many as leave room for two blocks on an SM where the rows are short, else what one block can have
+inline int decode_stages(int row, bool two_blocks) {
+  for (int n = MAX_STAGES; n > 2; n--)
+    if (attn_decode_smem(row, n) + 4096 <= (size_t)(two_blocks ? 113 : 226) * 1024) return n;
+  return 2;
 }
 
-template <int MT, int NW, int KSM, int NV>
-__global__ void __launch_bounds__(NW * 32) latent_attn_decode_kernel(const __grid_constant__ CUtensorMap map, AttnDecodeDev a) {
-  constexpr int R = MT * 16, SL = NW / 2, NT = NW * 32;
+__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
+__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
+__device__ __forceinline__ void tc_commit(uint32_t bar) {
+  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
+}
+__device__ __forceinline__ void tc_mma(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
+      :
+      : "r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(0u)
+      : "memory");
+}
+__device__ __forceinline__ void tc_ld16(uint32_t taddr, uint32_t* r) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]),
+        "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+      : "r"(taddr));
+}
+__device__ __forceinline__ void tc_st16(uint32_t taddr, const uint32_t* r) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]),
+      "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
+      : "memory");
+}
+__device__ __forceinline__ void tc_wait_ld() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
+__device__ __forceinline__ void tc_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+// K-major operand: 128-byte rows (64 elements of the reduction dimension, 128-byte swizzle), groups of 8 rows 1024 bytes apart.
+__device__ __forceinline__ uint64_t desc_kmajor(uint32_t addr) {
+  return (uint64_t)((addr >> 4) & 0x3FFF) | (1ull << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
+}
+// MN-major operand: rows are the reduction dimension, 64 contiguous elements of the other one per row; groups of 8 rows 1024
+// bytes apart, the next 64 elements in the next atom.
+__device__ __forceinline__ uint64_t desc_mnmajor(uint32_t addr) {
+  return (uint64_t)((addr >> 4) & 0x3FFF) | ((uint64_t)(ATOM >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
+}
+// Reduction of 16 values per lane over the 32 lanes of a warp, op = max or sum: afterwards lanes 2i and 2i + 1 hold the result
+// of value i. Every exchange halves the values a lane still carries.
+template <typename Op>
+__device__ __forceinline__ float transposed_reduce(const float* v, int lane, Op op) {
+  float a[8], b[4], c[2];
+#pragma unroll
+  for (int i = 0; i < 8; i++) {
+    const float keep = lane & 16 ? v[8 + i] : v[i], send = lane & 16 ? v[i] : v[8 + i];
+    a[i] = op(keep, __shfl_xor_sync(0xffffffffu, send, 16));
+  }
+#pragma unroll
+  for (int i = 0; i < 4; i++) {
+    const float keep = lane & 8 ? a[4 + i] : a[i], send = lane & 8 ? a[i] : a[4 + i];
+    b[i] = op(keep, __shfl_xor_sync(0xffffffffu, send, 8));
+  }
+#pragma unroll
+  for (int i = 0; i < 2; i++) {
+    const float keep = lane & 4 ? b[2 + i] : b[i], send = lane & 4 ? b[i] : b[2 + i];
+    c[i] = op(keep, __shfl_xor_sync(0xffffffffu, send, 4));
+  }
+  const float keep = lane & 2 ? c[1] : c[0], send = lane & 2 ? c[0] : c[1];
+  const float d = op(keep, __shfl_xor_sync(0xffffffffu, send, 2));
+  return op(d, __shfl_xor_sync(0xffffffffu, d, 1));
+}
+
+__global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_q, AttnDecodeDev a) {
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024 - (smem_u32(smem_raw) & 1023)) & 1023);
-  __shared__ __align__(8) uint64_t full[NS];
-  __shared__ float2 ml_s[R];
-  __shared__ float fs[R][MAX_SPLITS];
+  __shared__ __align__(8) uint64_t k_full[MAX_STAGES], k_empty[MAX_STAGES], q_full, bar_s[2], bar_p, bar_o[2];
+  __shared__ uint32_t tmem_slot;
+  __shared__ int grow_s[2][2];                                    // [tile parity][head half]: some maximum has to be followed
+  __shared__ __align__(16) float corr_s[2][LHEADS], mx_s[2][2][LHEADS];  // [tile parity], [tile parity][key half]
+  __shared__ float2 ml_s[LHEADS];
+  __shared__ float fs[LHEADS][MAX_SPLITS];
   SB_TRACE_BEGIN();
-  pdl_trigger();
-  const int split = blockIdx.x, h0 = blockIdx.y * R, b = blockIdx.z;
-  const int n_atoms = (a.row + 63) / 64, stage_bytes = n_atoms * ATOM;
-  float* sp = (float*)(smem + NS * stage_bytes);       // [SL][R][SP_LD], behind the ring of key tiles
-  bf16* pp = (bf16*)(sp + SL * R * SP_LD);             // [2][hi, lo][R][PP_LD]
-  float* corr_s = (float*)(pp + 2 * 2 * R * PP_LD);    // [2][R]
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tig = lane & 3, mi = lane >> 3, r8 = lane & 7;
+  const int split = blockIdx.x, h0 = blockIdx.y * LHEADS, b = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n_atoms = (a.row + 63) / 64, stage_bytes = n_atoms * ATOM, n_mb = (a.rank_p + 127) / 128;
+  const uint32_t sK = smem_u32(smem), sQ = sK + (uint32_t)(a.stages * stage_bytes), sP = sQ + (uint32_t)(n_atoms * Q_ATOM);
+  const uint32_t tmem_cols = n_mb <= 2 ? 256u : 512u;  // two S^T tiles of 32 columns, then 64 columns per block of latents
   if (threadIdx.x == 0) {
-    for (int i = 0; i < NS; i++) mbar_init(smem_u32(&full[i]), 1);
+    for (int i = 0; i < a.stages; i++) { mbar_init(smem_u32(&k_full[i]), 1); mbar_init(smem_u32(&k_empty[i]), 1); }
+    mbar_init(smem_u32(&q_full), 1);
+    mbar_init(smem_u32(&bar_p), 192);
+    for (int i = 0; i < 2; i++) { mbar_init(smem_u32(&bar_s[i]), 1); mbar_init(smem_u32(&bar_o[i]), 1); }
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
+  if (warp == 2) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(tmem_cols) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  tc_fence_before();
   __syncthreads();
-  const uint64_t policy = l2_evict_first_policy();
-  // One thread. Rows beyond the chunk are whatever the cache holds there (finite, or zeros beyond its end); their weights are zero.
-  auto load_tile = [&](int t, int kb) {
-    const uint32_t bar = smem_u32(&full[t & (NS - 1)]), dst = smem_u32(smem) + (uint32_t)((t & (NS - 1)) * stage_bytes);
-    mbar_expect_tx(bar, (uint32_t)stage_bytes);
-    for (int i = 0; i < n_atoms; i++) tma_load_2d(dst + i * ATOM, &map, i * 64, b * a.maxlen + kb + t * LKT, bar, policy);
-  };
+  tc_fence_after();
+  const uint32_t tmem = tmem_slot;
+  // Only now may the following kernels begin: one that also takes tensor memory and waits for this one must find this block's
+  // share already allocated.
+  pdl_trigger();
+
   auto range = [&](int len, int& kb, int& ke) {
     const int lo = a.window > 0 ? max(0, len - a.window) : 0;
     kb = lo + split * a.chunk;
     ke = min(len, kb + a.chunk);
   };
+  const uint64_t policy = l2_evict_first_policy();
+  // One thread. Rows beyond the chunk are whatever the cache holds there (finite, or zeros beyond its end); their weights are zero.
+  auto load_tile = [&](int t, int kb) {
+    const int st = t % a.stages;
+    mbar_expect_tx(smem_u32(&k_full[st]), (uint32_t)stage_bytes);
+    for (int i = 0; i < n_atoms; i++) tma_load_2d(sK + (uint32_t)(st * stage_bytes + i * ATOM), &map_k, i * 64, b * a.maxlen + kb + t * LKT, smem_u32(&k_full[st]), policy);
+  };
   // Tiles that hold rows of earlier steps only are requested before the dependency wait; the length they are derived from is
-  // read again after it. (It belongs to the previous step and has not changed; if it had, the sequence would be refused below.)
-  int kb, ke;
+  // read again after it. (It belongs to the previous step and has not changed; if it had, the step would report an error.)
+  int kb, ke, n_early = 0;
   const int len_early = min(ld_volatile_i32(a.lens + b) + 1, a.maxlen);
   range(len_early, kb, ke);
-  int n_early = 0;
   if (a.prefetch)
-    for (; n_early < NS - 2 && kb + (n_early + 1) * LKT <= min(ke, len_early - 1); n_early++)
-      if (threadIdx.x == 0) load_tile(n_early, kb);
+    for (; n_early < a.stages && kb + (n_early + 1) * LKT <= min(ke, len_early - 1); n_early++)
+      if (threadIdx.x == 96) load_tile(n_early, kb);
   pdl_wait();
   SB_TRACE_WAITED();
   const int len = min(ld_volatile_i32(a.lens + b) + 1, a.maxlen);
-  bool bad = len != len_early && n_early;
-  if (!bad) range(len, kb, ke);
+  int err = 0;
+  if (len != len_early && n_early) err = 17;
+  else range(len, kb, ke);
   const int ntiles = kb < ke ? (ke - kb + LKT - 1) / LKT : 0;
-  if (threadIdx.x == 0)
-    for (int t = n_early; t < min(NS - 2, ntiles); t++) load_tile(t, kb);
-  const int ks = warp % SL, kh = warp / SL;
-  const int nks = a.row / 16;
+  auto wait = [&](uint64_t* bar, int parity, int code) {
+    if (!err && !mbar_wait(smem_u32(bar), (uint32_t)parity & 1)) err = code;
+    return err == 0;
+  };
+  // O^T columns of this warp's lanes times the heads' corrections; part of parts: which share of the columns
+  auto rescale = [&](int t, int part, int parts) {
+    const float* cs = corr_s[t & 1];
+    const uint32_t base = tmem + 64u + ((uint32_t)((warp & 3) * 32) << 16);
+    for (int c = part; c < n_mb * 4; c += parts) {
+      uint32_t r[16];
+      tc_ld16(base + (uint32_t)(c * 16), r);
+      tc_wait_ld();
+#pragma unroll
+      for (int j = 0; j < 16; j++) r[j] = __float_as_uint(__uint_as_float(r[j]) * cs[(c & 1) * 16 + j]);
+      tc_st16(base + (uint32_t)(c * 16), r);
+    }
+    tc_wait_st();
+  };
 
-  uint32_t qf[MT][KSM][4];
-#pragma unroll
-  for (int m = 0; m < MT; m++)
-#pragma unroll
-    for (int k = 0; k < KSM; k++) {
-      const int step = ks + SL * k, ha = h0 + m * 16 + g, hb = ha + 8;
-      const bf16* q0 = a.q + ((int64_t)b * a.H + ha) * a.row + step * 16 + 2 * tig;
-      const bf16* q1 = q0 + 8 * (int64_t)a.row;
-      const bool v = step < nks;
-      qf[m][k][0] = v && ha < a.H ? *(const uint32_t*)q0 : 0u;
-      qf[m][k][1] = v && hb < a.H ? *(const uint32_t*)q1 : 0u;
-      qf[m][k][2] = v && ha < a.H ? *(const uint32_t*)(q0 + 8) : 0u;
-      qf[m][k][3] = v && hb < a.H ? *(const uint32_t*)(q1 + 8) : 0u;
-    }
-  float o[MT][NV][4];
-#pragma unroll
-  for (int m = 0; m < MT; m++)
-#pragma unroll
-    for (int j = 0; j < NV; j++)
-#pragma unroll
-      for (int i = 0; i < 4; i++) o[m][j][i] = 0.f;
-  constexpr int TPR = NT / R, KPT = LKT / TPR;  // softmax: threads per head row (16 or 32: never across warps), keys per thread
-  const int srow = threadIdx.x / TPR, skey = (threadIdx.x % TPR) * KPT;
-  float m_run = -INFINITY, l_run = 0.f;
-  const int dim0 = warp * NV * 8;
-  const bool has_cols = dim0 < a.rank_p;
-
-  float s[MT][2][4];
-  // this lane's place in an atom of the key tile: reduction steps ks, ks + SL, .. all lie in the same two 16-byte chunks
-  const uint32_t k_lane = smem_u32(smem) + (uint32_t)((ks >> 2) * ATOM + (kh * 16 + (mi >> 1) * 8 + r8) * 128 + ((((ks & 3) * 2 + (mi & 1)) ^ r8) << 4));
-  auto scores = [&](int t) {  // into registers
-    const uint32_t tile = k_lane + (uint32_t)((t & (NS - 1)) * stage_bytes);
-#pragma unroll
-    for (int k = 0; k < KSM; k++) {
-      if (ks + SL * k < nks) {
-        uint32_t kf[4];
-        ldsm_x4(tile + (uint32_t)(SL / 4 * k * ATOM), kf);
-#pragma unroll
-        for (int m = 0; m < MT; m++) {
-          if (k == 0) {
-            mma_bf16_zero(s[m][0], qf[m][k], kf[0], kf[1]);
-            mma_bf16_zero(s[m][1], qf[m][k], kf[2], kf[3]);
-          } else {
-            mma_bf16(s[m][0], qf[m][k], kf[0], kf[1]);
-            mma_bf16(s[m][1], qf[m][k], kf[2], kf[3]);
-          }
-        }
-      } else if (k == 0) {
-#pragma unroll
-        for (int m = 0; m < MT; m++)
-#pragma unroll
-          for (int i = 0; i < 4; i++) s[m][0][i] = s[m][1][i] = 0.f;
+  if (warp == 3) {
+    // ---- TMA producer
+    if (lane == 0 && ntiles > 0) {
+      mbar_expect_tx(smem_u32(&q_full), (uint32_t)(n_atoms * Q_ATOM));
+      for (int i = 0; i < n_atoms; i++)
+        asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(sQ + (uint32_t)(i * Q_ATOM)), "l"(&map_q),
+                     "r"(i * 64), "r"(b * a.H + h0), "r"(smem_u32(&q_full))
+                     : "memory");
+      for (int t = n_early; t < ntiles; t++) {
+        if (t >= a.stages && !wait(&k_empty[t % a.stages], (t / a.stages) + 1, 18)) break;
+        load_tile(t, kb);
       }
     }
-  };
-  float* const sp_w = sp + (ks * R + g) * SP_LD + kh * 16 + 2 * tig;
-  auto store_scores = [&]() {
+  } else if (warp == 2) {
+    // ---- MMA issue: S(0), then per tile S(t+1) and PV(t)
+    if (lane == 0 && ntiles > 0) {
+      // D = F32, A = B = BF16, M = 128; N = 32 heads, or N = 64 with both operands MN-major
+      constexpr uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(LHEADS >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+      constexpr uint32_t idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | (1u << 16) | ((uint32_t)(64 >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+      const int nks = (a.row + 15) / 16;
+      auto issue_s = [&](int t) {
+        if (!wait(&k_full[t % a.stages], t / a.stages, 19)) return;
+        tc_fence_after();
+        const uint32_t tile = sK + (uint32_t)((t % a.stages) * stage_bytes);
+        for (int s = 0; s < nks; s++)
+          tc_mma(tmem + (uint32_t)((t & 1) * LHEADS), desc_kmajor(tile + (uint32_t)((s >> 2) * ATOM + (s & 3) * 32)), desc_kmajor(sQ + (uint32_t)((s >> 2) * Q_ATOM + (s & 3) * 32)),
+                 idesc_s, s ? 1u : 0u);
+        tc_commit(smem_u32(&bar_s[t & 1]));
+      };
+      if (wait(&q_full, 0, 20)) issue_s(0);
+      for (int t = 0; t < ntiles && !err; t++) {
+        if (t + 1 < ntiles) issue_s(t + 1);
+        if (!wait(&bar_p, t, 21)) break;  // the weights are in shared memory, O^T follows the new maxima
+        tc_fence_after();
+        const uint32_t tile = sK + (uint32_t)((t % a.stages) * stage_bytes), p = sP + (uint32_t)((t & 1) * P_BYTES);
+        for (int mb = 0; mb < n_mb; mb++)
 #pragma unroll
-    for (int m = 0; m < MT; m++)
-#pragma unroll
-      for (int j = 0; j < 2; j++) {
-        float* w = sp_w + m * 16 * SP_LD + j * 8;
-        *(float2*)w = make_float2(s[m][j][0], s[m][j][1]);
-        *(float2*)(w + 8 * SP_LD) = make_float2(s[m][j][2], s[m][j][3]);
-      }
-  };
-  const float* const sp_r = sp + srow * SP_LD + skey;
-  float v[KPT];
-  auto fetch_scores = [&]() {  // the slices' sums, in slice order
-#pragma unroll
-    for (int i = 0; i < KPT; i++) v[i] = sp_r[i];
-#pragma unroll
-    for (int p = 1; p < SL; p++)
-#pragma unroll
-      for (int i = 0; i < KPT; i++) v[i] += sp_r[p * R * SP_LD + i];
-  };
-  auto softmax = [&](int t) {
-    const int lim = ke - kb - t * LKT;
-    float mx = -INFINITY;
-#pragma unroll
-    for (int i = 0; i < KPT; i++) {
-      v[i] = skey + i < lim ? v[i] * a.scale_log2 : -INFINITY;
-      mx = fmaxf(mx, v[i]);
-    }
-#pragma unroll
-    for (int off = 1; off < TPR; off <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-    const float m_new = fmaxf(m_run, mx);  // finite: every tile holds a visible key
-    const float corr = ex2_approx(m_run - m_new);
-    m_run = m_new;
-    float ls = 0.f;
-    bf16* ph = pp + ((t & 1) * 2 * R + srow) * PP_LD + skey;
-    if (KPT == 1) {
-      const float p0 = ex2_approx(v[0] - m_new), a0 = round_bf16(p0);
-      ls = p0;
-      ph[0] = __float2bfloat16_rn(a0);
-      ph[R * PP_LD] = __float2bfloat16_rn(p0 - a0);
-    } else {
-#pragma unroll
-      for (int i = 0; i + 1 < KPT; i += 2) {
-        const float p0 = ex2_approx(v[i] - m_new), p1 = ex2_approx(v[i + 1] - m_new);
-        ls += p0 + p1;
-        uint32_t hi, lo;
-        split_bf16x2(p0, p1, hi, lo);
-        *(uint32_t*)(ph + i) = hi;
-        *(uint32_t*)(ph + R * PP_LD + i) = lo;
+          for (int s = 0; s < LKT / 16; s++)  // 16 keys = 16 rows of 128 bytes
+            tc_mma(tmem + 64u + (uint32_t)(mb * 64), desc_mnmajor(tile + (uint32_t)(2 * mb * ATOM + s * 2048)), desc_mnmajor(p + (uint32_t)(s * 2048)), idesc_pv, (t | s) ? 1u : 0u);
+        tc_commit(smem_u32(&bar_o[t & 1]));
+        tc_commit(smem_u32(&k_empty[t % a.stages]));
       }
     }
-    l_run = l_run * corr + ls;
-    if (skey == 0) corr_s[(t & 1) * R + srow] = corr;
-  };
-  uint32_t v_chunk[NV / 2];  // swizzled place of this lane's 16-byte chunk of the warp's latent columns (all in one atom)
-#pragma unroll
-  for (int jp = 0; jp < NV / 2; jp++) v_chunk[jp] = (uint32_t)(((((dim0 >> 3) & 7) + jp * 2 + (mi >> 1)) ^ r8) << 4);
-  auto accumulate = [&](int t) {
-    if (!has_cols) return;
-    const float* cs = corr_s + (t & 1) * R;
-#pragma unroll
-    for (int m = 0; m < MT; m++) {
-      const float c0 = cs[m * 16 + g], c1 = cs[m * 16 + g + 8];
-      if (!__all_sync(0xffffffffu, c0 == 1.0f && c1 == 1.0f)) {
-#pragma unroll
-        for (int j = 0; j < NV; j++) { o[m][j][0] *= c0; o[m][j][1] *= c0; o[m][j][2] *= c1; o[m][j][3] *= c1; }
+  } else if (warp >= 6) {
+    for (int t = 0; t < ntiles; t++) {
+      asm volatile("bar.sync 2, 192;" ::: "memory");
+      if (t > 0 && (grow_s[t & 1][0] | grow_s[t & 1][1])) {
+        wait(&bar_o[(t - 1) & 1], (t - 1) >> 1, 22);
+        __syncwarp();
+        tc_fence_after();
+        rescale(t, 0, 1);
+        tc_fence_before();
       }
+      asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(&bar_p)) : "memory");
     }
-    const uint32_t tile = smem_u32(smem) + (uint32_t)((t & (NS - 1)) * stage_bytes + (dim0 >> 6) * ATOM + ((mi & 1) * 8 + r8) * 128);
-    const uint32_t ps = smem_u32(pp + (t & 1) * 2 * R * PP_LD + ((mi & 1) * 8 + r8) * PP_LD + (mi >> 1) * 8);
+  } else {
+    // ---- softmax: thread = key, 16 heads
+    const int kh = warp & 1, hg = warp >> 2, key = kh * 32 + lane;
+    float m_run[16], l_run[16];
 #pragma unroll
-    for (int kk = 0; kk < LKT / 16; kk++) {
-      uint32_t ph[MT][4], pl[MT][4];
+    for (int i = 0; i < 16; i++) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
+    const uint32_t p_row = (uint32_t)((key >> 3) * 1024 + (key & 7) * 128);
+    for (int t = 0; t < ntiles; t++) {
+      wait(&bar_s[t & 1], t >> 1, 23);
+      __syncwarp();
+      tc_fence_after();
+      uint32_t r[16];
+      tc_ld16(tmem + (uint32_t)((t & 1) * LHEADS + hg * 16) + ((uint32_t)(kh * 32) << 16), r);
+      tc_wait_ld();
+      const bool live = kb + t * LKT + key < ke;
+      float v[16];
 #pragma unroll
-      for (int m = 0; m < MT; m++) {
-        ldsm_x4(ps + (uint32_t)((m * 16 * PP_LD + kk * 16) * 2), ph[m]);
-        ldsm_x4(ps + (uint32_t)(((R + m * 16) * PP_LD + kk * 16) * 2), pl[m]);
-      }
+      for (int i = 0; i < 16; i++) v[i] = live ? __uint_as_float(r[i]) * a.scale_log2 : -INFINITY;
+      const float mx = transposed_reduce(v, lane, [](float x, float y) { return fmaxf(x, y); });
+      if (!(lane & 1)) mx_s[t & 1][kh][hg * 16 + (lane >> 1)] = mx;
+      asm volatile("bar.sync 1, 128;" ::: "memory");
+      bool grow = false;
+      float corr[16];
 #pragma unroll
-      for (int jp = 0; jp < NV / 2; jp++) {
-        if (dim0 + jp * 16 < a.rank_p) {
-          uint32_t vf[4];
-          ldsm_x4_t(tile + (uint32_t)(kk * 16 * 128) + v_chunk[jp], vf);
+      for (int i = 0; i < 16; i += 4) {
+        const float4 x = *(const float4*)&mx_s[t & 1][0][hg * 16 + i], y = *(const float4*)&mx_s[t & 1][1][hg * 16 + i];
+        const float m[4] = {fmaxf(x.x, y.x), fmaxf(x.y, y.y), fmaxf(x.z, y.z), fmaxf(x.w, y.w)};
 #pragma unroll
-          for (int m = 0; m < MT; m++) {
-            mma_bf16(o[m][2 * jp], ph[m], vf[0], vf[1]);
-            mma_bf16(o[m][2 * jp + 1], ph[m], vf[2], vf[3]);
-          }
-#pragma unroll
-          for (int m = 0; m < MT; m++) {
-            mma_bf16(o[m][2 * jp], pl[m], vf[0], vf[1]);
-            mma_bf16(o[m][2 * jp + 1], pl[m], vf[2], vf[3]);
-          }
+        for (int j = 0; j < 4; j++) {
+          const bool g = m[j] > m_run[i + j] + 8.0f;  // also for the first tile (m_run = -inf)
+          const float m_use = g ? m[j] : m_run[i + j];
+          corr[i + j] = g ? ex2_approx(m_run[i + j] - m_use) : 1.0f;
+          m_run[i + j] = m_use;
+          grow |= g;
         }
       }
+      if (grow) {  // the same in every thread of the head half
+        if (kh == 0) {
+#pragma unroll
+          for (int i = 0; i < 16; i++)
+            if (lane == i) corr_s[t & 1][hg * 16 + i] = corr[i];
+        }
+#pragma unroll
+        for (int i = 0; i < 16; i++) l_run[i] *= corr[i];
+      } else if (kh == 0 && lane < 16) {
+        corr_s[t & 1][hg * 16 + lane] = 1.0f;
+      }
+      if (kh == 0 && lane == 0) grow_s[t & 1][hg] = grow;
+      asm volatile("bar.sync 2, 192;" ::: "memory");
+      if (t > 0 && (grow_s[t & 1][0] | grow_s[t & 1][1])) {
+        wait(&bar_o[(t - 1) & 1], (t - 1) >> 1, 24);  // the previous product must have finished writing O^T
+        __syncwarp();
+        tc_fence_after();
+        rescale(t, hg, 2);
+      }
+      if (t >= 2) wait(&bar_o[t & 1], (t - 2) >> 1, 25);  // this half of the weight buffer is free
+      uint32_t hi[8], lo[8];
+#pragma unroll
+      for (int i = 0; i < 8; i++) {
+        const float p0 = ex2_approx(v[2 * i] - m_run[2 * i]), p1 = ex2_approx(v[2 * i + 1] - m_run[2 * i + 1]);
+        l_run[2 * i] += p0;
+        l_run[2 * i + 1] += p1;
+        split_bf16x2(p0, p1, hi[i], lo[i]);
+      }
+      uint8_t* prow = smem + (sP - sK) + (t & 1) * P_BYTES + p_row;
+#pragma unroll
+      for (int c = 0; c < 2; c++) {
+        *(uint4*)(prow + (((hg * 2 + c) ^ (key & 7)) << 4)) = make_uint4(hi[4 * c], hi[4 * c + 1], hi[4 * c + 2], hi[4 * c + 3]);
+        *(uint4*)(prow + (((4 + hg * 2 + c) ^ (key & 7)) << 4)) = make_uint4(lo[4 * c], lo[4 * c + 1], lo[4 * c + 2], lo[4 * c + 3]);
+      }
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // the tensor cores read what these stores wrote
+      tc_fence_before();
+      asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(&bar_p)) : "memory");
     }
-  };
-  auto arrived = [&](int t) {  // tile t has landed (bounded)
-    if (!mbar_wait(smem_u32(&full[t & (NS - 1)]), (uint32_t)(t / NS) & 1)) bad = true;
-  };
-
-  if (ntiles > 0) {
-    arrived(0);
-    scores(0);
-    store_scores();
-    for (int t = 0; t <= ntiles; t++) {
-      if (t + 1 < ntiles) arrived(t + 1);
-      __syncthreads();  // S(t) and P(t-1) of every thread; everyone has left tile t - 2
-      if (threadIdx.x == 0 && t + 2 < ntiles) load_tile(t + 2, kb);
-      if (t < ntiles) fetch_scores();
-      if (t + 1 < ntiles) scores(t + 1);
-      __syncthreads();  // everyone has fetched S(t)
-      if (t + 1 < ntiles) store_scores();
-      if (t < ntiles) softmax(t);
-      if (t > 0) accumulate(t - 1);
+    // sums over the keys
+    const float l = transposed_reduce(l_run, lane, [](float x, float y) { return x + y; });
+    if (!(lane & 1)) mx_s[0][kh][hg * 16 + (lane >> 1)] = l;  // its last readers are behind a barrier of the loop, or it was never used
+    if (kh == 0) {
+#pragma unroll
+      for (int i = 0; i < 16; i++)
+        if (lane == i) ml_s[hg * 16 + i].x = m_run[i];
     }
   }
-#pragma unroll
-  for (int off = 1; off < TPR; off <<= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, off);
+  __syncwarp();
+  if (ntiles > 0) wait(&bar_o[(ntiles - 1) & 1], (ntiles - 1) >> 1, 26);  // every product is complete
+  __syncwarp();
+  tc_fence_after();
   __syncthreads();  // the ring is free: it holds this block's sums now
-  float* so = (float*)smem;  // [R][rank_p + 4]
+  float* so = (float*)smem;  // [32][rank_p + 4]
   const int so_ld = a.rank_p + 4;
-  if (skey == 0) ml_s[srow] = make_float2(m_run, l_run);
+  if (ntiles > 0) {
+    for (int mb = warp >> 2; mb < n_mb; mb += 2) {
+      const int lat = mb * 128 + (warp & 3) * 32 + lane;
+      const uint32_t base = tmem + 64u + (uint32_t)(mb * 64) + ((uint32_t)((warp & 3) * 32) << 16);
 #pragma unroll
-  for (int m = 0; m < MT; m++)
+      for (int c = 0; c < 2; c++) {
+        uint32_t x[16], y[16];
+        tc_ld16(base + (uint32_t)(c * 16), x);
+        tc_ld16(base + (uint32_t)(32 + c * 16), y);
+        tc_wait_ld();
+        if (lat < a.rank_p) {
 #pragma unroll
-    for (int j = 0; j < NV; j++) {
-      const int col = dim0 + j * 8 + 2 * tig;
-      if (col < a.rank_p) {
-        *(float2*)(so + (m * 16 + g) * so_ld + col) = make_float2(o[m][j][0], o[m][j][1]);
-        *(float2*)(so + (m * 16 + g + 8) * so_ld + col) = make_float2(o[m][j][2], o[m][j][3]);
+          for (int j = 0; j < 16; j++) so[(c * 16 + j) * so_ld + lat] = __uint_as_float(x[j]) + __uint_as_float(y[j]);
+        }
       }
     }
+  }
+  if (threadIdx.x < LHEADS) {
+    const float l = ntiles > 0 ? mx_s[0][0][threadIdx.x] + mx_s[0][1][threadIdx.x] : 0.f;
+    ml_s[threadIdx.x] = make_float2(ntiles > 0 ? ml_s[threadIdx.x].x : -INFINITY, l);
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 2) {
+    tc_fence_after();
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(tmem_cols) : "memory");
+  }
   cluster_sync();
-  if (threadIdx.x < R) {
+  if (threadIdx.x < LHEADS) {
     float2 ml[MAX_SPLITS];
     float M = -INFINITY, L = 0.f;
 #pragma unroll
@@ -673,23 +753,23 @@ __global__ void __launch_bounds__(NW * 32) latent_attn_decode_kernel(const __gri
       if (i < a.nsplit) fs[threadIdx.x][i] = ml[i].x * inv;
   }
   __syncthreads();
-  const int c4n = a.rank_p / 4, heads = min(R, a.H - h0);
+  const int c4n = a.rank_p / 4, heads = min(LHEADS, a.H - h0);
   const uint32_t so_a = smem_u32(so);
-  for (int i = split * NT + (int)threadIdx.x; i < heads * c4n; i += a.nsplit * NT) {
+  for (int i = split * 256 + (int)threadIdx.x; i < heads * c4n; i += a.nsplit * 256) {
     const int h = i / c4n, c = (i - h * c4n) * 4;
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f), x[MAX_SPLITS];
 #pragma unroll
     for (int p = 0; p < MAX_SPLITS; p++)
-      if (p < a.nsplit) x[p] = ld_cluster4(map_to_rank(so_a + (uint32_t)((h * so_ld + c) * 4), p));
+      if (p < a.nsplit && fs[h][p] != 0.f) x[p] = ld_cluster4(map_to_rank(so_a + (uint32_t)((h * so_ld + c) * 4), p));
 #pragma unroll
     for (int p = 0; p < MAX_SPLITS; p++)
-      if (p < a.nsplit && fs[h][p] != 0.f) {  // a block without keys holds zeros; its weight is zero
+      if (p < a.nsplit && fs[h][p] != 0.f) {  // a block without keys has weight zero
         const float w = fs[h][p];
         acc.x += w * x[p].x; acc.y += w * x[p].y; acc.z += w * x[p].z; acc.w += w * x[p].w;
       }
     *(uint2*)(a.out + ((int64_t)b * a.H + h0 + h) * a.rank_p + c) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
   }
-  if (bad && lane == 0) { *(volatile int*)a.status = 17; __threadfence_system(); }
+  if (err) { *(volatile int*)a.status = err; __threadfence_system(); }
   cluster_sync();  // nobody leaves while another block may still read its shared memory
   SB_TRACE_END(SB_K_ATTN, 0);
 }
@@ -848,8 +928,8 @@ constexpr size_t SMEM_MAX = 227 * 1024 - 1024;  // what a block may take, less t
 
 typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
                              const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-// 2D map of a layer's cache rows [rows, row], box = 32 rows x 64 columns (128 bytes), 128-byte swizzle.
-int cache_map(CUtensorMap* map, const bf16* base, int64_t rows, int row) {
+// 2D map of bf16 rows [rows, row], box = box_rows x 64 columns (128 bytes), 128-byte swizzle.
+int rows_map(CUtensorMap* map, const bf16* base, int64_t rows, int row, int box_rows) {
   static EncodeFn encode = nullptr;
   if (!encode) {
     void* fn = nullptr;
@@ -860,30 +940,11 @@ int cache_map(CUtensorMap* map, const bf16* base, int64_t rows, int row) {
   }
   cuuint64_t dims[2] = {(cuuint64_t)row, (cuuint64_t)rows};
   cuuint64_t strides[1] = {(cuuint64_t)row * 2};
-  cuuint32_t box[2] = {64u, (cuuint32_t)LKT};
+  cuuint32_t box[2] = {64u, (cuuint32_t)box_rows};
   cuuint32_t estr[2] = {1, 1};
   CUresult r = encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<bf16*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                       CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   if (r != CUDA_SUCCESS) return sb_fail(STRICTB200_ERR_CUDA, "cuTensorMapEncodeTiled failed with code " + std::to_string((int)r));
-  return STRICTB200_OK;
-}
-
-// The kernel's shapes: warps, reduction steps per slice, latent columns per warp. Rows of up to 192 (rank 128), 384 (rank 256)
-// and 640 (rank 512) elements.
-int decode_shape(const LatentShape& s) {
-  const int rp = s.rank_p(), row = s.row();
-  return rp <= 128 && row <= 192 ? 0 : rp <= 256 && row <= 384 ? 1 : 2;
-}
-int decode_warps(const LatentShape& s) { return decode_shape(s) == 0 ? 8 : 16; }
-
-template <int MT, int NW, int KSM, int NV>
-int launch_attn_decode(strictb200_ctx* ctx, const CUtensorMap& map, const AttnDecodeDev& a, int B) {
-  static size_t have[64] = {};
-  const size_t smem = attn_decode_smem(MT, NW, a.row);
-  SB_TRY(allow_smem(ctx, latent_attn_decode_kernel<MT, NW, KSM, NV>, smem, have));
-  SB_CUDA(sb_launch_cluster(ctx, latent_attn_decode_kernel<MT, NW, KSM, NV>, dim3(a.nsplit, (a.H + MT * 16 - 1) / (MT * 16), B), dim3(NW * 32), smem,
-                            dim3(a.nsplit, 1, 1), map, a));
-  ctx->launches++;
   return STRICTB200_OK;
 }
 
@@ -910,7 +971,7 @@ int k_latent_gather(strictb200_ctx* ctx, const bf16* cache, int64_t maxlen, int 
 }
 
 bool sb_latent_decode_fits(const LatentShape& s) {
-  return s.rank_p() <= 512 && s.row() <= 640 && s.dim <= 512 && decode_in_smem(s.dim) <= (int)SMEM_MAX;
+  return s.rank_p() <= 512 && s.row() <= 640 && s.dim <= 512 && decode_in_smem(s.dim) <= (int)SMEM_MAX;  // 512 latents fill the tensor memory
 }
 
 int k_latent_decode_in(strictb200_ctx* ctx, const LatentDecodeInArgs& x, int64_t B) {
@@ -927,20 +988,21 @@ int k_latent_decode_in(strictb200_ctx* ctx, const LatentDecodeInArgs& x, int64_t
   return STRICTB200_OK;
 }
 
+// Two blocks on an SM: half of the tensor memory each, and a ring of at least three stages in half of the shared memory.
+bool two_decode_blocks(const LatentShape& s) { return s.rank_p() <= 256 && attn_decode_smem(s.row(), 3) + 4096 <= 113 * 1024; }
+
 // Keys per block: waves of blocks x (key tiles per block + what a block costs besides), over the multiples of the tile that
 // leave at most MAX_SPLITS chunks of the window (or of the planned length, where that is shorter). The chunks of a (sequence,
 // head group) are one cluster, and clusters of 3, 5, 6 or 7 blocks pack the SMs of a GPC badly: 1, 2, 4 or 8 chunks.
 int sb_latent_decode_chunk(strictb200_ctx* ctx, const LatentShape& s, int B, int len_plan) {
   const int n = s.window > 0 ? std::min(s.window, len_plan) : len_plan, tiles = std::max(1, (n + LKT - 1) / LKT);
-  const int mt = s.H <= 16 ? 1 : 2;
-  const int per_sm = std::max<int>(1, std::min<int>(2, (int)(227 * 1024 / (attn_decode_smem(mt, decode_warps(s), s.row()) + 2048))));
-  const int64_t slots = (int64_t)ctx->sm_count * per_sm, pairs = (int64_t)B * ((s.H + mt * 16 - 1) / (mt * 16));
+  const int64_t slots = (int64_t)ctx->sm_count * (two_decode_blocks(s) ? 2 : 1), pairs = (int64_t)B * ((s.H + LHEADS - 1) / LHEADS);
   int best = tiles;
   double best_cost = 1e30;
   for (int k = 1; k <= MAX_SPLITS && k <= tiles; k *= 2) {
     const int c = (tiles + k - 1) / k;
     const int64_t blocks = pairs * k, waves = (blocks + slots - 1) / slots;
-    const double cost = (double)waves * (c + 4);
+    const double cost = (double)waves * (c + 3);
     if (cost < best_cost - 1e-9) { best_cost = cost; best = c; }
   }
   return best * LKT;
@@ -952,15 +1014,20 @@ int k_latent_attn_decode(strictb200_ctx* ctx, const LatentShape& s, const bf16* 
   if (!sb_latent_decode_fits(s)) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "latent decode attention: rows too wide for the tensor-core kernel");
   if (nsplit < 1 || nsplit > MAX_SPLITS || chunk < LKT || chunk % LKT || B > 65535) return sb_fail(STRICTB200_ERR_INVALID_ARG, "latent decode attention: bad key chunks");
   if ((int64_t)B * maxlen > INT32_MAX) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "latent decode attention: cache too large for 32-bit tile coordinates");
-  CUtensorMap map;
-  SB_TRY(cache_map(&map, cache, (int64_t)B * maxlen, s.row()));
-  AttnDecodeDev a{q_abs, lens, s.H, s.row(), s.rank_p(), maxlen, s.window, chunk, nsplit, s.scale * LOG2E, scratch, ctx->opt.attn_prefetch, ctx->d_status};
-  const int rp = s.rank_p(), shape = decode_shape(s);
-#define LATENT_DECODE(NW, KSM, NV) SB_TRY((s.H <= 16 ? launch_attn_decode<1, NW, KSM, NV>(ctx, map, a, B) : launch_attn_decode<2, NW, KSM, NV>(ctx, map, a, B)))
-  if (shape == 0) LATENT_DECODE(8, 3, 2);
-  else if (shape == 1) LATENT_DECODE(16, 3, 2);
-  else LATENT_DECODE(16, 5, 4);
-#undef LATENT_DECODE
+  const int rp = s.rank_p(), stages = decode_stages(s.row(), two_decode_blocks(s));
+  CUtensorMap map_k, map_q;
+  SB_TRY(rows_map(&map_k, cache, (int64_t)B * maxlen, s.row(), LKT));
+  SB_TRY(rows_map(&map_q, q_abs, (int64_t)B * s.H, s.row(), LHEADS));
+  AttnDecodeDev a{lens, s.H, s.row(), rp, maxlen, s.window, chunk, nsplit, stages, s.scale * LOG2E, scratch, ctx->opt.attn_prefetch, ctx->d_status};
+  {
+    static size_t have[64] = {};
+    // The blocks of a cluster wait for one another, so no block may wait for tensor memory that a waiting block holds: shared
+    // memory admits no more blocks to an SM than its tensor memory does (one with all 512 columns, or two with 256).
+    const size_t smem = std::max(attn_decode_smem(s.row(), stages), (size_t)(rp > 256 ? 116 : 78) * 1024);
+    SB_TRY(allow_smem(ctx, latent_attn_decode_kernel, smem, have));
+    SB_CUDA(sb_launch_cluster(ctx, latent_attn_decode_kernel, dim3(nsplit, (s.H + LHEADS - 1) / LHEADS, B), dim3(256), smem, dim3(nsplit, 1, 1), map_k, map_q, a));
+    ctx->launches++;
+  }
   sb_prof_split(ctx, STRICTB200_K_ATTN_MERGE);
   static size_t have[64] = {};
   const size_t smem = (size_t)(64 + 16) * (rp + 8) * 2;
