@@ -59,10 +59,22 @@ __device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity) {
   }
   return false;
 }
-__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar, uint64_t policy) {
-  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes.L2::cache_hint [%0], [%1, {%2, %3}], [%4], %5;" ::"r"(dst),
-               "l"(map), "r"(x), "r"(y), "r"(bar), "l"(policy)
-               : "memory");
+// by one lane of a warp that runs converged (see tc_mma_warp)
+__device__ __forceinline__ void tma_load_2d_warp(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar, uint64_t policy) {
+  asm volatile(
+      "{\n\t.reg .pred e;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\t"
+      "@e cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes.L2::cache_hint [%0], [%1, {%2, %3}], [%4], %5;\n\t}" ::"r"(dst),
+      "l"(map), "r"(x), "r"(y), "r"(bar), "l"(policy)
+      : "memory");
+}
+__device__ __forceinline__ void mbar_expect_tx_warp(uint32_t bar, uint32_t bytes) {
+  asm volatile(
+      "{\n\t.reg .pred e;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\t"
+      "@e mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n\t}" ::"r"(bar),
+      "r"(bytes)
+      : "memory");
 }
 // the address of this block's shared-memory location in block `rank` of the cluster
 __device__ __forceinline__ uint32_t map_to_rank(uint32_t local, uint32_t rank) {
@@ -73,11 +85,6 @@ __device__ __forceinline__ uint32_t map_to_rank(uint32_t local, uint32_t rank) {
 __device__ __forceinline__ float2 ld_cluster2(uint32_t addr) {
   float2 v;
   asm volatile("ld.shared::cluster.v2.f32 {%0,%1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(addr) : "memory");
-  return v;
-}
-__device__ __forceinline__ float4 ld_cluster4(uint32_t addr) {
-  float4 v;
-  asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr) : "memory");
   return v;
 }
 __device__ __forceinline__ void cluster_sync() {
@@ -394,8 +401,9 @@ __global__ void __launch_bounds__(256) latent_decode_in_kernel(DecodeInDev d, in
 // 6, 7 help to rescale O^T (their lanes are out of the softmax warps' reach). S^T is double-buffered, so S^T(t+1) runs under
 // the softmax of tile t. A head's running maximum is followed lazily (only when it grew by more than 2^8, as in the prompt's
 // kernel), so O^T is hardly ever rescaled.
-// Key tiles are TMA atoms of 64 rows x 64 columns (128-byte swizzle) in a ring of NS stages. At the end the cluster's blocks
-// weigh each other's sums through distributed shared memory; what leaves is one bf16 row of latents per head.
+// Key tiles are TMA atoms of 64 columns (128-byte swizzle) in a ring; an atom group's part of S^T is issued as soon as it has
+// arrived. At the end every block of the cluster gets the others' sums of its share of the heads (bulk copies between the
+// blocks' shared memories) and weighs them; what leaves is one bf16 row of latents per head.
 // Every mbarrier wait is bounded: on expiry the error word is set and the block runs to its end.
 constexpr int LKT = 64, LHEADS = 32;
 constexpr int MAX_SPLITS = 8;               // blocks of a cluster
@@ -410,7 +418,7 @@ struct AttnDecodeDev {
   int prefetch;
   int* status;
 };
-constexpr int MAX_STAGES = 4;
+constexpr int MAX_STAGES = 4, GROUPS = 3;   // a tile's atoms arrive in up to three groups, each with a barrier of its own
 inline int decode_atoms(int row) { return (row + 63) / 64; }
 inline size_t attn_decode_smem(int row, int stages) {
   return 1024 /* round-up to the swizzle's alignment */ + (size_t)stages * decode_atoms(row) * ATOM + (size_t)decode_atoms(row) * Q_ATOM + 2 * P_BYTES;
@@ -424,14 +432,21 @@ inline int decode_stages(int row, bool two_blocks) {
 
 __device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
 __device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_commit(uint32_t bar) {
-  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ void tc_mma(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+// Issued by one lane of a warp that runs converged: its operands are then the same in all lanes and stay in uniform registers
+// (inside a one-lane branch every operand of every product is moved there first, which takes longer than a 128 x 32 product).
+__device__ __forceinline__ void tc_commit_warp(uint32_t bar) {
   asm volatile(
-      "{\n\t.reg .pred p;\n\t"
+      "{\n\t.reg .pred e;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\t"
+      "@e tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}" ::"r"(bar)
+      : "memory");
+}
+__device__ __forceinline__ void tc_mma_warp(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, e;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\t"
       "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
       :
       : "r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(0u)
       : "memory");
@@ -488,7 +503,7 @@ __device__ __forceinline__ float transposed_reduce(const float* v, int lane, Op 
 __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_q, AttnDecodeDev a) {
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024 - (smem_u32(smem_raw) & 1023)) & 1023);
-  __shared__ __align__(8) uint64_t k_full[MAX_STAGES], k_empty[MAX_STAGES], q_full, bar_s[2], bar_p, bar_o[2];
+  __shared__ __align__(8) uint64_t k_full[MAX_STAGES][GROUPS], k_empty[MAX_STAGES], q_full, bar_s[2], bar_p, bar_o[2], bar_m;
   __shared__ uint32_t tmem_slot;
   __shared__ int grow_s[2][2];                                    // [tile parity][head half]: some maximum has to be followed
   __shared__ __align__(16) float corr_s[2][LHEADS], mx_s[2][2][LHEADS];  // [tile parity], [tile parity][key half]
@@ -497,12 +512,16 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
   SB_TRACE_BEGIN();
   const int split = blockIdx.x, h0 = blockIdx.y * LHEADS, b = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n_atoms = (a.row + 63) / 64, stage_bytes = n_atoms * ATOM, n_mb = (a.rank_p + 127) / 128;
+  const int n_atoms = (a.row + 63) / 64, stage_bytes = n_atoms * ATOM, n_mb = (a.rank_p + 127) / 128, per_group = (n_atoms + GROUPS - 1) / GROUPS;
   const uint32_t sK = smem_u32(smem), sQ = sK + (uint32_t)(a.stages * stage_bytes), sP = sQ + (uint32_t)(n_atoms * Q_ATOM);
   const uint32_t tmem_cols = n_mb <= 2 ? 256u : 512u;  // two S^T tiles of 32 columns, then 64 columns per block of latents
   if (threadIdx.x == 0) {
-    for (int i = 0; i < a.stages; i++) { mbar_init(smem_u32(&k_full[i]), 1); mbar_init(smem_u32(&k_empty[i]), 1); }
+    for (int i = 0; i < a.stages; i++) {
+      for (int g = 0; g < GROUPS; g++) mbar_init(smem_u32(&k_full[i][g]), 1);
+      mbar_init(smem_u32(&k_empty[i]), 1);
+    }
     mbar_init(smem_u32(&q_full), 1);
+    mbar_init(smem_u32(&bar_m), 1);
     mbar_init(smem_u32(&bar_p), 192);
     for (int i = 0; i < 2; i++) { mbar_init(smem_u32(&bar_s[i]), 1); mbar_init(smem_u32(&bar_o[i]), 1); }
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -525,11 +544,20 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
     ke = min(len, kb + a.chunk);
   };
   const uint64_t policy = l2_evict_first_policy();
-  // One thread. Rows beyond the chunk are whatever the cache holds there (finite, or zeros beyond its end); their weights are zero.
-  auto load_tile = [&](int t, int kb) {
-    const int st = t % a.stages;
-    mbar_expect_tx(smem_u32(&k_full[st]), (uint32_t)stage_bytes);
-    for (int i = 0; i < n_atoms; i++) tma_load_2d(sK + (uint32_t)(st * stage_bytes + i * ATOM), &map_k, i * 64, b * a.maxlen + kb + t * LKT, smem_u32(&k_full[st]), policy);
+  uint64_t policy_q;  // the queries stay: the other blocks of the cluster read them too
+  asm volatile("createpolicy.fractional.L2::evict_last.b64 %0, 1.0;" : "=l"(policy_q));
+  // The producer warp. Rows beyond the chunk are whatever the cache holds there (finite, or zeros beyond its end); their
+  // weights are zero.
+  auto load_tile = [&](int st, int row) {
+#pragma unroll
+    for (int g = 0; g < GROUPS; g++) {
+      const int first = g * per_group, n = min(per_group, n_atoms - first);
+      if (n <= 0) break;
+      const uint32_t bar = smem_u32(&k_full[st][g]);
+      mbar_expect_tx_warp(bar, (uint32_t)(n * ATOM));
+#pragma unroll 1
+      for (int i = first; i < first + n; i++) tma_load_2d_warp(sK + (uint32_t)(st * stage_bytes + i * ATOM), &map_k, i * 64, row, bar, policy);
+    }
   };
   // Tiles that hold rows of earlier steps only are requested before the dependency wait; the length they are derived from is
   // read again after it. (It belongs to the previous step and has not changed; if it had, the step would report an error.)
@@ -538,7 +566,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
   range(len_early, kb, ke);
   if (a.prefetch)
     for (; n_early < a.stages && kb + (n_early + 1) * LKT <= min(ke, len_early - 1); n_early++)
-      if (threadIdx.x == 96) load_tile(n_early, kb);
+      if (warp == 3) load_tile(n_early, b * a.maxlen + kb + n_early * LKT);
   pdl_wait();
   SB_TRACE_WAITED();
   const int len = min(ld_volatile_i32(a.lens + b) + 1, a.maxlen);
@@ -566,46 +594,85 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
   };
 
   if (warp == 3) {
-    // ---- TMA producer
-    if (lane == 0 && ntiles > 0) {
-      mbar_expect_tx(smem_u32(&q_full), (uint32_t)(n_atoms * Q_ATOM));
-      for (int i = 0; i < n_atoms; i++)
-        asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(sQ + (uint32_t)(i * Q_ATOM)), "l"(&map_q),
-                     "r"(i * 64), "r"(b * a.H + h0), "r"(smem_u32(&q_full))
-                     : "memory");
+    // ---- TMA producer, the whole warp in step
+    if (ntiles > 0) {
+      mbar_expect_tx_warp(smem_u32(&q_full), (uint32_t)(n_atoms * Q_ATOM));
+#pragma unroll 1
+      for (int i = 0; i < n_atoms; i++) tma_load_2d_warp(sQ + (uint32_t)(i * Q_ATOM), &map_q, i * 64, b * a.H + h0, smem_u32(&q_full), policy_q);
+      int st = n_early == a.stages ? 0 : n_early, free_parity = 1;  // the first pass over the ring needs no waiting
       for (int t = n_early; t < ntiles; t++) {
-        if (t >= a.stages && !wait(&k_empty[t % a.stages], (t / a.stages) + 1, 18)) break;
-        load_tile(t, kb);
+        if (st == 0 && t > 0) free_parity ^= 1;
+        if (t >= a.stages && !__all_sync(0xffffffffu, wait(&k_empty[st], free_parity, 18))) break;
+        load_tile(st, b * a.maxlen + kb + t * LKT);
+        if (++st == a.stages) st = 0;
       }
     }
   } else if (warp == 2) {
-    // ---- MMA issue: S(0), then per tile S(t+1) and PV(t)
-    if (lane == 0 && ntiles > 0) {
-      // D = F32, A = B = BF16, M = 128; N = 32 heads, or N = 64 with both operands MN-major
-      constexpr uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(LHEADS >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-      constexpr uint32_t idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | (1u << 16) | ((uint32_t)(64 >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-      const int nks = (a.row + 15) / 16;
-      auto issue_s = [&](int t) {
-        if (!wait(&k_full[t % a.stages], t / a.stages, 19)) return;
+    // ---- MMA issue, the whole warp in step: O^T of the current tile when its weights are there, else S^T of the
+    // next one as far as its atoms have arrived
+    // D = F32, A = B = BF16, M = 128; N = 32 heads, or N = 64 with both operands MN-major
+    constexpr uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(LHEADS >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+    constexpr uint32_t idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | (1u << 16) | ((uint32_t)(64 >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+    // an operand advances by constants: 16 columns = 32 bytes, an atom = ATOM bytes, 16 keys = 2048 bytes (units of 16 bytes)
+    const uint64_t dk0 = desc_kmajor(sK), dq0 = desc_kmajor(sQ), dc0 = desc_mnmajor(sK), dp0 = desc_mnmajor(sP);
+    const uint32_t td = __shfl_sync(0xffffffffu, tmem, 0);
+    const int stage16 = stage_bytes >> 4;
+    int st = 0, ps = 0;  // ring stages of the next S^T and the next O^T product,
+    int sp = 0, pr = 0;  // the parities of their barriers,
+    int sg = 0;          // and the group of atoms the next S^T continues with
+    int ns = 0, np = 0;  // tiles whose S^T / O^T product has been issued
+    auto ready = [&](uint64_t* bar, int parity) {
+      uint32_t done;
+      asm volatile(
+          "{\n\t.reg .pred p;\n\t"
+          "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+          "selp.u32 %0, 1, 0, p;\n\t}"
+          : "=r"(done)
+          : "r"(smem_u32(bar)), "r"((uint32_t)parity)
+          : "memory");
+      return __all_sync(0xffffffffu, done);
+    };
+    if (ntiles > 0) wait(&q_full, 0, 20);
+    bool go = __all_sync(0xffffffffu, err == 0);
+    uint32_t spins = 0;
+    while (np < ntiles && go) {
+      if (ns > np && ready(&bar_p, pr)) {  // the weights are in shared memory, O^T follows the new maxima
         tc_fence_after();
-        const uint32_t tile = sK + (uint32_t)((t % a.stages) * stage_bytes);
-        for (int s = 0; s < nks; s++)
-          tc_mma(tmem + (uint32_t)((t & 1) * LHEADS), desc_kmajor(tile + (uint32_t)((s >> 2) * ATOM + (s & 3) * 32)), desc_kmajor(sQ + (uint32_t)((s >> 2) * Q_ATOM + (s & 3) * 32)),
-                 idesc_s, s ? 1u : 0u);
-        tc_commit(smem_u32(&bar_s[t & 1]));
-      };
-      if (wait(&q_full, 0, 20)) issue_s(0);
-      for (int t = 0; t < ntiles && !err; t++) {
-        if (t + 1 < ntiles) issue_s(t + 1);
-        if (!wait(&bar_p, t, 21)) break;  // the weights are in shared memory, O^T follows the new maxima
-        tc_fence_after();
-        const uint32_t tile = sK + (uint32_t)((t % a.stages) * stage_bytes), p = sP + (uint32_t)((t & 1) * P_BYTES);
-        for (int mb = 0; mb < n_mb; mb++)
+        const uint64_t dc = dc0 + (uint64_t)(uint32_t)(ps * stage16), dp = dp0 + (uint64_t)(uint32_t)((np & 1) * (P_BYTES >> 4));
 #pragma unroll
-          for (int s = 0; s < LKT / 16; s++)  // 16 keys = 16 rows of 128 bytes
-            tc_mma(tmem + 64u + (uint32_t)(mb * 64), desc_mnmajor(tile + (uint32_t)(2 * mb * ATOM + s * 2048)), desc_mnmajor(p + (uint32_t)(s * 2048)), idesc_pv, (t | s) ? 1u : 0u);
-        tc_commit(smem_u32(&bar_o[t & 1]));
-        tc_commit(smem_u32(&k_empty[t % a.stages]));
+        for (int s = 0; s < LKT / 16; s++)  // 16 keys = 16 rows of 128 bytes; the blocks of latents take turns
+#pragma unroll
+          for (int mb = 0; mb < 4; mb++)
+            if (mb < n_mb) tc_mma_warp(td + 64u + (uint32_t)(mb * 64), dc + (uint64_t)((2 * mb * ATOM + s * 2048) >> 4), dp + (uint64_t)(s * 2048 >> 4), idesc_pv, (np | s) ? 1u : 0u);
+        tc_commit_warp(smem_u32(&bar_o[np & 1]));
+        tc_commit_warp(smem_u32(&k_empty[ps]));
+        np++;
+        pr ^= 1;
+        if (++ps == a.stages) ps = 0;
+        spins = 0;
+      } else if (ns < ntiles && ns <= np + 1 && ready(&k_full[st][sg], sp)) {
+        tc_fence_after();
+        const int first = sg * per_group, last = min(n_atoms, first + per_group);
+        const uint32_t d = td + (uint32_t)((ns & 1) * LHEADS);
+#pragma unroll 1
+        for (int i = first; i < last; i++) {  // a row's last atom is zero beyond its width
+          const uint64_t dk = dk0 + (uint64_t)(uint32_t)(st * stage16 + i * (ATOM >> 4)), dq = dq0 + (uint64_t)(uint32_t)(i * (Q_ATOM >> 4));
+          tc_mma_warp(d, dk, dq, idesc_s, i ? 1u : 0u);
+          tc_mma_warp(d, dk + 2, dq + 2, idesc_s, 1u);
+          tc_mma_warp(d, dk + 4, dq + 4, idesc_s, 1u);
+          tc_mma_warp(d, dk + 6, dq + 6, idesc_s, 1u);
+        }
+        sg++;
+        if (last == n_atoms) {
+          tc_commit_warp(smem_u32(&bar_s[ns & 1]));
+          ns++;
+          sg = 0;
+          if (++st == a.stages) { st = 0; sp ^= 1; }
+        }
+        spins = 0;
+      } else if (++spins > (1u << 24)) {
+        err = 21;
+        go = false;
       }
     }
   } else if (warp >= 6) {
@@ -634,7 +701,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
       uint32_t r[16];
       tc_ld16(tmem + (uint32_t)((t & 1) * LHEADS + hg * 16) + ((uint32_t)(kh * 32) << 16), r);
       tc_wait_ld();
-      const bool live = kb + t * LKT + key < ke;
+      const bool live = key < LKT && kb + t * LKT + key < ke;
       float v[16];
 #pragma unroll
       for (int i = 0; i < 16; i++) v[i] = live ? __uint_as_float(r[i]) * a.scale_log2 : -INFINITY;
@@ -685,6 +752,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
         split_bf16x2(p0, p1, hi[i], lo[i]);
       }
       uint8_t* prow = smem + (sP - sK) + (t & 1) * P_BYTES + p_row;
+      if (LKT == 64 || key < LKT)
 #pragma unroll
       for (int c = 0; c < 2; c++) {
         *(uint4*)(prow + (((hg * 2 + c) ^ (key & 7)) << 4)) = make_uint4(hi[4 * c], hi[4 * c + 1], hi[4 * c + 2], hi[4 * c + 3]);
@@ -731,43 +799,56 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
     const float l = ntiles > 0 ? mx_s[0][0][threadIdx.x] + mx_s[0][1][threadIdx.x] : 0.f;
     ml_s[threadIdx.x] = make_float2(ntiles > 0 ? ml_s[threadIdx.x].x : -INFINITY, l);
   }
+  asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // the copies below read what the stores above wrote
   tc_fence_before();
   __syncthreads();
   if (warp == 2) {
     tc_fence_after();
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(tmem_cols) : "memory");
   }
-  cluster_sync();
-  if (threadIdx.x < LHEADS) {
-    float2 ml[MAX_SPLITS];
-    float M = -INFINITY, L = 0.f;
+  // Every block owns some of the heads: the others' rows of those heads come as one bulk copy each, [source][own head][rank_p + 4].
+  const int own = (LHEADS + a.nsplit - 1) / a.nsplit, first = split * own, n_own = max(0, min(own, LHEADS - first));
+  const uint32_t slot_bytes = (uint32_t)(own * so_ld * 4);
+  uint8_t* recv = smem + LHEADS * so_ld * 4;
+  if (threadIdx.x == 0 && a.nsplit > 1) mbar_expect_tx(smem_u32(&bar_m), (uint32_t)((a.nsplit - 1) * n_own * so_ld * 4));
+  cluster_sync();  // every block's sums are complete and every ring is free
+  if (threadIdx.x < a.nsplit && (int)threadIdx.x != split) {
+    const int to = threadIdx.x, n = max(0, min(own, LHEADS - to * own));
+    if (n > 0)
+      asm volatile("cp.async.bulk.shared::cluster.shared::cta.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(map_to_rank(smem_u32(recv) + (uint32_t)split * slot_bytes, to)),
+                   "r"(smem_u32(so + to * own * so_ld)), "r"((uint32_t)(n * so_ld * 4)), "r"(map_to_rank(smem_u32(&bar_m), to))
+                   : "memory");
+  }
+  {  // weights of the chunks: eight neighbouring threads per head, one per chunk
+    const int h = threadIdx.x >> 3, p = threadIdx.x & 7;
+    float2 ml = make_float2(-INFINITY, 0.f);
+    if (h < n_own && p < a.nsplit) ml = ld_cluster2(map_to_rank(smem_u32(&ml_s[first + h]), p));
+    float M = ml.x;
 #pragma unroll
-    for (int i = 0; i < MAX_SPLITS; i++)
-      if (i < a.nsplit) { ml[i] = ld_cluster2(map_to_rank(smem_u32(&ml_s[threadIdx.x]), i)); M = fmaxf(M, ml[i].x); }
+    for (int off = 1; off < 8; off <<= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, off));
+    const float f = ml.y > 0.f ? ex2_approx(ml.x - M) : 0.f;
+    float L = f * ml.y;
 #pragma unroll
-    for (int i = 0; i < MAX_SPLITS; i++)
-      if (i < a.nsplit) { ml[i].x = ml[i].y > 0.f ? exp2f(ml[i].x - M) : 0.f; L += ml[i].x * ml[i].y; }
-    const float inv = 1.0f / L;
-#pragma unroll
-    for (int i = 0; i < MAX_SPLITS; i++)
-      if (i < a.nsplit) fs[threadIdx.x][i] = ml[i].x * inv;
+    for (int off = 1; off < 8; off <<= 1) L += __shfl_xor_sync(0xffffffffu, L, off);
+    fs[h][p] = f > 0.f ? f / L : 0.f;
   }
   __syncthreads();
-  const int c4n = a.rank_p / 4, heads = min(LHEADS, a.H - h0);
-  const uint32_t so_a = smem_u32(so);
-  for (int i = split * 256 + (int)threadIdx.x; i < heads * c4n; i += a.nsplit * 256) {
+  if (a.nsplit > 1) wait(&bar_m, 0, 27);
+  const int c4n = a.rank_p / 4, heads = min(n_own, a.H - h0 - first);
+  for (int i = threadIdx.x; i < heads * c4n; i += 256) {
     const int h = i / c4n, c = (i - h * c4n) * 4;
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f), x[MAX_SPLITS];
-#pragma unroll
-    for (int p = 0; p < MAX_SPLITS; p++)
-      if (p < a.nsplit && fs[h][p] != 0.f) x[p] = ld_cluster4(map_to_rank(so_a + (uint32_t)((h * so_ld + c) * 4), p));
-#pragma unroll
-    for (int p = 0; p < MAX_SPLITS; p++)
-      if (p < a.nsplit && fs[h][p] != 0.f) {  // a block without keys has weight zero
-        const float w = fs[h][p];
-        acc.x += w * x[p].x; acc.y += w * x[p].y; acc.z += w * x[p].z; acc.w += w * x[p].w;
+    const float* mine = so + (first + h) * so_ld + c;
+    const float* theirs = (const float*)recv + h * so_ld + c;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 1
+    for (int p = 0; p < a.nsplit; p++, theirs += own * so_ld) {
+      const float w = fs[h][p];
+      if (w != 0.f) {  // a block without keys has weight zero
+        const float4 x = *(const float4*)(p == split ? mine : theirs);
+        acc.x += w * x.x; acc.y += w * x.y; acc.z += w * x.z; acc.w += w * x.w;
       }
-    *(uint2*)(a.out + ((int64_t)b * a.H + h0 + h) * a.rank_p + c) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
+    }
+    *(uint2*)(a.out + ((int64_t)b * a.H + h0 + first + h) * a.rank_p + c) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
   }
   if (err) { *(volatile int*)a.status = err; __threadfence_system(); }
   cluster_sync();  // nobody leaves while another block may still read its shared memory
