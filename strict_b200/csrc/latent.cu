@@ -393,19 +393,18 @@ __global__ void __launch_bounds__(256) latent_decode_in_kernel(DecodeInDev d, in
 // grid (nsplit, ceil(H / 32), B), 256 threads; the nsplit blocks of a (sequence, head group) are one cluster. The work is two
 // products per tile of 64 keys on the tcgen05 tensor cores, with the long dimension of each as the tensor-memory lanes:
 //   S^T = K Q^T      A = the key tile [64 keys x row] (K-major), B = the queries [32 heads x row] (K-major, staged once);
-//                    lane = key, column = head. M is 128: lanes 64.. read past the tile and are ignored.
+//                    key 16 q + r = lane r of quarter q of tensor memory (M = 64), column = head.
 //   O^T += c^T P     A = the same tile read MN-major, [128 latents x 64 keys] per block of 128 latents, B = the weights
 //                    [64 keys x 64], MN-major: columns 0..31 the heads' hi terms, 32..63 their lo terms (P = hi + lo);
 //                    lane = latent, column = head; the two halves are added at the end
-// Roles by warp: 0, 1, 4, 5 softmax (warp & 1 = which 32 keys, warp >> 2 = which 16 heads), 2 MMA issue, 3 TMA producer,
-// 6, 7 help to rescale O^T (their lanes are out of the softmax warps' reach). S^T is double-buffered, so S^T(t+1) runs under
-// the softmax of tile t. A head's running maximum is followed lazily (only when it grew by more than 2^8, as in the prompt's
-// kernel), so O^T is hardly ever rescaled.
+// Roles by warp: 0..3 softmax (16 keys each, all heads), 4 MMA issue, 5 TMA producer. S^T is double-buffered, so S^T(t+1)
+// runs under the softmax of tile t. A head's running maximum is followed lazily (only when it grew by more than 2^8, as in the
+// prompt's kernel), so O^T is hardly ever rescaled.
 // Key tiles are TMA atoms of 64 columns (128-byte swizzle) in a ring; an atom group's part of S^T is issued as soon as it has
 // arrived. At the end every block of the cluster gets the others' sums of its share of the heads (bulk copies between the
 // blocks' shared memories) and weighs them; what leaves is one bf16 row of latents per head.
 // Every mbarrier wait is bounded: on expiry the error word is set and the block runs to its end.
-constexpr int LKT = 64, LHEADS = 32;
+constexpr int LKT = 64, LHEADS = 32;         // keys per tile (M of the first product), heads per block
 constexpr int MAX_SPLITS = 8;               // blocks of a cluster
 constexpr int ATOM = LKT * 128;             // bytes of a key tile's 64-column atom
 constexpr int Q_ATOM = LHEADS * 128;        // ... and of the queries'
@@ -458,6 +457,14 @@ __device__ __forceinline__ void tc_ld16(uint32_t taddr, uint32_t* r) {
         "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
       : "r"(taddr));
 }
+// 16 lanes x 32 columns as four 16 x 8 tiles, each laid out like an mma.sync accumulator (rows lane / 4 and + 8, two columns)
+__device__ __forceinline__ void tc_ld_16x256(uint32_t taddr, uint32_t* r) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.16x256b.x4.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]),
+        "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+      : "r"(taddr));
+}
 __device__ __forceinline__ void tc_st16(uint32_t taddr, const uint32_t* r) {
   asm volatile(
       "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]),
@@ -475,29 +482,23 @@ __device__ __forceinline__ uint64_t desc_kmajor(uint32_t addr) {
 __device__ __forceinline__ uint64_t desc_mnmajor(uint32_t addr) {
   return (uint64_t)((addr >> 4) & 0x3FFF) | ((uint64_t)(ATOM >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
 }
-// Reduction of 16 values per lane over the 32 lanes of a warp, op = max or sum: afterwards lanes 2i and 2i + 1 hold the result
-// of value i. Every exchange halves the values a lane still carries.
+// Reduction of 8 values per lane over the 8 lanes of the same lane % 4, op = max or sum: afterwards lane 4 g + i holds the
+// result of value g. Every exchange halves the values a lane still carries.
 template <typename Op>
 __device__ __forceinline__ float transposed_reduce(const float* v, int lane, Op op) {
-  float a[8], b[4], c[2];
+  float a[4], b[2];
 #pragma unroll
-  for (int i = 0; i < 8; i++) {
-    const float keep = lane & 16 ? v[8 + i] : v[i], send = lane & 16 ? v[i] : v[8 + i];
+  for (int i = 0; i < 4; i++) {
+    const float keep = lane & 16 ? v[4 + i] : v[i], send = lane & 16 ? v[i] : v[4 + i];
     a[i] = op(keep, __shfl_xor_sync(0xffffffffu, send, 16));
   }
 #pragma unroll
-  for (int i = 0; i < 4; i++) {
-    const float keep = lane & 8 ? a[4 + i] : a[i], send = lane & 8 ? a[i] : a[4 + i];
+  for (int i = 0; i < 2; i++) {
+    const float keep = lane & 8 ? a[2 + i] : a[i], send = lane & 8 ? a[i] : a[2 + i];
     b[i] = op(keep, __shfl_xor_sync(0xffffffffu, send, 8));
   }
-#pragma unroll
-  for (int i = 0; i < 2; i++) {
-    const float keep = lane & 4 ? b[2 + i] : b[i], send = lane & 4 ? b[i] : b[2 + i];
-    c[i] = op(keep, __shfl_xor_sync(0xffffffffu, send, 4));
-  }
-  const float keep = lane & 2 ? c[1] : c[0], send = lane & 2 ? c[0] : c[1];
-  const float d = op(keep, __shfl_xor_sync(0xffffffffu, send, 2));
-  return op(d, __shfl_xor_sync(0xffffffffu, d, 1));
+  const float keep = lane & 4 ? b[1] : b[0], send = lane & 4 ? b[0] : b[1];
+  return op(keep, __shfl_xor_sync(0xffffffffu, send, 4));
 }
 
 __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_q, AttnDecodeDev a) {
@@ -505,8 +506,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
   uint8_t* smem = smem_raw + ((1024 - (smem_u32(smem_raw) & 1023)) & 1023);
   __shared__ __align__(8) uint64_t k_full[MAX_STAGES][GROUPS], k_empty[MAX_STAGES], q_full, bar_s[2], bar_p, bar_o[2], bar_m;
   __shared__ uint32_t tmem_slot;
-  __shared__ int grow_s[2][2];                                    // [tile parity][head half]: some maximum has to be followed
-  __shared__ __align__(16) float corr_s[2][LHEADS], mx_s[2][2][LHEADS];  // [tile parity], [tile parity][key half]
+  __shared__ float corr_s[4][LHEADS], mx_s[2][4][LHEADS];  // [softmax warp], [tile parity][softmax warp]
   __shared__ float2 ml_s[LHEADS];
   __shared__ float fs[LHEADS][MAX_SPLITS];
   SB_TRACE_BEGIN();
@@ -522,11 +522,11 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
     }
     mbar_init(smem_u32(&q_full), 1);
     mbar_init(smem_u32(&bar_m), 1);
-    mbar_init(smem_u32(&bar_p), 192);
+    mbar_init(smem_u32(&bar_p), 128);
     for (int i = 0; i < 2; i++) { mbar_init(smem_u32(&bar_s[i]), 1); mbar_init(smem_u32(&bar_o[i]), 1); }
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
-  if (warp == 2) {
+  if (warp == 4) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(tmem_cols) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
@@ -566,7 +566,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
   range(len_early, kb, ke);
   if (a.prefetch)
     for (; n_early < a.stages && kb + (n_early + 1) * LKT <= min(ke, len_early - 1); n_early++)
-      if (warp == 3) load_tile(n_early, b * a.maxlen + kb + n_early * LKT);
+      if (warp == 5) load_tile(n_early, b * a.maxlen + kb + n_early * LKT);
   pdl_wait();
   SB_TRACE_WAITED();
   const int len = min(ld_volatile_i32(a.lens + b) + 1, a.maxlen);
@@ -578,22 +578,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
     if (!err && !mbar_wait(smem_u32(bar), (uint32_t)parity & 1)) err = code;
     return err == 0;
   };
-  // O^T columns of this warp's lanes times the heads' corrections; part of parts: which share of the columns
-  auto rescale = [&](int t, int part, int parts) {
-    const float* cs = corr_s[t & 1];
-    const uint32_t base = tmem + 64u + ((uint32_t)((warp & 3) * 32) << 16);
-    for (int c = part; c < n_mb * 4; c += parts) {
-      uint32_t r[16];
-      tc_ld16(base + (uint32_t)(c * 16), r);
-      tc_wait_ld();
-#pragma unroll
-      for (int j = 0; j < 16; j++) r[j] = __float_as_uint(__uint_as_float(r[j]) * cs[(c & 1) * 16 + j]);
-      tc_st16(base + (uint32_t)(c * 16), r);
-    }
-    tc_wait_st();
-  };
-
-  if (warp == 3) {
+  if (warp == 5) {
     // ---- TMA producer, the whole warp in step
     if (ntiles > 0) {
       mbar_expect_tx_warp(smem_u32(&q_full), (uint32_t)(n_atoms * Q_ATOM));
@@ -607,11 +592,11 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
         if (++st == a.stages) st = 0;
       }
     }
-  } else if (warp == 2) {
+  } else if (warp == 4) {
     // ---- MMA issue, the whole warp in step: O^T of the current tile when its weights are there, else S^T of the
     // next one as far as its atoms have arrived
-    // D = F32, A = B = BF16, M = 128; N = 32 heads, or N = 64 with both operands MN-major
-    constexpr uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(LHEADS >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+    // D = F32, A = B = BF16; M = 64 keys, N = 32 heads, or M = 128 latents, N = 64 with both operands MN-major
+    constexpr uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(LHEADS >> 3) << 17) | ((uint32_t)(LKT >> 4) << 24);
     constexpr uint32_t idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | (1u << 16) | ((uint32_t)(64 >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
     // an operand advances by constants: 16 columns = 32 bytes, an atom = ATOM bytes, 16 keys = 2048 bytes (units of 16 bytes)
     const uint64_t dk0 = desc_kmajor(sK), dq0 = desc_kmajor(sQ), dc0 = desc_mnmajor(sK), dp0 = desc_mnmajor(sP);
@@ -675,101 +660,82 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
         go = false;
       }
     }
-  } else if (warp >= 6) {
-    for (int t = 0; t < ntiles; t++) {
-      asm volatile("bar.sync 2, 192;" ::: "memory");
-      if (t > 0 && (grow_s[t & 1][0] | grow_s[t & 1][1])) {
-        wait(&bar_o[(t - 1) & 1], (t - 1) >> 1, 22);
-        __syncwarp();
-        tc_fence_after();
-        rescale(t, 0, 1);
-        tc_fence_before();
-      }
-      asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(&bar_p)) : "memory");
-    }
-  } else {
-    // ---- softmax: thread = key, 16 heads
-    const int kh = warp & 1, hg = warp >> 2, key = kh * 32 + lane;
-    float m_run[16], l_run[16];
+  } else if (warp < 4) {
+    // ---- softmax. A thread has two keys (rows g and g + 8 of its warp's 16) of eight heads (columns 8 j + 2 tig, + 1); lane L
+    // also keeps head L's running maximum, the same in all four warps.
+    const int g = lane >> 2, tig = lane & 3, key = warp * 16 + g;
+    float m_run = -INFINITY, l_run[8];
 #pragma unroll
-    for (int i = 0; i < 16; i++) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
-    const uint32_t p_row = (uint32_t)((key >> 3) * 1024 + (key & 7) * 128);
+    for (int i = 0; i < 8; i++) l_run[i] = 0.f;
+    uint8_t* const p_row = smem + (sP - sK) + warp * 2048 + g * 128 + tig * 4;
     for (int t = 0; t < ntiles; t++) {
       wait(&bar_s[t & 1], t >> 1, 23);
       __syncwarp();
       tc_fence_after();
       uint32_t r[16];
-      tc_ld16(tmem + (uint32_t)((t & 1) * LHEADS + hg * 16) + ((uint32_t)(kh * 32) << 16), r);
+      tc_ld_16x256(tmem + (uint32_t)((t & 1) * LHEADS) + ((uint32_t)(warp * 32) << 16), r);
       tc_wait_ld();
-      const bool live = key < LKT && kb + t * LKT + key < ke;
-      float v[16];
+      const int left = ke - kb - t * LKT - key;
+      float v[16], mx[8];
 #pragma unroll
-      for (int i = 0; i < 16; i++) v[i] = live ? __uint_as_float(r[i]) * a.scale_log2 : -INFINITY;
-      const float mx = transposed_reduce(v, lane, [](float x, float y) { return fmaxf(x, y); });
-      if (!(lane & 1)) mx_s[t & 1][kh][hg * 16 + (lane >> 1)] = mx;
+      for (int j = 0; j < 4; j++)
+#pragma unroll
+        for (int k = 0; k < 2; k++) {
+          v[4 * j + k] = left > 0 ? __uint_as_float(r[4 * j + k]) * a.scale_log2 : -INFINITY;
+          v[4 * j + 2 + k] = left > 8 ? __uint_as_float(r[4 * j + 2 + k]) * a.scale_log2 : -INFINITY;
+          mx[2 * j + k] = fmaxf(v[4 * j + k], v[4 * j + 2 + k]);
+        }
+      mx_s[t & 1][warp][8 * (g >> 1) + 2 * tig + (g & 1)] = transposed_reduce(mx, lane, [](float x, float y) { return fmaxf(x, y); });
       asm volatile("bar.sync 1, 128;" ::: "memory");
-      bool grow = false;
-      float corr[16];
+      const float m_tile = fmaxf(fmaxf(mx_s[t & 1][0][lane], mx_s[t & 1][1][lane]), fmaxf(mx_s[t & 1][2][lane], mx_s[t & 1][3][lane]));
+      const bool grow = m_tile > m_run + 8.0f;  // also for the first tile (m_run = -inf)
+      if (__any_sync(0xffffffffu, grow)) {      // the same in all four warps
+        const float m_use = grow ? m_tile : m_run, corr = grow ? ex2_approx(m_run - m_use) : 1.0f;
+        m_run = m_use;
 #pragma unroll
-      for (int i = 0; i < 16; i += 4) {
-        const float4 x = *(const float4*)&mx_s[t & 1][0][hg * 16 + i], y = *(const float4*)&mx_s[t & 1][1][hg * 16 + i];
-        const float m[4] = {fmaxf(x.x, y.x), fmaxf(x.y, y.y), fmaxf(x.z, y.z), fmaxf(x.w, y.w)};
+        for (int i = 0; i < 8; i++) l_run[i] *= __shfl_sync(0xffffffffu, corr, 8 * (i >> 1) + 2 * tig + (i & 1));
+        if (t > 0) {
+          corr_s[warp][lane] = corr;
+          wait(&bar_o[(t - 1) & 1], (t - 1) >> 1, 24);  // the previous product must have finished writing O^T
+          __syncwarp();
+          tc_fence_after();
+          const uint32_t base = tmem + 64u + ((uint32_t)(warp * 32) << 16);
+          for (int c = 0; c < n_mb * 4; c++) {
+            uint32_t x[16];
+            tc_ld16(base + (uint32_t)(c * 16), x);
+            tc_wait_ld();
 #pragma unroll
-        for (int j = 0; j < 4; j++) {
-          const bool g = m[j] > m_run[i + j] + 8.0f;  // also for the first tile (m_run = -inf)
-          const float m_use = g ? m[j] : m_run[i + j];
-          corr[i + j] = g ? ex2_approx(m_run[i + j] - m_use) : 1.0f;
-          m_run[i + j] = m_use;
-          grow |= g;
+            for (int j = 0; j < 16; j++) x[j] = __float_as_uint(__uint_as_float(x[j]) * corr_s[warp][(c & 1) * 16 + j]);
+            tc_st16(base + (uint32_t)(c * 16), x);
+          }
+          tc_wait_st();
         }
-      }
-      if (grow) {  // the same in every thread of the head half
-        if (kh == 0) {
-#pragma unroll
-          for (int i = 0; i < 16; i++)
-            if (lane == i) corr_s[t & 1][hg * 16 + i] = corr[i];
-        }
-#pragma unroll
-        for (int i = 0; i < 16; i++) l_run[i] *= corr[i];
-      } else if (kh == 0 && lane < 16) {
-        corr_s[t & 1][hg * 16 + lane] = 1.0f;
-      }
-      if (kh == 0 && lane == 0) grow_s[t & 1][hg] = grow;
-      asm volatile("bar.sync 2, 192;" ::: "memory");
-      if (t > 0 && (grow_s[t & 1][0] | grow_s[t & 1][1])) {
-        wait(&bar_o[(t - 1) & 1], (t - 1) >> 1, 24);  // the previous product must have finished writing O^T
-        __syncwarp();
-        tc_fence_after();
-        rescale(t, hg, 2);
       }
       if (t >= 2) wait(&bar_o[t & 1], (t - 2) >> 1, 25);  // this half of the weight buffer is free
-      uint32_t hi[8], lo[8];
+      __syncwarp();
+      uint8_t* const pw = p_row + (t & 1) * P_BYTES;
 #pragma unroll
-      for (int i = 0; i < 8; i++) {
-        const float p0 = ex2_approx(v[2 * i] - m_run[2 * i]), p1 = ex2_approx(v[2 * i + 1] - m_run[2 * i + 1]);
-        l_run[2 * i] += p0;
-        l_run[2 * i + 1] += p1;
-        split_bf16x2(p0, p1, hi[i], lo[i]);
-      }
-      uint8_t* prow = smem + (sP - sK) + (t & 1) * P_BYTES + p_row;
-      if (LKT == 64 || key < LKT)
+      for (int j = 0; j < 4; j++) {
+        const float m0 = __shfl_sync(0xffffffffu, m_run, 8 * j + 2 * tig), m1 = __shfl_sync(0xffffffffu, m_run, 8 * j + 2 * tig + 1);
 #pragma unroll
-      for (int c = 0; c < 2; c++) {
-        *(uint4*)(prow + (((hg * 2 + c) ^ (key & 7)) << 4)) = make_uint4(hi[4 * c], hi[4 * c + 1], hi[4 * c + 2], hi[4 * c + 3]);
-        *(uint4*)(prow + (((4 + hg * 2 + c) ^ (key & 7)) << 4)) = make_uint4(lo[4 * c], lo[4 * c + 1], lo[4 * c + 2], lo[4 * c + 3]);
+        for (int k = 0; k < 2; k++) {
+          const float p0 = ex2_approx(v[4 * j + 2 * k] - m0), p1 = ex2_approx(v[4 * j + 2 * k + 1] - m1);
+          l_run[2 * j] += p0;
+          l_run[2 * j + 1] += p1;
+          uint32_t hi, lo;
+          split_bf16x2(p0, p1, hi, lo);
+          *(uint32_t*)(pw + k * 1024 + ((j ^ g) << 4)) = hi;
+          *(uint32_t*)(pw + k * 1024 + (((4 + j) ^ g) << 4)) = lo;
+        }
       }
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // the tensor cores read what these stores wrote
       tc_fence_before();
       asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(&bar_p)) : "memory");
     }
-    // sums over the keys
-    const float l = transposed_reduce(l_run, lane, [](float x, float y) { return x + y; });
-    if (!(lane & 1)) mx_s[0][kh][hg * 16 + (lane >> 1)] = l;  // its last readers are behind a barrier of the loop, or it was never used
-    if (kh == 0) {
-#pragma unroll
-      for (int i = 0; i < 16; i++)
-        if (lane == i) ml_s[hg * 16 + i].x = m_run[i];
-    }
+    // sums over the keys; the barrier keeps them out of maxima that are still being read
+    asm volatile("bar.sync 1, 128;" ::: "memory");
+    mx_s[0][warp][8 * (g >> 1) + 2 * tig + (g & 1)] = transposed_reduce(l_run, lane, [](float x, float y) { return x + y; });
+    if (warp == 0) ml_s[lane].x = m_run;
   }
   __syncwarp();
   if (ntiles > 0) wait(&bar_o[(ntiles - 1) & 1], (ntiles - 1) >> 1, 26);  // every product is complete
@@ -796,13 +762,13 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
     }
   }
   if (threadIdx.x < LHEADS) {
-    const float l = ntiles > 0 ? mx_s[0][0][threadIdx.x] + mx_s[0][1][threadIdx.x] : 0.f;
-    ml_s[threadIdx.x] = make_float2(ntiles > 0 ? ml_s[threadIdx.x].x : -INFINITY, l);
+    const float l = (mx_s[0][0][threadIdx.x] + mx_s[0][1][threadIdx.x]) + (mx_s[0][2][threadIdx.x] + mx_s[0][3][threadIdx.x]);
+    ml_s[threadIdx.x].y = l;  // without keys: (-inf, 0)
   }
   asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // the copies below read what the stores above wrote
   tc_fence_before();
   __syncthreads();
-  if (warp == 2) {
+  if (warp == 4) {
     tc_fence_after();
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(tmem_cols) : "memory");
   }
