@@ -526,6 +526,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
     for (int i = 0; i < 2; i++) { mbar_init(smem_u32(&bar_s[i]), 1); mbar_init(smem_u32(&bar_o[i]), 1); }
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
+  if (warp == 5 && lane < 2) asm volatile("prefetch.tensormap [%0];" ::"l"(lane ? &map_q : &map_k) : "memory");
   if (warp == 4) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(tmem_cols) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
@@ -670,6 +671,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
     uint8_t* const p_row = smem + (sP - sK) + warp * 2048 + g * 128 + tig * 4;
     for (int t = 0; t < ntiles; t++) {
       wait(&bar_s[t & 1], t >> 1, 23);
+      if (t == 0) SB_TRACE_MARK(0);
       __syncwarp();
       tc_fence_after();
       uint32_t r[16];
@@ -741,6 +743,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
   if (ntiles > 0) wait(&bar_o[(ntiles - 1) & 1], (ntiles - 1) >> 1, 26);  // every product is complete
   __syncwarp();
   tc_fence_after();
+  SB_TRACE_MARK(1);
   __syncthreads();  // the ring is free: it holds this block's sums now
   float* so = (float*)smem;  // [32][rank_p + 4]
   const int so_ld = a.rank_p + 4;
@@ -800,6 +803,7 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
   }
   __syncthreads();
   if (a.nsplit > 1) wait(&bar_m, 0, 27);
+  SB_TRACE_MARK(2);
   const int c4n = a.rank_p / 4, heads = min(n_own, a.H - h0 - first);
   for (int i = threadIdx.x; i < heads * c4n; i += 256) {
     const int h = i / c4n, c = (i - h * c4n) * 4;

@@ -8,14 +8,15 @@ Prints one JSON line. Times are CUDA events on the library's stream (prefill: th
 host ids in, greedy ids out; decode: graph-replayed steps with ids resident on the device). A step streams
 more than L2 holds in every configuration but the few-layer ones of --layers. `kernels` are plain launches
 of the decode step, one pair of events per call, with the bytes a call must move and their share of the
-copy bandwidth; `flops_frac` is a prefill's useful matrix work over the measured bf16 throughput.
+copy bandwidth, and beside it the same inside the replayed step (`exposed_us`, `hbm_frac_in_step`: how
+far a launch moved the end of the chain, from per-block time stamps); `flops_frac` is a prefill's useful matrix work over the measured bf16 throughput.
 """
 import json
 import os
 
 import numpy as np
 
-from . import clocks, native as N
+from . import clocks, native as N, timeline
 from .kernel import Context, DeviceVariable
 from .model import CONFIGS, STACK, Model, latent_layer, stack_config
 
@@ -80,6 +81,23 @@ def call_bytes(cfg, B, length):
             "attn_decode": B * length * Hkv * D * 4}
 
 
+TRACE_CLASS = {"rope": "rope_kvappend", "attn_combine": "attn_merge"}
+
+
+def gemm_names(cfg):
+    """(N, K) of the decode step's GEMM launches -> kernel class, to label them in a trace."""
+    d = cfg["d_model"]
+    if cfg["arch"] != STACK:
+        D, H, Hkv, I = cfg["head_dim"], cfg["n_q_heads"], cfg["n_kv_heads"], cfg["d_ff"]
+        return {((H + 2 * Hkv) * D, d): "gemm_qkv", (d, H * D): "gemm_o", (2 * I, d): "gemm_gate_up", (d, I): "gemm_down", (cfg["vocab"], d): "head"}
+    out = {(cfg["vocab"], d): "head"}
+    for y in cfg["layers"]:
+        n0 = y["heads"] * (y["dim"] + y["rot_dim"]) + (y["kv_rank"] + y["rot_dim"] if y["kv_from"] < 0 else 0)
+        out[(-(-n0 // 256) * 256 + y["d_ff"], d)] = "gemm_qkv"
+        out[(d, y["heads"] * y["vdim"] + y["d_ff"])] = "gemm_o"
+    return out
+
+
 def ids(ctx, n, vocab, seed):
     v = DeviceVariable(ctx, n, np.int32)
     N.check(N.lib().strictb200_gen_tokens(ctx.h, seed, 1, n, vocab, v.p))
@@ -132,6 +150,17 @@ def run_model(ctx, cfg, decode, prefill, steps, warmup):
                 if k in per_call:
                     calls_of_bytes = calls / 3 if k != "head" else 1  # the head's product and its pick are two calls
                     kernels[k]["hbm_frac"] = per_call[k] / (tot * 1e3 / (3 * calls_of_bytes) * 1e-6) / 1e9 / hbm
+        # the same classes inside the replayed step, from the kernels' own time stamps: how far each launch moved the end of the chain
+        with ctx.trace(1 << 20) as tr:
+            kv.decode_steps_device(1)
+        for k, (ns, calls) in timeline.per_kernel(timeline.launches(tr.records, gemm_names(cfg))).items():
+            k = TRACE_CLASS.get(k, k)
+            if k in kernels:
+                e = kernels[k]
+                e["exposed_us"] = e.get("exposed_us", 0.0) + ns / 1e3 / e["calls_per_step"]
+        for k, e in kernels.items():
+            if k in per_call and e.get("exposed_us") and k != "head":
+                e["hbm_frac_in_step"] = per_call[k] / (e["exposed_us"] * 1e-6) / 1e9 / hbm
         out["decode"].append({"batch": B, "context": S, "ms": ms, "tokens_per_s": B / ms * 1e3, "step_gb": nbytes / 1e9,
                               "hbm_frac": nbytes / (ms * 1e-3) / 1e9 / hbm, "kernels": kernels, "clocks": clk})
         kv.dispose()
