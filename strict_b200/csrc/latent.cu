@@ -5,7 +5,7 @@
 //  * prompts: keys and values are rebuilt per head by one GEMM over the visible latents, then the tcgen05 prefill kernel
 //    runs on them (attention_tc.cu). Here: the projection's rows into rotated queries and cache rows.
 //  * decode: nothing is rebuilt. A head's query is carried into latent space (q' = q W_uk), so that q' . c replaces
-//    q . W_uk c, all heads read the same cache row (the heads are the rows of the MMA tile) and the weighted sum of latents
+//    q . W_uk c, all heads read the same cache row (the heads are the columns of the MMA tile) and the weighted sum of latents
 //    goes through W_uv once per head. Three launches: queries into latent space beside everything else the projection
 //    feeds (rotation, cache append, activation); split-key attention, merged inside a cluster; W_uv.
 //  * any other width, and fp32: one block per row and head, straight from the cache.
@@ -59,7 +59,7 @@ __device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity) {
   }
   return false;
 }
-// by one lane of a warp that runs converged (see tc_mma_warp)
+// by one elected lane of a warp that runs converged
 __device__ __forceinline__ void tma_load_2d_warp(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar, uint64_t policy) {
   asm volatile(
       "{\n\t.reg .pred e;\n\t"
@@ -431,8 +431,8 @@ inline int decode_stages(int row, bool two_blocks) {
 
 __device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
 __device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-// Issued by one lane of a warp that runs converged: its operands are then the same in all lanes and stay in uniform registers
-// (inside a one-lane branch every operand of every product is moved there first, which takes longer than a 128 x 32 product).
+// The issuing warps run converged, so that addresses and descriptors stay in uniform registers: one elected lane issues (a
+// whole batch of products inside one elected branch measured fastest; an election per product costs 10 % of the kernel).
 __device__ __forceinline__ void tc_commit_warp(uint32_t bar) {
   asm volatile(
       "{\n\t.reg .pred e;\n\t"
@@ -440,12 +440,16 @@ __device__ __forceinline__ void tc_commit_warp(uint32_t bar) {
       "@e tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}" ::"r"(bar)
       : "memory");
 }
-__device__ __forceinline__ void tc_mma_warp(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+__device__ __forceinline__ bool elect_one() {
+  uint32_t e;
+  asm volatile("{\n\t.reg .pred e;\n\telect.sync _|e, 0xffffffff;\n\tselp.u32 %0, 1, 0, e;\n\t}" : "=r"(e));
+  return e != 0;
+}
+__device__ __forceinline__ void tc_mma(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
   asm volatile(
-      "{\n\t.reg .pred p, e;\n\t"
-      "elect.sync _|e, 0xffffffff;\n\t"
+      "{\n\t.reg .pred p;\n\t"
       "setp.ne.b32 p, %4, 0;\n\t"
-      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
       :
       : "r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(0u)
       : "memory");
@@ -625,11 +629,14 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
       if (ns > np && ready(&bar_p, pr)) {  // the weights are in shared memory, O^T follows the new maxima
         tc_fence_after();
         const uint64_t dc = dc0 + (uint64_t)(uint32_t)(ps * stage16), dp = dp0 + (uint64_t)(uint32_t)((np & 1) * (P_BYTES >> 4));
+        if (elect_one()) {
 #pragma unroll
-        for (int s = 0; s < LKT / 16; s++)  // 16 keys = 16 rows of 128 bytes; the blocks of latents take turns
+          for (int s = 0; s < LKT / 16; s++)  // 16 keys = 16 rows of 128 bytes; the blocks of latents take turns
 #pragma unroll
-          for (int mb = 0; mb < 4; mb++)
-            if (mb < n_mb) tc_mma_warp(td + 64u + (uint32_t)(mb * 64), dc + (uint64_t)((2 * mb * ATOM + s * 2048) >> 4), dp + (uint64_t)(s * 2048 >> 4), idesc_pv, (np | s) ? 1u : 0u);
+            for (int mb = 0; mb < 4; mb++)
+              if (mb < n_mb) tc_mma(td + 64u + (uint32_t)(mb * 64), dc + (uint64_t)((2 * mb * ATOM + s * 2048) >> 4), dp + (uint64_t)(s * 2048 >> 4), idesc_pv, (np | s) ? 1u : 0u);
+        }
+        __syncwarp();
         tc_commit_warp(smem_u32(&bar_o[np & 1]));
         tc_commit_warp(smem_u32(&k_empty[ps]));
         np++;
@@ -640,14 +647,19 @@ __global__ void __launch_bounds__(256) latent_attn_decode_kernel(const __grid_co
         tc_fence_after();
         const int first = sg * per_group, last = min(n_atoms, first + per_group);
         const uint32_t d = td + (uint32_t)((ns & 1) * LHEADS);
-#pragma unroll 1
-        for (int i = first; i < last; i++) {  // a row's last atom is zero beyond its width
-          const uint64_t dk = dk0 + (uint64_t)(uint32_t)(st * stage16 + i * (ATOM >> 4)), dq = dq0 + (uint64_t)(uint32_t)(i * (Q_ATOM >> 4));
-          tc_mma_warp(d, dk, dq, idesc_s, i ? 1u : 0u);
-          tc_mma_warp(d, dk + 2, dq + 2, idesc_s, 1u);
-          tc_mma_warp(d, dk + 4, dq + 4, idesc_s, 1u);
-          tc_mma_warp(d, dk + 6, dq + 6, idesc_s, 1u);
+        const uint64_t dkb = dk0 + (uint64_t)(uint32_t)(st * stage16 + first * (ATOM >> 4)), dqb = dq0 + (uint64_t)(uint32_t)(first * (Q_ATOM >> 4));
+        if (elect_one()) {
+#pragma unroll
+          for (int i = 0; i < 4; i++)  // a group is at most four atoms; a row's last one is zero beyond its width
+            if (first + i < last) {
+              const uint64_t dk = dkb + (uint64_t)(i * (ATOM >> 4)), dq = dqb + (uint64_t)(i * (Q_ATOM >> 4));
+              tc_mma(d, dk, dq, idesc_s, first + i ? 1u : 0u);
+              tc_mma(d, dk + 2, dq + 2, idesc_s, 1u);
+              tc_mma(d, dk + 4, dq + 4, idesc_s, 1u);
+              tc_mma(d, dk + 6, dq + 6, idesc_s, 1u);
+            }
         }
+        __syncwarp();
         sg++;
         if (last == n_atoms) {
           tc_commit_warp(smem_u32(&bar_s[ns & 1]));
