@@ -458,9 +458,14 @@ __device__ __forceinline__ void sb_bf16_store16(const Bf16Epilogue& e, int M, in
   if (!act && e.out_f32) {
     if (n >= N) return;
     float* o = e.out_f32 + (int64_t)m0 * e.ldo + n;
+    float old[16];  // all read before the first store, so that the sixteen reads overlap
+    if (e.accumulate) {
+#pragma unroll
+      for (int j = 0; j < 16; j++) old[j] = m0 + j < M ? o[j * e.ldo] : 0.f;
+    }
 #pragma unroll
     for (int j = 0; j < 16; j++, o += e.ldo)
-      if (m0 + j < M) *o = e.accumulate ? *o + __uint_as_float(r[j]) : __uint_as_float(r[j]);
+      if (m0 + j < M) *o = e.accumulate ? old[j] + __uint_as_float(r[j]) : __uint_as_float(r[j]);
     return;
   }
   const int64_t ld = act ? e.ld_act : e.ldo;
