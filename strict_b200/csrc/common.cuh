@@ -472,7 +472,11 @@ __device__ __forceinline__ void sb_bf16_store16(const Bf16Epilogue& e, int M, in
   bf16* o = act ? e.act_out + (n - e.n_switch) : e.out_bf16 + n;
   float v[16];
 #pragma unroll
-  for (int j = 0; j < 16; j++) v[j] = act ? sb_xielu_bf16(__uint_as_float(r[j]), e.act_pos, e.act_neg) : __uint_as_float(r[j]);
+  for (int j = 0; j < 16; j++) v[j] = __uint_as_float(r[j]);
+  if (act) {
+#pragma unroll
+    for (int j = 0; j < 16; j++) v[j] = sb_xielu_bf16(v[j], e.act_pos, e.act_neg);
+  }
   if ((ld & 1) == 0 && (N & 1) == 0 && ((uintptr_t)(act ? e.act_out : e.out_bf16) & 3) == 0) {  // the same for every lane
     const bool odd = n & 1;
     o += (int64_t)(m0 + (odd ? 8 : 0)) * ld - (odd ? 1 : 0);

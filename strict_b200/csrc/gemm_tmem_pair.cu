@@ -106,6 +106,14 @@ __device__ __forceinline__ void tc_ld16(uint32_t taddr, uint32_t* r) {
       : "r"(taddr));
 }
 __device__ __forceinline__ void tc_wait_ld() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
+// The same, and the sixteen values of a load are not touched before it.
+__device__ __forceinline__ void tc_wait_ld16(uint32_t* r) {
+  asm volatile("tcgen05.wait::ld.sync.aligned;"
+               : "+r"(r[0]), "+r"(r[1]), "+r"(r[2]), "+r"(r[3]), "+r"(r[4]), "+r"(r[5]), "+r"(r[6]), "+r"(r[7]), "+r"(r[8]), "+r"(r[9]),
+                 "+r"(r[10]), "+r"(r[11]), "+r"(r[12]), "+r"(r[13]), "+r"(r[14]), "+r"(r[15])
+               :
+               : "memory");
+}
 // Barrier over the 4 epilogue warps that also ORs a predicate (all 128 leave the tile loop together).
 __device__ __forceinline__ bool epi_any(bool pred) {
   uint32_t out;
@@ -249,24 +257,33 @@ __global__ void __launch_bounds__(192) gemm_pair_kernel(const __grid_constant__ 
       const int n = (tile % a.tiles_n) * 2 * BN + (int)rank * BN + ch;
       const int tok_base = (tile / a.tiles_n) * BTH;  // 256 operand rows = 128 tokens per tile
       const float swn = !BF16 && n < a.N ? a.sw[n] : 0.f;
+      if constexpr (BF16) {  // 256 tokens per tile, 32 at a time
 #pragma unroll 1
-      for (int grp = 0; grp < ACC_COLS / 16; grp++) {
-        uint32_t r[16];
-        tc_ld16(acc + (uint32_t)(grp * 16), r);
-        tc_wait_ld();
-        if constexpr (BF16) {
-          sb_bf16_store16(a.e, a.M, a.N, 2 * tok_base + grp * 16, n, r);  // 256 tokens per tile
-        } else {
-#pragma unroll
-        for (int j = 0; j < 8; j++) {
-          const int tok = tok_base + grp * 8 + j;  // operand rows 16g.. hold tokens 8g..
-          if (tok < a.M && n < a.N) {
-            float v = __fadd_rn(__uint_as_float(r[j]), __fmul_rn(0.0625f, __uint_as_float(r[8 + j])));
-            float y = __fmul_rn(__fmul_rn(v, a.sx[tok]), swn);
-            if (a.out_f32) ((float*)a.out)[(int64_t)tok * a.N + n] = y;
-            else ((bf16*)a.out)[(int64_t)tok * a.N + n] = __float2bfloat16_rn(y);
-          }
+        for (int grp = 0; grp < ACC_COLS / 16; grp += 2) {
+          uint32_t r[32];
+          tc_ld16(acc + (uint32_t)(grp * 16), r);
+          tc_ld16(acc + (uint32_t)(grp * 16 + 16), r + 16);
+          tc_wait_ld16(r);
+          tc_wait_ld16(r + 16);
+          sb_bf16_store16(a.e, a.M, a.N, 2 * tok_base + grp * 16, n, r);
+          sb_bf16_store16(a.e, a.M, a.N, 2 * tok_base + grp * 16 + 16, n, r + 16);
         }
+      } else {
+#pragma unroll 1
+        for (int grp = 0; grp < ACC_COLS / 16; grp++) {
+          uint32_t r[16];
+          tc_ld16(acc + (uint32_t)(grp * 16), r);
+          tc_wait_ld();
+#pragma unroll
+          for (int j = 0; j < 8; j++) {
+            const int tok = tok_base + grp * 8 + j;  // operand rows 16g.. hold tokens 8g..
+            if (tok < a.M && n < a.N) {
+              float v = __fadd_rn(__uint_as_float(r[j]), __fmul_rn(0.0625f, __uint_as_float(r[8 + j])));
+              float y = __fmul_rn(__fmul_rn(v, a.sx[tok]), swn);
+              if (a.out_f32) ((float*)a.out)[(int64_t)tok * a.N + n] = y;
+              else ((bf16*)a.out)[(int64_t)tok * a.N + n] = __float2bfloat16_rn(y);
+            }
+          }
         }
       }
       // the accumulator is drained in this block: tell the leader's MMA warp
