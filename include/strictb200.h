@@ -304,31 +304,47 @@ typedef struct strictb200_model_config {
 int strictb200_model_create(strictb200_ctx* ctx, const strictb200_model_config* cfg, strictb200_model** out);
 int strictb200_model_destroy(strictb200_model* m);
 /* ---- models described layer by layer (single GPU) ----
- * Every layer: x <- x + mixer(norm1(x)) + ff(norm2(x)), both norms of the same x, each an RMS norm over norm_groups equal
- * consecutive parts of the row. The model is strictb200_model like any other: the cache, prefill, decode, generate and
+ * Every layer: x <- x + residual_mult * (ls1 * mixer(norm1(x)) + ls2 * ff(norm2(x))), both norms of the same x, each an RMS
+ * norm over norm_groups equal consecutive parts of the row; with shared_norm there is only norm1, without layer_scale ls1 and
+ * ls2 (vectors over the width) are 1. The logits are multiplied by logit_scale. The model is strictb200_model like any other: the cache, prefill, decode, generate and
  * tensor calls below take it.
  * Mixer "latent attention": per head `dim` unrotated and `rot_dim` rotated query/key dimensions and `vdim` value
  * dimensions; a position leaves one RMS-normed latent of kv_rank values and one rotated key part that all heads share
  * (what the cache holds); keys and values of a head are linear in the latent. Rotation pairs (2i, 2i+1), angle
  * pos * rot_base^(-2i/rot_dim). Scores are multiplied by `scale`; a position sees `window` keys, itself included
  * (0: every earlier one). kv_from >= 0: no latents of its own, it reads those of that earlier layer.
- * Feed-forward: down(xIELU(up(h))), or none.
+ * Mixer "attention": softmax attention of `heads` query heads over kv_heads key/value heads (dim, vdim). Rotation of the
+ * first rot_dim dimensions, i with i + rot_dim / 2; rot_factor > 0 stretches the frequencies (YaRN: rot_original, rot_fast,
+ * rot_slow). qk_norm: rotated queries and keys divided by their root mean square; sink: one more key of score 0 and no value
+ * in the softmax; gate: a head's output times sigmoid(g(h)) of its own. A position sees every earlier one and itself.
+ * Mixer "gated": y = gelu(Wy h + by), u = causal convolution of Wx h + bx (`conv` taps per channel), r and i sigmoids of
+ * block-diagonal products of u (`blocks` matrices), log a = -8 r softplus(lam), S <- a S + sqrt(1 - a^2) i u, output S * y;
+ * `width` channels.
+ * Mixer "retention": per head S <- decay[h] S + k v^T, o = S^T q, q and k rotated as above, k times dim^-1/2, o divided by its
+ * root mean square and multiplied by silu(g(h)). The states live in the cache object, in fp32.
+ * Feed-forward: down(xIELU(up(h))), down(relu(gate(h)) * up(h)), or none.
  * dtype BF16: bf16 weights, cache and matrix operands; fp32 residual, norms, scores and softmax. FP32: all fp32. */
-enum strictb200_mixer { STRICTB200_MIXER_LATENT = 1 };
-enum strictb200_mlp { STRICTB200_MLP_NONE = 0, STRICTB200_MLP_XIELU = 1 };
+enum strictb200_mixer { STRICTB200_MIXER_LATENT = 1, STRICTB200_MIXER_ATTENTION = 2, STRICTB200_MIXER_GATED = 3, STRICTB200_MIXER_RETENTION = 4 };
+enum strictb200_mlp { STRICTB200_MLP_NONE = 0, STRICTB200_MLP_XIELU = 1, STRICTB200_MLP_RELU_GLU = 2 };
 enum strictb200_dtype { STRICTB200_BF16 = 0, STRICTB200_FP32 = 1 };
 typedef struct strictb200_layer_config {
   int32_t mixer; /* strictb200_mixer */
   int32_t heads, dim, rot_dim, vdim, kv_rank;
   int32_t window, kv_from; /* 0: no window; -1: latents of its own */
   int32_t mlp, d_ff;       /* strictb200_mlp */
+  int32_t kv_heads, qk_norm, sink, gate; /* attention */
+  int32_t width, blocks, conv;           /* gated */
+  int32_t reserved;
   double scale, rot_base;
+  double rot_factor, rot_original, rot_fast, rot_slow; /* rot_factor 0: plain rotation */
+  const double* decay;                   /* retention: [heads], read by strictb200_stack_create */
 } strictb200_layer_config;
 typedef struct strictb200_stack_config {
   int32_t n_layers, d_model, vocab, max_pos;
   int32_t norm_groups;
   int32_t dtype; /* strictb200_dtype */
-  double eps;
+  int32_t shared_norm, layer_scale;
+  double eps, residual_mult, logit_scale;
 } strictb200_stack_config;
 int strictb200_stack_create(strictb200_ctx* ctx, const strictb200_stack_config* cfg, const strictb200_layer_config* layers, strictb200_model** out);
 /* Fill every tensor from the seeded generator (std 0.02, norm gains 1, biases 0). Under
@@ -389,7 +405,9 @@ enum strictb200_kernel_class {
   STRICTB200_K_HEAD = 9,      /* LM head GEMM + argmax */
   STRICTB200_K_ALLREDUCE = 10,
   STRICTB200_K_ATTN_MERGE = 11, /* merge of the key chunks + quantise */
-  STRICTB200_K_COUNT = 12
+  STRICTB200_K_GATES = 12,      /* gate product of a gated recurrence */
+  STRICTB200_K_RECURRENCE = 13, /* gated recurrence, retention (the kernels that stream a state) */
+  STRICTB200_K_COUNT = 14
 };
 /* Runs n_steps greedy decode steps as plain launches with a pair of CUDA events around every
  * call, and returns the summed device milliseconds and the number of calls per kernel class

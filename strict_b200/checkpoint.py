@@ -78,8 +78,32 @@ def kipatar_config(cfg, max_pos, dtype):
                           eps=cfg["norm"]["eps"], dtype=dtype)
 
 
+def morarax_config(cfg, max_pos, dtype):
+    """Morarax: softmax attention with a sink and gated heads, real-gated linear recurrences and retention in any order, each
+    parallel with a ReLU-gated feed-forward under one norm, with a scale per channel on both."""
+    layers = []
+    for i, e in enumerate(cfg["layers"]):
+        mix, mlp = e["mixer"], e.get("mlp")
+        if mlp and mlp["kind"] != "dense":
+            raise _unknown(f"layer {i}: feed-forward", mlp["kind"])
+        d_ff = mlp["ff"] if mlp else 0
+        rot = mix.get("rot")
+        rotation = dict(rot_dim=rot["dims"], rot_base=rot["base"], rot_scaling=rot.get("scaling")) if rot else {}
+        if e["type"] == "attention":
+            layers.append(M.attention_layer(heads=mix["heads"], kv_heads=mix["kv_heads"], dim=mix["dim"], vdim=mix["vdim"], scale=mix["scale"],
+                                            qk_norm=True, sink=True, gate=True, d_ff=d_ff, **rotation))
+        elif e["type"] == "rglru":
+            layers.append(M.gated_layer(width=mix["width"], blocks=mix["blocks"], conv=mix["conv"], d_ff=d_ff))
+        elif e["type"] == "retention":
+            layers.append(M.retention_layer(heads=mix["heads"], dim=mix["dim"], vdim=mix["vdim"], decay=mix["decay"], d_ff=d_ff, **rotation))
+        else:
+            raise _unknown(f"layer {i}: mixer", e["type"])
+    return M.stack_config(layers, d_model=cfg["width"], vocab=cfg["vocab"], max_pos=max_pos, norm_groups=1, eps=cfg["norm"]["eps"], dtype=dtype,
+                          shared_norm=True, layer_scale=True, residual_mult=cfg["residual_mult"], logit_scale=cfg["logit_scale"])
+
+
 # architecture named by config.json -> configuration of the library's model
-ARCHITECTURES = {"Kipatar": kipatar_config}
+ARCHITECTURES = {"Kipatar": kipatar_config, "Morarax": morarax_config}
 
 
 def read_config(folder, max_pos, dtype=M.BF16):
@@ -91,25 +115,63 @@ def read_config(folder, max_pos, dtype=M.BF16):
     return ARCHITECTURES[name](cfg, max_pos, dtype)
 
 
+def _latent_tensors(y, d):
+    H = y["heads"]
+    out = {"q": (H * (y["dim"] + y["rot_dim"]), d), "uk": (H * y["dim"], y["kv_rank"]), "uv": (H * y["vdim"], y["kv_rank"]), "o": (d, H * y["vdim"])}
+    if y["kv_from"] < 0:
+        out["dkv"] = (y["kv_rank"] + y["rot_dim"], d)
+        out["dkv.norm"] = (y["kv_rank"],)
+    return out
+
+
+def _attention_tensors(y, d):
+    H, G = y["heads"], y["kv_heads"]
+    out = {"q": (H * y["dim"], d), "k": (G * y["dim"], d), "v": (G * y["vdim"], d), "o": (d, H * y["vdim"])}
+    if y["gate"]:
+        out["g"] = (H, d)
+    return out
+
+
+def _gated_tensors(y, d):
+    w, b = y["width"], y["blocks"]
+    out = {"y": (w, d), "y.b": (w,), "x": (w, d), "x.b": (w,), "conv": (w, y["conv"]), "conv.b": (w,), "lam": (w,), "o": (d, w)}
+    for k in ("ra", "ri"):
+        out[k] = (b, w // b, w // b)
+        out[k + ".b"] = (b, w // b)
+    return out
+
+
+def _retention_tensors(y, d):
+    n, v = y["heads"] * y["dim"], y["heads"] * y["vdim"]
+    return {"q": (n, d), "k": (n, d), "v": (v, d), "g": (v, d), "o": (d, v)}
+
+
+_MIXER_TENSORS = {M.MIXER_LATENT: _latent_tensors, M.MIXER_ATTENTION: _attention_tensors, M.MIXER_GATED: _gated_tensors,
+                  M.MIXER_RETENTION: _retention_tensors}
+
+
 def expected_tensors(cfg):
     """Names a STACK configuration needs, with their shapes."""
     d = cfg["d_model"]
     out = {"embed": (cfg["vocab"], d), "head": (cfg["vocab"], d), "final.norm": (d,)}
     for i, y in enumerate(cfg["layers"]):
-        p, H = f"l{i}.", y["heads"]
+        p = f"l{i}."
         out[p + "norm1"] = (d,)
-        out[p + "mix.q"] = (H * (y["dim"] + y["rot_dim"]), d)
-        if y["kv_from"] < 0:
-            out[p + "mix.dkv"] = (y["kv_rank"] + y["rot_dim"], d)
-            out[p + "mix.dkv.norm"] = (y["kv_rank"],)
-        out[p + "mix.uk"] = (H * y["dim"], y["kv_rank"])
-        out[p + "mix.uv"] = (H * y["vdim"], y["kv_rank"])
-        out[p + "mix.o"] = (d, H * y["vdim"])
-        if y["mlp"] != M.MLP_NONE:
+        out.update({p + "mix." + k: v for k, v in _MIXER_TENSORS[y["mixer"]](y, d).items()})
+        if cfg["layer_scale"]:
+            out[p + "ls1"] = (d,)
+        if y["mlp"] == M.MLP_NONE:
+            continue
+        if not cfg["shared_norm"]:
             out[p + "norm2"] = (d,)
-            out[p + "mlp.up"] = (y["d_ff"], d)
-            out[p + "mlp.down"] = (d, y["d_ff"])
+        if cfg["layer_scale"]:
+            out[p + "ls2"] = (d,)
+        out[p + "mlp.up"] = (y["d_ff"], d)
+        out[p + "mlp.down"] = (d, y["d_ff"])
+        if y["mlp"] == M.MLP_XIELU:
             out[p + "mlp.act"] = (2,)
+        else:
+            out[p + "mlp.gate"] = (y["d_ff"], d)
     return out
 
 

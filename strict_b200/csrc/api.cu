@@ -129,8 +129,11 @@ int sb_trace_set_norm(const SbTraceDev&);
 int sb_trace_set_rope(const SbTraceDev&);
 int sb_trace_set_attention(const SbTraceDev&);
 int sb_trace_set_latent(const SbTraceDev&);
+int sb_trace_set_heads(const SbTraceDev&);
+int sb_trace_set_recurrent(const SbTraceDev&);
 static int trace_set_all(const SbTraceDev& t) {
-  return sb_trace_set_gemm_split(t) | sb_trace_set_norm(t) | sb_trace_set_rope(t) | sb_trace_set_attention(t) | sb_trace_set_latent(t);
+  return sb_trace_set_gemm_split(t) | sb_trace_set_norm(t) | sb_trace_set_rope(t) | sb_trace_set_attention(t) | sb_trace_set_latent(t) |
+         sb_trace_set_heads(t) | sb_trace_set_recurrent(t);
 }
 
 extern "C" {

@@ -61,7 +61,9 @@ __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint3
   hi = pack_bf16(ah, bh);
   lo = pack_bf16(a - ah, b - bh);
 }
-__device__ __forceinline__ uint32_t tile_off(int row, int chunk) { return (uint32_t)(row * 256 + ((chunk ^ (row & 7)) << 4)); }
+// HD = dims of a row (64 or 128): rows of HD / 8 chunks of 16 bytes, chunk c of row r at chunk c ^ (r & 7)
+template <int HD = D>
+__device__ __forceinline__ uint32_t tile_off(int row, int chunk) { return (uint32_t)(row * 2 * HD + ((chunk ^ (row & 7)) << 4)); }
 
 // Copy `rows` rows of 128 bf16 (global row stride 128 elements) into a swizzled tile; rows at
 // or beyond `valid_rows` are zero-filled.
@@ -73,13 +75,14 @@ __device__ __forceinline__ void load_tile(uint32_t tile, const bf16* src, int ro
   }
 }
 
-// Same, with an L2 eviction policy on the global reads (the decode kernel reads every key and
+// Same for rows of HD dims, with an L2 eviction policy on the global reads (the decode kernel reads every key and
 // value exactly once).
+template <int HD>
 __device__ __forceinline__ void load_tile_hint(uint32_t tile, const bf16* src, int rows, int valid_rows, int nthreads, uint64_t policy) {
-  for (int c = threadIdx.x; c < rows * 16; c += nthreads) {
-    int r = c >> 4, cc = c & 15;
+  for (int c = threadIdx.x; c < rows * (HD / 8); c += nthreads) {
+    int r = c / (HD / 8), cc = c % (HD / 8);
     bool v = r < valid_rows;
-    cp_async16_hint(tile + tile_off(r, cc), src + (int64_t)(v ? r : 0) * D + cc * 8, v, policy);
+    cp_async16_hint(tile + tile_off<HD>(r, cc), src + (int64_t)(v ? r : 0) * HD + cc * 8, v, policy);
   }
 }
 
@@ -292,27 +295,29 @@ __device__ __forceinline__ int ld_volatile_i32(const int32_t* p) {
 }
 
 // grid (nsplit, Hkv, B), 128 threads. Warp w owns keys [16w,16w+16) of every 64-key tile.
-// scratch: o_part [B][Hq][nsplit][128] then ml_part [B][Hq][nsplit][2].
+// HD = dims of a cache row (64 or 128).
+// scratch: o_part [B][Hq][nsplit][HD] then ml_part [B][Hq][nsplit][2].
 // FUSED: the queries do not come from memory; every block computes the (at most 16) query heads of
 // its KV head from the qkv projection's partial results (sum, scales, QK-norm, RoPE), and the block
 // whose key chunk holds the new token's position also computes that token's key and value rows,
 // appends them to the cache and patches them into its own shared-memory tile (its tile load may
 // have read that row before the append). One kernel less per layer of the decode step.
-template <bool FUSED>
+template <int HD, bool FUSED>
 __global__ void __launch_bounds__(128) attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
                                                           const int32_t* __restrict__ lens, int len_add, int B, int Hq, int Hkv, int maxlen,
                                                           int chunk, int nsplit, float scale_log2, float* __restrict__ o_part,
                                                           float* __restrict__ ml_part, RopeFuseArgs rf, int prefetch) {
+  static_assert(!FUSED || HD == D, "the RoPE prologue is for 128 dims");
   extern __shared__ __align__(128) uint8_t smem[];
-  __shared__ __align__(16) bf16 q_s[FUSED ? 16 * D : 8];    // the query heads of this KV head
-  __shared__ __align__(16) bf16 kv_new[FUSED ? 2 * D : 8];  // the new token's key row, then its value row
+  __shared__ __align__(16) bf16 q_s[FUSED ? 16 * HD : 8];    // the query heads of this KV head
+  __shared__ __align__(16) bf16 kv_new[FUSED ? 2 * HD : 8];  // the new token's key row, then its value row
   SB_TRACE_BEGIN();
   pdl_trigger();
   const int split = blockIdx.x, hk = blockIdx.y, b = blockIdx.z;
   const int k_begin = split * chunk;
-  const uint32_t sK = smem_u32(smem), sV = sK + DEC_STAGES * KT * 256;
-  const bf16* kbase = kc + ((int64_t)b * Hkv + hk) * maxlen * D;
-  const bf16* vbase = vc + ((int64_t)b * Hkv + hk) * maxlen * D;
+  const uint32_t sK = smem_u32(smem), sV = sK + DEC_STAGES * KT * 2 * HD;
+  const bf16* kbase = kc + ((int64_t)b * Hkv + hk) * maxlen * HD;
+  const bf16* vbase = vc + ((int64_t)b * Hkv + hk) * maxlen * HD;
   const uint64_t kv_policy = l2_evict_first_policy();
   // Before the dependency wait: the first tiles of this block's keys and values start to stream
   // while the preceding kernels (the qkv projection's tail, RoPE) still run. Only rows that were
@@ -326,8 +331,8 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const bf16* __restrict
     npre = min(DEC_STAGES - 1, nt - 1);
     for (int t = 0; t < npre; t++) {
       const int k0 = k_begin + t * KT;
-      load_tile_hint(sK + t * KT * 256, kbase + (int64_t)k0 * D, KT, KT, 128, kv_policy);
-      load_tile_hint(sV + t * KT * 256, vbase + (int64_t)k0 * D, KT, KT, 128, kv_policy);
+      load_tile_hint<HD>(sK + t * KT * 2 * HD, kbase + (int64_t)k0 * HD, KT, KT, 128, kv_policy);
+      load_tile_hint<HD>(sV + t * KT * 2 * HD, vbase + (int64_t)k0 * HD, KT, KT, 128, kv_policy);
       cp_async_commit();
     }
   }
@@ -352,46 +357,46 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const bf16* __restrict
   for (int t = npre; t < DEC_STAGES - 1; t++) {
     if (t < ntiles) {
       int k0 = k_begin + t * KT;
-      load_tile_hint(sK + t * KT * 256, kbase + (int64_t)k0 * D, KT, min(KT, k_end - k0), 128, kv_policy);
-      load_tile_hint(sV + t * KT * 256, vbase + (int64_t)k0 * D, KT, min(KT, k_end - k0), 128, kv_policy);
+      load_tile_hint<HD>(sK + t * KT * 2 * HD, kbase + (int64_t)k0 * HD, KT, min(KT, k_end - k0), 128, kv_policy);
+      load_tile_hint<HD>(sV + t * KT * 2 * HD, vbase + (int64_t)k0 * HD, KT, min(KT, k_end - k0), 128, kv_policy);
     }
     cp_async_commit();
   }
 
   if (FUSED) {
-    const int64_t nqkv = (int64_t)(Hq + 2 * Hkv) * D;
+    const int64_t nqkv = (int64_t)(Hq + 2 * Hkv) * HD;
     const int pos = min(p_new, rf.max_pos - 1);
     // items 0..G-1: the query heads; for the owner of the new position also G: the key head, G+1: the value head
     for (int i = warp; i < G + (owns_new ? 2 : 0); i += 4) {
       if (i < G) {
-        const uint2 w = rope_head_bf16(rf, B, b, nqkv, (int64_t)(hk * G + i) * D, rf.qgain, pos, false, lane);
-        *(uint2*)(q_s + i * D + lane * 4) = w;
+        const uint2 w = rope_head_bf16(rf, B, b, nqkv, (int64_t)(hk * G + i) * HD, rf.qgain, pos, false, lane);
+        *(uint2*)(q_s + i * HD + lane * 4) = w;
       } else {
         const bool is_v = i == G + 1;
-        const uint2 w = rope_head_bf16(rf, B, b, nqkv, (int64_t)(Hq + (is_v ? Hkv : 0) + hk) * D, rf.kgain, pos, is_v, lane);
-        *(uint2*)(kv_new + (is_v ? D : 0) + lane * 4) = w;
+        const uint2 w = rope_head_bf16(rf, B, b, nqkv, (int64_t)(Hq + (is_v ? Hkv : 0) + hk) * HD, rf.kgain, pos, is_v, lane);
+        *(uint2*)(kv_new + (is_v ? HD : 0) + lane * 4) = w;
         bf16* cache = is_v ? rf.vcache : rf.kcache;
-        *(uint2*)(cache + (((int64_t)b * Hkv + hk) * maxlen + p_new) * D + lane * 4) = w;
+        *(uint2*)(cache + (((int64_t)b * Hkv + hk) * maxlen + p_new) * HD + lane * 4) = w;
       }
     }
     __syncthreads();
   }
   // Q fragments: rows = the G query heads of this KV head (zero beyond), from memory or from the prologue above
-  uint32_t qf[8][4];
+  uint32_t qf[HD / 16][4];
   {
-    const bf16* q0 = FUSED ? q_s : q + ((int64_t)b * Hq + hk * G) * D;
+    const bf16* q0 = FUSED ? q_s : q + ((int64_t)b * Hq + hk * G) * HD;
 #pragma unroll
-    for (int ks = 0; ks < 8; ks++) {
+    for (int ks = 0; ks < HD / 16; ks++) {
       int d0 = ks * 16 + 2 * tig;
-      qf[ks][0] = g < G ? *(const uint32_t*)(q0 + g * D + d0) : 0u;
-      qf[ks][1] = g + 8 < G ? *(const uint32_t*)(q0 + (g + 8) * D + d0) : 0u;
-      qf[ks][2] = g < G ? *(const uint32_t*)(q0 + g * D + d0 + 8) : 0u;
-      qf[ks][3] = g + 8 < G ? *(const uint32_t*)(q0 + (g + 8) * D + d0 + 8) : 0u;
+      qf[ks][0] = g < G ? *(const uint32_t*)(q0 + g * HD + d0) : 0u;
+      qf[ks][1] = g + 8 < G ? *(const uint32_t*)(q0 + (g + 8) * HD + d0) : 0u;
+      qf[ks][2] = g < G ? *(const uint32_t*)(q0 + g * HD + d0 + 8) : 0u;
+      qf[ks][3] = g + 8 < G ? *(const uint32_t*)(q0 + (g + 8) * HD + d0 + 8) : 0u;
     }
   }
-  float o[16][4];
+  float o[HD / 8][4];
 #pragma unroll
-  for (int j = 0; j < 16; j++)
+  for (int j = 0; j < HD / 8; j++)
 #pragma unroll
     for (int i = 0; i < 4; i++) o[j][i] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
@@ -402,28 +407,28 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const bf16* __restrict
       const int tn = t + DEC_STAGES - 1;  // refill the stage consumed in the previous iteration
       if (tn < ntiles) {
         int k0 = k_begin + tn * KT;
-        load_tile_hint(sK + (tn % DEC_STAGES) * KT * 256, kbase + (int64_t)k0 * D, KT, min(KT, k_end - k0), 128, kv_policy);
-        load_tile_hint(sV + (tn % DEC_STAGES) * KT * 256, vbase + (int64_t)k0 * D, KT, min(KT, k_end - k0), 128, kv_policy);
+        load_tile_hint<HD>(sK + (tn % DEC_STAGES) * KT * 2 * HD, kbase + (int64_t)k0 * HD, KT, min(KT, k_end - k0), 128, kv_policy);
+        load_tile_hint<HD>(sV + (tn % DEC_STAGES) * KT * 2 * HD, vbase + (int64_t)k0 * HD, KT, min(KT, k_end - k0), 128, kv_policy);
       }
       cp_async_commit();
       cp_async_wait<DEC_STAGES - 1>();  // all but the newest DEC_STAGES-1 groups: tile t has landed
     }
     __syncthreads();
-    const uint32_t tK = sK + (t % DEC_STAGES) * KT * 256, tV = sV + (t % DEC_STAGES) * KT * 256;
+    const uint32_t tK = sK + (t % DEC_STAGES) * KT * 2 * HD, tV = sV + (t % DEC_STAGES) * KT * 2 * HD;
     if (FUSED && owns_new && p_new >= k_begin + t * KT && p_new < k_begin + (t + 1) * KT) {
       // the tile copy may have read the new token's row before it was appended: put the rows computed above in its place
       if (warp == 0) {
         const int row = p_new - (k_begin + t * KT), cc = lane & 15;
-        const uint4 w = *(const uint4*)(kv_new + (lane < 16 ? 0 : D) + cc * 8);
-        *(uint4*)(smem + ((lane < 16 ? tK : tV) - sK) + tile_off(row, cc)) = w;
+        const uint4 w = *(const uint4*)(kv_new + (lane < 16 ? 0 : HD) + cc * 8);
+        *(uint4*)(smem + ((lane < 16 ? tK : tV) - sK) + tile_off<HD>(row, cc)) = w;
       }
       __syncthreads();
     }
     float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
-    for (int ks = 0; ks < 8; ks++) {
+    for (int ks = 0; ks < HD / 16; ks++) {
       uint32_t kb[4];
-      ldsm_x4(tK + tile_off(warp * 16 + (mi >> 1) * 8 + r8, 2 * ks + (mi & 1)), kb);
+      ldsm_x4(tK + tile_off<HD>(warp * 16 + (mi >> 1) * 8 + r8, 2 * ks + (mi & 1)), kb);
       mma_bf16(s[0], qf[ks], kb[0], kb[1]);
       mma_bf16(s[1], qf[ks], kb[2], kb[3]);
     }
@@ -462,14 +467,14 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const bf16* __restrict
       split_bf16(p[1][0], p[1][1], pf[2], pl[2]); split_bf16(p[1][2], p[1][3], pf[3], pl[3]);
     }
 #pragma unroll
-    for (int j = 0; j < 16; j++) {
+    for (int j = 0; j < HD / 8; j++) {
       o[j][0] *= corr[0]; o[j][1] *= corr[0];
       o[j][2] *= corr[1]; o[j][3] *= corr[1];
     }
 #pragma unroll
-    for (int jj = 0; jj < 8; jj++) {
+    for (int jj = 0; jj < HD / 16; jj++) {
       uint32_t vb[4];
-      ldsm_x4_t(tV + tile_off(warp * 16 + (mi & 1) * 8 + r8, 2 * jj + (mi >> 1)), vb);
+      ldsm_x4_t(tV + tile_off<HD>(warp * 16 + (mi & 1) * 8 + r8, 2 * jj + (mi >> 1)), vb);
       mma_bf16(o[2 * jj], pf, vb[0], vb[1]);
       mma_bf16(o[2 * jj + 1], pf, vb[2], vb[3]);
       mma_bf16(o[2 * jj], pl, vb[0], vb[1]);
@@ -483,23 +488,23 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const bf16* __restrict
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
   }
   // merge the four warps through shared memory (tiles are free after the last barrier)
-  float* so = (float*)smem;                       // [4 warps][16 rows][128]
-  float* sml = so + 4 * 16 * D;                   // [4 warps][16 rows][2]
+  float* so = (float*)smem;                       // [4 warps][16 rows][HD]
+  float* sml = so + 4 * 16 * HD;                   // [4 warps][16 rows][2]
 #pragma unroll
   for (int r = 0; r < 2; r++) {
     int row = g + 8 * r;
     if (row < G) {
 #pragma unroll
-      for (int j = 0; j < 16; j++) {
-        so[(warp * 16 + row) * D + 8 * j + 2 * tig] = o[j][2 * r];
-        so[(warp * 16 + row) * D + 8 * j + 2 * tig + 1] = o[j][2 * r + 1];
+      for (int j = 0; j < HD / 8; j++) {
+        so[(warp * 16 + row) * HD + 8 * j + 2 * tig] = o[j][2 * r];
+        so[(warp * 16 + row) * HD + 8 * j + 2 * tig + 1] = o[j][2 * r + 1];
       }
       if (tig == 0) { sml[(warp * 16 + row) * 2] = m_run[r]; sml[(warp * 16 + row) * 2 + 1] = l_run[r]; }
     }
   }
   __syncthreads();
-  for (int e = threadIdx.x; e < G * D; e += 128) {
-    int row = e / D, d = e - row * D;
+  for (int e = threadIdx.x; e < G * HD; e += 128) {
+    int row = e / HD, d = e - row * HD;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; w++) M = fmaxf(M, sml[(w * 16 + row) * 2]);
@@ -509,10 +514,10 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const bf16* __restrict
       float mw = sml[(w * 16 + row) * 2];
       float f = mw == -INFINITY ? 0.f : exp2f(mw - M);
       L += sml[(w * 16 + row) * 2 + 1] * f;
-      O += so[(w * 16 + row) * D + d] * f;
+      O += so[(w * 16 + row) * HD + d] * f;
     }
     int64_t idx = ((int64_t)b * Hq + hk * G + row) * nsplit + split;
-    o_part[idx * D + d] = O;
+    o_part[idx * HD + d] = O;
     if (d == 0) { ml_part[idx * 2] = M; ml_part[idx * 2 + 1] = L; }
   }
   SB_TRACE_END(SB_K_ATTN, 0);
@@ -788,12 +793,12 @@ static int decode_chunk(strictb200_ctx* ctx, int B, int Hkv, int maxlen, int len
   const size_t smem_dec = 2 * DEC_STAGES * KT * 256;
   static int resident_fused_of[64] = {};
   once.run(ctx->device, [&] {
-    cudaFuncSetAttribute(attn_decode_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_dec);
-    cudaFuncSetAttribute(attn_decode_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_dec);
+    cudaFuncSetAttribute(attn_decode_kernel<D, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_dec);
+    cudaFuncSetAttribute(attn_decode_kernel<D, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_dec);
     int r = 0;
-    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&r, attn_decode_kernel<false>, 128, smem_dec) != cudaSuccess || r < 1) r = 1;
+    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&r, attn_decode_kernel<D, false>, 128, smem_dec) != cudaSuccess || r < 1) r = 1;
     resident_of[ctx->device & 63] = r;
-    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&r, attn_decode_kernel<true>, 128, smem_dec) != cudaSuccess || r < 1) r = 1;
+    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&r, attn_decode_kernel<D, true>, 128, smem_dec) != cudaSuccess || r < 1) r = 1;
     resident_fused_of[ctx->device & 63] = r;
     return cudaSuccess;
   });
@@ -822,6 +827,21 @@ int sb_attn_decode_splits(strictb200_ctx* ctx, int B, int Hkv, int maxlen) {
 int sb_attn_decode_chunk(strictb200_ctx* ctx, int B, int Hkv, int maxlen, int len_plan) { return decode_chunk(ctx, B, Hkv, maxlen, len_plan); }
 size_t sb_attn_decode_scratch(int B, int Hq, int Dh, int nsplit) { return (size_t)B * Hq * nsplit * (Dh + 2) * sizeof(float); }
 
+// The key chunks alone, for a merge of the caller's: rows of HD = 64 or 128 dims, len_add = 1 (the new token's row is in the cache).
+int k_attn_decode_chunks(strictb200_ctx* ctx, int HD, const bf16* q, const bf16* kc, const bf16* vc, const int32_t* lens, int B, int Hq, int Hkv, int maxlen,
+                         float scale, int nsplit, int chunk, float* o_part, float* ml_part) {
+  if ((HD != 64 && HD != 128) || Hq / Hkv > 16 || Hkv > 65535 || B > 65535) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "attention: head shape the split-key kernel does not take");
+  if (chunk <= 0 || chunk % KT || nsplit < 1) return sb_fail(STRICTB200_ERR_INVALID_ARG, "attention: bad key chunks");
+  const size_t smem = 2 * DEC_STAGES * KT * 2 * HD;  // (for 128 dims decode_chunk has raised the kernel's limit)
+  auto go = [&](auto kernel) {
+    return sb_launch(ctx, kernel, dim3(nsplit, Hkv, B), dim3(128), smem, q, kc, vc, lens, 1, B, Hq, Hkv, maxlen, chunk, nsplit, scale * LOG2E, o_part, ml_part,
+                     RopeFuseArgs{}, ctx->opt.attn_prefetch);
+  };
+  SB_CUDA(HD == 64 ? go(attn_decode_kernel<64, false>) : go(attn_decode_kernel<128, false>));
+  ctx->launches++;
+  return STRICTB200_OK;
+}
+
 int k_attn_decode(strictb200_ctx* ctx, const bf16* q, const bf16* kc, const bf16* vc, const int32_t* lens, int len_add, int B, int Hq, int Hkv,
                   int Dh, int maxlen, float scale, int nsplit, float* scratch, bf16* out, uint8_t* q_out, float* qscale_out, const RopeArgs* rope,
                   int chunk) {
@@ -842,10 +862,10 @@ int k_attn_decode(strictb200_ctx* ctx, const bf16* q, const bf16* kc, const bf16
       return sb_fail(STRICTB200_ERR_INVALID_ARG, "attention: the fused RoPE prologue needs split-K partials (at most 8), one new token and the same caches");
     RopeFuseArgs rf{rope->part, rope->splits, rope->sx, rope->sw, rope->cos_t, rope->sin_t, rope->qgain, rope->kgain, rope->eps, rope->max_pos,
                     rope->kcache, rope->vcache};
-    SB_CUDA(sb_launch(ctx, attn_decode_kernel<true>, grid, dim3(128), smem, (const bf16*)nullptr, kc, vc, lens, len_add, B, Hq, Hkv, maxlen, chunk, nsplit,
+    SB_CUDA(sb_launch(ctx, attn_decode_kernel<D, true>, grid, dim3(128), smem, (const bf16*)nullptr, kc, vc, lens, len_add, B, Hq, Hkv, maxlen, chunk, nsplit,
                       scale * LOG2E, o_part, ml_part, rf, ctx->opt.attn_prefetch));
   } else {
-    SB_CUDA(sb_launch(ctx, attn_decode_kernel<false>, grid, dim3(128), smem, q, kc, vc, lens, len_add, B, Hq, Hkv, maxlen, chunk, nsplit, scale * LOG2E,
+    SB_CUDA(sb_launch(ctx, attn_decode_kernel<D, false>, grid, dim3(128), smem, q, kc, vc, lens, len_add, B, Hq, Hkv, maxlen, chunk, nsplit, scale * LOG2E,
                       o_part, ml_part, RopeFuseArgs{}, ctx->opt.attn_prefetch));
   }
   ctx->launches++;

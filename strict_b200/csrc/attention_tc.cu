@@ -23,127 +23,18 @@
 // an SM (96 KB of shared memory, 256 tensor-memory columns each) and fill each other's gaps.
 // Every mbarrier wait is bounded: on expiry the block records an error word in host-visible
 // memory, stops, frees its tensor memory and returns.
-#include <cuda.h>
-
 #include <cstdlib>
 
-#include "common.cuh"
+#include "tcgen05.cuh"
+
+using namespace tc;
 
 namespace {
 
 constexpr int D = 128;
 constexpr int BQ = 128;   // query rows per block
 constexpr int BKV = 128;  // keys per tile
-constexpr int HALF_BYTES = 128 * 128;       // 128 rows x 64 bf16: one TMA box
-constexpr int TILE_BYTES = 2 * HALF_BYTES;  // 128 x 128 bf16
-constexpr uint32_t WAIT_LIMIT = 1u << 22;
 constexpr float LOG2E = 1.4426950408889634f;
-
-__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void mbar_init(uint32_t bar, uint32_t count) {
-  asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count));
-}
-__device__ __forceinline__ void mbar_expect_tx(uint32_t bar, uint32_t bytes) {
-  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity) {
-  for (uint32_t i = 0; i < WAIT_LIMIT; i++) {
-    uint32_t done;
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-        "selp.u32 %0, 1, 0, p;\n\t}"
-        : "=r"(done)
-        : "r"(bar), "r"(parity)
-        : "memory");
-    if (done) return true;
-  }
-  return false;
-}
-__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
-  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst),
-               "l"(map), "r"(x), "r"(y), "r"(bar)
-               : "memory");
-}
-__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
-  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];" ::"r"(dst),
-               "l"(map), "r"(x), "r"(y), "r"(z), "r"(bar)
-               : "memory");
-}
-__device__ __forceinline__ void set_status(int* status, int code) {
-  *(volatile int*)status = code;
-  __threadfence_system();
-}
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_commit(uint32_t bar) {
-  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-// D[tmem] (+)= A[smem desc] * B[smem desc]
-__device__ __forceinline__ void tc_mma_ss(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
-      :
-      : "r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(0u)
-      : "memory");
-}
-// D[tmem] (+)= A[tmem] * B[smem desc]
-__device__ __forceinline__ void tc_mma_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, {%5, %5, %5, %5}, p;\n\t}"
-      :
-      : "r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate), "r"(0u)
-      : "memory");
-}
-__device__ __forceinline__ void tc_ld32(uint32_t taddr, uint32_t* r) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-      "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]),
-        "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]),
-        "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]),
-        "=r"(r[31])
-      : "r"(taddr));
-}
-__device__ __forceinline__ void tc_st16(uint32_t taddr, const uint32_t* r) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(taddr),
-      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]),
-      "r"(r[13]), "r"(r[14]), "r"(r[15])
-      : "memory");
-}
-__device__ __forceinline__ void tc_st32(uint32_t taddr, const uint32_t* r) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-      "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};" ::"r"(taddr),
-      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]),
-      "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]), "r"(r[24]),
-      "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
-      : "memory");
-}
-__device__ __forceinline__ float ex2_approx(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ void tc_wait_ld() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ void tc_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-
-// K-major operand (rows of 128 bytes = 64 bf16 of the reduction dimension, 128-byte swizzle,
-// groups of 8 rows 1024 bytes apart): Q and K tiles for S = Q K^T.
-__device__ __forceinline__ uint64_t desc_kmajor(uint32_t addr) {
-  return (uint64_t)((addr >> 4) & 0x3FFF) | (1ull << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
-}
-// MN-major operand: the V tile for O = P V. Its rows are keys (the reduction dimension), each row
-// holds 64 contiguous output dims (128 bytes, swizzled); 8-key groups are 1024 bytes apart
-// (stride offset), the second 64 dims live in the next 16 KB box (leading offset).
-__device__ __forceinline__ uint64_t desc_mnmajor(uint32_t addr) {
-  return (uint64_t)((addr >> 4) & 0x3FFF) | ((uint64_t)(HALF_BYTES >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
-}
 
 struct TcAttnArgs {
   const int32_t* lens;
@@ -160,6 +51,9 @@ struct TcAttnArgs {
   int nks_q, nks_r;      // 16-wide reduction steps of the unrotated and of the rotated part
   int dv;                // value width
   int64_t ldo;           // row stride of out
+  // heads with a sink and an output gate
+  int sink;              // 1: the softmax denominator counts one more key, of score 0 and without a value
+  const float* gate;     // [rows, Hq] factor of a head's output; may be null
 };
 
 __global__ void __launch_bounds__(128) attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
@@ -403,12 +297,15 @@ __global__ void __launch_bounds__(128) attn_prefill_tc_kernel(const __grid_const
 // tensor maps (dims x heads x rows), which fill with zeros; reduction steps beyond the width are not
 // issued. KST = stages of the K ring. WIN adds a sliding window: the walk over the key tiles begins
 // at the first tile any row of the block sees, and rows drop keys below their own window.
+//
+// PLAIN: grouped heads of 128 dims, output rows [Hq, 128]. Otherwise the output goes to rows of ldo with heads of dv dims, and
+// without a shared part (RA = 0: grouped heads over cache rows of 64 * QA dims) the sink and the gate of TcAttnArgs apply.
 constexpr int TC2_THREADS = 576;  // 16 softmax warps + MMA warp + TMA warp
 
 template <int QA, int RA, int VA, int KST>
 constexpr int tc2_tile_bytes() { return (2 * (QA + RA) + KST * (QA + RA) + 2 * VA) * HALF_BYTES; }
 
-template <int QA, int RA, int VA, int KST, bool WIN>
+template <int QA, int RA, int VA, int KST, bool WIN, bool PLAIN>
 __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_qr,
                                                                       const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_kr,
                                                                       const __grid_constant__ CUtensorMap map_v, TcAttnArgs a) {
@@ -636,9 +533,15 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
     wg_sync();
     if (ok && nt[w] > 0) {
       const bool live = qw + row < n_new;
-      const float inv = 1.0f / x_sum[w][row];
-      bf16* dst = RA ? a.out + (row0 + qw + row) * a.ldo + (int64_t)h * a.dv : a.out + ((row0 + qw + row) * a.Hq + h) * D;
-      const bool whole = !RA || (((a.dv & 7) == 0) && ((a.ldo & 7) == 0));
+      float inv;
+      if constexpr (!PLAIN && !RA) {
+        inv = 1.0f / (x_sum[w][row] + (a.sink ? exp2f(-m_run) : 0.f));  // the sums are relative to 2^m_run
+        if (a.gate && live) inv *= a.gate[(row0 + qw + row) * a.Hq + h];
+      } else {
+        inv = 1.0f / x_sum[w][row];
+      }
+      bf16* dst = !PLAIN ? a.out + (row0 + qw + row) * a.ldo + (int64_t)h * a.dv : a.out + ((row0 + qw + row) * a.Hq + h) * D;
+      const bool whole = PLAIN || (((a.dv & 7) == 0) && ((a.ldo & 7) == 0));
 #pragma unroll 1
       for (int c = VA * half; c < VA * half + VA; c++) {
         uint32_t r[32];
@@ -651,7 +554,7 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
         } else if (live) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
-            if (RA && c * 32 + i >= a.dv) break;
+            if (!PLAIN && c * 32 + i >= a.dv) break;
             uint4 wv;
             wv.x = f32_to_bf16_bits(__uint_as_float(r[i]) * inv) | (f32_to_bf16_bits(__uint_as_float(r[i + 1]) * inv) << 16);
             wv.y = f32_to_bf16_bits(__uint_as_float(r[i + 2]) * inv) | (f32_to_bf16_bits(__uint_as_float(r[i + 3]) * inv) << 16);
@@ -671,51 +574,13 @@ __global__ void __launch_bounds__(TC2_THREADS) attn_prefill_tc2_kernel(const __g
   }
 }
 
-typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
-                             const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-EncodeFn g_encode = nullptr;
-
-int get_encode() {
-  if (g_encode) return STRICTB200_OK;
-  void* fn = nullptr;
-  cudaDriverEntryPointQueryResult q;
-  SB_CUDA(cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &q));
-  if (!fn || q != cudaDriverEntryPointSuccess) return sb_fail(STRICTB200_ERR_CUDA, "cuTensorMapEncodeTiled is not available from this driver");
-  g_encode = (EncodeFn)fn;
-  return STRICTB200_OK;
-}
-
-// 2D map of a row-major bf16 matrix [rows, cols] (row stride ld elements), box = 128 rows x 64 columns (128 bytes), 128-byte swizzle.
-int make_map(CUtensorMap* map, const void* base, int64_t rows, int64_t cols, int64_t ld) {
-  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
-  cuuint32_t box[2] = {64u, 128u};
-  cuuint32_t estr[2] = {1, 1};
-  CUresult r = g_encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                        CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  if (r != CUDA_SUCCESS) return sb_fail(STRICTB200_ERR_CUDA, "cuTensorMapEncodeTiled failed with code " + std::to_string((int)r));
-  return STRICTB200_OK;
-}
-
-// 3D map of bf16 rows of `heads` heads (width x heads x rows, strides in elements), box = 64 x 1 x 128, 128-byte swizzle.
-int make_map3(CUtensorMap* map, const void* base, int64_t width, int64_t heads, int64_t rows, int64_t head_stride, int64_t row_stride) {
-  cuuint64_t dims[3] = {(cuuint64_t)width, (cuuint64_t)heads, (cuuint64_t)rows};
-  cuuint64_t strides[2] = {(cuuint64_t)head_stride * 2, (cuuint64_t)row_stride * 2};
-  cuuint32_t box[3] = {64u, 1u, 128u};
-  cuuint32_t estr[3] = {1, 1, 1};
-  CUresult r = g_encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                        CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  if (r != CUDA_SUCCESS) return sb_fail(STRICTB200_ERR_CUDA, "cuTensorMapEncodeTiled failed with code " + std::to_string((int)r));
-  return STRICTB200_OK;
-}
-
-template <int QA, int RA, int VA, int KST, bool WIN>
+template <int QA, int RA, int VA, int KST, bool WIN, bool PLAIN>
 int launch_tc2(strictb200_ctx* ctx, const CUtensorMap* m, const TcAttnArgs& a, int B, int S) {
   const size_t smem = tc2_tile_bytes<QA, RA, VA, KST>() + 1024;
   static SbDeviceOnce once;  // one per instantiation
-  SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(attn_prefill_tc2_kernel<QA, RA, VA, KST, WIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
+  SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(attn_prefill_tc2_kernel<QA, RA, VA, KST, WIN, PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
   dim3 grid((unsigned)((S + 2 * BQ - 1) / (2 * BQ)), (unsigned)a.Hq, (unsigned)B);
-  attn_prefill_tc2_kernel<QA, RA, VA, KST, WIN><<<grid, TC2_THREADS, smem, ctx->stream>>>(m[0], m[1], m[2], m[3], m[4], a);
+  attn_prefill_tc2_kernel<QA, RA, VA, KST, WIN, PLAIN><<<grid, TC2_THREADS, smem, ctx->stream>>>(m[0], m[1], m[2], m[3], m[4], a);
   SB_LAUNCHED(ctx);
   return STRICTB200_OK;
 }
@@ -728,8 +593,7 @@ int k_attn_prefill_tc(strictb200_ctx* ctx, const bf16* q, const bf16* kc, const 
   if (Hq > 65535 || B > 65535 || Hq % Hkv) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "attention: too many heads or sequences");
   if ((int64_t)B * Hkv * maxlen > INT32_MAX || q_rows > INT32_MAX) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "attention: cache too large for 32-bit tile coordinates");
   if (((uintptr_t)q | (uintptr_t)kc | (uintptr_t)vc) & 15) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "attention: operands must be 16-byte aligned");
-  SB_TRY(get_encode());
-  TcAttnArgs a{lens, past, qstart, S, Hq, Hkv, maxlen, scale * LOG2E, out, ctx->d_status, nullptr, nullptr, 0, 0, 0, D, (int64_t)Hq * D};
+  TcAttnArgs a{lens, past, qstart, S, Hq, Hkv, maxlen, scale * LOG2E, out, ctx->d_status, nullptr, nullptr, 0, 0, 0, D, (int64_t)Hq * D, 0, nullptr};
   // two query tiles per block (ping-pong) from 256 new tokens per sequence on; the attn_tc option (1 / 2) forces a kernel
   const int forced = ctx->opt.attn_tc;
   if (forced == 2 || (forced != 1 && S >= 2 * BQ)) {
@@ -738,7 +602,7 @@ int k_attn_prefill_tc(strictb200_ctx* ctx, const bf16* q, const bf16* kc, const 
     SB_TRY(make_map3(&m[2], kc, D, 1, (int64_t)B * Hkv * maxlen, D, D));
     SB_TRY(make_map3(&m[4], vc, D, 1, (int64_t)B * Hkv * maxlen, D, D));
     m[1] = m[0]; m[3] = m[2];
-    return launch_tc2<2, 0, 2, 2, false>(ctx, m, a, B, S);
+    return launch_tc2<2, 0, 2, 2, false, true>(ctx, m, a, B, S);
   }
   CUtensorMap mq, mk, mv;
   SB_TRY(make_map(&mq, q, q_rows, (int64_t)Hq * D, (int64_t)Hq * D));
@@ -753,13 +617,29 @@ int k_attn_prefill_tc(strictb200_ctx* ctx, const bf16* q, const bf16* kc, const 
   return STRICTB200_OK;
 }
 
+// Grouped heads over cache rows of row_dims = 64 or 128 dims (narrower heads are filled up with zeros), values of vdim dims.
+int k_attn_prefill_heads(strictb200_ctx* ctx, const HeadPrefillArgs& p) {
+  const int HD = p.row_dims;
+  if (HD != 64 && HD != 128) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "prefill attention: rows of 64 or 128 dims");
+  if (p.H > 65535 || p.B > 65535 || p.H % p.Hkv || p.q_rows > INT32_MAX || (int64_t)p.B * p.Hkv * p.maxlen > INT32_MAX)
+    return sb_fail(STRICTB200_ERR_UNSUPPORTED, "prefill attention: too many heads, sequences or rows");
+  TcAttnArgs a{};
+  a.lens = p.lens; a.past = p.past; a.qstart = p.qstart; a.S = p.S; a.Hq = p.H; a.Hkv = p.Hkv; a.maxlen = p.maxlen;
+  a.scale_log2 = p.scale * LOG2E; a.out = p.out; a.status = ctx->d_status; a.dv = p.vdim; a.ldo = p.ldo; a.sink = p.sink; a.gate = p.gate;
+  CUtensorMap m[5];
+  SB_TRY(make_map3(&m[0], p.q, HD, p.H, p.q_rows, HD, (int64_t)p.H * HD));
+  SB_TRY(make_map3(&m[2], p.k, HD, 1, (int64_t)p.B * p.Hkv * p.maxlen, HD, HD));
+  SB_TRY(make_map3(&m[4], p.v, HD, 1, (int64_t)p.B * p.Hkv * p.maxlen, HD, HD));
+  m[1] = m[0]; m[3] = m[2];
+  return HD == 64 ? launch_tc2<1, 0, 1, 2, false, false>(ctx, m, a, p.B, p.S) : launch_tc2<2, 0, 2, 2, false, false>(ctx, m, a, p.B, p.S);
+}
+
 bool sb_latent_prefill_fits(int dim, int rot, int vdim) { return dim <= 128 && rot <= 64 && vdim <= 128; }
 
 int k_attn_prefill_latent(strictb200_ctx* ctx, const LatentPrefillArgs& p) {
   if (!sb_latent_prefill_fits(p.dim, p.rot, p.vdim)) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "latent prefill attention: head too wide for the tensor-core kernel");
   if (p.H > 65535 || p.B > 65535 || p.q_rows > INT32_MAX || p.k_rows > INT32_MAX)
     return sb_fail(STRICTB200_ERR_UNSUPPORTED, "latent prefill attention: too many heads, sequences or rows");
-  SB_TRY(get_encode());
   TcAttnArgs a{};
   a.lens = p.lens; a.past = p.past; a.qstart = p.qstart; a.S = p.S; a.Hq = p.H; a.Hkv = p.H;
   a.scale_log2 = p.scale * LOG2E; a.out = p.out; a.status = ctx->d_status;
@@ -771,7 +651,7 @@ int k_attn_prefill_latent(strictb200_ctx* ctx, const LatentPrefillArgs& p) {
   SB_TRY(make_map3(&m[3], p.k_rot, p.rot, 1, p.k_rows, p.ld_rot, p.ld_rot));
   SB_TRY(make_map3(&m[4], p.v, p.vdim, p.H, p.k_rows, p.v_head, p.ldk));
   const int S = p.S, B = p.B;
-#define LATENT_TC2(QA, VA, KST) return p.window > 0 ? launch_tc2<QA, 1, VA, KST, true>(ctx, m, a, B, S) : launch_tc2<QA, 1, VA, KST, false>(ctx, m, a, B, S)
+#define LATENT_TC2(QA, VA, KST) return p.window > 0 ? launch_tc2<QA, 1, VA, KST, true, false>(ctx, m, a, B, S) : launch_tc2<QA, 1, VA, KST, false, false>(ctx, m, a, B, S)
   if (p.dim <= 64) {
     if (p.vdim <= 64) LATENT_TC2(1, 1, 2);
     LATENT_TC2(1, 2, 2);

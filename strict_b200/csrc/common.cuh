@@ -219,6 +219,12 @@ struct GroupNormArgs {
   void *y1 = nullptr, *y2 = nullptr;
   int64_t ldy = 0;
   bool f32 = false;              // y in fp32
+  // Two sublayers that feed the residual under scales of their own: the first splits0 partial sums belong to the first one;
+  // x += mult * (scale0 * (sum of those) + scale1 * (sum of the rest)). Scales are [d], null: 1.
+  int splits0 = 8;
+  const float *scale0 = nullptr, *scale1 = nullptr;
+  float mult = 1.f;
+  float out_scale = 1.f;         // factor on y1 and y2
 };
 int k_group_norm(strictb200_ctx*, const GroupNormArgs& a, int64_t M, int64_t d);
 void sb_xielu_coefficients(float p, float q, float* pos, float* neg);
@@ -271,7 +277,14 @@ struct RopeArgs {
   bf16* vcache = nullptr;
 };
 int k_rope_qknorm_kvappend(strictb200_ctx*, const RopeArgs& a, int64_t T);
-int sb_rope_table(strictb200_ctx*, int max_pos, int D, double theta, float** d_cos, float** d_sin);
+// Frequencies stretched for longer contexts (YaRN): a pair that turns more than `fast` times within `original` positions
+// keeps its frequency, one that turns less than `slow` times has it divided by `factor`, a linear ramp in between; cos and
+// sin are multiplied by 0.1 ln(factor) + 1. factor 0: none.
+struct RopeScaling {
+  double factor = 0, original = 0, fast = 0, slow = 0;
+  bool operator==(const RopeScaling& o) const { return factor == o.factor && original == o.original && fast == o.fast && slow == o.slow; }
+};
+int sb_rope_table(strictb200_ctx*, int max_pos, int D, double theta, float** d_cos, float** d_sin, const RopeScaling& scaling = RopeScaling());
 // gemm_fp8.cu
 struct GemmArgs {
   int64_t M = 0, N = 0, K = 0;
@@ -299,11 +312,14 @@ struct Bf16Epilogue {
   float* out_f32 = nullptr;   // [M, ldo]
   bf16* out_bf16 = nullptr;   // [M, ldo] (used when out_f32 is null)
   int64_t ldo = 0;
-  int accumulate = 0;         // out_f32 += value (the residual stream)
+  int accumulate = 0;         // out_f32 += value (the residual stream), times alpha * col_scale[n] when col_scale is given
+  const float* col_scale = nullptr;
+  float alpha = 1.f;
   int n_switch = 0, x_row_off = 0;
   bf16* act_out = nullptr;    // [M, ld_act], column n - n_switch
   int64_t ld_act = 0;
   float act_pos = 0.f, act_neg = 0.f;  // xIELU coefficients (sb_xielu)
+  int glu = 0;                // 1: from n_switch on columns are (gate, up) pairs; act_out column (n - n_switch) / 2 = relu(gate) * up
 };
 struct GemmBf16Args {
   int64_t M = 0, N = 0, K = 0;  // K in elements; rows may end inside a 64-element block (the copies fill with zeros)
@@ -313,6 +329,10 @@ struct GemmBf16Args {
   int64_t ldw = 0;
   float* part = nullptr;        // [splits][M,N] raw sums instead of an epilogue
   int splits = 1;
+  int64_t k_switch = 0;         // > 0 (a multiple of 64, with part): the first splits0 splits share the columns of K before it, the others those after it
+  int splits0 = 0;
+  int group_n = 0;              // > 0: block-diagonal product, columns [g * group_n, (g + 1) * group_n) read x from its column g * group_k on
+  int64_t group_k = 0;          // (group_n must be a multiple of the kernel's channel tile: 128 up to 128 tokens, 256 beyond)
   Bf16Epilogue e;
 };
 int k_gemm_bf16(strictb200_ctx*, const GemmBf16Args& g);
@@ -329,8 +349,10 @@ struct GemmF32Args {
   const float* bias = nullptr;
   float* y = nullptr;
   int64_t ldy = 0;
-  int mode = 0;  // 0 store, 1 add to y, 2 GELU, 3 xIELU
+  int mode = 0;  // 0 store, 1 add to y, 2 GELU, 3 xIELU, 4 add alpha * col_scale[n] * value to y (col_scale null: 1)
   float act_pos = 0.f, act_neg = 0.f;
+  const float* col_scale = nullptr;
+  float alpha = 1.f;
 };
 int k_gemm_f32(strictb200_ctx*, const GemmF32Args& g);
 // attention.cu
@@ -353,6 +375,20 @@ struct LatentPrefillArgs {
   bf16* out = nullptr;          // row t, head h: out + t * ldo + h * vdim
   int64_t ldo = 0;
 };
+// the same kernel over grouped heads straight from the cache, with a sink and a gate per head
+struct HeadPrefillArgs {
+  const bf16* q = nullptr;      // [q_rows, H, row_dims]
+  int64_t q_rows = 0;
+  const bf16 *k = nullptr, *v = nullptr;  // [B, Hkv, maxlen, row_dims]
+  const int32_t *lens = nullptr, *past = nullptr, *qstart = nullptr;  // [B]
+  int B = 0, S = 0, H = 0, Hkv = 0, maxlen = 0, row_dims = 128, vdim = 128;
+  float scale = 1.f;
+  int sink = 0;
+  const float* gate = nullptr;  // [q_rows, H]
+  bf16* out = nullptr;          // row t, head h: out + t * ldo + h * vdim
+  int64_t ldo = 0;
+};
+int k_attn_prefill_heads(strictb200_ctx*, const HeadPrefillArgs& a);
 bool sb_latent_prefill_fits(int dim, int rot, int vdim);
 int k_attn_prefill_latent(strictb200_ctx*, const LatentPrefillArgs& a);
 // latent.cu: latent attention (one low-rank vector and one rotated key part per position instead of keys and values per head)
@@ -415,6 +451,111 @@ int k_latent_attn_any(strictb200_ctx*, const LatentShape& s, bool f32, const voi
 // rows of the cache of several sequences one after the other: dst row koff[j] + i = cache row kpos0[j] + i of sequence j, i < n[j]
 int k_latent_gather(strictb200_ctx*, const bf16* cache, int64_t maxlen, int row, const int32_t* koff, const int32_t* kpos0, const int32_t* lens, int nb,
                     int max_n, bf16* dst);
+// heads.cu: softmax attention over grouped heads of any width (optional RMS norm of the rotated queries and keys, sink, output
+// gate per head), and the projection rows of every mixer that has rotated heads
+struct HeadShape {
+  int H = 0, G = 0, dim = 0, vdim = 0, rot = 0;  // query heads, key/value heads, query/key and value dims, rotated dims (first ones, i with i + rot/2)
+  float scale = 1.f;
+  float k_scale = 1.f;  // factor on the rotated keys
+  int qk_norm = 0;      // 1: rotated queries and keys divided by their root mean square
+  int sink = 0;         // 1: one more key in the softmax denominator, score 0, no value
+  int gate = 0;         // 1: a column per head; its sigmoid multiplies the head's output
+  SB_HD int row() const {  // dims of a query, key or value row in memory (zeros beyond dim or vdim)
+    const int m = dim > vdim ? dim : vdim;
+    return m <= 64 ? 64 : m <= 128 ? 128 : (m + 7) & ~7;
+  }
+  SB_HD int n_in() const { return H * dim + G * (dim + vdim) + (gate ? H : 0); }
+};
+// The feed-forward's columns of a projection, finished: kind 1 xIELU of columns [col, col + n), kind 2 relu(gate) * up of
+// the n column pairs from col on. out[t * ld + i], bf16 or fp32 like the rest of the launch.
+struct ActArgs {
+  int kind = 0, col = 0, n = 0;
+  float pos = 0.f, neg = 0.f;
+  void* out = nullptr;
+  int64_t ld = 0;
+};
+// Rows of a projection: column c of row t is the sum over splits of in[(split * T + t) * ld + c].
+struct ProjRows {
+  const float* in = nullptr;
+  int64_t ld = 0;
+  int splits = 1;  // at most 8
+};
+// Columns [q heads | k heads | v heads | gates] become rotated rows.
+struct HeadSplitArgs {
+  HeadShape s;
+  ProjRows p;
+  const int32_t *seq = nullptr, *pos = nullptr, *lens = nullptr;  // row t: sequence seq[t] (null: t) at pos[t] (null: lens[seq])
+  const float *cos_t = nullptr, *sin_t = nullptr;                 // [max_pos, rot/2]
+  int max_pos = 0, maxlen = 0;
+  float eps = 1e-5f;
+  void* q_out = nullptr;               // [T, H, row]
+  void *k_out = nullptr, *v_out = nullptr;  // caches [B, G, maxlen, row], or [T, G, row] with dense
+  bool dense = false;
+  float* gate_out = nullptr;           // [T, H]
+  bool f32 = false;
+  ActArgs act;
+};
+int k_head_split(strictb200_ctx*, const HeadSplitArgs& a, int64_t T);
+// one block per row and head, straight from the cache; prompt rows (seq, pos) and decode rows (lens)
+int k_head_attn_any(strictb200_ctx*, const HeadShape& s, bool f32, const void* q, const void* kc, const void* vc, const float* gate, const int32_t* seq,
+                    const int32_t* pos, const int32_t* lens, int64_t T, int maxlen, void* out, int64_t ldo);
+// merge of the key chunks of k_attn_decode_chunks
+int k_head_combine(strictb200_ctx*, const HeadShape& s, const float* o_part, const float* ml_part, const float* gate, const int32_t* lens, int B, int maxlen,
+                   int chunk, int nsplit, bf16* out, int64_t ldo);
+int k_act_rows(strictb200_ctx*, const ProjRows& p, const ActArgs& a, bool f32, int64_t T);
+// recurrent.cu: layers with a state per sequence instead of a cache (all states fp32)
+// Real-gated linear recurrence behind a causal convolution per channel. Projection columns [y | x], `width` each.
+struct GatedShape {
+  int width = 0, taps = 1, blocks = 1;
+  SB_HD int bs() const { return width / blocks; }
+  SB_HD int bs_p() const { return (bs() + 7) & ~7; }       // columns of a block in the convolution's output, which the gate product reads
+  SB_HD int64_t ld_u() const { return (int64_t)blocks * bs_p(); }
+};
+struct GatedArgs {
+  GatedShape s;
+  ProjRows p;
+  const float *y_bias = nullptr, *x_bias = nullptr;          // [width]
+  const float *conv = nullptr, *conv_bias = nullptr;         // [width, taps], [width]
+  const float *r_bias = nullptr, *i_bias = nullptr;          // [width]
+  const float* decay = nullptr;                              // [width] -8 softplus(lam)
+  float* hist = nullptr;                                     // [B, taps - 1, width] the convolution's last inputs
+  float* state = nullptr;                                    // [B, width]
+  const int32_t *seq = nullptr, *qstart = nullptr, *lens = nullptr, *past = nullptr;  // prompt rows; null: row t is the next token of sequence t
+  int nb = 0, max_new = 0;
+  void* u = nullptr;                                         // [T, ld_u]
+  const float* gates = nullptr;                              // [T, 2 width]: block by block, its bs values for r, then those for i
+  void* out = nullptr;                                       // [T, ldo]
+  int64_t ldo = 0;
+  bool f32 = false;
+  ActArgs act;
+};
+int k_gated_conv(strictb200_ctx*, const GatedArgs& a, int64_t T);   // u, and the new hist; with act, the feed-forward's columns too
+int k_gated_scan(strictb200_ctx*, const GatedArgs& a, int64_t T);   // the recurrence and out = S * gelu(y)
+// Retention: S <- decay S + k v^T, o = S^T q, per head; o over its root mean square, times silu(g). Projection columns [q | k | v | g].
+struct RetentionArgs {
+  HeadShape s;
+  ProjRows p;
+  const float* decay = nullptr;      // [H]
+  const float* log2_decay = nullptr; // [H]
+  float* state = nullptr;            // [B, H, dim, vdim]
+  const void *q = nullptr, *k = nullptr, *v = nullptr;  // [T, H, row] (k_head_split, dense)
+  const int32_t *qstart = nullptr, *lens = nullptr, *past = nullptr;  // prompt rows of nb sequences; null: row t is the next token of sequence t
+  int nb = 0, max_new = 0;
+  float eps = 1e-5f;
+  void* out = nullptr;
+  int64_t ldo = 0;
+  bool f32 = false;
+  // k_retention_decode: straight from the projection
+  const float *cos_t = nullptr, *sin_t = nullptr;
+  const int32_t* cache_lens = nullptr;  // [B] positions of the new tokens
+  int max_pos = 0;
+  ActArgs act;
+};
+int k_retention_any(strictb200_ctx*, const RetentionArgs& a);            // any widths, token by token
+bool sb_retention_prefill_fits(const HeadShape& s);
+int k_retention_prefill(strictb200_ctx*, const RetentionArgs& a, int64_t T);  // retention_tc.cu: chunks of 128 tokens
+bool sb_retention_decode_fits(const HeadShape& s);
+int k_retention_decode(strictb200_ctx*, const RetentionArgs& a, int64_t B);
 size_t sb_attn_decode_scratch(int B, int Hq, int D, int nsplit);
 int sb_attn_decode_splits(strictb200_ctx*, int B, int Hkv, int maxlen);
 int sb_attn_decode_chunk(strictb200_ctx*, int B, int Hkv, int maxlen, int len_plan);  // keys per block for sequences of about len_plan keys (at most 8 chunks cover maxlen)
@@ -423,6 +564,8 @@ int sb_attn_decode_chunk(strictb200_ctx*, int B, int Hkv, int maxlen, int len_pl
 int k_attn_decode(strictb200_ctx*, const bf16* q, const bf16* kc, const bf16* vc, const int32_t* lens, int len_add, int B, int Hq,
                   int Hkv, int D, int maxlen, float scale, int nsplit, float* scratch, bf16* out, uint8_t* q_out, float* qscale_out,
                   const RopeArgs* rope = nullptr, int chunk = 0);
+int k_attn_decode_chunks(strictb200_ctx*, int HD, const bf16* q, const bf16* kc, const bf16* vc, const int32_t* lens, int B, int Hq, int Hkv, int maxlen,
+                         float scale, int nsplit, int chunk, float* o_part, float* ml_part);
 int k_attn_f32(strictb200_ctx*, const float* qkv, float* kc, float* vc, const int32_t* seq, const int32_t* pos, const int32_t* lens,
                int64_t T, int H, int D, int maxlen, float scale, float* out);
 // sampling.cu
@@ -455,8 +598,32 @@ __device__ __forceinline__ uint32_t f32_to_bf16_bits(float f);
 // same side of n_switch). bf16 rows: neighbouring lanes trade tokens so that each stores two channels at a time.
 __device__ __forceinline__ void sb_bf16_store16(const Bf16Epilogue& e, int M, int N, int m0, int n, const uint32_t* r) {
   const bool act = e.act_out && n >= e.n_switch;
+  if (act && e.glu) {
+    // The lanes of a pair hold the gate and the up value of one channel. Each takes eight tokens, then the lanes of two
+    // neighbouring channels trade so that each stores both channels of four tokens.
+    const int odd = n & 1, second = (n >> 1) & 1, j = (n - e.n_switch) >> 1, nf = (N - e.n_switch) >> 1;
+    float p[8];
+#pragma unroll
+    for (int i = 0; i < 8; i++) {
+      const float got = __uint_as_float(__shfl_xor_sync(0xffffffffu, odd ? r[i] : r[8 + i], 1));
+      const float gate = odd ? got : __uint_as_float(r[i]), up = odd ? __uint_as_float(r[8 + i]) : got;
+      p[i] = fmaxf(gate, 0.f) * up;
+    }
+    bf16* o = e.act_out + (int64_t)(m0 + odd * 8 + second * 4) * e.ld_act + (j - second);
+#pragma unroll
+    for (int i = 0; i < 4; i++, o += e.ld_act) {
+      const float got = __shfl_xor_sync(0xffffffffu, second ? p[i] : p[4 + i], 2);
+      const float lo = second ? got : p[i], hi = second ? p[4 + i] : got;
+      if (m0 + odd * 8 + second * 4 + i < M && j - second < nf) {
+        if (j - second + 1 < nf) *(uint32_t*)o = f32_to_bf16_bits(lo) | (f32_to_bf16_bits(hi) << 16);
+        else *o = __float2bfloat16_rn(lo);
+      }
+    }
+    return;
+  }
   if (!act && e.out_f32) {
     if (n >= N) return;
+    const float cs = e.col_scale ? e.alpha * e.col_scale[n] : e.alpha;
     float* o = e.out_f32 + (int64_t)m0 * e.ldo + n;
     float old[16];  // all read before the first store, so that the sixteen reads overlap
     if (e.accumulate) {
@@ -465,7 +632,7 @@ __device__ __forceinline__ void sb_bf16_store16(const Bf16Epilogue& e, int M, in
     }
 #pragma unroll
     for (int j = 0; j < 16; j++, o += e.ldo)
-      if (m0 + j < M) *o = e.accumulate ? old[j] + __uint_as_float(r[j]) : __uint_as_float(r[j]);
+      if (m0 + j < M) *o = e.accumulate ? fmaf(cs, __uint_as_float(r[j]), old[j]) : __uint_as_float(r[j]);
     return;
   }
   const int64_t ld = act ? e.ld_act : e.ldo;

@@ -1,7 +1,8 @@
 // fp32 linear layer of the GPT-2 path: Y[M,N] = X[M,K] . W[N,K]^T + bias. Decode (M = 1) is
 // a pure HBM stream over W; one warp (or 2-8 for a long row) per output channel, lanes split K with 128-bit loads,
 // warp-shuffle reduction. Up to 8 token rows share one pass over a weight row. `accumulate`: 0
-// stores the result, 1 adds it to Y (residual), 2 stores GELU(result) (the MLP's first layer), 3 xIELU(result).
+// stores the result, 1 adds it to Y (residual), 2 stores GELU(result) (the MLP's first layer), 3 xIELU(result), 4 adds
+// alpha * col_scale[n] * result to Y.
 // Rows of X, W and Y may be wider than the product (ldx, ldw, ldy).
 #include "common.cuh"
 
@@ -12,7 +13,7 @@ constexpr int F32_PRE = 8;  // float4 of its weight row a lane fetches before th
 
 __global__ void __launch_bounds__(256) gemm_f32_kernel(int M, int N, int K, const float* __restrict__ x, int64_t ldx, const float* __restrict__ w,
                                                        int64_t ldw, const float* __restrict__ bias, float* __restrict__ y, int64_t ldy, int accumulate, int ks,
-                                                       float act_pos, float act_neg) {
+                                                       float act_pos, float act_neg, const float* __restrict__ col_scale, float alpha) {
   // The block's 8 warps are 8/ks output channels x ks slices of K: a long row (K > 1024) is
   // walked by several warps at once so that every lane still has all its loads in flight in one
   // round trip; the slices' sums meet in shared memory and are added in slice order.
@@ -66,6 +67,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(int M, int N, int K, cons
     for (int s2 = 0; s2 < ks; s2++) v += part[warp + s2][lane];
     const int64_t o = (int64_t)(m0 + lane) * ldy + n;
     v += bn;
+    if (accumulate == 4) { y[o] += alpha * (col_scale ? col_scale[n] : 1.f) * v; return; }
     y[o] = accumulate == 1 ? y[o] + v : accumulate == 2 ? sb_gelu_tanh(v) : accumulate == 3 ? sb_xielu(v, act_pos, act_neg) : v;
   }
 }
@@ -87,7 +89,7 @@ int k_gemm_f32(strictb200_ctx* ctx, const GemmF32Args& g) {
   dim3 grid((unsigned)((N + rows - 1) / rows), (unsigned)((M + F32_MT - 1) / F32_MT));
   if (grid.y > 65535) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_f32: M too large");
   SB_CUDA(sb_launch(ctx, gemm_f32_kernel, grid, dim3(256), 0, (int)M, (int)N, (int)K, g.x, g.ldx, g.w, g.ldw, g.bias, g.y, g.ldy, g.mode, ks, g.act_pos,
-                    g.act_neg));
+                    g.act_neg, g.col_scale, g.alpha));
   ctx->launches++;
   return STRICTB200_OK;
 }

@@ -155,7 +155,8 @@ struct PairArgs {
   int* status;   // host-visible error word
   int tiles_n;   // 256-channel tiles; tile = tt * tiles_n + tn
   int tiles;
-  Bf16Epilogue e;  // BF16 only
+  Bf16Epilogue e;        // BF16 only, and so are the rest
+  int group_n, group_k;  // block-diagonal product: channels per group, bytes of an operand row per group (0: dense)
 };
 
 // BF16: plain bf16 operands, one operand row (accumulator column) per token, so a tile is 256 channels x 256 tokens; K
@@ -210,7 +211,8 @@ __global__ void __launch_bounds__(192) gemm_pair_kernel(const __grid_constant__ 
         if (leader) mbar_expect_tx(smem_u32(&bar_full[s]), 2 * STAGE_BYTES);  // the bytes of both blocks
         const uint32_t dst = smem_u32(smem + (size_t)s * STAGE_BYTES);
         tma_load_2d_pair(dst, &map_w, kb * BK, wy, full_leader);
-        tma_load_2d_pair(dst + BN * BK, &map_x, kb * BK, xy, full_leader);
+        const int xk = BF16 && a.group_n > 0 ? (tile % a.tiles_n) * 2 * BN / a.group_n * a.group_k : 0;
+        tma_load_2d_pair(dst + BN * BK, &map_x, xk + kb * BK, xy, full_leader);
       }
     }
   } else if (warp == 1) {
@@ -343,7 +345,7 @@ int k_gemm_fp8_tmem_pair(strictb200_ctx* ctx, const GemmArgs& g) {
   CUtensorMap mw, mx;
   SB_TRY(make_map(&mw, g.wq, g.N, g.K, g.ldw));
   SB_TRY(make_map(&mx, g.xq, Mq, g.K, g.ldx));
-  PairArgs pa{(int)g.M, (int)Mq, (int)g.N, (int)g.K, g.sx, g.sw, g.out, g.out_f32, ctx->d_status, (int)tiles_n, (int)tiles, {}};
+  PairArgs pa{(int)g.M, (int)Mq, (int)g.N, (int)g.K, g.sx, g.sw, g.out, g.out_f32, ctx->d_status, (int)tiles_n, (int)tiles, {}, 0, 0};
   int64_t pairs = ctx->sm_count / 2;
   if (pairs > tiles) pairs = tiles;
   SB_CUDA(sb_launch_cluster(ctx, gemm_pair_kernel<false>, dim3((unsigned)(2 * pairs)), dim3(192), smem, dim3(2, 1, 1), mw, mx, pa));
@@ -360,9 +362,10 @@ int k_gemm_bf16_tmem_pair(strictb200_ctx* ctx, const GemmBf16Args& b) {
   static SbDeviceOnce once;
   SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(gemm_pair_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
   CUtensorMap mw, mx;
+  if (b.group_n && (b.group_n % (2 * BN) || b.group_k % 8)) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_bf16: groups must fill channel tiles");
   SB_TRY(make_map(&mw, b.w, b.N, kbytes, 2 * b.ldw));
-  SB_TRY(make_map(&mx, b.x, b.x_rows ? b.x_rows : b.M, kbytes, 2 * b.ldx));
-  PairArgs pa{(int)b.M, (int)b.M, (int)b.N, (int)kbytes, nullptr, nullptr, nullptr, 1, ctx->d_status, (int)tiles_n, (int)tiles, b.e};
+  SB_TRY(make_map(&mx, b.x, b.x_rows ? b.x_rows : b.M, b.group_n ? 2 * ((b.N + b.group_n - 1) / b.group_n) * b.group_k : kbytes, 2 * b.ldx));
+  PairArgs pa{(int)b.M, (int)b.M, (int)b.N, (int)kbytes, nullptr, nullptr, nullptr, 1, ctx->d_status, (int)tiles_n, (int)tiles, b.e, b.group_n, (int)(2 * b.group_k)};
   int64_t pairs = ctx->sm_count / 2;
   if (pairs > tiles) pairs = tiles;
   SB_CUDA(sb_launch_cluster(ctx, gemm_pair_kernel<true>, dim3((unsigned)(2 * pairs)), dim3(192), smem, dim3(2, 1, 1), mw, mx, pa));

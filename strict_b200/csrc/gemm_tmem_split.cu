@@ -122,7 +122,9 @@ struct TmemArgs {
   int raw;
   int* status;  // host-visible error word
   int prefetch;  // issue the first ring of weight loads before the dependency wait
-  Bf16Epilogue e;  // BF16 only
+  Bf16Epilogue e;  // BF16 only, and so are the rest
+  int kb_switch, splits0;  // K blocks of the first part of K, and the splits that share it (0: one part)
+  int group_n, group_k;    // block-diagonal product: channels per group, bytes of an operand row per group (0: dense)
 };
 enum { KIND_F8 = 0, KIND_I8 = 1, KIND_BF16 = 2 };
 
@@ -150,8 +152,19 @@ __global__ void __launch_bounds__(192) gemm_tmem_kernel(const __grid_constant__ 
   // split z owns the k-blocks [z * nkb_all / splits, (z + 1) * nkb_all / splits): sizes differ by at most one
   const int nkb_all = (a.K + BK - 1) / BK;
   const int x0 = KIND == KIND_BF16 && a.e.n_switch > 0 && n0 >= a.e.n_switch ? a.e.x_row_off + t0 : t0;  // first operand row
-  const int kb_first = (int)((int64_t)blockIdx.z * nkb_all / a.splits), kb_last = (int)((int64_t)(blockIdx.z + 1) * nkb_all / a.splits);
+  int kb_first, kb_last;
+  if (KIND == KIND_BF16 && a.splits0 > 0) {
+    const bool first = (int)blockIdx.z < a.splits0;
+    const int base = first ? 0 : a.kb_switch, count = first ? a.kb_switch : nkb_all - a.kb_switch;
+    const int z = first ? (int)blockIdx.z : (int)blockIdx.z - a.splits0, nz = first ? a.splits0 : a.splits - a.splits0;
+    kb_first = base + (int)((int64_t)z * count / nz);
+    kb_last = base + (int)((int64_t)(z + 1) * count / nz);
+  } else {
+    kb_first = (int)((int64_t)blockIdx.z * nkb_all / a.splits);
+    kb_last = (int)((int64_t)(blockIdx.z + 1) * nkb_all / a.splits);
+  }
   const int k_begin = kb_first * BK, nkb = kb_last - kb_first;
+  const int xk = KIND == KIND_BF16 && a.group_n > 0 ? n0 / a.group_n * a.group_k + k_begin : k_begin;  // the same columns in the operand rows
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < STAGES; s++) { mbar_init(smem_u32(&bar_full[s]), 1); mbar_init(smem_u32(&bar_empty[s]), 1); }
@@ -185,7 +198,7 @@ __global__ void __launch_bounds__(192) gemm_tmem_kernel(const __grid_constant__ 
       pdl_wait();
       SB_TRACE_WAITED();
       for (int kb = 0; kb < npre; kb++)
-        tma_load_2d(smem_u32(smem + (size_t)kb * STAGE_BYTES) + BN * BK, &map_x, k_begin + kb * BK, x0, smem_u32(&bar_full[kb]));
+        tma_load_2d(smem_u32(smem + (size_t)kb * STAGE_BYTES) + BN * BK, &map_x, xk + kb * BK, x0, smem_u32(&bar_full[kb]));
       for (int kb = npre; kb < nkb; kb++) {
         int s = kb % STAGES;
         if (!mbar_wait(smem_u32(&bar_empty[s]), ((kb / STAGES) & 1) ^ 1)) { set_status(a.status, 1); abort_flag = 1; break; }
@@ -194,7 +207,7 @@ __global__ void __launch_bounds__(192) gemm_tmem_kernel(const __grid_constant__ 
         uint32_t dst = smem_u32(smem + (size_t)s * STAGE_BYTES);
         mbar_expect_tx(full, STAGE_BYTES);
         tma_load_2d_hint(dst, &map_w, k_begin + kb * BK, n0, full, w_policy);
-        tma_load_2d(dst + BN * BK, &map_x, k_begin + kb * BK, x0, full);
+        tma_load_2d(dst + BN * BK, &map_x, xk + kb * BK, x0, full);
       }
     }
   } else if (warp == 1) {
@@ -320,14 +333,14 @@ int make_map(CUtensorMap* map, const void* base, int64_t rows, int64_t K, int64_
 }
 
 template <int BT, int STAGES, int KIND = KIND_F8>
-int launch(strictb200_ctx* ctx, const GemmArgs& g, const TmemArgs& ta, int64_t x_rows = 0) {
+int launch(strictb200_ctx* ctx, const GemmArgs& g, const TmemArgs& ta, int64_t x_rows = 0, int64_t x_cols = 0) {
   constexpr int STAGE_BYTES = BN * BK + BT * BK;
   size_t smem = (size_t)STAGES * STAGE_BYTES + 1024;  // + slack for the 1024-byte round-up
   static SbDeviceOnce once;  // one per instantiation
   SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(gemm_tmem_kernel<BT, STAGES, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
   CUtensorMap mw, mx;
   SB_TRY(make_map(&mw, g.wq, g.N, g.K, g.ldw, BN));
-  SB_TRY(make_map(&mx, g.xq, x_rows ? x_rows : ta.Mq, g.K, g.ldx, BT));
+  SB_TRY(make_map(&mx, g.xq, x_rows ? x_rows : ta.Mq, x_cols ? x_cols : g.K, g.ldx, BT));
   dim3 grid((unsigned)((g.N + BN - 1) / BN), (unsigned)((ta.Mq + BT - 1) / BT), (unsigned)g.splits);
   if (grid.y > 65535) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_fp8: M too large for one launch");
   SB_CUDA(sb_launch(ctx, gemm_tmem_kernel<BT, STAGES, KIND>, grid, dim3(192), smem, mw, mx, ta));
@@ -372,15 +385,21 @@ int k_gemm_bf16_tmem_split(strictb200_ctx* ctx, const GemmBf16Args& b) {
   if (b.splits < 1 || b.splits > nkb) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_bf16: more K splits than K blocks");
   if (b.splits > 1 && !b.part) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_bf16: split-K needs a partial buffer");
   if (b.M > 256) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "the split bf16 GEMM takes at most 256 tokens");
+  if (b.k_switch && (!b.part || b.k_switch % 64 || b.k_switch >= b.K || b.splits0 < 1 || b.splits0 >= b.splits || b.splits0 > b.k_switch / 64 ||
+                     b.splits - b.splits0 > nkb - b.k_switch / 64))
+    return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_bf16: bad split of a K of two parts");
+  if (b.group_n && (b.group_n % BN || b.group_k % 8)) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gemm_bf16: groups must fill channel tiles");
   SB_TRY(get_encode());
-  TmemArgs ta{(int)b.M, (int)b.M, (int)b.N, (int)kbytes, nullptr, nullptr, nullptr, 1, b.part, b.splits, b.part ? 1 : 0, ctx->d_status, ctx->opt.prefetch, b.e};
+  TmemArgs ta{(int)b.M, (int)b.M, (int)b.N, (int)kbytes, nullptr, nullptr, nullptr, 1, b.part, b.splits, b.part ? 1 : 0, ctx->d_status, ctx->opt.prefetch, b.e,
+              (int)(b.k_switch / 64), b.k_switch ? b.splits0 : 0, b.group_n, (int)(2 * b.group_k)};
   GemmArgs g;
   g.M = b.M; g.N = b.N; g.K = kbytes;
   g.xq = (const uint8_t*)b.x; g.ldx = 2 * b.ldx; g.wq = (const uint8_t*)b.w; g.ldw = 2 * b.ldw; g.splits = b.splits;
   const int64_t blocks = ((b.N + BN - 1) / BN) * b.splits, x_rows = b.x_rows ? b.x_rows : b.M;
+  const int64_t x_cols = b.group_n ? 2 * ((b.N + b.group_n - 1) / b.group_n) * b.group_k : 0;
   const bool deep = ctx->opt.deep_ring && blocks <= ctx->sm_count;
-  if (b.M <= 32) return deep ? launch<32, 10, KIND_BF16>(ctx, g, ta, x_rows) : launch<32, 5, KIND_BF16>(ctx, g, ta, x_rows);
-  if (b.M <= 64) return deep ? launch<64, 9, KIND_BF16>(ctx, g, ta, x_rows) : launch<64, 4, KIND_BF16>(ctx, g, ta, x_rows);
-  if (b.M <= 128) return launch<128, 4, KIND_BF16>(ctx, g, ta, x_rows);
-  return launch<256, 4, KIND_BF16>(ctx, g, ta, x_rows);
+  if (b.M <= 32) return deep ? launch<32, 10, KIND_BF16>(ctx, g, ta, x_rows, x_cols) : launch<32, 5, KIND_BF16>(ctx, g, ta, x_rows, x_cols);
+  if (b.M <= 64) return deep ? launch<64, 9, KIND_BF16>(ctx, g, ta, x_rows, x_cols) : launch<64, 4, KIND_BF16>(ctx, g, ta, x_rows, x_cols);
+  if (b.M <= 128) return launch<128, 4, KIND_BF16>(ctx, g, ta, x_rows, x_cols);
+  return launch<256, 4, KIND_BF16>(ctx, g, ta, x_rows, x_cols);
 }

@@ -909,8 +909,8 @@ int strictb200_kv_create(strictb200_model* m, int batch, int maxlen, strictb200_
   const size_t esz = qwen ? 2 : 4;
   kv->layer_stride = (size_t)batch * (qwen ? m->Hkv_l : m->c.n_kv_heads) * kv->maxlen * m->c.head_dim;
   size_t bytes = kv->layer_stride * m->c.n_layers * esz;
-  if (m->stack) {  // one array of latent rows; nothing in v
-    SB_TRY(sb_stack_kv_layout(m, kv, &kv->layer_stride));
+  if (m->stack) {  // one array of rows, nothing in v; states apart
+    SB_TRY(sb_stack_kv_layout(m, kv, &kv->layer_stride, &kv->state_floats));
     bytes = kv->layer_stride * (m->c.n_layers ? sb_stack_esz(m) : 0);
   }
   auto fail = [&](int s) { strictb200_kv_destroy(kv); return s; };
@@ -923,6 +923,10 @@ int strictb200_kv_create(strictb200_model* m, int batch, int maxlen, strictb200_
 #define K_TRY(e) do { st = (e); if (st != STRICTB200_OK) return fail(st); } while (0)
   K_TRY(alloc(&kv->k, bytes));
   if (!m->stack) K_TRY(alloc(&kv->v, bytes));
+  if (kv->state_floats) {
+    K_TRY(alloc((void**)&kv->state, kv->state_floats * 4));
+    cudaMemsetAsync(kv->state, 0, kv->state_floats * 4, ctx->stream);
+  }
   // zero so that the padding rows of a partly filled 64-key tile are finite
   if (cudaMemsetAsync(kv->k, 0, bytes, ctx->stream) != cudaSuccess ||
       (kv->v && cudaMemsetAsync(kv->v, 0, bytes, ctx->stream) != cudaSuccess))
@@ -960,6 +964,7 @@ int strictb200_kv_reset(strictb200_kv* kv) {
   strictb200_ctx* ctx = kv->m->ctx;
   SB_ENTER(ctx);
   SB_CUDA(cudaMemsetAsync(kv->d_lens, 0, (size_t)kv->B * 4, ctx->stream));
+  if (kv->state) SB_CUDA(cudaMemsetAsync(kv->state, 0, kv->state_floats * 4, ctx->stream));
   SB_CUDA(cudaStreamSynchronize(ctx->stream));
   std::fill(kv->h_lens.begin(), kv->h_lens.end(), 0);
   kv->plan_until = 0;  // the next decode step plans the attention's key chunks for the new lengths
@@ -985,6 +990,7 @@ int strictb200_kv_fill_synthetic(strictb200_kv* kv, uint64_t seed, int len) {
   if (m->stack) {
     if (sb_stack_esz(m) == 2) SB_TRY(k_gen_normal_bf16(ctx, sb_stream_key(seed, 0x4B00), 0, (int64_t)kv->layer_stride, 1.0f, (bf16*)kv->k));
     else SB_TRY(k_gen_normal_f32(ctx, sb_stream_key(seed, 0x4B00), 0, (int64_t)kv->layer_stride, 1.0f, (float*)kv->k));
+    if (kv->state) SB_TRY(k_gen_normal_f32(ctx, sb_stream_key(seed, 0x5300), 0, (int64_t)kv->state_floats, 1.0f, kv->state));
   } else if (m->c.arch == STRICTB200_QWEN3) {
     SB_TRY(k_gen_normal_bf16(ctx, sb_stream_key(seed, 0x4B00 + m->rank), 0, (int64_t)n, 1.0f, (bf16*)kv->k));
     SB_TRY(k_gen_normal_bf16(ctx, sb_stream_key(seed, 0x5600 + m->rank), 0, (int64_t)n, 1.0f, (bf16*)kv->v));

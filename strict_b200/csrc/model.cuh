@@ -69,6 +69,9 @@ struct strictb200_kv {
   int plan_until = 0;    // the plan is kept until a sequence grows beyond this length
   std::vector<void*> allocs;
   std::vector<size_t> layer_off;           // stack models: first element of a layer's rows in k
+  float* state = nullptr;                  // stack models: states of the recurrent layers (zero before a sequence's first token)
+  size_t state_floats = 0;
+  std::vector<size_t> state_off;           // first float of a layer's states
   std::vector<int> layer_chunk;            // stack models: keys per chunk (x 32) + chunks of every layer's decode attention
   uint64_t plan_version = 0;               // stack models: constants the recorded step was made with
 };
@@ -180,7 +183,7 @@ struct PrefillChunk {  // the rows of one prefill chunk: nb sequences from b0 on
 int sb_stack_init_random(strictb200_model* m, uint64_t seed);
 int sb_stack_tensor(strictb200_model* m, const char* name, const void* h_in, void* h_out, size_t bytes);
 void sb_stack_destroy(strictb200_model* m);
-int sb_stack_kv_layout(strictb200_model* m, strictb200_kv* kv, size_t* elements);  // layer offsets of the cache
+int sb_stack_kv_layout(strictb200_model* m, strictb200_kv* kv, size_t* elements, size_t* state_floats);  // layer offsets of the cache and of the states
 bool sb_stack_plan(strictb200_model* m, strictb200_kv* kv, int longest);           // true: the decode step changed, record it again
 size_t sb_stack_esz(strictb200_model* m);                                          // bytes of a weight or cache element
 size_t sb_stack_decode_bytes(strictb200_model* m, strictb200_kv* kv);              // bytes of the decode buffers

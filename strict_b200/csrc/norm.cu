@@ -800,7 +800,12 @@ struct GroupNormDev {
   int gw;  // columns per group
   int cb;  // blocks (one cluster) per group
   int* status;
+  int splits0;
+  const float *scale0, *scale1;
+  float mult, out_scale;
 };
+// what the partial sums of a column add to the residual: the sublayers' sums under their scales
+__device__ __forceinline__ float residual_gain(const float* scale, float mult, int k) { return scale ? mult * scale[k] : mult; }
 template <typename T>
 __device__ __forceinline__ void store4(T* p, float a, float b, float c, float d);
 template <>
@@ -847,14 +852,19 @@ __global__ void __launch_bounds__(NI == 1 ? 1024 : 512) group_norm_kernel(GroupN
       float* xp = a.x + row * a.ldx + c0 + k;
       float4 x = *(const float4*)xp;
       if (a.part) {
-        float4 p[8], t = make_float4(0.f, 0.f, 0.f, 0.f);
+        float4 p[8], t = make_float4(0.f, 0.f, 0.f, 0.f), u = t;
 #pragma unroll
         for (int s = 0; s < 8; s++)
           if (s < a.splits) p[s] = *(const float4*)(a.part + ((int64_t)s * M + row) * a.ldp + c0 + k);
 #pragma unroll
         for (int s = 0; s < 8; s++)
-          if (s < a.splits) { t.x += p[s].x; t.y += p[s].y; t.z += p[s].z; t.w += p[s].w; }
-        x.x += t.x; x.y += t.y; x.z += t.z; x.w += t.w;
+          if (s < a.splits) {
+            float4& o = s < a.splits0 ? t : u;
+            o.x += p[s].x; o.y += p[s].y; o.z += p[s].z; o.w += p[s].w;
+          }
+        if (a.scale0) { const float4 c = *(const float4*)(a.scale0 + c0 + k); t.x *= c.x; t.y *= c.y; t.z *= c.z; t.w *= c.w; }
+        if (a.scale1) { const float4 c = *(const float4*)(a.scale1 + c0 + k); u.x *= c.x; u.y *= c.y; u.z *= c.z; u.w *= c.w; }
+        x.x = fmaf(a.mult, t.x + u.x, x.x); x.y = fmaf(a.mult, t.y + u.y, x.y); x.z = fmaf(a.mult, t.z + u.z, x.z); x.w = fmaf(a.mult, t.w + u.w, x.w);
         *(float4*)xp = x;
       }
       v[i] = x;
@@ -869,7 +879,7 @@ __global__ void __launch_bounds__(NI == 1 ? 1024 : 512) group_norm_kernel(GroupN
     ss = 0.f;
     for (int r = 0; r < a.cb; r++) ss += ((volatile float*)xch.slot[0])[r];
   }
-  const float r = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.gw), a.eps)));
+  const float r = __fdiv_rn(a.out_scale, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.gw), a.eps)));
 #pragma unroll
   for (int i = 0; i < NI; i++) {
     const int k = (i * (int)blockDim.x + (int)threadIdx.x) * 4;
@@ -913,7 +923,7 @@ __global__ void __launch_bounds__(256) group_norm_rows_kernel(GroupNormDev a, in
       const int first = k / a.gw * per;
       float ss = 0.f;
       for (int j = 0; j < per; j++) ss += sums[first + j];
-      const float r = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.gw), a.eps)));
+      const float r = __fdiv_rn(a.out_scale, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.gw), a.eps)));
       const float4 g = *(const float4*)(a.g1 + k), t = make_float4(v[i].x * r, v[i].y * r, v[i].z * r, v[i].w * r);
       store4<T>((T*)a.y1 + row * a.ldy + k, t.x * g.x, t.y * g.y, t.z * g.z, t.w * g.w);
       if (a.g2) {
@@ -937,16 +947,16 @@ __global__ void __launch_bounds__(256) group_norm_any_kernel(GroupNormDev a, int
     float* xp = a.x + row * a.ldx + c0 + k;
     float x = *xp;
     if (a.part) {
-      float t = 0.f;
-      for (int s = 0; s < a.splits; s++) t += a.part[((int64_t)s * M + row) * a.ldp + c0 + k];
-      x += t;
+      float t = 0.f, u = 0.f;
+      for (int s = 0; s < a.splits; s++) (s < a.splits0 ? t : u) += a.part[((int64_t)s * M + row) * a.ldp + c0 + k];
+      x += t * residual_gain(a.scale0, a.mult, c0 + k) + u * residual_gain(a.scale1, a.mult, c0 + k);
       *xp = x;
     }
     ss += x * x;
   }
   if (!a.g1) return;
   ss = block_sum(ss, red);
-  const float r = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.gw), a.eps)));
+  const float r = __fdiv_rn(a.out_scale, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.gw), a.eps)));
   for (int k = threadIdx.x; k < a.gw; k += blockDim.x) {
     const float t = a.x[row * a.ldx + c0 + k] * r;  // this thread's own column
     ((T*)a.y1)[row * a.ldy + c0 + k] = from_f32<T>(t * a.g1[c0 + k]);
@@ -958,7 +968,8 @@ __global__ void __launch_bounds__(256) group_norm_any_kernel(GroupNormDev a, int
 int k_group_norm(strictb200_ctx* ctx, const GroupNormArgs& a, int64_t M, int64_t d) {
   if (a.groups < 1 || d % a.groups) return sb_fail(STRICTB200_ERR_INVALID_ARG, "group_norm: the width must be a multiple of the groups");
   if (a.groups > 16383 || a.splits < 1 || a.splits > 8) return sb_fail(STRICTB200_ERR_INVALID_ARG, "group_norm: at most 16383 groups and 8 partial sums");
-  GroupNormDev v{a.x, a.ldx, a.part, a.ldp, a.splits, a.g1, a.g2, a.eps, a.y1, a.y2, a.ldy, (int)(d / a.groups), 1, ctx->d_status};
+  GroupNormDev v{a.x, a.ldx, a.part, a.ldp, a.splits, a.g1, a.g2, a.eps, a.y1, a.y2, a.ldy, (int)(d / a.groups), 1, ctx->d_status,
+                 a.splits0, a.scale0, a.scale1, a.mult, a.out_scale};
   const bool vec = v.gw % 4 == 0 && a.ldx % 4 == 0 && a.ldp % 4 == 0 && a.ldy % 4 == 0 && v.gw <= 8192;
   if (!vec) {
     dim3 grid((unsigned)M, (unsigned)a.groups);

@@ -1,0 +1,354 @@
+// Layers that carry a state per sequence instead of a cache. All states are fp32 and are advanced in place, so a prompt may be
+// cut anywhere.
+//
+// Real-gated linear recurrence: u = causal convolution of x per channel; r, i = sigmoid of block-diagonal products of u;
+//   log a = -8 r softplus(lam), S <- a S + sqrt(1 - a^2) i u, out = S gelu(y).
+//   * k_gated_conv: u as the operand of the gate product (rounded to bf16 there, so that the product of bf16 matrices with fp32
+//     sums is the exact product of what the recurrence uses), and the convolution's last inputs.
+//   * k_gated_scan: prompts run 256 tokens at a time in a block of 32 channels: every warp folds eight tokens into one (a, b)
+//     pair, the pairs meet in shared memory, and each warp replays its tokens from the state before them. Decode is one
+//     step per channel. sqrt(1 - a^2) is taken as sqrt(-expm1(2 log a)), which stays exact where a is close to one.
+// Retention: S <- decay S + k v^T, o = S^T q.
+//   * k_retention_decode: one block per head streams the state once, from the projection's partial sums to the gated output.
+//   * k_retention_any: any widths, token by token. Prompts of usual widths: retention_tc.cu.
+#include "mixers.cuh"
+
+using namespace mix;
+
+namespace {
+
+// ------------------------------------------------------------------ convolution
+// grid rows * (channel blocks + activation blocks), 256 threads
+template <typename T>
+__global__ void __launch_bounds__(256) gated_conv_kernel(GatedArgs a, int64_t rows, int ch_blocks, int act_blks) {
+  SB_TRACE_BEGIN();
+  pdl_trigger();
+  const int per_row = ch_blocks + act_blks;
+  const int64_t t = blockIdx.x / per_row;
+  const int blk = blockIdx.x % per_row, w = a.s.width, taps = a.s.taps;
+  pdl_wait();
+  SB_TRACE_WAITED();
+  if (blk >= ch_blocks) {
+    act_block<T>(a.act, a.p, rows, t, blk - ch_blocks);
+  } else {
+    const int c = blk * 256 + (int)threadIdx.x;
+    if (c < w) {
+      const int b = a.seq ? a.seq[t] : (int)t;
+      const int64_t li = a.seq ? t - a.qstart[b] : 0;  // tokens of this launch before the row
+      float* hist = a.hist + (int64_t)b * (taps - 1) * w + c;
+      const float* k = a.conv + (int64_t)c * taps;
+      const float xb = a.x_bias[c], now = proj(a.p, rows, t, w + c) + xb;
+      float acc = a.conv_bias[c];
+      for (int j = 0; j < taps - 1; j++) {  // oldest first
+        const int64_t back = taps - 1 - j;
+        const float x = back <= li ? proj(a.p, rows, t - back, w + c) + xb : hist[(taps - 1 + li - back) * w];
+        acc = fmaf(k[j], x, acc);
+      }
+      acc = fmaf(k[taps - 1], now, acc);
+      const int bs = a.s.bs(), g = c / bs;
+      ((T*)a.u)[t * a.s.ld_u() + g * a.s.bs_p() + c - g * bs] = to_t<T>(acc);
+      if (!a.seq) {  // decode: the row is its sequence's only one, nobody else reads this history
+        for (int j = 0; j < taps - 2; j++) hist[(int64_t)j * w] = hist[(int64_t)(j + 1) * w];
+        if (taps > 1) hist[(int64_t)(taps - 2) * w] = now;
+      }
+    }
+  }
+  SB_TRACE_END(SB_K_ROPE, 0);
+}
+// the convolution's last inputs after a prompt's rows; grid (channel blocks, nb)
+__global__ void __launch_bounds__(256) conv_hist_kernel(GatedArgs a, int64_t rows) {
+  pdl_trigger();
+  pdl_wait();
+  const int c = blockIdx.x * 256 + threadIdx.x, b = blockIdx.y, w = a.s.width, keep = a.s.taps - 1;
+  if (c >= w) return;
+  const int n = a.lens[b] - a.past[b];
+  float* hist = a.hist + (int64_t)b * keep * w + c;
+  for (int j = 0; j < keep; j++) {  // ascending: slot j takes slot j + n, which has not been written yet
+    const int from = n + j - keep;  // row of this launch, or (negative) a slot from the end
+    hist[(int64_t)j * w] = from >= 0 ? proj(a.p, rows, a.qstart[b] + from, w + c) + a.x_bias[c] : hist[(int64_t)(j + n) * w];
+  }
+}
+
+// ------------------------------------------------------------------ gated recurrence
+struct Step { float a, b; };  // S <- a S + b
+template <typename T>
+__device__ __forceinline__ Step gated_step(const GatedArgs& g, int64_t t, int c, int64_t gr, int64_t gi, int64_t uo, float rb, float ib, float decay) {
+  const float r = sigmoid(g.gates[t * 2 * g.s.width + gr] + rb), i = sigmoid(g.gates[t * 2 * g.s.width + gi] + ib);
+  const float la = decay * r;
+  const float u = to_f(((const T*)g.u)[t * g.s.ld_u() + uo]);
+  return Step{expf(la), sqrtf(-expm1f(2.f * la)) * i * u};
+}
+constexpr int SCAN_WARPS = 32, SCAN_PER = 8;  // tokens per warp and pass
+// grid (ceil(width / 32), nb), 1024 threads: lane = channel, warp = run of tokens
+template <typename T>
+__global__ void __launch_bounds__(1024) gated_scan_kernel(GatedArgs g, int64_t rows) {
+  __shared__ Step fold[SCAN_WARPS][32];
+  __shared__ float carry[32];
+  SB_TRACE_BEGIN();
+  pdl_trigger();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, w = g.s.width;
+  const int c = blockIdx.x * 32 + lane, seq = blockIdx.y;
+  const bool live = c < w;
+  const int bs = g.s.bs(), blk = live ? c / bs : 0, in_blk = c - blk * bs;
+  const int64_t gr = (int64_t)blk * 2 * bs + in_blk, gi = gr + bs, uo = (int64_t)blk * g.s.bs_p() + in_blk;
+  const float rb = live ? g.r_bias[c] : 0.f, ib = live ? g.i_bias[c] : 0.f, decay = live ? g.decay[c] : 0.f, yb = live ? g.y_bias[c] : 0.f;
+  pdl_wait();
+  SB_TRACE_WAITED();
+  const int n = g.lens[seq] - g.past[seq];
+  const int64_t row0 = g.qstart[seq];
+  if (warp == 0) carry[lane] = live ? g.state[(int64_t)seq * w + c] : 0.f;
+  for (int t0 = 0; t0 < n; t0 += SCAN_WARPS * SCAN_PER) {
+    const int first = t0 + warp * SCAN_PER;
+    Step st[SCAN_PER];
+    float y[SCAN_PER];
+#pragma unroll
+    for (int j = 0; j < SCAN_PER; j++) {
+      const bool on = live && first + j < n;
+      st[j] = on ? gated_step<T>(g, row0 + first + j, c, gr, gi, uo, rb, ib, decay) : Step{1.f, 0.f};
+      y[j] = on ? proj(g.p, rows, row0 + first + j, c) : 0.f;
+    }
+    Step all{1.f, 0.f};
+#pragma unroll
+    for (int j = 0; j < SCAN_PER; j++) { all.b = fmaf(st[j].a, all.b, st[j].b); all.a *= st[j].a; }
+    fold[warp][lane] = all;
+    __syncthreads();
+    float s = carry[lane];
+    for (int v = 0; v < warp; v++) s = fmaf(fold[v][lane].a, s, fold[v][lane].b);
+#pragma unroll
+    for (int j = 0; j < SCAN_PER; j++) {
+      s = fmaf(st[j].a, s, st[j].b);
+      if (live && first + j < n) ((T*)g.out)[(row0 + first + j) * g.ldo + c] = to_t<T>(s * sb_gelu_tanh(y[j] + yb));
+    }
+    __syncthreads();  // everybody has read the state before this pass
+    if (warp == SCAN_WARPS - 1) carry[lane] = s;
+    __syncthreads();
+  }
+  if (warp == 0 && live) g.state[(int64_t)seq * w + c] = carry[lane];
+  SB_TRACE_END(SB_K_ATTN, 0);
+}
+// decode: grid (ceil(width / 256), rows)
+template <typename T>
+__global__ void __launch_bounds__(256) gated_step_kernel(GatedArgs g, int64_t rows) {
+  SB_TRACE_BEGIN();
+  pdl_trigger();
+  const int c = blockIdx.x * 256 + threadIdx.x, w = g.s.width;
+  const int64_t t = blockIdx.y;
+  pdl_wait();
+  SB_TRACE_WAITED();
+  if (c < w) {
+    const int bs = g.s.bs(), blk = c / bs, in_blk = c - blk * bs;
+    const int64_t gr = (int64_t)blk * 2 * bs + in_blk;
+    const Step st = gated_step<T>(g, t, c, gr, gr + bs, (int64_t)blk * g.s.bs_p() + in_blk, g.r_bias[c], g.i_bias[c], g.decay[c]);
+    const float s = fmaf(st.a, g.state[t * w + c], st.b);
+    g.state[t * w + c] = s;
+    ((T*)g.out)[t * g.ldo + c] = to_t<T>(s * sb_gelu_tanh(proj(g.p, rows, t, c) + g.y_bias[c]));
+  }
+  SB_TRACE_END(SB_K_ATTN, 0);
+}
+
+// ------------------------------------------------------------------ retention, any widths
+// grid (H, sequences), 256 threads. A state element belongs to one thread for the whole launch.
+template <typename T>
+__global__ void __launch_bounds__(256) retention_any_kernel(RetentionArgs a, int64_t rows) {
+  extern __shared__ float sm[];
+  __shared__ float red[32];
+  pdl_trigger();
+  pdl_wait();
+  const HeadShape& s = a.s;
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, row = s.row();
+  const int n = a.qstart ? a.lens[b] - a.past[b] : 1;
+  const int64_t t0 = a.qstart ? a.qstart[b] : b;
+  float *qs = sm, *ks = qs + s.dim, *vs = ks + s.dim, *os = vs + s.vdim, *part = os + s.vdim;  // part [256]
+  float* S = a.state + ((int64_t)b * s.H + h) * s.dim * s.vdim;
+  const float decay = a.decay[h];
+  const int parts = s.vdim <= 256 ? 256 / s.vdim : 1;  // threads that share a value column
+  const int64_t gcol = (int64_t)s.H * (2 * s.dim + s.vdim) + (int64_t)h * s.vdim;
+  for (int i = 0; i < n; i++) {
+    const int64_t t = t0 + i, at = (t * s.H + h) * row;
+    for (int e = tid; e < s.dim; e += 256) { qs[e] = to_f(((const T*)a.q)[at + e]); ks[e] = to_f(((const T*)a.k)[at + e]); }
+    for (int e = tid; e < s.vdim; e += 256) vs[e] = to_f(((const T*)a.v)[at + e]);
+    __syncthreads();
+    for (int v0 = 0; v0 < s.vdim; v0 += 256) {
+      const int v = parts > 1 ? tid % s.vdim : v0 + tid, p = parts > 1 ? tid / s.vdim : 0;
+      float acc = 0.f;
+      if (v < s.vdim && p < parts) {
+        const float vv = vs[v];
+#pragma unroll 4
+        for (int d = p; d < s.dim; d += parts) {
+          const float x = fmaf(decay, S[(int64_t)d * s.vdim + v], ks[d] * vv);
+          S[(int64_t)d * s.vdim + v] = x;
+          acc = fmaf(qs[d], x, acc);
+        }
+      }
+      if (parts > 1) {
+        part[tid] = acc;
+        __syncthreads();
+        if (p == 0) {
+          for (int j = 1; j < parts; j++) acc += part[j * s.vdim + v];
+          os[v] = acc;
+        }
+      } else if (v < s.vdim) {
+        os[v] = acc;
+      }
+    }
+    __syncthreads();
+    float ss = 0.f;
+    for (int v = tid; v < s.vdim; v += 256) ss += os[v] * os[v];
+    ss = block_sum(ss, red);
+    const float r = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)s.vdim), a.eps)));
+    for (int v = tid; v < s.vdim; v += 256) {
+      const float g = proj(a.p, rows, t, gcol + v);
+      ((T*)a.out)[t * a.ldo + (int64_t)h * s.vdim + v] = to_t<T>(os[v] * r * (g * sigmoid(g)));
+    }
+    __syncthreads();
+  }
+}
+
+// ------------------------------------------------------------------ retention, decode
+// B * H blocks of one head each, then B * act_blks for the feed-forward's columns; 256 threads. The threads of a block form
+// 256 / (vdim / 4) groups; a thread owns four value columns of every group-th state row.
+constexpr int RET_UNROLL = 8;
+__global__ void __launch_bounds__(256) retention_decode_kernel(RetentionArgs a, int64_t B, int act_blks) {
+  extern __shared__ float sm[];
+  __shared__ float red[32];
+  SB_TRACE_BEGIN();
+  pdl_trigger();
+  const HeadShape& s = a.s;
+  const int tid = threadIdx.x;
+  const int64_t heads = B * s.H;
+  if (blockIdx.x >= heads) {
+    pdl_wait();
+    SB_TRACE_WAITED();
+    act_block<bf16>(a.act, a.p, B, (blockIdx.x - heads) / act_blks, (int)((blockIdx.x - heads) % act_blks));
+    SB_TRACE_END(SB_K_ATTN, 0);
+    return;
+  }
+  const int h = (int)(blockIdx.x % s.H);
+  const int64_t b = blockIdx.x / s.H;
+  float* S = a.state + (b * s.H + h) * (int64_t)s.dim * s.vdim;
+  // the state starts on its way to L2 while the projection still runs (a hint: nothing is read before the wait)
+  for (int i = tid * 32; i < s.dim * s.vdim; i += 256 * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(S + i));
+  const float decay = a.decay[h];
+  pdl_wait();
+  SB_TRACE_WAITED();
+  float *x = sm, *qs = x + 2 * s.dim, *ks = qs + s.dim, *vs = ks + s.dim, *gs = vs + s.vdim, *po = gs + s.vdim;  // po [groups][vdim]
+  const int p = a.cache_lens[b];
+  if (p < 0 || p >= a.max_pos) return;
+  const int64_t HD = (int64_t)s.H * s.dim;
+  const int n4 = (2 * s.dim + 2 * s.vdim) / 4;
+  for (int i = tid; i < n4; i += 256) {  // q, k (before rotation), v, g of this head
+    int e = i * 4;
+    float* dst;
+    int64_t col;
+    if (e < s.dim) { col = (int64_t)h * s.dim + e; dst = x + e; }
+    else if (e < 2 * s.dim) { col = HD + (int64_t)h * s.dim + e - s.dim; dst = x + e; }
+    else if (e < 2 * s.dim + s.vdim) { e -= 2 * s.dim; col = 2 * HD + (int64_t)h * s.vdim + e; dst = vs + e; }
+    else { e -= 2 * s.dim + s.vdim; col = 2 * HD + (int64_t)(s.H + h) * s.vdim + e; dst = gs + e; }
+    *(float4*)dst = proj4(a.p, B, b, col);
+  }
+  __syncthreads();
+  const int half = s.rot / 2;
+  for (int e = tid; e < 2 * s.dim; e += 256) {
+    const int d = e < s.dim ? e : e - s.dim;
+    const float* src = e < s.dim ? x : x + s.dim;
+    float v = src[d];
+    if (d < s.rot) {
+      const int i = d < half ? d : d - half;
+      const float c = a.cos_t[(int64_t)p * half + i], n = a.sin_t[(int64_t)p * half + i];
+      v = d < half ? src[d] * c - src[d + half] * n : src[d] * c + src[d - half] * n;
+    }
+    if (e < s.dim) qs[d] = v;
+    else ks[d] = v * s.k_scale;
+  }
+  __syncthreads();
+  const int vq = s.vdim / 4, groups = 256 / vq, g = tid / vq, c4 = (tid % vq) * 4;
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (g < groups) {
+    const float4 v = *(const float4*)(vs + c4);
+    for (int d0 = g; d0 < s.dim; d0 += groups * RET_UNROLL) {
+      float4 st[RET_UNROLL];
+#pragma unroll
+      for (int j = 0; j < RET_UNROLL; j++)
+        if (d0 + j * groups < s.dim) st[j] = __ldcs((const float4*)(S + (int64_t)(d0 + j * groups) * s.vdim + c4));
+#pragma unroll
+      for (int j = 0; j < RET_UNROLL; j++) {
+        const int d = d0 + j * groups;
+        if (d < s.dim) {
+          const float k = ks[d], q = qs[d];
+          st[j].x = fmaf(decay, st[j].x, k * v.x); st[j].y = fmaf(decay, st[j].y, k * v.y);
+          st[j].z = fmaf(decay, st[j].z, k * v.z); st[j].w = fmaf(decay, st[j].w, k * v.w);
+          __stcs((float4*)(S + (int64_t)d * s.vdim + c4), st[j]);
+          o.x = fmaf(q, st[j].x, o.x); o.y = fmaf(q, st[j].y, o.y); o.z = fmaf(q, st[j].z, o.z); o.w = fmaf(q, st[j].w, o.w);
+        }
+      }
+    }
+    *(float4*)(po + g * s.vdim + c4) = o;
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int v = tid; v < s.vdim; v += 256) {
+    float t = 0.f;
+    for (int j = 0; j < groups; j++) t += po[j * s.vdim + v];
+    po[v] = t;  // this thread's column
+    ss += t * t;
+  }
+  ss = block_sum(ss, red);
+  const float r = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)s.vdim), a.eps)));
+  for (int v = tid; v < s.vdim; v += 256) ((bf16*)a.out)[b * a.ldo + (int64_t)h * s.vdim + v] = __float2bfloat16_rn(po[v] * r * (gs[v] * sigmoid(gs[v])));
+  SB_TRACE_END(SB_K_ATTN, 0);
+}
+size_t retention_decode_smem(const HeadShape& s) { return (size_t)(4 * s.dim + 2 * s.vdim + 256 / (s.vdim / 4) * s.vdim) * sizeof(float); }
+
+}  // namespace
+
+SB_TRACE_TU(recurrent)
+
+int k_gated_conv(strictb200_ctx* ctx, const GatedArgs& a, int64_t T) {
+  const int ch = (a.s.width + 255) / 256, act = act_blocks(a.act);
+  if (T * (ch + act) > INT32_MAX || a.p.splits > 8) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gated recurrence: too many rows or partial sums");
+  const dim3 grid((unsigned)(T * (ch + act)));
+  if (a.f32) SB_CUDA(sb_launch(ctx, gated_conv_kernel<float>, grid, dim3(256), 0, a, T, ch, act));
+  else SB_CUDA(sb_launch(ctx, gated_conv_kernel<bf16>, grid, dim3(256), 0, a, T, ch, act));
+  ctx->launches++;
+  if (!a.seq || a.s.taps < 2) return STRICTB200_OK;
+  SB_CUDA(sb_launch(ctx, conv_hist_kernel, dim3((unsigned)ch, (unsigned)a.nb), dim3(256), 0, a, T));
+  ctx->launches++;
+  return STRICTB200_OK;
+}
+
+int k_gated_scan(strictb200_ctx* ctx, const GatedArgs& a, int64_t T) {
+  if (!a.seq) {
+    const dim3 grid((unsigned)((a.s.width + 255) / 256), (unsigned)T);
+    if (a.f32) SB_CUDA(sb_launch(ctx, gated_step_kernel<float>, grid, dim3(256), 0, a, T));
+    else SB_CUDA(sb_launch(ctx, gated_step_kernel<bf16>, grid, dim3(256), 0, a, T));
+  } else {
+    const dim3 grid((unsigned)((a.s.width + 31) / 32), (unsigned)a.nb);
+    if (a.f32) SB_CUDA(sb_launch(ctx, gated_scan_kernel<float>, grid, dim3(1024), 0, a, T));
+    else SB_CUDA(sb_launch(ctx, gated_scan_kernel<bf16>, grid, dim3(1024), 0, a, T));
+  }
+  ctx->launches++;
+  return STRICTB200_OK;
+}
+
+int k_retention_any(strictb200_ctx* ctx, const RetentionArgs& a) {
+  const HeadShape& s = a.s;
+  const size_t smem = (size_t)(2 * s.dim + 2 * s.vdim + 256) * sizeof(float);
+  if (smem > 40 * 1024) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "retention: heads too wide");
+  const dim3 grid((unsigned)s.H, (unsigned)a.nb);
+  const int64_t rows = a.qstart ? 0 : a.nb;  // (stride of partial sums; a prompt's projection is one finished array)
+  if (a.f32) SB_CUDA(sb_launch(ctx, retention_any_kernel<float>, grid, dim3(256), smem, a, rows));
+  else SB_CUDA(sb_launch(ctx, retention_any_kernel<bf16>, grid, dim3(256), smem, a, rows));
+  ctx->launches++;
+  return STRICTB200_OK;
+}
+
+bool sb_retention_decode_fits(const HeadShape& s) {
+  return s.dim % 4 == 0 && s.vdim % 4 == 0 && s.vdim <= 1024 && retention_decode_smem(s) <= 40 * 1024;
+}
+int k_retention_decode(strictb200_ctx* ctx, const RetentionArgs& a, int64_t B) {
+  if (!sb_retention_decode_fits(a.s) || a.p.ld % 4 || a.p.splits > 8) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "retention: widths the decode kernel does not take");
+  const int act = act_blocks(a.act);
+  SB_CUDA(sb_launch(ctx, retention_decode_kernel, dim3((unsigned)(B * (a.s.H + act))), dim3(256), retention_decode_smem(a.s), a, B, act));
+  ctx->launches++;
+  return STRICTB200_OK;
+}

@@ -1,0 +1,332 @@
+// Retention over prompts on the tcgen05 tensor cores: S <- decay S + k v^T, o = S^T q per head (heads of up to 128 dims), then o
+// over its root mean square times silu(g).
+// One block owns one head of one sequence and walks its tokens in chunks of 128; with n tokens in the chunk and rows i, j:
+//   P = Q K^T                           P_ij *= decay^(i - j) for j <= i, else 0; kept as two bf16 terms (hi + lo)
+//   O = P V,  O2 = Q S                  o_i = O_i + decay^(i + 1) O2_i
+//   S <- decay^n S + K^T V'             V'_j = decay^(n - 1 - j) v_j
+// The state stays in tensor memory in fp32 from the first chunk to the last (lane = query/key dim, column = value dim). As the
+// operand of Q S it is written to shared memory as two bf16 terms, and so is V'; q, k and v themselves are bf16, the powers of
+// the decay fp32. Tensor memory: P, O, O2 and S, 128 columns each.
+//   warps 0..7  rows: thread (row, half) owns 64 columns of row `row` of every tile
+//   warp 8      one lane issues copies and products
+// Every mbarrier wait is bounded: on expiry the block records an error word in host-visible memory, stops, frees its tensor
+// memory and returns.
+#include "mixers.cuh"
+#include "tcgen05.cuh"
+
+using namespace tc;
+
+namespace {
+
+constexpr int CHUNK = 128;
+constexpr int RT_THREADS = 288;
+
+struct RtArgs {
+  int H, dim, vdim;
+  const int32_t *lens, *past, *qstart;
+  const float* decay;
+  float* state;
+  const float* g;   // first gate column of the projection
+  int64_t ld_g;
+  float eps;
+  bf16* out;
+  int64_t ldo;
+  int* status;
+};
+
+// two bf16 terms by truncation: hi = the upper 16 bits, lo = the upper 16 bits of the exact remainder
+__device__ __forceinline__ void split2(float p0, float p1, uint32_t& hi, uint32_t& lo) {
+  const uint32_t b0 = __float_as_uint(p0), b1 = __float_as_uint(p1);
+  hi = __byte_perm(b0, b1, 0x7632);
+  lo = __byte_perm(__float_as_uint(p0 - __uint_as_float(b0 & 0xFFFF0000u)), __float_as_uint(p1 - __uint_as_float(b1 & 0xFFFF0000u)), 0x7632);
+}
+__device__ __forceinline__ void arrive(uint64_t* bar) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory"); }
+// 16 bytes `chunk` of row `row` of a swizzled box
+__device__ __forceinline__ uint32_t box_off(int row, int chunk) { return (uint32_t)(row * 128 + ((chunk ^ (row & 7)) << 4)); }
+
+__global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+                                                                      const __grid_constant__ CUtensorMap map_v, RtArgs a) {
+  extern __shared__ __align__(1024) uint8_t smem_raw[];
+  uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+  __shared__ __align__(8) uint64_t bar_qk, bar_v, bar_s, bar_o, bar_state, s_ready, vp_ready, p_ready;
+  __shared__ uint32_t tmem_base_slot;
+  __shared__ float pw[CHUNK + 1], x_sum[2][CHUNK];
+
+  const int h = blockIdx.x, b = blockIdx.y;
+  const int n_all = a.lens[b] - a.past[b], chunks = (n_all + CHUNK - 1) / CHUNK;
+  const int64_t row0 = a.qstart[b];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  uint8_t *bQ = smem, *bK = bQ + TILE_BYTES, *bV = bK + TILE_BYTES, *bVh = bV + TILE_BYTES, *bVl = bVh + TILE_BYTES, *bSh = bVl + TILE_BYTES, *bSl = bSh + TILE_BYTES;
+  const uint32_t sQ = smem_u32(bQ), sK = smem_u32(bK), sV = smem_u32(bV), sVh = smem_u32(bVh), sVl = smem_u32(bVl), sSh = smem_u32(bSh), sSl = smem_u32(bSl);
+  if (threadIdx.x == 0) {
+    mbar_init(smem_u32(&bar_qk), 1); mbar_init(smem_u32(&bar_v), 1);
+    mbar_init(smem_u32(&bar_s), 1); mbar_init(smem_u32(&bar_o), 1); mbar_init(smem_u32(&bar_state), 1);
+    mbar_init(smem_u32(&s_ready), 256); mbar_init(smem_u32(&vp_ready), 256); mbar_init(smem_u32(&p_ready), 256);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (threadIdx.x <= CHUNK) pw[threadIdx.x] = (float)pow((double)a.decay[h], (double)threadIdx.x);
+  if (warp == 8) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_base_slot)), "r"(512u) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tP = tmem_base_slot, tO = tP + 128, tO2 = tP + 256, tS = tP + 384;
+  // D = F32, A = B = bf16, M = N = 128; bit 15: A is MN-major (its rows are the reduction), bit 16: B is
+  constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(128 >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+  constexpr uint32_t idesc_b = idesc | (1u << 16), idesc_ab = idesc_b | (1u << 15);
+
+  if (warp == 8) {
+    if (lane == 0) {
+      auto load = [&](int c) {
+        const int row = (int)row0 + c * CHUNK;
+        mbar_expect_tx(smem_u32(&bar_qk), 2 * TILE_BYTES);
+        for (int i = 0; i < 2; i++) {
+          tma_load_3d(sQ + i * HALF_BYTES, &map_q, i * 64, h, row, smem_u32(&bar_qk));
+          tma_load_3d(sK + i * HALF_BYTES, &map_k, i * 64, h, row, smem_u32(&bar_qk));
+        }
+        mbar_expect_tx(smem_u32(&bar_v), TILE_BYTES);
+        for (int i = 0; i < 2; i++) tma_load_3d(sV + i * HALF_BYTES, &map_v, i * 64, h, row, smem_u32(&bar_v));
+      };
+      load(0);
+      bool good = true;
+      for (int c = 0; c < chunks && good; c++) {
+        const uint32_t ph = (uint32_t)(c & 1);
+        good = mbar_wait(smem_u32(&bar_qk), ph) && mbar_wait(smem_u32(&s_ready), ph);
+        if (!good) break;
+        tc_fence_after();
+#pragma unroll
+        for (int s = 0; s < 8; s++) {
+          const uint32_t off = (uint32_t)((s >> 2) * HALF_BYTES + (s & 3) * 32);
+          tc_mma_ss(tP, desc_kmajor(sQ + off), desc_kmajor(sK + off), idesc, s ? 1u : 0u);
+        }
+        tc_commit(smem_u32(&bar_s));
+#pragma unroll
+        for (int s = 0; s < 8; s++) {
+          const uint64_t dq = desc_kmajor(sQ + (uint32_t)((s >> 2) * HALF_BYTES + (s & 3) * 32));
+          tc_mma_ss(tO2, dq, desc_mnmajor(sSh + (uint32_t)(s * 2048)), idesc_b, s ? 1u : 0u);
+          tc_mma_ss(tO2, dq, desc_mnmajor(sSl + (uint32_t)(s * 2048)), idesc_b, 1u);
+        }
+        good = mbar_wait(smem_u32(&p_ready), ph) && mbar_wait(smem_u32(&bar_v), ph);
+        if (!good) break;
+        tc_fence_after();
+#pragma unroll
+        for (int s = 0; s < 8; s++) {
+          const uint64_t dv = desc_mnmajor(sV + (uint32_t)(s * 2048));
+          const uint32_t pcol = (uint32_t)((s >> 1) * 32 + (s & 1) * 8);
+          tc_mma_ts(tO, tP + pcol, dv, idesc_b, s ? 1u : 0u);
+          tc_mma_ts(tO, tP + pcol + 16, dv, idesc_b, 1u);
+        }
+        tc_commit(smem_u32(&bar_o));
+        good = mbar_wait(smem_u32(&vp_ready), ph);
+        if (!good) break;
+        tc_fence_after();
+#pragma unroll
+        for (int s = 0; s < 8; s++) {
+          const uint64_t dk = desc_mnmajor(sK + (uint32_t)(s * 2048));
+          tc_mma_ss(tS, dk, desc_mnmajor(sVh + (uint32_t)(s * 2048)), idesc_ab, 1u);
+          tc_mma_ss(tS, dk, desc_mnmajor(sVl + (uint32_t)(s * 2048)), idesc_ab, 1u);
+        }
+        tc_commit(smem_u32(&bar_state));
+        if (c + 1 < chunks) {
+          good = mbar_wait(smem_u32(&bar_state), ph);  // every product of the chunk has read its tiles, every row its part of V
+          if (good) load(c + 1);
+        }
+      }
+      if (!good) set_status(a.status, 17);
+    }
+  } else {
+    const int row = (int)threadIdx.x & (CHUNK - 1), half = (int)threadIdx.x >> 7;
+    const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
+    const int c0 = half * 64;  // first of this thread's columns, in every tile
+    auto rows_sync = [&]() { asm volatile("bar.sync 1, 256;" ::: "memory"); };
+    float* S = a.state + (((int64_t)b * a.H + h) * a.dim + row) * a.vdim;  // state row `row` (where it exists)
+    bool ok = true;
+    for (int c = 0; c < chunks; c++) {
+      const uint32_t ph = (uint32_t)(c & 1);
+      const int n = min(CHUNK, n_all - c * CHUNK);
+      if (c > 0 && !mbar_wait(smem_u32(&bar_state), ph ^ 1)) { ok = false; break; }
+      tc_fence_after();
+      // ---- the state before the chunk: operand tiles, and decay^n times it back to tensor memory
+      const float dn = pw[n];
+#pragma unroll
+      for (int q = 0; q < 2; q++) {
+        uint32_t r[32];
+        if (c > 0) {
+          tc_ld32(tS + lane_base + (uint32_t)(c0 + q * 32), r);
+          tc_wait_ld();
+        } else {
+#pragma unroll
+          for (int j = 0; j < 32; j++) {
+            const int v = c0 + q * 32 + j;
+            r[j] = __float_as_uint(row < a.dim && v < a.vdim ? S[v] : 0.f);
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+          uint4 hi, lo;
+          split2(__uint_as_float(r[8 * j]), __uint_as_float(r[8 * j + 1]), hi.x, lo.x);
+          split2(__uint_as_float(r[8 * j + 2]), __uint_as_float(r[8 * j + 3]), hi.y, lo.y);
+          split2(__uint_as_float(r[8 * j + 4]), __uint_as_float(r[8 * j + 5]), hi.z, lo.z);
+          split2(__uint_as_float(r[8 * j + 6]), __uint_as_float(r[8 * j + 7]), hi.w, lo.w);
+          const uint32_t off = (uint32_t)(half * HALF_BYTES) + box_off(row, q * 4 + j);
+          *(uint4*)(bSh + off) = hi;
+          *(uint4*)(bSl + off) = lo;
+        }
+#pragma unroll
+        for (int j = 0; j < 32; j++) r[j] = __float_as_uint(__uint_as_float(r[j]) * dn);
+        tc_st32(tS + lane_base + (uint32_t)(c0 + q * 32), r);
+      }
+      tc_wait_st();
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+      tc_fence_before();
+      arrive(&s_ready);
+      // ---- V' = the values under their powers of the decay at the end of the chunk
+      if (!mbar_wait(smem_u32(&bar_v), ph)) { ok = false; break; }
+      const float wv = row < n ? pw[n - 1 - row] : 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; j++) {
+        const uint32_t off = (uint32_t)(half * HALF_BYTES) + box_off(row, j);
+        const uint4 v = *(const uint4*)(bV + off);
+        uint4 hi, lo;
+        auto both = [&](uint32_t x, uint32_t& o_hi, uint32_t& o_lo) {
+          split2(__uint_as_float(x << 16) * wv, __uint_as_float(x & 0xFFFF0000u) * wv, o_hi, o_lo);
+        };
+        both(v.x, hi.x, lo.x); both(v.y, hi.y, lo.y); both(v.z, hi.z, lo.z); both(v.w, hi.w, lo.w);
+        *(uint4*)(bVh + off) = hi;
+        *(uint4*)(bVl + off) = lo;
+      }
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+      arrive(&vp_ready);
+      // ---- P under the decay
+      if (!mbar_wait(smem_u32(&bar_s), ph)) { ok = false; break; }
+      tc_fence_after();
+#pragma unroll 1
+      for (int q = 2 * half; q < 2 * half + 2; q++) {
+        uint32_t r[32], hi[16], lo[16];
+        tc_ld32(tP + lane_base + (uint32_t)(q * 32), r);
+        tc_wait_ld();
+#pragma unroll
+        for (int j = 0; j < 16; j++) {
+          const int k = q * 32 + 2 * j;
+          const float p0 = k <= row ? __uint_as_float(r[2 * j]) * pw[row - k] : 0.f;
+          const float p1 = k + 1 <= row ? __uint_as_float(r[2 * j + 1]) * pw[row - k - 1] : 0.f;
+          split2(p0, p1, hi[j], lo[j]);
+        }
+        tc_st16(tP + lane_base + (uint32_t)(q * 32), hi);
+        tc_st16(tP + lane_base + (uint32_t)(q * 32 + 16), lo);
+      }
+      tc_wait_st();
+      tc_fence_before();
+      arrive(&p_ready);
+      // ---- output of the chunk; the gates are on their way while the products run
+      const bool live = row < n;
+      const int64_t t = row0 + c * CHUNK + row;
+      const float* g = a.g + t * a.ld_g + (int64_t)h * a.vdim + c0;
+      const bool vec = ((a.vdim | (int)(a.ld_g & 3)) & 3) == 0 && ((uintptr_t)a.g & 15) == 0;
+      float gv[64];
+#pragma unroll
+      for (int j = 0; j < 16; j++) {
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (live && c0 + 4 * j < a.vdim) {
+          if (vec) x = *(const float4*)(g + 4 * j);
+          else {
+            x.x = g[4 * j];
+            if (c0 + 4 * j + 1 < a.vdim) x.y = g[4 * j + 1];
+            if (c0 + 4 * j + 2 < a.vdim) x.z = g[4 * j + 2];
+            if (c0 + 4 * j + 3 < a.vdim) x.w = g[4 * j + 3];
+          }
+        }
+        gv[4 * j] = x.x; gv[4 * j + 1] = x.y; gv[4 * j + 2] = x.z; gv[4 * j + 3] = x.w;
+      }
+      if (!mbar_wait(smem_u32(&bar_o), ph)) { ok = false; break; }
+      tc_fence_after();
+      const float d1 = pw[min(row + 1, CHUNK)];
+      float ss = 0.f;
+      float o[64];
+#pragma unroll
+      for (int q = 0; q < 2; q++) {
+        uint32_t r[32], r2[32];
+        tc_ld32(tO + lane_base + (uint32_t)(c0 + q * 32), r);
+        tc_ld32(tO2 + lane_base + (uint32_t)(c0 + q * 32), r2);
+        tc_wait_ld();
+#pragma unroll
+        for (int j = 0; j < 32; j++) {
+          const float v = fmaf(d1, __uint_as_float(r2[j]), __uint_as_float(r[j]));
+          o[q * 32 + j] = v;
+          ss = fmaf(v, v, ss);  // columns beyond vdim are zero
+        }
+      }
+      x_sum[half][row] = ss;
+      rows_sync();
+      ss = x_sum[0][row] + x_sum[1][row];
+      rows_sync();
+      const float rn = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.vdim), a.eps)));
+      bf16* dst = a.out + t * a.ldo + (int64_t)h * a.vdim + c0;
+      const bool wide = ((a.vdim | (int)(a.ldo & 7)) & 7) == 0 && ((uintptr_t)a.out & 15) == 0;
+      if (live) {
+#pragma unroll
+        for (int j = 0; j < 64; j += 8) {
+          float y[8];
+#pragma unroll
+          for (int i = 0; i < 8; i++) y[i] = o[j + i] * rn * (gv[j + i] * mix::sigmoid(gv[j + i]));
+          if (wide) {
+            if (c0 + j < a.vdim)
+              *(uint4*)(dst + j) = make_uint4(mix::pack_bf16(y[0], y[1]), mix::pack_bf16(y[2], y[3]), mix::pack_bf16(y[4], y[5]), mix::pack_bf16(y[6], y[7]));
+          } else {
+#pragma unroll
+            for (int i = 0; i < 8; i++)
+              if (c0 + j + i < a.vdim) dst[j + i] = __float2bfloat16_rn(y[i]);
+          }
+        }
+      }
+    }
+    if (ok && chunks > 0) {
+      ok = mbar_wait(smem_u32(&bar_state), (uint32_t)((chunks - 1) & 1));
+      tc_fence_after();
+      if (ok) {
+#pragma unroll 1
+        for (int q = 0; q < 2; q++) {
+          uint32_t r[32];
+          tc_ld32(tS + lane_base + (uint32_t)(c0 + q * 32), r);
+          tc_wait_ld();
+#pragma unroll
+          for (int j = 0; j < 32; j++) {
+            const int v = c0 + q * 32 + j;
+            if (row < a.dim && v < a.vdim) S[v] = __uint_as_float(r[j]);
+          }
+        }
+      }
+    }
+    if (!ok && row == 0) set_status(a.status, 18);
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 8) {
+    tc_fence_after();
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tP), "r"(512u) : "memory");
+  }
+}
+
+}  // namespace
+
+bool sb_retention_prefill_fits(const HeadShape& s) { return s.dim <= 128 && s.vdim <= 128; }
+
+int k_retention_prefill(strictb200_ctx* ctx, const RetentionArgs& p, int64_t T) {
+  const HeadShape& s = p.s;
+  if (!sb_retention_prefill_fits(s) || p.f32 || p.p.splits != 1) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "retention: heads the tensor-core kernel does not take");
+  if (s.H > INT32_MAX / 2 || p.nb > 65535 || T > INT32_MAX) return sb_fail(STRICTB200_ERR_INVALID_ARG, "retention: too many sequences or rows");
+  RtArgs a{s.H, s.dim, s.vdim, p.lens, p.past, p.qstart, p.decay, p.state, p.p.in + (int64_t)s.H * (2 * s.dim + s.vdim), p.p.ld, p.eps, (bf16*)p.out, p.ldo, ctx->d_status};
+  const int row = s.row();
+  CUtensorMap mq, mk, mv;
+  SB_TRY(make_map3(&mq, p.q, row, s.H, T, row, (int64_t)s.H * row));
+  SB_TRY(make_map3(&mk, p.k, row, s.H, T, row, (int64_t)s.H * row));
+  SB_TRY(make_map3(&mv, p.v, row, s.H, T, row, (int64_t)s.H * row));
+  const size_t smem = 7 * TILE_BYTES + 1024;
+  static SbDeviceOnce once;
+  SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(retention_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
+  retention_prefill_kernel<<<dim3((unsigned)s.H, (unsigned)p.nb), RT_THREADS, smem, ctx->stream>>>(mq, mk, mv, a);
+  SB_LAUNCHED(ctx);
+  return STRICTB200_OK;
+}

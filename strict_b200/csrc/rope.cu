@@ -203,16 +203,27 @@ int k_rope_qknorm_kvappend(strictb200_ctx* ctx, const RopeArgs& a, int64_t T) {
 
 // cos/sin of pos * theta^(-2i/D), evaluated in double on the host and rounded to fp32: part of
 // the model constants (like the weights), not of the per-token path.
-int sb_rope_table(strictb200_ctx* ctx, int max_pos, int D, double theta, float** d_cos, float** d_sin) {
+int sb_rope_table(strictb200_ctx* ctx, int max_pos, int D, double theta, float** d_cos, float** d_sin, const RopeScaling& sc) {
   int h = D / 2;
   std::vector<float> c((size_t)max_pos * h), s((size_t)max_pos * h);
   std::vector<double> inv(h);
   for (int i = 0; i < h; i++) inv[i] = std::pow(theta, -2.0 * (double)i / (double)D);
+  double gain = 1.0;
+  if (sc.factor > 0) {
+    // pair index (times two) at which a pair turns `turns` times within the original length
+    auto pair_of = [&](double turns) { return D * std::log(sc.original / (2.0 * M_PI * turns)) / (2.0 * std::log(theta)); };
+    const double lo = std::max(std::floor(pair_of(sc.fast)), 0.0), hi = std::min(std::ceil(pair_of(sc.slow)), (double)(D - 1));
+    for (int i = 0; i < h; i++) {
+      const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+      inv[i] = inv[i] / sc.factor * ramp + inv[i] * (1.0 - ramp);
+    }
+    gain = 0.1 * std::log(sc.factor) + 1.0;
+  }
   for (int p = 0; p < max_pos; p++)
     for (int i = 0; i < h; i++) {
       double ang = (double)p * inv[i];
-      c[(size_t)p * h + i] = (float)std::cos(ang);
-      s[(size_t)p * h + i] = (float)std::sin(ang);
+      c[(size_t)p * h + i] = (float)(gain * std::cos(ang));
+      s[(size_t)p * h + i] = (float)(gain * std::sin(ang));
     }
   size_t bytes = c.size() * sizeof(float);
   SB_CUDA(cudaMalloc((void**)d_cos, bytes));

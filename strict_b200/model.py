@@ -14,8 +14,8 @@ from . import native as N
 
 GPT2, QWEN3, STACK = 0, 1, 2
 BF16, FP32 = 0, 1            # strictb200_dtype
-MIXER_LATENT = 1             # strictb200_mixer
-MLP_NONE, MLP_XIELU = 0, 1   # strictb200_mlp
+MIXER_LATENT, MIXER_ATTENTION, MIXER_GATED, MIXER_RETENTION = 1, 2, 3, 4  # strictb200_mixer
+MLP_NONE, MLP_XIELU, MLP_RELU_GLU = 0, 1, 2                               # strictb200_mlp
 
 CONFIGS = {
     # GPT-2 small: 12 layers, d 768, 12 heads x 64, MLP 3072, LN eps 1e-5, 1024 positions, tied
@@ -45,21 +45,52 @@ def latent_layer(heads, dim, rot_dim, vdim, kv_rank, scale, rot_base, window=0, 
                 mlp=MLP_XIELU if d_ff else MLP_NONE, d_ff=d_ff, scale=scale, rot_base=rot_base)
 
 
-def stack_config(layers, d_model, vocab, max_pos, norm_groups, eps, dtype=BF16):
+def _rotation(rot_dim, rot_base, scaling):
+    """scaling: dict of factor, original, fast and slow (YaRN), or None."""
+    s = scaling or {}
+    return dict(rot_dim=rot_dim, rot_base=rot_base, rot_factor=s.get("factor", 0.0), rot_original=s.get("original", 0.0),
+                rot_fast=s.get("fast", 0.0), rot_slow=s.get("slow", 0.0))
+
+
+def attention_layer(heads, kv_heads, dim, vdim, scale, rot_dim=0, rot_base=0.0, rot_scaling=None, qk_norm=False, sink=False, gate=False, d_ff=0,
+                    mlp=MLP_RELU_GLU):
+    """Softmax attention over grouped heads, and a feed-forward when d_ff > 0."""
+    return dict(mixer=MIXER_ATTENTION, heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale, qk_norm=int(qk_norm), sink=int(sink),
+                gate=int(gate), mlp=mlp if d_ff else MLP_NONE, d_ff=d_ff, **_rotation(rot_dim, rot_base, rot_scaling))
+
+
+def gated_layer(width, blocks, conv, d_ff=0, mlp=MLP_RELU_GLU):
+    """Real-gated linear recurrence behind a causal convolution of `conv` taps."""
+    return dict(mixer=MIXER_GATED, width=width, blocks=blocks, conv=conv, mlp=mlp if d_ff else MLP_NONE, d_ff=d_ff)
+
+
+def retention_layer(heads, dim, vdim, decay, rot_dim=0, rot_base=0.0, rot_scaling=None, d_ff=0, mlp=MLP_RELU_GLU):
+    """Retention with a fixed decay per head."""
+    if len(decay) != heads:
+        raise ValueError("retention needs one decay per head")
+    return dict(mixer=MIXER_RETENTION, heads=heads, dim=dim, vdim=vdim, decay=list(decay), mlp=mlp if d_ff else MLP_NONE, d_ff=d_ff,
+                **_rotation(rot_dim, rot_base, rot_scaling))
+
+
+def stack_config(layers, d_model, vocab, max_pos, norm_groups, eps, dtype=BF16, shared_norm=False, layer_scale=False, residual_mult=1.0,
+                 logit_scale=1.0):
     """Configuration of a model described layer by layer (strictb200_stack_create)."""
     return dict(arch=STACK, n_layers=len(layers), d_model=d_model, vocab=vocab, max_pos=max_pos, norm_groups=norm_groups, eps=eps, dtype=dtype,
-                layers=list(layers))
+                shared_norm=int(shared_norm), layer_scale=int(layer_scale), residual_mult=residual_mult, logit_scale=logit_scale, layers=list(layers))
 
 
 def make_stack_config(cfg):
     c = N.StackConfig()
-    for k in ("n_layers", "d_model", "vocab", "max_pos", "norm_groups", "dtype"):
-        setattr(c, k, int(cfg[k]))
-    c.eps = float(cfg["eps"])
+    for k, t in N.StackConfig._fields_:
+        setattr(c, k, float(cfg[k]) if t is C.c_double else int(cfg[k]))
     layers = (N.LayerConfig * len(cfg["layers"]))()
     for dst, src in zip(layers, cfg["layers"]):
-        for k, t in N.LayerConfig._fields_:
-            setattr(dst, k, float(src[k]) if t is C.c_double else int(src[k]))
+        for k, t in N.LayerConfig._fields_:  # what a layer does not name stays 0
+            if k == "decay":
+                if "decay" in src:
+                    dst.decay = (C.c_double * len(src[k]))(*src[k])
+            elif k in src:
+                setattr(dst, k, float(src[k]) if t is C.c_double else int(src[k]))
     return c, layers
 
 
@@ -164,7 +195,7 @@ class KvCache:
         N.check(N.lib().strictb200_decode_steps_device(self.model.h, self.h, None, n_steps))
 
     KERNEL_CLASSES = ("embed", "gemm_qkv", "rope_kvappend", "attn_decode", "gemm_o", "rownorm", "gemm_gate_up", "swiglu",
-                      "gemm_down", "head", "allreduce", "attn_merge")
+                      "gemm_down", "head", "allreduce", "attn_merge", "gates", "recurrence")
 
     def profile_decode(self, n_steps):
         """Per-kernel-class device time of n plain-launch decode steps: {class: (total_ms, calls)}."""

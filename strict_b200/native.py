@@ -30,13 +30,16 @@ class ModelConfig(C.Structure):
 
 class LayerConfig(C.Structure):
     """strictb200_layer_config"""
-    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "rot_dim", "vdim", "kv_rank", "window", "kv_from", "mlp", "d_ff")] + \
-               [("scale", C.c_double), ("rot_base", C.c_double)]
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "rot_dim", "vdim", "kv_rank", "window", "kv_from", "mlp", "d_ff",
+                                         "kv_heads", "qk_norm", "sink", "gate", "width", "blocks", "conv", "reserved")] + \
+               [(n, C.c_double) for n in ("scale", "rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")] + \
+               [("decay", C.POINTER(C.c_double))]
 
 
 class StackConfig(C.Structure):
     """strictb200_stack_config"""
-    _fields_ = [(n, C.c_int32) for n in ("n_layers", "d_model", "vocab", "max_pos", "norm_groups", "dtype")] + [("eps", C.c_double)]
+    _fields_ = [(n, C.c_int32) for n in ("n_layers", "d_model", "vocab", "max_pos", "norm_groups", "dtype", "shared_norm", "layer_scale")] + \
+               [(n, C.c_double) for n in ("eps", "residual_mult", "logit_scale")]
 
 
 _lib = None

@@ -95,4 +95,4 @@ def test_safetensors_round_trip(tmp_path):
 
 def test_struct_layouts():
     import ctypes
-    assert ctypes.sizeof(sb.native.LayerConfig) == 10 * 4 + 2 * 8 and ctypes.sizeof(sb.native.StackConfig) == 6 * 4 + 8
+    assert ctypes.sizeof(sb.native.LayerConfig) == 18 * 4 + 6 * 8 + 8 and ctypes.sizeof(sb.native.StackConfig) == 8 * 4 + 3 * 8
