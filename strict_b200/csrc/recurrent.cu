@@ -46,7 +46,10 @@ __global__ void __launch_bounds__(256) gated_conv_kernel(GatedArgs a, int64_t ro
       }
       acc = fmaf(k[taps - 1], now, acc);
       const int bs = a.s.bs(), g = c / bs;
-      ((T*)a.u)[t * a.s.ld_u() + g * a.s.bs_p() + c - g * bs] = to_t<T>(acc);
+      T* u = (T*)a.u + t * a.s.ld_u() + (int64_t)g * a.s.bs_p() + c - g * bs;
+      *u = to_t<T>(acc);
+      if (c - g * bs == bs - 1)  // columns that fill the block up meet zero weights, but they must be finite
+        for (int j = 1; j <= a.s.bs_p() - bs; j++) u[j] = to_t<T>(0.f);
       if (!a.seq) {  // decode: the row is its sequence's only one, nobody else reads this history
         for (int j = 0; j < taps - 2; j++) hist[(int64_t)j * w] = hist[(int64_t)(j + 1) * w];
         if (taps > 1) hist[(int64_t)(taps - 2) * w] = now;

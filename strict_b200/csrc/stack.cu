@@ -693,7 +693,7 @@ int sb_stack_decode_body(strictb200_model* m, strictb200_kv* kv) {
       continue;
     }
     if (!w.fast_decode) {  // fp32, and widths the tensor-core kernels do not take: the prompt's kernels on B rows
-      const int64_t ld_in = w.ff ? w.n_switch : w.n_in;
+      const int64_t ld_in = ld_in_of(st, w);
       PROF(STRICTB200_K_GEMM_QKV, project_in(m, w, B, b.h, b.part, ld_in, b.oa));
       LatentSplitArgs a = split_args(m, kv, l, 0);
       a.in = b.part; a.ld_in = ld_in; a.lens = kv->d_lens; a.q_out = b.q;
@@ -930,6 +930,7 @@ extern "C" int strictb200_stack_create(strictb200_ctx* ctx, const strictb200_sta
   if (ctx->tp_world != 1) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "models described layer by layer are single-GPU");
   SB_REQUIRE(c.n_layers > 0 && c.d_model > 0 && c.vocab > 0 && c.max_pos > 0 && c.eps > 0, "non-positive dimension");
   SB_REQUIRE(c.norm_groups > 0 && c.d_model % c.norm_groups == 0, "the width must be a multiple of the norm groups");
+  SB_REQUIRE(c.residual_mult != 0 && c.logit_scale != 0, "the residual and the logits need a factor");
   SB_REQUIRE(c.dtype == STRICTB200_BF16 || c.dtype == STRICTB200_FP32, "unknown dtype");
   for (int l = 0; l < c.n_layers; l++) {
     const strictb200_layer_config& y = layers[l];
