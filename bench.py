@@ -361,13 +361,13 @@ def main():
     ap.add_argument("--timeline", default=None, help="also write the per-launch timeline of one graph-replayed decode step (per-block time stamps) to this file")
     ap.add_argument("--no-timeline", action="store_true", help="skip the traced replay (outside every timed region) that gives the per-kernel exposed times")
     ap.add_argument("--no-graph", action="store_true", help="plain launches instead of CUDA-graph replay of the decode step")
-    ap.add_argument("--design", default=None, choices=["kipatar"], help="instead of the headline workload: prefill and decode throughput of this design "
+    ap.add_argument("--design", default=None, choices=["kipatar", "morarax"], help="instead of the headline workload: prefill and decode throughput of this design "
                     "beside the closest existing model at equal size (strict_b200/layered_bench.py; one GPU)")
     ap.add_argument("--sizes", default="8b,0.6b", help="with --design: sizes to run")
     args = ap.parse_args()
     if args.design:
         from strict_b200 import layered_bench
-        layered_bench.run(args.sizes.split(","), args.steps, args.warmup, args.layers)
+        layered_bench.run(args.design, args.sizes.split(","), args.steps, args.warmup, args.layers)
         return
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))

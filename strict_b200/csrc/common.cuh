@@ -682,7 +682,7 @@ struct SbTraceDev {
 static __device__ SbTraceDev sb_trace_dev;
 #define SB_TRACE_TU(name) \
   int sb_trace_set_##name(const SbTraceDev& t) { return cudaMemcpyToSymbol(sb_trace_dev, &t, sizeof t) == cudaSuccess ? 0 : 1; }
-enum { SB_K_GEMM = 1, SB_K_ROWNORM = 2, SB_K_ROPE = 3, SB_K_ATTN = 4, SB_K_COMBINE = 5, SB_K_SWIGLU = 6, SB_K_ROWNORM_TP = 7 };
+enum { SB_K_GEMM = 1, SB_K_ROWNORM = 2, SB_K_ROPE = 3, SB_K_ATTN = 4, SB_K_COMBINE = 5, SB_K_SWIGLU = 6, SB_K_ROWNORM_TP = 7, SB_K_RECURRENCE = 8 };
 __device__ __forceinline__ unsigned long long sb_globaltimer() {
   unsigned long long t;
   asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(t));

@@ -13,10 +13,75 @@ using namespace mix;
 
 namespace {
 
-// grid rows * (item blocks + activation blocks), 256 threads: warp w of an item block owns item 8 * block + w of the row:
-// a query head, a key head, a value head, or (the last item) all gates.
-// VEC: four dims per lane; widths multiples of 4, at most 128 (the rotated half too).
-template <typename T, bool VEC>
+// One head of a row. VEC: four dims per lane (widths multiples of 4, at most 128; so is the rotated half).
+struct HeadItem {
+  bool is_q, is_v;
+  int n;          // dims
+  int64_t col;    // first column of the projection
+  int64_t dst;    // element of q_out, k_out or v_out
+};
+__device__ __forceinline__ HeadItem head_item(const HeadSplitArgs& a, int64_t t, int b, int p, int item) {
+  const HeadShape& s = a.s;
+  HeadItem i;
+  i.is_q = item < s.H; i.is_v = item >= s.H + s.G;
+  const int h = i.is_q ? item : i.is_v ? item - s.H - s.G : item - s.H, row = s.row();
+  i.n = i.is_v ? s.vdim : s.dim;
+  i.col = i.is_q ? (int64_t)h * s.dim : i.is_v ? (int64_t)(s.H + s.G) * s.dim + (int64_t)h * s.vdim : (int64_t)(s.H + h) * s.dim;
+  i.dst = i.is_q ? (t * s.H + h) * row : a.dense ? (t * s.G + h) * row : (((int64_t)b * s.G + h) * a.maxlen + p) * row;
+  return i;
+}
+template <typename T>
+__device__ __forceinline__ void head_vec(const HeadSplitArgs& a, const HeadItem& it, float4 x, const float* cs, const float* sn, int lane) {
+  const HeadShape& s = a.s;
+  const int e = lane * 4, half = s.rot / 2;
+  if (!it.is_v) {
+    const int src = e < half ? lane + half / 4 : lane - half / 4;  // the lane that holds the other half of the pairs
+    float4 o;
+    o.x = __shfl_sync(0xffffffffu, x.x, src & 31); o.y = __shfl_sync(0xffffffffu, x.y, src & 31);
+    o.z = __shfl_sync(0xffffffffu, x.z, src & 31); o.w = __shfl_sync(0xffffffffu, x.w, src & 31);
+    if (e < s.rot) {
+      const int i = e < half ? e : e - half;
+      const float4 c = *(const float4*)(cs + i), d = *(const float4*)(sn + i);
+      const float g = e < half ? -1.f : 1.f;
+      x.x = fmaf(x.x, c.x, g * o.x * d.x); x.y = fmaf(x.y, c.y, g * o.y * d.y);
+      x.z = fmaf(x.z, c.z, g * o.z * d.z); x.w = fmaf(x.w, c.w, g * o.w * d.w);
+    }
+    float r = it.is_q ? 1.f : s.k_scale;
+    if (s.qk_norm) {
+      const float ss = warp_sum(x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w);
+      r *= __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)s.dim), a.eps)));
+    }
+    x.x *= r; x.y *= r; x.z *= r; x.w *= r;
+  }
+  T* dst = (T*)(it.is_q ? a.q_out : it.is_v ? a.v_out : a.k_out) + it.dst;
+  if (e < s.row()) store4<T>(dst + e, x);
+}
+template <typename T>
+__device__ __forceinline__ void head_any(const HeadSplitArgs& a, const HeadItem& it, int64_t rows, int64_t t, const float* cs, const float* sn, float* buf, int lane) {
+  const HeadShape& s = a.s;
+  const int half = s.rot / 2;
+  for (int e = lane; e < it.n; e += 32) buf[e] = proj(a.p, rows, t, it.col + e);
+  __syncwarp();
+  auto value = [&](int e) {
+    if (it.is_v || e >= s.rot) return buf[e];
+    const int i = e < half ? e : e - half;
+    return e < half ? buf[e] * cs[i] - buf[e + half] * sn[i] : buf[e] * cs[i] + buf[e - half] * sn[i];
+  };
+  float r = it.is_q || it.is_v ? 1.f : s.k_scale;
+  if (s.qk_norm && !it.is_v) {
+    float ss = 0.f;
+    for (int e = lane; e < it.n; e += 32) { const float v = value(e); ss += v * v; }
+    r *= __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(warp_sum(ss), (float)s.dim), a.eps)));
+  }
+  T* dst = (T*)(it.is_q ? a.q_out : it.is_v ? a.v_out : a.k_out) + it.dst;
+  const int row = s.row();
+  for (int e = lane; e < row; e += 32) dst[e] = to_t<T>(e < it.n ? value(e) * r : 0.f);
+}
+
+// grid rows * (item blocks + activation blocks), 256 threads: warp w of an item block owns the PER items of the row from
+// (8 * block + w) * PER on: query heads, key heads, value heads, and as the last item all gates. A decode step takes PER = 1 (few
+// rows, short chains), a prompt more, so that a warp has several heads' loads in flight.
+template <typename T, bool VEC, int PER>
 __global__ void __launch_bounds__(256) head_split_kernel(HeadSplitArgs a, int64_t rows, int item_blocks, int act_blks) {
   extern __shared__ float sm[];
   SB_TRACE_BEGIN();
@@ -30,66 +95,29 @@ __global__ void __launch_bounds__(256) head_split_kernel(HeadSplitArgs a, int64_
   if (blk >= item_blocks) {
     act_block<T>(a.act, a.p, rows, t, blk - item_blocks);
   } else {
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int item = blk * 8 + warp;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_heads = s.H + 2 * s.G;
+    const int first = (blk * 8 + warp) * PER;
     const int b = a.seq ? a.seq[t] : (int)t, p = a.pos ? a.pos[t] : a.lens[b];
-    const int row = s.row();
     if (p >= 0 && p < a.max_pos && (a.dense || p < a.maxlen)) {  // the host validates; never index outside the cache
-      const int n_heads = s.H + 2 * s.G;
-      if (item < n_heads) {
-        const bool is_q = item < s.H, is_v = item >= s.H + s.G;
-        const int h = is_q ? item : is_v ? item - s.H - s.G : item - s.H;
-        const int n = is_v ? s.vdim : s.dim;
-        const int64_t col = is_q ? (int64_t)h * s.dim : is_v ? (int64_t)(s.H + s.G) * s.dim + (int64_t)h * s.vdim : (int64_t)(s.H + h) * s.dim;
-        T* dst = is_q ? (T*)a.q_out + (t * s.H + h) * row
-                      : (T*)(is_v ? a.v_out : a.k_out) + (a.dense ? (t * s.G + h) * row : (((int64_t)b * s.G + h) * a.maxlen + p) * row);
-        const float post = is_q || is_v ? 1.f : s.k_scale;
-        const int half = s.rot / 2;
-        const float *cs = a.cos_t + (int64_t)p * half, *sn = a.sin_t + (int64_t)p * half;
-        if constexpr (VEC) {
-          const int e = lane * 4;
-          float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (e < n) x = proj4(a.p, rows, t, col + e);
-          if (!is_v) {
-            const int src = e < half ? lane + half / 4 : lane - half / 4;  // the lane that holds the other half of the pairs
-            float4 o;
-            o.x = __shfl_sync(0xffffffffu, x.x, src & 31); o.y = __shfl_sync(0xffffffffu, x.y, src & 31);
-            o.z = __shfl_sync(0xffffffffu, x.z, src & 31); o.w = __shfl_sync(0xffffffffu, x.w, src & 31);
-            if (e < s.rot) {
-              const int i = e < half ? e : e - half;
-              const float4 c = *(const float4*)(cs + i), d = *(const float4*)(sn + i);
-              const float g = e < half ? -1.f : 1.f;
-              x.x = fmaf(x.x, c.x, g * o.x * d.x); x.y = fmaf(x.y, c.y, g * o.y * d.y);
-              x.z = fmaf(x.z, c.z, g * o.z * d.z); x.w = fmaf(x.w, c.w, g * o.w * d.w);
-            }
-            float r = post;
-            if (s.qk_norm) {
-              const float ss = warp_sum(x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w);
-              r *= __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)s.dim), a.eps)));
-            }
-            x.x *= r; x.y *= r; x.z *= r; x.w *= r;
-          }
-          if (e < row) store4<T>(dst + e, x);
-        } else {
-          float* buf = sm + warp * (s.dim > s.vdim ? s.dim : s.vdim);
-          for (int e = lane; e < n; e += 32) buf[e] = proj(a.p, rows, t, col + e);
-          __syncwarp();
-          auto value = [&](int e) {
-            if (is_v || e >= s.rot) return buf[e];
-            const int i = e < half ? e : e - half;
-            return e < half ? buf[e] * cs[i] - buf[e + half] * sn[i] : buf[e] * cs[i] + buf[e - half] * sn[i];
-          };
-          float r = post;
-          if (s.qk_norm && !is_v) {
-            float ss = 0.f;
-            for (int e = lane; e < n; e += 32) { const float v = value(e); ss += v * v; }
-            r *= __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(warp_sum(ss), (float)s.dim), a.eps)));
-          }
-          for (int e = lane; e < row; e += 32) dst[e] = to_t<T>(e < n ? value(e) * r : 0.f);
+      const float *cs = a.cos_t + (int64_t)p * (s.rot / 2), *sn = a.sin_t + (int64_t)p * (s.rot / 2);
+      HeadItem it[PER];
+      float4 x[PER];
+#pragma unroll
+      for (int i = 0; i < PER; i++)
+        if (first + i < n_heads) {
+          it[i] = head_item(a, t, b, p, first + i);
+          x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (VEC && lane * 4 < it[i].n) x[i] = proj4(a.p, rows, t, it[i].col + lane * 4);
         }
-      } else if (item == n_heads && s.gate) {
-        const int64_t col = (int64_t)(s.H + s.G) * s.dim + (int64_t)s.G * s.vdim;
-        for (int h = lane; h < s.H; h += 32) a.gate_out[t * s.H + h] = sigmoid(proj(a.p, rows, t, col + h));
+#pragma unroll
+      for (int i = 0; i < PER; i++) {
+        if (first + i < n_heads) {
+          if (VEC) head_vec<T>(a, it[i], x[i], cs, sn, lane);
+          else head_any<T>(a, it[i], rows, t, cs, sn, sm + warp * max(s.dim, s.vdim), lane);
+        } else if (first + i == n_heads && s.gate) {
+          const int64_t col = (int64_t)(s.H + s.G) * s.dim + (int64_t)s.G * s.vdim;
+          for (int h = lane; h < s.H; h += 32) a.gate_out[t * s.H + h] = sigmoid(proj(a.p, rows, t, col + h));
+        }
       }
     }
   }
@@ -222,15 +250,17 @@ SB_TRACE_TU(heads)
 
 int k_head_split(strictb200_ctx* ctx, const HeadSplitArgs& a, int64_t T) {
   const HeadShape& s = a.s;
-  const int items = s.H + 2 * s.G + (s.gate ? 1 : 0), item_blocks = (items + 7) / 8, act_blks = act_blocks(a.act);
+  const int per = a.seq && a.p.splits == 1 ? 4 : 1;
+  const int items = s.H + 2 * s.G + (s.gate ? 1 : 0), act_blks = act_blocks(a.act);
   const bool vec = s.dim <= 128 && s.vdim <= 128 && ((s.dim | s.vdim | (s.rot / 2) | (int)(a.p.ld & 3)) & 3) == 0;
+  const int item_blocks = (items + 8 * (vec ? per : 1) - 1) / (8 * (vec ? per : 1));
   const int64_t blocks = T * (item_blocks + act_blks);
   if (blocks > INT32_MAX || a.p.splits > 8) return sb_fail(STRICTB200_ERR_INVALID_ARG, "head split: too many rows or partial sums");
   const size_t smem = vec ? 0 : (size_t)8 * std::max(s.dim, s.vdim) * sizeof(float);
   if (smem > 48 * 1024) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "heads of more than 1536 dims");
   auto go = [&](auto kernel) { return sb_launch(ctx, kernel, dim3((unsigned)blocks), dim3(256), smem, a, T, item_blocks, act_blks); };
-  if (a.f32) SB_CUDA(vec ? go(head_split_kernel<float, true>) : go(head_split_kernel<float, false>));
-  else SB_CUDA(vec ? go(head_split_kernel<bf16, true>) : go(head_split_kernel<bf16, false>));
+  if (a.f32) SB_CUDA(!vec ? go(head_split_kernel<float, false, 1>) : per > 1 ? go(head_split_kernel<float, true, 4>) : go(head_split_kernel<float, true, 1>));
+  else SB_CUDA(!vec ? go(head_split_kernel<bf16, false, 1>) : per > 1 ? go(head_split_kernel<bf16, true, 4>) : go(head_split_kernel<bf16, true, 1>));
   ctx->launches++;
   return STRICTB200_OK;
 }

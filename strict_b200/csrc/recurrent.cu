@@ -5,7 +5,7 @@
 //   log a = -8 r softplus(lam), S <- a S + sqrt(1 - a^2) i u, out = S gelu(y).
 //   * k_gated_conv: u as the operand of the gate product (rounded to bf16 there, so that the product of bf16 matrices with fp32
 //     sums is the exact product of what the recurrence uses), and the convolution's last inputs.
-//   * k_gated_scan: prompts run 256 tokens at a time in a block of 32 channels: every warp folds eight tokens into one (a, b)
+//   * k_gated_scan: prompts run 128 tokens at a time in a block of 32 channels: every warp folds eight tokens into one (a, b)
 //     pair, the pairs meet in shared memory, and each warp replays its tokens from the state before them. Decode is one
 //     step per channel. sqrt(1 - a^2) is taken as sqrt(-expm1(2 log a)), which stays exact where a is close to one.
 // Retention: S <- decay S + k v^T, o = S^T q.
@@ -58,6 +58,60 @@ __global__ void __launch_bounds__(256) gated_conv_kernel(GatedArgs a, int64_t ro
   }
   SB_TRACE_END(SB_K_ROPE, 0);
 }
+// Prompt rows, four channels of CONV_ROWS consecutive rows per thread: the taps slide over registers. Blocks of 8 k channels.
+constexpr int CONV_ROWS = 16;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) gated_conv_rows_kernel(GatedArgs a, int64_t rows) {
+  const int w = a.s.width, c = ((int)blockIdx.x * 128 + (int)threadIdx.x) * 4;
+  const int64_t t0 = (int64_t)blockIdx.y * CONV_ROWS;
+  pdl_trigger();
+  pdl_wait();
+  if (c >= w) return;
+  const int n = (int)min((int64_t)CONV_ROWS, rows - t0);
+  const float4 xb = *(const float4*)(a.x_bias + c), cb = *(const float4*)(a.conv_bias + c);
+  float k[4][TAPS];
+#pragma unroll
+  for (int j = 0; j < 4; j++)
+#pragma unroll
+    for (int i = 0; i < TAPS; i++) k[j][i] = a.conv[(int64_t)(c + j) * TAPS + i];
+  auto row = [&](int64_t t) {
+    const float4 v = *(const float4*)(a.p.in + t * a.p.ld + w + c);
+    return make_float4(v.x + xb.x, v.y + xb.y, v.z + xb.z, v.w + xb.w);
+  };
+  float4 x[CONV_ROWS];
+#pragma unroll
+  for (int i = 0; i < CONV_ROWS; i++)
+    if (i < n) x[i] = row(t0 + i);
+  float4 win[TAPS];  // the row and the ones before it, oldest first
+  int b = a.seq[t0];
+  int64_t li = t0 - a.qstart[b];
+#pragma unroll
+  for (int i = 0; i < CONV_ROWS; i++) {
+    if (i >= n) break;
+    const int64_t t = t0 + i;
+    if (i > 0) {
+      const int b1 = a.seq[t];
+      li = b1 == b ? li + 1 : 0;
+      b = b1;
+    }
+    if (i == 0 || li == 0) {
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; j++) {
+        const int64_t back = TAPS - 1 - j;
+        win[j] = back <= li ? row(t - back) : *(const float4*)(a.hist + ((int64_t)b * (TAPS - 1) + TAPS - 1 + li - back) * w + c);
+      }
+    }
+    win[TAPS - 1] = x[i];
+    float4 o = cb;
+#pragma unroll
+    for (int j = 0; j < TAPS; j++) {
+      o.x = fmaf(k[0][j], win[j].x, o.x); o.y = fmaf(k[1][j], win[j].y, o.y); o.z = fmaf(k[2][j], win[j].z, o.z); o.w = fmaf(k[3][j], win[j].w, o.w);
+    }
+    store4<T>((T*)a.u + t * a.s.ld_u() + c, o);
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; j++) win[j] = win[j + 1];
+  }
+}
 // the convolution's last inputs after a prompt's rows; grid (channel blocks, nb)
 __global__ void __launch_bounds__(256) conv_hist_kernel(GatedArgs a, int64_t rows) {
   pdl_trigger();
@@ -74,17 +128,42 @@ __global__ void __launch_bounds__(256) conv_hist_kernel(GatedArgs a, int64_t row
 
 // ------------------------------------------------------------------ gated recurrence
 struct Step { float a, b; };  // S <- a S + b
+// The gates' functions, for fp32 results, and for results that end in bf16: exponentials through ex2.approx (2^-22), and the
+// series of 1 - exp(x) where that would cancel (x > -1/4; the first term left out is below 2^-23 of the sum).
 template <typename T>
-__device__ __forceinline__ Step gated_step(const GatedArgs& g, int64_t t, int c, int64_t gr, int64_t gi, int64_t uo, float rb, float ib, float decay) {
-  const float r = sigmoid(g.gates[t * 2 * g.s.width + gr] + rb), i = sigmoid(g.gates[t * 2 * g.s.width + gi] + ib);
+struct Gates {
+  static __device__ __forceinline__ float sig(float z) { return sigmoid(z); }
+  static __device__ __forceinline__ float ex(float z) { return expf(z); }
+  static __device__ __forceinline__ float one_minus_exp(float x) { return -expm1f(x); }
+  static __device__ __forceinline__ float gelu(float z) { return sb_gelu_tanh(z); }
+};
+template <>
+struct Gates<bf16> {
+  static __device__ __forceinline__ float ex(float z) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(z * 1.4426950408889634f));
+    return y;
+  }
+  static __device__ __forceinline__ float sig(float z) { return __fdividef(1.0f, 1.0f + ex(-z)); }
+  static __device__ __forceinline__ float one_minus_exp(float x) {  // x <= 0
+    const float series = -x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 720.f, 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
+    return x > -0.25f ? series : 1.f - ex(x);
+  }
+  // 1/2 (1 + tanh(y)) = sigmoid(2 y)
+  static __device__ __forceinline__ float gelu(float z) { return z * sig(1.5957691216f * fmaf(0.044715f * z * z, z, z)); }
+};
+template <typename T>
+__device__ __forceinline__ Step gated_step(const GatedArgs& g, int64_t t, int64_t gr, int64_t gi, int64_t uo, float rb, float ib, float decay) {
+  typedef Gates<T> G;
+  const float* gates = g.gates + t * 2 * g.s.width;
+  const float r = G::sig(gates[gr] + rb), i = G::sig(gates[gi] + ib), u = to_f(((const T*)g.u)[t * g.s.ld_u() + uo]);
   const float la = decay * r;
-  const float u = to_f(((const T*)g.u)[t * g.s.ld_u() + uo]);
-  return Step{expf(la), sqrtf(-expm1f(2.f * la)) * i * u};
+  return Step{G::ex(la), sqrtf(G::one_minus_exp(2.f * la)) * i * u};
 }
-constexpr int SCAN_WARPS = 32, SCAN_PER = 8;  // tokens per warp and pass
-// grid (ceil(width / 32), nb), 1024 threads: lane = channel, warp = run of tokens
+constexpr int SCAN_WARPS = 16, SCAN_PER = 8;  // tokens per warp and pass
+// grid (ceil(width / 32), nb), 512 threads: lane = channel, warp = run of tokens
 template <typename T>
-__global__ void __launch_bounds__(1024) gated_scan_kernel(GatedArgs g, int64_t rows) {
+__global__ void __launch_bounds__(SCAN_WARPS * 32, 2) gated_scan_kernel(GatedArgs g, int64_t rows) {
   __shared__ Step fold[SCAN_WARPS][32];
   __shared__ float carry[32];
   SB_TRACE_BEGIN();
@@ -107,8 +186,8 @@ __global__ void __launch_bounds__(1024) gated_scan_kernel(GatedArgs g, int64_t r
 #pragma unroll
     for (int j = 0; j < SCAN_PER; j++) {
       const bool on = live && first + j < n;
-      st[j] = on ? gated_step<T>(g, row0 + first + j, c, gr, gi, uo, rb, ib, decay) : Step{1.f, 0.f};
-      y[j] = on ? proj(g.p, rows, row0 + first + j, c) : 0.f;
+      st[j] = on ? gated_step<T>(g, row0 + first + j, gr, gi, uo, rb, ib, decay) : Step{1.f, 0.f};
+      y[j] = on ? g.p.in[(row0 + first + j) * g.p.ld + c] : 0.f;  // a prompt's projection is finished
     }
     Step all{1.f, 0.f};
 #pragma unroll
@@ -120,14 +199,14 @@ __global__ void __launch_bounds__(1024) gated_scan_kernel(GatedArgs g, int64_t r
 #pragma unroll
     for (int j = 0; j < SCAN_PER; j++) {
       s = fmaf(st[j].a, s, st[j].b);
-      if (live && first + j < n) ((T*)g.out)[(row0 + first + j) * g.ldo + c] = to_t<T>(s * sb_gelu_tanh(y[j] + yb));
+      if (live && first + j < n) ((T*)g.out)[(row0 + first + j) * g.ldo + c] = to_t<T>(s * Gates<T>::gelu(y[j] + yb));
     }
     __syncthreads();  // everybody has read the state before this pass
     if (warp == SCAN_WARPS - 1) carry[lane] = s;
     __syncthreads();
   }
   if (warp == 0 && live) g.state[(int64_t)seq * w + c] = carry[lane];
-  SB_TRACE_END(SB_K_ATTN, 0);
+  SB_TRACE_END(SB_K_RECURRENCE, 0);
 }
 // decode: grid (ceil(width / 256), rows)
 template <typename T>
@@ -141,12 +220,12 @@ __global__ void __launch_bounds__(256) gated_step_kernel(GatedArgs g, int64_t ro
   if (c < w) {
     const int bs = g.s.bs(), blk = c / bs, in_blk = c - blk * bs;
     const int64_t gr = (int64_t)blk * 2 * bs + in_blk;
-    const Step st = gated_step<T>(g, t, c, gr, gr + bs, (int64_t)blk * g.s.bs_p() + in_blk, g.r_bias[c], g.i_bias[c], g.decay[c]);
+    const Step st = gated_step<T>(g, t, gr, gr + bs, (int64_t)blk * g.s.bs_p() + in_blk, g.r_bias[c], g.i_bias[c], g.decay[c]);
     const float s = fmaf(st.a, g.state[t * w + c], st.b);
     g.state[t * w + c] = s;
-    ((T*)g.out)[t * g.ldo + c] = to_t<T>(s * sb_gelu_tanh(proj(g.p, rows, t, c) + g.y_bias[c]));
+    ((T*)g.out)[t * g.ldo + c] = to_t<T>(s * Gates<T>::gelu(proj(g.p, rows, t, c) + g.y_bias[c]));
   }
-  SB_TRACE_END(SB_K_ATTN, 0);
+  SB_TRACE_END(SB_K_RECURRENCE, 0);
 }
 
 // ------------------------------------------------------------------ retention, any widths
@@ -223,7 +302,7 @@ __global__ void __launch_bounds__(256) retention_decode_kernel(RetentionArgs a, 
     pdl_wait();
     SB_TRACE_WAITED();
     act_block<bf16>(a.act, a.p, B, (blockIdx.x - heads) / act_blks, (int)((blockIdx.x - heads) % act_blks));
-    SB_TRACE_END(SB_K_ATTN, 0);
+    SB_TRACE_END(SB_K_RECURRENCE, 0);
     return;
   }
   const int h = (int)(blockIdx.x % s.H);
@@ -298,7 +377,7 @@ __global__ void __launch_bounds__(256) retention_decode_kernel(RetentionArgs a, 
   ss = block_sum(ss, red);
   const float r = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)s.vdim), a.eps)));
   for (int v = tid; v < s.vdim; v += 256) ((bf16*)a.out)[b * a.ldo + (int64_t)h * s.vdim + v] = __float2bfloat16_rn(po[v] * r * (gs[v] * sigmoid(gs[v])));
-  SB_TRACE_END(SB_K_ATTN, 0);
+  SB_TRACE_END(SB_K_RECURRENCE, 0);
 }
 size_t retention_decode_smem(const HeadShape& s) { return (size_t)(4 * s.dim + 2 * s.vdim + 256 / (s.vdim / 4) * s.vdim) * sizeof(float); }
 
@@ -310,7 +389,15 @@ int k_gated_conv(strictb200_ctx* ctx, const GatedArgs& a, int64_t T) {
   const int ch = (a.s.width + 255) / 256, act = act_blocks(a.act);
   if (T * (ch + act) > INT32_MAX || a.p.splits > 8) return sb_fail(STRICTB200_ERR_INVALID_ARG, "gated recurrence: too many rows or partial sums");
   const dim3 grid((unsigned)(T * (ch + act)));
-  if (a.f32) SB_CUDA(sb_launch(ctx, gated_conv_kernel<float>, grid, dim3(256), 0, a, T, ch, act));
+  const GatedShape& s = a.s;
+  const bool rows = a.seq && !a.act.kind && a.p.splits == 1 && s.width % 4 == 0 && s.bs() % 8 == 0 && a.p.ld % 4 == 0 && s.taps >= 2 && s.taps <= 4 &&
+                    T <= (int64_t)65535 * CONV_ROWS;
+  if (rows) {
+    const dim3 g((unsigned)((s.width / 4 + 127) / 128), (unsigned)((T + CONV_ROWS - 1) / CONV_ROWS));
+    auto go = [&](auto kernel) { return sb_launch(ctx, kernel, g, dim3(128), 0, a, T); };
+    if (a.f32) SB_CUDA(s.taps == 2 ? go(gated_conv_rows_kernel<float, 2>) : s.taps == 3 ? go(gated_conv_rows_kernel<float, 3>) : go(gated_conv_rows_kernel<float, 4>));
+    else SB_CUDA(s.taps == 2 ? go(gated_conv_rows_kernel<bf16, 2>) : s.taps == 3 ? go(gated_conv_rows_kernel<bf16, 3>) : go(gated_conv_rows_kernel<bf16, 4>));
+  } else if (a.f32) SB_CUDA(sb_launch(ctx, gated_conv_kernel<float>, grid, dim3(256), 0, a, T, ch, act));
   else SB_CUDA(sb_launch(ctx, gated_conv_kernel<bf16>, grid, dim3(256), 0, a, T, ch, act));
   ctx->launches++;
   if (!a.seq || a.s.taps < 2) return STRICTB200_OK;
@@ -326,8 +413,8 @@ int k_gated_scan(strictb200_ctx* ctx, const GatedArgs& a, int64_t T) {
     else SB_CUDA(sb_launch(ctx, gated_step_kernel<bf16>, grid, dim3(256), 0, a, T));
   } else {
     const dim3 grid((unsigned)((a.s.width + 31) / 32), (unsigned)a.nb);
-    if (a.f32) SB_CUDA(sb_launch(ctx, gated_scan_kernel<float>, grid, dim3(1024), 0, a, T));
-    else SB_CUDA(sb_launch(ctx, gated_scan_kernel<bf16>, grid, dim3(1024), 0, a, T));
+    if (a.f32) SB_CUDA(sb_launch(ctx, gated_scan_kernel<float>, grid, dim3(SCAN_WARPS * 32), 0, a, T));
+    else SB_CUDA(sb_launch(ctx, gated_scan_kernel<bf16>, grid, dim3(SCAN_WARPS * 32), 0, a, T));
   }
   ctx->launches++;
   return STRICTB200_OK;

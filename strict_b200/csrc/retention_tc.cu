@@ -7,8 +7,10 @@
 // The state stays in tensor memory in fp32 from the first chunk to the last (lane = query/key dim, column = value dim). As the
 // operand of Q S it is written to shared memory as two bf16 terms, and so is V'; q, k and v themselves are bf16, the powers of
 // the decay fp32. Tensor memory: P, O, O2 and S, 128 columns each.
-//   warps 0..7  rows: thread (row, half) owns 64 columns of row `row` of every tile
-//   warp 8      one lane issues copies and products
+//   warps 0..15  rows: thread (row, quarter) owns 32 columns of row `row` of every tile
+//   warp 16      one lane issues copies and products
+// A row thread takes its sums of a chunk out of tensor memory, prepares the operands of the next chunk (state, V'), and only
+// then norms, gates and stores, while the next chunk's products run.
 // Every mbarrier wait is bounded: on expiry the block records an error word in host-visible memory, stops, frees its tensor
 // memory and returns.
 #include "mixers.cuh"
@@ -19,7 +21,8 @@ using namespace tc;
 namespace {
 
 constexpr int CHUNK = 128;
-constexpr int RT_THREADS = 288;
+constexpr int ROW_THREADS = 4 * CHUNK;
+constexpr int RT_THREADS = ROW_THREADS + 32;
 
 struct RtArgs {
   int H, dim, vdim;
@@ -61,11 +64,11 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
   if (threadIdx.x == 0) {
     mbar_init(smem_u32(&bar_qk), 1); mbar_init(smem_u32(&bar_v), 1);
     mbar_init(smem_u32(&bar_s), 1); mbar_init(smem_u32(&bar_o), 1); mbar_init(smem_u32(&bar_state), 1);
-    mbar_init(smem_u32(&s_ready), 256); mbar_init(smem_u32(&vp_ready), 256); mbar_init(smem_u32(&p_ready), 256);
+    mbar_init(smem_u32(&s_ready), ROW_THREADS); mbar_init(smem_u32(&vp_ready), ROW_THREADS); mbar_init(smem_u32(&p_ready), ROW_THREADS);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   if (threadIdx.x <= CHUNK) pw[threadIdx.x] = (float)pow((double)a.decay[h], (double)threadIdx.x);
-  if (warp == 8) {
+  if (warp == 16) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_base_slot)), "r"(512u) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
@@ -77,7 +80,7 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
   constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(128 >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
   constexpr uint32_t idesc_b = idesc | (1u << 16), idesc_ab = idesc_b | (1u << 15);
 
-  if (warp == 8) {
+  if (warp == 16) {
     if (lane == 0) {
       auto load = [&](int c) {
         const int row = (int)row0 + c * CHUNK;
@@ -137,57 +140,45 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
       if (!good) set_status(a.status, 17);
     }
   } else {
-    const int row = (int)threadIdx.x & (CHUNK - 1), half = (int)threadIdx.x >> 7;
+    const int row = (int)threadIdx.x & (CHUNK - 1), quarter = (int)threadIdx.x >> 7;
     const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
-    const int c0 = half * 64;  // first of this thread's columns, in every tile
-    auto rows_sync = [&]() { asm volatile("bar.sync 1, 256;" ::: "memory"); };
-    float* S = a.state + (((int64_t)b * a.H + h) * a.dim + row) * a.vdim;  // state row `row` (where it exists)
-    bool ok = true;
-    for (int c = 0; c < chunks; c++) {
-      const uint32_t ph = (uint32_t)(c & 1);
+    const int c0 = quarter * 32;  // first of this thread's columns, in every tile
+    const uint32_t box = (uint32_t)((quarter >> 1) * HALF_BYTES);
+    const int chunk0 = (quarter & 1) * 4;  // first of its 16-byte chunks in the box's row
+    auto rows_sync = [&]() { asm volatile("bar.sync 1, 512;" ::: "memory"); };
+    float* S = a.state + (((int64_t)b * a.H + h) * a.dim + row) * a.vdim + c0;  // this thread's part of the state (where it exists)
+    const bool s_vec = (a.vdim & 3) == 0;
+    const bool g_vec = ((a.vdim | (int)(a.ld_g & 3)) & 3) == 0 && ((uintptr_t)a.g & 15) == 0;
+    const bool o_vec = ((a.vdim | (int)(a.ldo & 7)) & 7) == 0 && ((uintptr_t)a.out & 15) == 0;
+
+    // Operands of a chunk of n tokens: the state before it as two bf16 tiles, decay^n times it back to tensor memory; the values
+    // under their powers of the decay at the chunk's end.
+    auto operands = [&](int c, uint32_t* r) -> bool {
       const int n = min(CHUNK, n_all - c * CHUNK);
-      if (c > 0 && !mbar_wait(smem_u32(&bar_state), ph ^ 1)) { ok = false; break; }
-      tc_fence_after();
-      // ---- the state before the chunk: operand tiles, and decay^n times it back to tensor memory
       const float dn = pw[n];
 #pragma unroll
-      for (int q = 0; q < 2; q++) {
-        uint32_t r[32];
-        if (c > 0) {
-          tc_ld32(tS + lane_base + (uint32_t)(c0 + q * 32), r);
-          tc_wait_ld();
-        } else {
-#pragma unroll
-          for (int j = 0; j < 32; j++) {
-            const int v = c0 + q * 32 + j;
-            r[j] = __float_as_uint(row < a.dim && v < a.vdim ? S[v] : 0.f);
-          }
-        }
-#pragma unroll
-        for (int j = 0; j < 4; j++) {
-          uint4 hi, lo;
-          split2(__uint_as_float(r[8 * j]), __uint_as_float(r[8 * j + 1]), hi.x, lo.x);
-          split2(__uint_as_float(r[8 * j + 2]), __uint_as_float(r[8 * j + 3]), hi.y, lo.y);
-          split2(__uint_as_float(r[8 * j + 4]), __uint_as_float(r[8 * j + 5]), hi.z, lo.z);
-          split2(__uint_as_float(r[8 * j + 6]), __uint_as_float(r[8 * j + 7]), hi.w, lo.w);
-          const uint32_t off = (uint32_t)(half * HALF_BYTES) + box_off(row, q * 4 + j);
-          *(uint4*)(bSh + off) = hi;
-          *(uint4*)(bSl + off) = lo;
-        }
-#pragma unroll
-        for (int j = 0; j < 32; j++) r[j] = __float_as_uint(__uint_as_float(r[j]) * dn);
-        tc_st32(tS + lane_base + (uint32_t)(c0 + q * 32), r);
+      for (int j = 0; j < 4; j++) {
+        uint4 hi, lo;
+        split2(__uint_as_float(r[8 * j]), __uint_as_float(r[8 * j + 1]), hi.x, lo.x);
+        split2(__uint_as_float(r[8 * j + 2]), __uint_as_float(r[8 * j + 3]), hi.y, lo.y);
+        split2(__uint_as_float(r[8 * j + 4]), __uint_as_float(r[8 * j + 5]), hi.z, lo.z);
+        split2(__uint_as_float(r[8 * j + 6]), __uint_as_float(r[8 * j + 7]), hi.w, lo.w);
+        const uint32_t off = box + box_off(row, chunk0 + j);
+        *(uint4*)(bSh + off) = hi;
+        *(uint4*)(bSl + off) = lo;
       }
+#pragma unroll
+      for (int j = 0; j < 32; j++) r[j] = __float_as_uint(__uint_as_float(r[j]) * dn);
+      tc_st32(tS + lane_base + (uint32_t)c0, r);
       tc_wait_st();
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       tc_fence_before();
       arrive(&s_ready);
-      // ---- V' = the values under their powers of the decay at the end of the chunk
-      if (!mbar_wait(smem_u32(&bar_v), ph)) { ok = false; break; }
+      if (!mbar_wait(smem_u32(&bar_v), (uint32_t)(c & 1))) return false;
       const float wv = row < n ? pw[n - 1 - row] : 0.f;
 #pragma unroll
-      for (int j = 0; j < 8; j++) {
-        const uint32_t off = (uint32_t)(half * HALF_BYTES) + box_off(row, j);
+      for (int j = 0; j < 4; j++) {
+        const uint32_t off = box + box_off(row, chunk0 + j);
         const uint4 v = *(const uint4*)(bV + off);
         uint4 hi, lo;
         auto both = [&](uint32_t x, uint32_t& o_hi, uint32_t& o_lo) {
@@ -199,38 +190,61 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
       }
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       arrive(&vp_ready);
+      return true;
+    };
+
+    bool ok = true;
+    {
+      uint32_t r[32];
+#pragma unroll
+      for (int j = 0; j < 8; j++) {
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (row < a.dim && c0 + 4 * j < a.vdim) {
+          if (s_vec) x = *(const float4*)(S + 4 * j);
+          else {
+            x.x = S[4 * j];
+            if (c0 + 4 * j + 1 < a.vdim) x.y = S[4 * j + 1];
+            if (c0 + 4 * j + 2 < a.vdim) x.z = S[4 * j + 2];
+            if (c0 + 4 * j + 3 < a.vdim) x.w = S[4 * j + 3];
+          }
+        }
+        r[4 * j] = __float_as_uint(x.x); r[4 * j + 1] = __float_as_uint(x.y); r[4 * j + 2] = __float_as_uint(x.z); r[4 * j + 3] = __float_as_uint(x.w);
+      }
+      ok = operands(0, r);
+    }
+    for (int c = 0; c < chunks && ok; c++) {
+      const uint32_t ph = (uint32_t)(c & 1);
+      const int n = min(CHUNK, n_all - c * CHUNK);
       // ---- P under the decay
       if (!mbar_wait(smem_u32(&bar_s), ph)) { ok = false; break; }
       tc_fence_after();
-#pragma unroll 1
-      for (int q = 2 * half; q < 2 * half + 2; q++) {
+      {
         uint32_t r[32], hi[16], lo[16];
-        tc_ld32(tP + lane_base + (uint32_t)(q * 32), r);
+        tc_ld32(tP + lane_base + (uint32_t)c0, r);
         tc_wait_ld();
 #pragma unroll
         for (int j = 0; j < 16; j++) {
-          const int k = q * 32 + 2 * j;
+          const int k = c0 + 2 * j;
           const float p0 = k <= row ? __uint_as_float(r[2 * j]) * pw[row - k] : 0.f;
           const float p1 = k + 1 <= row ? __uint_as_float(r[2 * j + 1]) * pw[row - k - 1] : 0.f;
           split2(p0, p1, hi[j], lo[j]);
         }
-        tc_st16(tP + lane_base + (uint32_t)(q * 32), hi);
-        tc_st16(tP + lane_base + (uint32_t)(q * 32 + 16), lo);
+        tc_st16(tP + lane_base + (uint32_t)c0, hi);
+        tc_st16(tP + lane_base + (uint32_t)(c0 + 16), lo);
       }
       tc_wait_st();
       tc_fence_before();
       arrive(&p_ready);
-      // ---- output of the chunk; the gates are on their way while the products run
+      // ---- the gates are on their way while the products run
       const bool live = row < n;
       const int64_t t = row0 + c * CHUNK + row;
       const float* g = a.g + t * a.ld_g + (int64_t)h * a.vdim + c0;
-      const bool vec = ((a.vdim | (int)(a.ld_g & 3)) & 3) == 0 && ((uintptr_t)a.g & 15) == 0;
-      float gv[64];
+      float gv[32];
 #pragma unroll
-      for (int j = 0; j < 16; j++) {
+      for (int j = 0; j < 8; j++) {
         float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
         if (live && c0 + 4 * j < a.vdim) {
-          if (vec) x = *(const float4*)(g + 4 * j);
+          if (g_vec) x = *(const float4*)(g + 4 * j);
           else {
             x.x = g[4 * j];
             if (c0 + 4 * j + 1 < a.vdim) x.y = g[4 * j + 1];
@@ -240,38 +254,52 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
         }
         gv[4 * j] = x.x; gv[4 * j + 1] = x.y; gv[4 * j + 2] = x.z; gv[4 * j + 3] = x.w;
       }
+      // ---- sums of the chunk
       if (!mbar_wait(smem_u32(&bar_o), ph)) { ok = false; break; }
       tc_fence_after();
       const float d1 = pw[min(row + 1, CHUNK)];
-      float ss = 0.f;
-      float o[64];
-#pragma unroll
-      for (int q = 0; q < 2; q++) {
+      float o[32], ss = 0.f;
+      {
         uint32_t r[32], r2[32];
-        tc_ld32(tO + lane_base + (uint32_t)(c0 + q * 32), r);
-        tc_ld32(tO2 + lane_base + (uint32_t)(c0 + q * 32), r2);
+        tc_ld32(tO + lane_base + (uint32_t)c0, r);
+        tc_ld32(tO2 + lane_base + (uint32_t)c0, r2);
         tc_wait_ld();
 #pragma unroll
         for (int j = 0; j < 32; j++) {
-          const float v = fmaf(d1, __uint_as_float(r2[j]), __uint_as_float(r[j]));
-          o[q * 32 + j] = v;
-          ss = fmaf(v, v, ss);  // columns beyond vdim are zero
+          o[j] = fmaf(d1, __uint_as_float(r2[j]), __uint_as_float(r[j]));
+          ss = fmaf(o[j], o[j], ss);  // columns beyond vdim are zero
         }
       }
-      x_sum[half][row] = ss;
+      if (quarter >= 2) x_sum[quarter - 2][row] = ss;
+      if (!mbar_wait(smem_u32(&bar_state), ph)) { ok = false; break; }
+      tc_fence_after();
+      {
+        uint32_t r[32];
+        tc_ld32(tS + lane_base + (uint32_t)c0, r);
+        tc_wait_ld();
+        if (c + 1 < chunks) {
+          ok = operands(c + 1, r);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 32; j++)
+            if (row < a.dim && c0 + j < a.vdim) S[j] = __uint_as_float(r[j]);
+        }
+      }
+      // ---- norm, gate, store (the sums of the four threads of a row meet in two steps)
+      rows_sync();
+      if (quarter < 2) x_sum[quarter][row] += ss;
       rows_sync();
       ss = x_sum[0][row] + x_sum[1][row];
       rows_sync();
-      const float rn = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)a.vdim), a.eps)));
-      bf16* dst = a.out + t * a.ldo + (int64_t)h * a.vdim + c0;
-      const bool wide = ((a.vdim | (int)(a.ldo & 7)) & 7) == 0 && ((uintptr_t)a.out & 15) == 0;
+      const float rn = rsqrtf(ss / (float)a.vdim + a.eps);
       if (live) {
+        bf16* dst = a.out + t * a.ldo + (int64_t)h * a.vdim + c0;
 #pragma unroll
-        for (int j = 0; j < 64; j += 8) {
+        for (int j = 0; j < 32; j += 8) {
           float y[8];
 #pragma unroll
-          for (int i = 0; i < 8; i++) y[i] = o[j + i] * rn * (gv[j + i] * mix::sigmoid(gv[j + i]));
-          if (wide) {
+          for (int i = 0; i < 8; i++) y[i] = o[j + i] * rn * __fdividef(gv[j + i], 1.0f + __expf(-gv[j + i]));
+          if (o_vec) {
             if (c0 + j < a.vdim)
               *(uint4*)(dst + j) = make_uint4(mix::pack_bf16(y[0], y[1]), mix::pack_bf16(y[2], y[3]), mix::pack_bf16(y[4], y[5]), mix::pack_bf16(y[6], y[7]));
           } else {
@@ -282,28 +310,11 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
         }
       }
     }
-    if (ok && chunks > 0) {
-      ok = mbar_wait(smem_u32(&bar_state), (uint32_t)((chunks - 1) & 1));
-      tc_fence_after();
-      if (ok) {
-#pragma unroll 1
-        for (int q = 0; q < 2; q++) {
-          uint32_t r[32];
-          tc_ld32(tS + lane_base + (uint32_t)(c0 + q * 32), r);
-          tc_wait_ld();
-#pragma unroll
-          for (int j = 0; j < 32; j++) {
-            const int v = c0 + q * 32 + j;
-            if (row < a.dim && v < a.vdim) S[v] = __uint_as_float(r[j]);
-          }
-        }
-      }
-    }
     if (!ok && row == 0) set_status(a.status, 18);
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 8) {
+  if (warp == 16) {
     tc_fence_after();
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tP), "r"(512u) : "memory");
   }

@@ -8,7 +8,7 @@ dependent launches overlap (programmatic dependent launch, loads issued before t
 wait), which per-kernel timings of separate launches cannot."""
 import numpy as np
 
-KERNELS = {1: "gemm", 2: "rownorm", 3: "rope", 4: "attn_decode", 5: "attn_combine", 6: "swiglu", 7: "rownorm_allreduce"}
+KERNELS = {1: "gemm", 2: "rownorm", 3: "rope", 4: "attn_decode", 5: "attn_combine", 6: "swiglu", 7: "rownorm_allreduce", 8: "recurrence"}
 
 
 def launches(records, gemm_names=None):
