@@ -545,6 +545,7 @@ struct RetentionArgs {
   void* out = nullptr;
   int64_t ldo = 0;
   bool f32 = false;
+  float* seg_state = nullptr;  // k_retention_prefill: scratch [sb_retention_segments, nb, H, dim, vdim] when that is more than one
   // k_retention_decode: straight from the projection
   const float *cos_t = nullptr, *sin_t = nullptr;
   const int32_t* cache_lens = nullptr;  // [B] positions of the new tokens
@@ -554,6 +555,7 @@ struct RetentionArgs {
 int k_retention_any(strictb200_ctx*, const RetentionArgs& a);            // any widths, token by token
 bool sb_retention_prefill_fits(const HeadShape& s);
 int k_retention_prefill(strictb200_ctx*, const RetentionArgs& a, int64_t T);  // retention_tc.cu: chunks of 128 tokens
+int sb_retention_segments(strictb200_ctx*, const HeadShape& s, int nb, int max_new);
 bool sb_retention_decode_fits(const HeadShape& s);
 int k_retention_decode(strictb200_ctx*, const RetentionArgs& a, int64_t B);
 size_t sb_attn_decode_scratch(int B, int Hq, int D, int nsplit);

@@ -31,20 +31,16 @@ __device__ __forceinline__ HeadItem head_item(const HeadSplitArgs& a, int64_t t,
   return i;
 }
 template <typename T>
-__device__ __forceinline__ void head_vec(const HeadSplitArgs& a, const HeadItem& it, float4 x, const float* cs, const float* sn, int lane) {
+__device__ __forceinline__ void head_vec(const HeadSplitArgs& a, const HeadItem& it, float4 x, const float4& c, const float4& d, int src, int lane) {
   const HeadShape& s = a.s;
-  const int e = lane * 4, half = s.rot / 2;
+  const int e = lane * 4;
   if (!it.is_v) {
-    const int src = e < half ? lane + half / 4 : lane - half / 4;  // the lane that holds the other half of the pairs
     float4 o;
     o.x = __shfl_sync(0xffffffffu, x.x, src & 31); o.y = __shfl_sync(0xffffffffu, x.y, src & 31);
     o.z = __shfl_sync(0xffffffffu, x.z, src & 31); o.w = __shfl_sync(0xffffffffu, x.w, src & 31);
     if (e < s.rot) {
-      const int i = e < half ? e : e - half;
-      const float4 c = *(const float4*)(cs + i), d = *(const float4*)(sn + i);
-      const float g = e < half ? -1.f : 1.f;
-      x.x = fmaf(x.x, c.x, g * o.x * d.x); x.y = fmaf(x.y, c.y, g * o.y * d.y);
-      x.z = fmaf(x.z, c.z, g * o.z * d.z); x.w = fmaf(x.w, c.w, g * o.w * d.w);
+      x.x = fmaf(x.x, c.x, o.x * d.x); x.y = fmaf(x.y, c.y, o.y * d.y);
+      x.z = fmaf(x.z, c.z, o.z * d.z); x.w = fmaf(x.w, c.w, o.w * d.w);
     }
     float r = it.is_q ? 1.f : s.k_scale;
     if (s.qk_norm) {
@@ -101,7 +97,13 @@ __global__ void __launch_bounds__(256) head_split_kernel(HeadSplitArgs a, int64_
     if (p >= 0 && p < a.max_pos && (a.dense || p < a.maxlen)) {  // the host validates; never index outside the cache
       const float *cs = a.cos_t + (int64_t)p * (s.rot / 2), *sn = a.sin_t + (int64_t)p * (s.rot / 2);
       HeadItem it[PER];
-      float4 x[PER];
+      float4 x[PER], c = make_float4(0.f, 0.f, 0.f, 0.f), d = c;  // this lane's cosines, and its sines with the sign of its half
+      const int e = lane * 4, half = s.rot / 2, src = e < half ? lane + half / 4 : lane - half / 4;  // the lane of the other half of its pairs
+      if (VEC && e < s.rot && first < s.H + s.G) {
+        c = *(const float4*)(cs + (e < half ? e : e - half));
+        d = *(const float4*)(sn + (e < half ? e : e - half));
+        if (e < half) d = make_float4(-d.x, -d.y, -d.z, -d.w);
+      }
 #pragma unroll
       for (int i = 0; i < PER; i++)
         if (first + i < n_heads) {
@@ -112,7 +114,7 @@ __global__ void __launch_bounds__(256) head_split_kernel(HeadSplitArgs a, int64_
 #pragma unroll
       for (int i = 0; i < PER; i++) {
         if (first + i < n_heads) {
-          if (VEC) head_vec<T>(a, it[i], x[i], cs, sn, lane);
+          if (VEC) head_vec<T>(a, it[i], x[i], c, d, src, lane);
           else head_any<T>(a, it[i], rows, t, cs, sn, sm + warp * max(s.dim, s.vdim), lane);
         } else if (first + i == n_heads && s.gate) {
           const int64_t col = (int64_t)(s.H + s.G) * s.dim + (int64_t)s.G * s.vdim;

@@ -5,7 +5,7 @@
 //   log a = -8 r softplus(lam), S <- a S + sqrt(1 - a^2) i u, out = S gelu(y).
 //   * k_gated_conv: u as the operand of the gate product (rounded to bf16 there, so that the product of bf16 matrices with fp32
 //     sums is the exact product of what the recurrence uses), and the convolution's last inputs.
-//   * k_gated_scan: prompts run 128 tokens at a time in a block of 32 channels: every warp folds eight tokens into one (a, b)
+//   * k_gated_scan: prompts run 64 or 256 tokens at a time in a block of 32 channels: every warp folds eight tokens into one (a, b)
 //     pair, the pairs meet in shared memory, and each warp replays its tokens from the state before them. Decode is one
 //     step per channel. sqrt(1 - a^2) is taken as sqrt(-expm1(2 log a)), which stays exact where a is close to one.
 // Retention: S <- decay S + k v^T, o = S^T q.
@@ -135,6 +135,7 @@ struct Gates {
   static __device__ __forceinline__ float sig(float z) { return sigmoid(z); }
   static __device__ __forceinline__ float ex(float z) { return expf(z); }
   static __device__ __forceinline__ float one_minus_exp(float x) { return -expm1f(x); }
+  static __device__ __forceinline__ float root(float x) { return sqrtf(x); }
   static __device__ __forceinline__ float gelu(float z) { return sb_gelu_tanh(z); }
 };
 template <>
@@ -149,6 +150,11 @@ struct Gates<bf16> {
     const float series = -x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 720.f, 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
     return x > -0.25f ? series : 1.f - ex(x);
   }
+  static __device__ __forceinline__ float root(float x) {
+    float y;
+    asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+  }
   // 1/2 (1 + tanh(y)) = sigmoid(2 y)
   static __device__ __forceinline__ float gelu(float z) { return z * sig(1.5957691216f * fmaf(0.044715f * z * z, z, z)); }
 };
@@ -158,12 +164,13 @@ __device__ __forceinline__ Step gated_step(const GatedArgs& g, int64_t t, int64_
   const float* gates = g.gates + t * 2 * g.s.width;
   const float r = G::sig(gates[gr] + rb), i = G::sig(gates[gi] + ib), u = to_f(((const T*)g.u)[t * g.s.ld_u() + uo]);
   const float la = decay * r;
-  return Step{G::ex(la), sqrtf(G::one_minus_exp(2.f * la)) * i * u};
+  return Step{G::ex(la), G::root(G::one_minus_exp(2.f * la)) * i * u};
 }
-constexpr int SCAN_WARPS = 16, SCAN_PER = 8;  // tokens per warp and pass
-// grid (ceil(width / 32), nb), 512 threads: lane = channel, warp = run of tokens
-template <typename T>
-__global__ void __launch_bounds__(SCAN_WARPS * 32, 2) gated_scan_kernel(GatedArgs g, int64_t rows) {
+constexpr int SCAN_PER = 8;  // tokens per warp and pass
+// grid (ceil(width / 32), nb), SCAN_WARPS warps: lane = channel, warp = run of tokens. Few blocks take many warps, a grid that fills
+// the GPU takes small blocks, whose loads and sums overlap each other's.
+template <typename T, int SCAN_WARPS>
+__global__ void __launch_bounds__(SCAN_WARPS * 32, 32 / SCAN_WARPS) gated_scan_kernel(GatedArgs g, int64_t rows) {
   __shared__ Step fold[SCAN_WARPS][32];
   __shared__ float carry[32];
   SB_TRACE_BEGIN();
@@ -413,8 +420,10 @@ int k_gated_scan(strictb200_ctx* ctx, const GatedArgs& a, int64_t T) {
     else SB_CUDA(sb_launch(ctx, gated_step_kernel<bf16>, grid, dim3(256), 0, a, T));
   } else {
     const dim3 grid((unsigned)((a.s.width + 31) / 32), (unsigned)a.nb);
-    if (a.f32) SB_CUDA(sb_launch(ctx, gated_scan_kernel<float>, grid, dim3(SCAN_WARPS * 32), 0, a, T));
-    else SB_CUDA(sb_launch(ctx, gated_scan_kernel<bf16>, grid, dim3(SCAN_WARPS * 32), 0, a, T));
+    const bool many = (int64_t)grid.x * grid.y > 2 * ctx->sm_count;
+    auto go = [&](auto kernel) { return sb_launch(ctx, kernel, grid, dim3(many ? 256 : 1024), 0, a, T); };
+    if (a.f32) SB_CUDA(many ? go(gated_scan_kernel<float, 8>) : go(gated_scan_kernel<float, 32>));
+    else SB_CUDA(many ? go(gated_scan_kernel<bf16, 8>) : go(gated_scan_kernel<bf16, 32>));
   }
   ctx->launches++;
   return STRICTB200_OK;

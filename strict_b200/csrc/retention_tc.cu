@@ -9,10 +9,15 @@
 // the decay fp32. Tensor memory: P, O, O2 and S, 128 columns each.
 //   warps 0..15  rows: thread (row, quarter) owns 32 columns of row `row` of every tile
 //   warp 16      one lane issues copies and products
+// Few (sequence, head) pairs leave most SMs idle, so a prompt is then cut into segments of whole chunks, in two launches: the first
+// walks every segment but the last for its own contribution to the state alone; the second starts each segment from the state
+// that the contributions before it add up to.
 // A row thread takes its sums of a chunk out of tensor memory, prepares the operands of the next chunk (state, V'), and only
 // then norms, gates and stores, while the next chunk's products run.
 // Every mbarrier wait is bounded: on expiry the block records an error word in host-visible memory, stops, frees its tensor
 // memory and returns.
+#include <algorithm>
+
 #include "mixers.cuh"
 #include "tcgen05.cuh"
 
@@ -35,6 +40,10 @@ struct RtArgs {
   bf16* out;
   int64_t ldo;
   int* status;
+  // segments: chunks of each, how many there are, and per segment [nb, H, dim, vdim] of scratch: the state that a segment leaves
+  // (segment 0 with what came before it); the last one holds a copy of the state before the launch
+  int seg_chunks, segs;
+  float* seg_state;
 };
 
 // two bf16 terms by truncation: hi = the upper 16 bits, lo = the upper 16 bits of the exact remainder
@@ -47,17 +56,23 @@ __device__ __forceinline__ void arrive(uint64_t* bar) { asm volatile("mbarrier.a
 // 16 bytes `chunk` of row `row` of a swizzled box
 __device__ __forceinline__ uint32_t box_off(int row, int chunk) { return (uint32_t)(row * 128 + ((chunk ^ (row & 7)) << 4)); }
 
+// STATE: the first launch of a prompt in segments. grid (H, nb, segments)
+template <bool STATE>
 __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                                                                       const __grid_constant__ CUtensorMap map_v, RtArgs a) {
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   __shared__ __align__(8) uint64_t bar_qk, bar_v, bar_s, bar_o, bar_state, s_ready, vp_ready, p_ready;
   __shared__ uint32_t tmem_base_slot;
-  __shared__ float pw[CHUNK + 1], x_sum[2][CHUNK];
+  __shared__ float pw[CHUNK + 1], x_sum[2][CHUNK], pw_seg;
 
-  const int h = blockIdx.x, b = blockIdx.y;
-  const int n_all = a.lens[b] - a.past[b], chunks = (n_all + CHUNK - 1) / CHUNK;
-  const int64_t row0 = a.qstart[b];
+  const int h = blockIdx.x, b = blockIdx.y, seg = blockIdx.z;
+  const int first = seg * a.seg_chunks * CHUNK, n_seq = a.lens[b] - a.past[b];
+  if (first >= n_seq) return;  // whole block, before anything is allocated
+  const bool last = first + a.seg_chunks * CHUNK >= n_seq;
+  if (STATE && last) return;   // nobody starts from the state the last segment leaves
+  const int n_all = last ? n_seq - first : a.seg_chunks * CHUNK, chunks = (n_all + CHUNK - 1) / CHUNK;
+  const int64_t row0 = a.qstart[b] + first;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   uint8_t *bQ = smem, *bK = bQ + TILE_BYTES, *bV = bK + TILE_BYTES, *bVh = bV + TILE_BYTES, *bVl = bVh + TILE_BYTES, *bSh = bVl + TILE_BYTES, *bSl = bSh + TILE_BYTES;
   const uint32_t sQ = smem_u32(bQ), sK = smem_u32(bK), sV = smem_u32(bV), sVh = smem_u32(bVh), sVl = smem_u32(bVl), sSh = smem_u32(bSh), sSl = smem_u32(bSl);
@@ -67,6 +82,7 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
     mbar_init(smem_u32(&s_ready), ROW_THREADS); mbar_init(smem_u32(&vp_ready), ROW_THREADS); mbar_init(smem_u32(&p_ready), ROW_THREADS);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
+  if (threadIdx.x == CHUNK + 1) pw_seg = (float)pow((double)a.decay[h], (double)(a.seg_chunks * CHUNK));
   if (threadIdx.x <= CHUNK) pw[threadIdx.x] = (float)pow((double)a.decay[h], (double)threadIdx.x);
   if (warp == 16) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_base_slot)), "r"(512u) : "memory");
@@ -84,9 +100,9 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
     if (lane == 0) {
       auto load = [&](int c) {
         const int row = (int)row0 + c * CHUNK;
-        mbar_expect_tx(smem_u32(&bar_qk), 2 * TILE_BYTES);
+        mbar_expect_tx(smem_u32(&bar_qk), (STATE ? 1 : 2) * TILE_BYTES);
         for (int i = 0; i < 2; i++) {
-          tma_load_3d(sQ + i * HALF_BYTES, &map_q, i * 64, h, row, smem_u32(&bar_qk));
+          if (!STATE) tma_load_3d(sQ + i * HALF_BYTES, &map_q, i * 64, h, row, smem_u32(&bar_qk));
           tma_load_3d(sK + i * HALF_BYTES, &map_k, i * 64, h, row, smem_u32(&bar_qk));
         }
         mbar_expect_tx(smem_u32(&bar_v), TILE_BYTES);
@@ -99,29 +115,31 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
         good = mbar_wait(smem_u32(&bar_qk), ph) && mbar_wait(smem_u32(&s_ready), ph);
         if (!good) break;
         tc_fence_after();
+        if (!STATE) {
 #pragma unroll
-        for (int s = 0; s < 8; s++) {
-          const uint32_t off = (uint32_t)((s >> 2) * HALF_BYTES + (s & 3) * 32);
-          tc_mma_ss(tP, desc_kmajor(sQ + off), desc_kmajor(sK + off), idesc, s ? 1u : 0u);
-        }
-        tc_commit(smem_u32(&bar_s));
+          for (int s = 0; s < 8; s++) {
+            const uint32_t off = (uint32_t)((s >> 2) * HALF_BYTES + (s & 3) * 32);
+            tc_mma_ss(tP, desc_kmajor(sQ + off), desc_kmajor(sK + off), idesc, s ? 1u : 0u);
+          }
+          tc_commit(smem_u32(&bar_s));
 #pragma unroll
-        for (int s = 0; s < 8; s++) {
-          const uint64_t dq = desc_kmajor(sQ + (uint32_t)((s >> 2) * HALF_BYTES + (s & 3) * 32));
-          tc_mma_ss(tO2, dq, desc_mnmajor(sSh + (uint32_t)(s * 2048)), idesc_b, s ? 1u : 0u);
-          tc_mma_ss(tO2, dq, desc_mnmajor(sSl + (uint32_t)(s * 2048)), idesc_b, 1u);
-        }
-        good = mbar_wait(smem_u32(&p_ready), ph) && mbar_wait(smem_u32(&bar_v), ph);
-        if (!good) break;
-        tc_fence_after();
+          for (int s = 0; s < 8; s++) {
+            const uint64_t dq = desc_kmajor(sQ + (uint32_t)((s >> 2) * HALF_BYTES + (s & 3) * 32));
+            tc_mma_ss(tO2, dq, desc_mnmajor(sSh + (uint32_t)(s * 2048)), idesc_b, s ? 1u : 0u);
+            tc_mma_ss(tO2, dq, desc_mnmajor(sSl + (uint32_t)(s * 2048)), idesc_b, 1u);
+          }
+          good = mbar_wait(smem_u32(&p_ready), ph) && mbar_wait(smem_u32(&bar_v), ph);
+          if (!good) break;
+          tc_fence_after();
 #pragma unroll
-        for (int s = 0; s < 8; s++) {
-          const uint64_t dv = desc_mnmajor(sV + (uint32_t)(s * 2048));
-          const uint32_t pcol = (uint32_t)((s >> 1) * 32 + (s & 1) * 8);
-          tc_mma_ts(tO, tP + pcol, dv, idesc_b, s ? 1u : 0u);
-          tc_mma_ts(tO, tP + pcol + 16, dv, idesc_b, 1u);
+          for (int s = 0; s < 8; s++) {
+            const uint64_t dv = desc_mnmajor(sV + (uint32_t)(s * 2048));
+            const uint32_t pcol = (uint32_t)((s >> 1) * 32 + (s & 1) * 8);
+            tc_mma_ts(tO, tP + pcol, dv, idesc_b, s ? 1u : 0u);
+            tc_mma_ts(tO, tP + pcol + 16, dv, idesc_b, 1u);
+          }
+          tc_commit(smem_u32(&bar_o));
         }
-        tc_commit(smem_u32(&bar_o));
         good = mbar_wait(smem_u32(&vp_ready), ph);
         if (!good) break;
         tc_fence_after();
@@ -146,7 +164,10 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
     const uint32_t box = (uint32_t)((quarter >> 1) * HALF_BYTES);
     const int chunk0 = (quarter & 1) * 4;  // first of its 16-byte chunks in the box's row
     auto rows_sync = [&]() { asm volatile("bar.sync 1, 512;" ::: "memory"); };
-    float* S = a.state + (((int64_t)b * a.H + h) * a.dim + row) * a.vdim + c0;  // this thread's part of the state (where it exists)
+    const int64_t head = ((int64_t)b * a.H + h) * a.dim * a.vdim, per_seg = (int64_t)gridDim.y * a.H * a.dim * a.vdim, mine = (int64_t)row * a.vdim + c0;
+    // this thread's part of a state (where it exists): what the segment begins with, and where it leaves its own
+    const float* S_in = (STATE || (seg == 0 && last) || a.segs == 1 ? a.state : a.seg_state + (seg ? 0 : a.segs - 1) * per_seg) + head + mine;
+    float* S_out = (STATE ? a.seg_state + seg * per_seg : a.state) + head + mine;
     const bool s_vec = (a.vdim & 3) == 0;
     const bool g_vec = ((a.vdim | (int)(a.ld_g & 3)) & 3) == 0 && ((uintptr_t)a.g & 15) == 0;
     const bool o_vec = ((a.vdim | (int)(a.ldo & 7)) & 7) == 0 && ((uintptr_t)a.out & 15) == 0;
@@ -157,7 +178,7 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
       const int n = min(CHUNK, n_all - c * CHUNK);
       const float dn = pw[n];
 #pragma unroll
-      for (int j = 0; j < 4; j++) {
+      for (int j = 0; j < 4 && !STATE; j++) {
         uint4 hi, lo;
         split2(__uint_as_float(r[8 * j]), __uint_as_float(r[8 * j + 1]), hi.x, lo.x);
         split2(__uint_as_float(r[8 * j + 2]), __uint_as_float(r[8 * j + 3]), hi.y, lo.y);
@@ -193,9 +214,7 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
       return true;
     };
 
-    bool ok = true;
-    {
-      uint32_t r[32];
+    auto read_state = [&](const float* S, float* r) {
 #pragma unroll
       for (int j = 0; j < 8; j++) {
         float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -208,10 +227,54 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
             if (c0 + 4 * j + 3 < a.vdim) x.w = S[4 * j + 3];
           }
         }
-        r[4 * j] = __float_as_uint(x.x); r[4 * j + 1] = __float_as_uint(x.y); r[4 * j + 2] = __float_as_uint(x.z); r[4 * j + 3] = __float_as_uint(x.w);
+        r[4 * j] = x.x; r[4 * j + 1] = x.y; r[4 * j + 2] = x.z; r[4 * j + 3] = x.w;
       }
+    };
+    auto write_state = [&](float* S, const uint32_t* r) {
+#pragma unroll
+      for (int j = 0; j < 8; j++) {
+        if (row >= a.dim || c0 + 4 * j >= a.vdim) continue;
+        if (s_vec) *(uint4*)(S + 4 * j) = make_uint4(r[4 * j], r[4 * j + 1], r[4 * j + 2], r[4 * j + 3]);
+        else
+#pragma unroll
+          for (int i = 0; i < 4; i++)
+            if (c0 + 4 * j + i < a.vdim) S[4 * j + i] = __uint_as_float(r[4 * j + i]);
+      }
+    };
+    bool ok = true;
+    {
+      float x[32];
+      uint32_t r[32];
+      if (STATE && seg > 0) {
+#pragma unroll
+        for (int j = 0; j < 32; j++) x[j] = 0.f;
+      } else {
+        read_state(S_in, x);
+      }
+      if (!STATE && seg > 0) {  // segment 0 left a whole state, the others what they add
+        for (int i = 1; i < seg; i++) {
+          float y[32];
+          read_state(a.seg_state + i * per_seg + head + mine, y);
+#pragma unroll
+          for (int j = 0; j < 32; j++) x[j] = fmaf(pw_seg, x[j], y[j]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 32; j++) r[j] = __float_as_uint(x[j]);
+      if (STATE && seg == 0) write_state(a.seg_state + (a.segs - 1) * per_seg + head + mine, r);
       ok = operands(0, r);
     }
+    if constexpr (STATE) {
+      for (int c = 0; c < chunks && ok; c++) {
+        if (!mbar_wait(smem_u32(&bar_state), (uint32_t)(c & 1))) { ok = false; break; }
+        tc_fence_after();
+        uint32_t r[32];
+        tc_ld32(tS + lane_base + (uint32_t)c0, r);
+        tc_wait_ld();
+        if (c + 1 < chunks) ok = operands(c + 1, r);
+        else write_state(S_out, r);
+      }
+    } else
     for (int c = 0; c < chunks && ok; c++) {
       const uint32_t ph = (uint32_t)(c & 1);
       const int n = min(CHUNK, n_all - c * CHUNK);
@@ -279,10 +342,8 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
         tc_wait_ld();
         if (c + 1 < chunks) {
           ok = operands(c + 1, r);
-        } else {
-#pragma unroll
-          for (int j = 0; j < 32; j++)
-            if (row < a.dim && c0 + j < a.vdim) S[j] = __uint_as_float(r[j]);
+        } else if (last) {
+          write_state(S_out, r);
         }
       }
       // ---- norm, gate, store (the sums of the four threads of a row meet in two steps)
@@ -324,11 +385,23 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
 
 bool sb_retention_prefill_fits(const HeadShape& s) { return s.dim <= 128 && s.vdim <= 128; }
 
+// Segments a prompt is cut into: as many as the SMs take at once (one block per SM), of at least two chunks each.
+int sb_retention_segments(strictb200_ctx* ctx, const HeadShape& s, int nb, int max_new) {
+  const int chunks = (max_new + CHUNK - 1) / CHUNK;
+  int segs = std::min((int)(ctx->sm_count / std::max<int64_t>((int64_t)s.H * nb, 1)), chunks / 2);
+  if (segs < 2) return 1;
+  const int per = (chunks + segs - 1) / segs;
+  return (chunks + per - 1) / per;
+}
+
 int k_retention_prefill(strictb200_ctx* ctx, const RetentionArgs& p, int64_t T) {
   const HeadShape& s = p.s;
   if (!sb_retention_prefill_fits(s) || p.f32 || p.p.splits != 1) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "retention: heads the tensor-core kernel does not take");
   if (s.H > INT32_MAX / 2 || p.nb > 65535 || T > INT32_MAX) return sb_fail(STRICTB200_ERR_INVALID_ARG, "retention: too many sequences or rows");
-  RtArgs a{s.H, s.dim, s.vdim, p.lens, p.past, p.qstart, p.decay, p.state, p.p.in + (int64_t)s.H * (2 * s.dim + s.vdim), p.p.ld, p.eps, (bf16*)p.out, p.ldo, ctx->d_status};
+  const int segs = sb_retention_segments(ctx, s, p.nb, p.max_new), chunks = (p.max_new + CHUNK - 1) / CHUNK;
+  if (segs > 1 && !p.seg_state) return sb_fail(STRICTB200_ERR_INVALID_ARG, "retention: segments need scratch");
+  RtArgs a{s.H, s.dim, s.vdim, p.lens, p.past, p.qstart, p.decay, p.state, p.p.in + (int64_t)s.H * (2 * s.dim + s.vdim), p.p.ld, p.eps, (bf16*)p.out, p.ldo, ctx->d_status,
+           (chunks + segs - 1) / segs, segs, p.seg_state};
   const int row = s.row();
   CUtensorMap mq, mk, mv;
   SB_TRY(make_map3(&mq, p.q, row, s.H, T, row, (int64_t)s.H * row));
@@ -336,8 +409,15 @@ int k_retention_prefill(strictb200_ctx* ctx, const RetentionArgs& p, int64_t T) 
   SB_TRY(make_map3(&mv, p.v, row, s.H, T, row, (int64_t)s.H * row));
   const size_t smem = 7 * TILE_BYTES + 1024;
   static SbDeviceOnce once;
-  SB_CUDA(once.run(ctx->device, [&] { return cudaFuncSetAttribute(retention_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); }));
-  retention_prefill_kernel<<<dim3((unsigned)s.H, (unsigned)p.nb), RT_THREADS, smem, ctx->stream>>>(mq, mk, mv, a);
+  SB_CUDA(once.run(ctx->device, [&] {
+    const cudaError_t e = cudaFuncSetAttribute(retention_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    return e != cudaSuccess ? e : cudaFuncSetAttribute(retention_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  }));
+  if (segs > 1) {
+    retention_prefill_kernel<true><<<dim3((unsigned)s.H, (unsigned)p.nb, (unsigned)segs - 1), RT_THREADS, smem, ctx->stream>>>(mq, mk, mv, a);
+    SB_LAUNCHED(ctx);
+  }
+  retention_prefill_kernel<false><<<dim3((unsigned)s.H, (unsigned)p.nb, (unsigned)segs), RT_THREADS, smem, ctx->stream>>>(mq, mk, mv, a);
   SB_LAUNCHED(ctx);
   return STRICTB200_OK;
 }

@@ -372,9 +372,10 @@ struct MixRows {
 };
 struct MixBufs {
   char *q = nullptr, *k = nullptr, *v = nullptr, *u = nullptr;
-  float *gate = nullptr, *gates = nullptr, *o_part = nullptr, *ml_part = nullptr;
+  float *gate = nullptr, *gates = nullptr, *o_part = nullptr, *ml_part = nullptr, *seg_state = nullptr;
 };
-void carve_mix(const StackLayer& w, int64_t T, bool prompt, size_t esz, char* base, MixBufs* o, size_t* total) {
+void carve_mix(strictb200_model* m, const StackLayer& w, int64_t T, bool prompt, int nb, int max_new, char* base, MixBufs* o, size_t* total) {
+  const size_t esz = m->stack->esz();
   Carver cv{base};
   if (w.kind == STRICTB200_MIXER_GATED) {
     o->u = cv.take<char>(T * w.gs.ld_u() * esz);
@@ -385,6 +386,8 @@ void carve_mix(const StackLayer& w, int64_t T, bool prompt, size_t esz, char* ba
     if (w.kind == STRICTB200_MIXER_RETENTION) {
       o->k = cv.take<char>(rows * esz);
       o->v = cv.take<char>(rows * esz);
+      const int segs = prompt && !m->stack->f32 && sb_retention_prefill_fits(w.hs) ? sb_retention_segments(m->ctx, w.hs, nb, max_new) : 1;
+      if (segs > 1) o->seg_state = cv.take<float>((size_t)segs * nb * w.state);
     } else {
       o->gate = cv.take<float>((size_t)T * w.hs.H);
       if (!prompt && w.fast_decode) {
@@ -427,7 +430,7 @@ int mix_rows(strictb200_model* m, strictb200_kv* kv, int l, const MixRows& r, co
   const StackLayer& w = st.L[l];
   MixBufs b;
   size_t total;
-  carve_mix(w, r.T, r.prompt(), st.esz(), scratch, &b, &total);
+  carve_mix(m, w, r.T, r.prompt(), r.nb, r.max_new, scratch, &b, &total);
   float* state = kv->state ? kv->state + kv->state_off[l] + (size_t)r.b0 * w.state : nullptr;
   if (w.kind == STRICTB200_MIXER_GATED) {
     GatedArgs a;
@@ -445,7 +448,7 @@ int mix_rows(strictb200_model* m, strictb200_kv* kv, int l, const MixRows& r, co
   const HeadShape& s = w.hs;
   RetentionArgs t;
   if (w.kind == STRICTB200_MIXER_RETENTION) {
-    t.s = s; t.p = p; t.decay = w.decay; t.state = state; t.q = b.q; t.k = b.k; t.v = b.v; t.nb = r.nb; t.max_new = r.max_new;
+    t.s = s; t.p = p; t.decay = w.decay; t.state = state; t.q = b.q; t.k = b.k; t.v = b.v; t.seg_state = b.seg_state; t.nb = r.nb; t.max_new = r.max_new;
     t.eps = m->c.eps; t.out = oa; t.ldo = w.ldo; t.f32 = st.f32; t.cos_t = w.cos_t; t.sin_t = w.sin_t; t.max_pos = m->c.max_pos;
     if (r.prompt()) { t.qstart = r.qstart; t.lens = r.lens; t.past = r.past; }
     else if (!st.f32 && sb_retention_decode_fits(s) && p.ld % 4 == 0) {
@@ -519,7 +522,7 @@ void carve_dec(strictb200_model* m, strictb200_kv* kv, char* base, StackDec* o, 
     if (w.kind != STRICTB200_MIXER_LATENT) {
       MixBufs t;
       size_t n;
-      carve_mix(w, B, false, st.esz(), nullptr, &t, &n);
+      carve_mix(m, w, B, false, (int)B, 1, nullptr, &t, &n);
       mix = std::max(mix, n);
       continue;
     }
@@ -570,7 +573,7 @@ void carve_pre(strictb200_model* m, const PrefillChunk& c, char* base, StackPre*
     if (w.kind != STRICTB200_MIXER_LATENT) {
       MixBufs t;
       size_t n;
-      carve_mix(w, T, true, st.esz(), nullptr, &t, &n);
+      carve_mix(m, w, T, true, c.nb, c.max_new, nullptr, &t, &n);
       mix = std::max(mix, n);
       continue;
     }

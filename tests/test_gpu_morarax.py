@@ -256,6 +256,32 @@ def test_two_caches_side_by_side(models):
     ka.dispose(), kb.dispose()
 
 
+@pytest.mark.parametrize("lens", [[700], [1100, 300, 129, 5], [513, 512, 511, 1]])
+def test_long_prompts_in_segments(ctx, lens):
+    """Few heads and long prompts: retention cuts them into segments that run side by side; whole, continued, and decoded on."""
+    cfg = MM.config([MM.retention(2, 64, 96, MM.rot(800.0, 64), 24, decay=[0.98, 0.9997]), MM.retention(3, 128, 40, MM.rot(800.0, 32), 0)], 96, 50)
+    w = MM.weights(cfg, 12)
+    rng = np.random.default_rng(6)
+    seqs = [rng.integers(0, 50, n + 290).astype(np.int32) for n in lens]
+    want = [P.forward(cfg, w, t) for t in seqs]
+    m = make(ctx, cfg, w, sb.BF16)
+    kv = m.new_cache(len(lens), max(lens) + 320)
+
+    def feed(lo, n):
+        tok = np.zeros((len(seqs), max(n)), np.int32)
+        for row, t, a, k in zip(tok, seqs, lo, n):
+            row[:k] = t[a:a + k]
+        _, logits = kv.prefill_rows(tok, [range(k) for k in n], n)
+        check(logits, np.concatenate([x[a:a + k] for x, a, k in zip(want, lo, n)]), sb.BF16, (lo, n))
+
+    feed([0] * len(lens), lens)
+    feed(lens, [280] * len(lens))
+    for i in range(10):
+        _, logits = kv.decode_step([t[n + 280 + i] for t, n in zip(seqs, lens)], want_logits=True)
+        check(logits, np.stack([x[n + 280 + i] for x, n in zip(want, lens)]), sb.BF16, i)
+    kv.dispose(), m.dispose()
+
+
 # ------------------------------------------------------------------ keys and memories that stand out
 def standing_out(seed):
     """One attention layer in which one token's key stands out for one query token, whatever the distance: little of a head is
