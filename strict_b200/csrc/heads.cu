@@ -13,71 +13,59 @@ using namespace mix;
 
 namespace {
 
-// One head of a row. VEC: four dims per lane (widths multiples of 4, at most 128; so is the rotated half).
-struct HeadItem {
-  bool is_q, is_v;
-  int n;          // dims
-  int64_t col;    // first column of the projection
-  int64_t dst;    // element of q_out, k_out or v_out
-};
-__device__ __forceinline__ HeadItem head_item(const HeadSplitArgs& a, int64_t t, int b, int p, int item) {
-  const HeadShape& s = a.s;
-  HeadItem i;
-  i.is_q = item < s.H; i.is_v = item >= s.H + s.G;
-  const int h = i.is_q ? item : i.is_v ? item - s.H - s.G : item - s.H, row = s.row();
-  i.n = i.is_v ? s.vdim : s.dim;
-  i.col = i.is_q ? (int64_t)h * s.dim : i.is_v ? (int64_t)(s.H + s.G) * s.dim + (int64_t)h * s.vdim : (int64_t)(s.H + h) * s.dim;
-  i.dst = i.is_q ? (t * s.H + h) * row : a.dense ? (t * s.G + h) * row : (((int64_t)b * s.G + h) * a.maxlen + p) * row;
-  return i;
-}
-template <typename T>
-__device__ __forceinline__ void head_vec(const HeadSplitArgs& a, const HeadItem& it, float4 x, const float4& c, const float4& d, int src, int lane) {
-  const HeadShape& s = a.s;
-  const int e = lane * 4;
-  if (!it.is_v) {
-    float4 o;
-    o.x = __shfl_sync(0xffffffffu, x.x, src & 31); o.y = __shfl_sync(0xffffffffu, x.y, src & 31);
-    o.z = __shfl_sync(0xffffffffu, x.z, src & 31); o.w = __shfl_sync(0xffffffffu, x.w, src & 31);
-    if (e < s.rot) {
-      x.x = fmaf(x.x, c.x, o.x * d.x); x.y = fmaf(x.y, c.y, o.y * d.y);
-      x.z = fmaf(x.z, c.z, o.z * d.z); x.w = fmaf(x.w, c.w, o.w * d.w);
-    }
-    float r = it.is_q ? 1.f : s.k_scale;
-    if (s.qk_norm) {
-      const float ss = warp_sum(x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w);
-      r *= __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)s.dim), a.eps)));
-    }
-    x.x *= r; x.y *= r; x.z *= r; x.w *= r;
+// One head of four dims per lane (widths multiples of 4, at most 128; so is the rotated half): rotation, norm, factor. c and d are
+// this lane's cosines, and its sines with the sign of its half; src the lane that holds the other half of its pairs.
+__device__ __forceinline__ float4 rotate_head(const HeadShape& s, float4 x, const float4& c, const float4& d, int src, float post, float eps, int lane) {
+  float4 o;
+  o.x = __shfl_sync(0xffffffffu, x.x, src); o.y = __shfl_sync(0xffffffffu, x.y, src);
+  o.z = __shfl_sync(0xffffffffu, x.z, src); o.w = __shfl_sync(0xffffffffu, x.w, src);
+  if (lane * 4 < s.rot) {
+    x.x = fmaf(x.x, c.x, o.x * d.x); x.y = fmaf(x.y, c.y, o.y * d.y);
+    x.z = fmaf(x.z, c.z, o.z * d.z); x.w = fmaf(x.w, c.w, o.w * d.w);
   }
-  T* dst = (T*)(it.is_q ? a.q_out : it.is_v ? a.v_out : a.k_out) + it.dst;
-  if (e < s.row()) store4<T>(dst + e, x);
+  float r = post;
+  if (s.qk_norm) {
+    const float ss = warp_sum(x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w);
+    r *= __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(ss, (float)s.dim), eps)));
+  }
+  return make_float4(x.x * r, x.y * r, x.z * r, x.w * r);
 }
+__device__ __forceinline__ void lane_angles(const HeadSplitArgs& a, int p, int lane, float4* c, float4* d, int* src) {
+  const int e = lane * 4, half = a.s.rot / 2;
+  *src = (e < half ? lane + half / 4 : lane - half / 4) & 31;
+  *c = *d = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (e < a.s.rot) {
+    const int64_t i = (int64_t)p * half + (e < half ? e : e - half);
+    *c = *(const float4*)(a.cos_t + i);
+    *d = *(const float4*)(a.sin_t + i);
+    if (e < half) *d = make_float4(-d->x, -d->y, -d->z, -d->w);
+  }
+}
+// any width: one head through shared memory
 template <typename T>
-__device__ __forceinline__ void head_any(const HeadSplitArgs& a, const HeadItem& it, int64_t rows, int64_t t, const float* cs, const float* sn, float* buf, int lane) {
+__device__ __forceinline__ void head_any(const HeadSplitArgs& a, int64_t rows, int64_t t, int64_t col, int n, bool is_v, float post, int p, T* dst, float* buf, int lane) {
   const HeadShape& s = a.s;
-  const int half = s.rot / 2;
-  for (int e = lane; e < it.n; e += 32) buf[e] = proj(a.p, rows, t, it.col + e);
+  const int half = s.rot / 2, row = s.row();
+  const float *cs = a.cos_t + (int64_t)p * half, *sn = a.sin_t + (int64_t)p * half;
+  for (int e = lane; e < n; e += 32) buf[e] = proj(a.p, rows, t, col + e);
   __syncwarp();
   auto value = [&](int e) {
-    if (it.is_v || e >= s.rot) return buf[e];
+    if (is_v || e >= s.rot) return buf[e];
     const int i = e < half ? e : e - half;
     return e < half ? buf[e] * cs[i] - buf[e + half] * sn[i] : buf[e] * cs[i] + buf[e - half] * sn[i];
   };
-  float r = it.is_q || it.is_v ? 1.f : s.k_scale;
-  if (s.qk_norm && !it.is_v) {
+  float r = post;
+  if (s.qk_norm && !is_v) {
     float ss = 0.f;
-    for (int e = lane; e < it.n; e += 32) { const float v = value(e); ss += v * v; }
+    for (int e = lane; e < n; e += 32) { const float v = value(e); ss += v * v; }
     r *= __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(warp_sum(ss), (float)s.dim), a.eps)));
   }
-  T* dst = (T*)(it.is_q ? a.q_out : it.is_v ? a.v_out : a.k_out) + it.dst;
-  const int row = s.row();
-  for (int e = lane; e < row; e += 32) dst[e] = to_t<T>(e < it.n ? value(e) * r : 0.f);
+  for (int e = lane; e < row; e += 32) dst[e] = to_t<T>(e < n ? value(e) * r : 0.f);
 }
 
-// grid rows * (item blocks + activation blocks), 256 threads: warp w of an item block owns the PER items of the row from
-// (8 * block + w) * PER on: query heads, key heads, value heads, and as the last item all gates. A decode step takes PER = 1 (few
-// rows, short chains), a prompt more, so that a warp has several heads' loads in flight.
-template <typename T, bool VEC, int PER>
+// grid rows * (item blocks + activation blocks), 256 threads: warp w of an item block owns item 8 * block + w of the row: a query
+// head, a key head, a value head, or (the last item) all gates. For decode steps and any widths.
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) head_split_kernel(HeadSplitArgs a, int64_t rows, int item_blocks, int act_blks) {
   extern __shared__ float sm[];
   SB_TRACE_BEGIN();
@@ -91,39 +79,79 @@ __global__ void __launch_bounds__(256) head_split_kernel(HeadSplitArgs a, int64_
   if (blk >= item_blocks) {
     act_block<T>(a.act, a.p, rows, t, blk - item_blocks);
   } else {
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_heads = s.H + 2 * s.G;
-    const int first = (blk * 8 + warp) * PER;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_heads = s.H + 2 * s.G, item = blk * 8 + warp;
     const int b = a.seq ? a.seq[t] : (int)t, p = a.pos ? a.pos[t] : a.lens[b];
+    const int row = s.row();
     if (p >= 0 && p < a.max_pos && (a.dense || p < a.maxlen)) {  // the host validates; never index outside the cache
-      const float *cs = a.cos_t + (int64_t)p * (s.rot / 2), *sn = a.sin_t + (int64_t)p * (s.rot / 2);
-      HeadItem it[PER];
-      float4 x[PER], c = make_float4(0.f, 0.f, 0.f, 0.f), d = c;  // this lane's cosines, and its sines with the sign of its half
-      const int e = lane * 4, half = s.rot / 2, src = e < half ? lane + half / 4 : lane - half / 4;  // the lane of the other half of its pairs
-      if (VEC && e < s.rot && first < s.H + s.G) {
-        c = *(const float4*)(cs + (e < half ? e : e - half));
-        d = *(const float4*)(sn + (e < half ? e : e - half));
-        if (e < half) d = make_float4(-d.x, -d.y, -d.z, -d.w);
-      }
-#pragma unroll
-      for (int i = 0; i < PER; i++)
-        if (first + i < n_heads) {
-          it[i] = head_item(a, t, b, p, first + i);
-          x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (VEC && lane * 4 < it[i].n) x[i] = proj4(a.p, rows, t, it[i].col + lane * 4);
+      if (item < n_heads) {
+        const bool is_q = item < s.H, is_v = item >= s.H + s.G;
+        const int h = is_q ? item : is_v ? item - s.H - s.G : item - s.H, n = is_v ? s.vdim : s.dim;
+        const int64_t col = is_v ? (int64_t)(s.H + s.G) * s.dim + (int64_t)h * s.vdim : (int64_t)item * s.dim;
+        T* dst = is_q ? (T*)a.q_out + (t * s.H + h) * row
+                      : (T*)(is_v ? a.v_out : a.k_out) + (a.dense ? (t * s.G + h) * row : (((int64_t)b * s.G + h) * a.maxlen + p) * row);
+        const float post = is_q ? 1.f : s.k_scale;
+        if constexpr (VEC) {
+          float4 x = make_float4(0.f, 0.f, 0.f, 0.f), c, d;
+          int src;
+          if (lane * 4 < n) x = proj4(a.p, rows, t, col + lane * 4);
+          if (!is_v) {
+            lane_angles(a, p, lane, &c, &d, &src);
+            x = rotate_head(s, x, c, d, src, post, a.eps, lane);
+          }
+          if (lane * 4 < row) store4<T>(dst + lane * 4, x);
+        } else {
+          head_any<T>(a, rows, t, col, n, is_v, is_v ? 1.f : post, p, dst, sm + warp * max(s.dim, s.vdim), lane);
         }
-#pragma unroll
-      for (int i = 0; i < PER; i++) {
-        if (first + i < n_heads) {
-          if (VEC) head_vec<T>(a, it[i], x[i], c, d, src, lane);
-          else head_any<T>(a, it[i], rows, t, cs, sn, sm + warp * max(s.dim, s.vdim), lane);
-        } else if (first + i == n_heads && s.gate) {
-          const int64_t col = (int64_t)(s.H + s.G) * s.dim + (int64_t)s.G * s.vdim;
-          for (int h = lane; h < s.H; h += 32) a.gate_out[t * s.H + h] = sigmoid(proj(a.p, rows, t, col + h));
-        }
+      } else if (item == n_heads && s.gate) {
+        const int64_t col = (int64_t)(s.H + s.G) * s.dim + (int64_t)s.G * s.vdim;
+        for (int h = lane; h < s.H; h += 32) a.gate_out[t * s.H + h] = sigmoid(proj(a.p, rows, t, col + h));
       }
     }
   }
   SB_TRACE_END(SB_K_ROPE, 0);
+}
+
+// Prompt rows of a finished projection, four dims per lane: one block per row, a warp walks every eighth head with four heads'
+// loads in flight.
+template <typename T>
+__device__ __forceinline__ void walk_heads(const HeadShape& s, const float* in, int n, int heads, int warp, int lane, bool rotated, const float4& c, const float4& d,
+                                           int src, float post, float eps, T* dst, int64_t stride) {
+  const int row = s.row(), e = lane * 4;
+  for (int h0 = warp; h0 < heads; h0 += 32) {
+    float4 x[4];
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (h0 + 8 * i < heads && e < n) x[i] = __ldcs((const float4*)(in + (h0 + 8 * i) * n + e));
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      const int h = h0 + 8 * i;
+      if (h >= heads) break;
+      if (rotated) x[i] = rotate_head(s, x[i], c, d, src, post, eps, lane);
+      if (e < row) store4<T>(dst + h * stride + e, x[i]);
+    }
+  }
+}
+template <typename T>
+__global__ void __launch_bounds__(256) head_rows_kernel(HeadSplitArgs a) {
+  const HeadShape& s = a.s;
+  const int64_t t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = s.row();
+  pdl_trigger();
+  pdl_wait();
+  const int b = a.seq[t], p = a.pos[t];
+  if (p < 0 || p >= a.max_pos || (!a.dense && p >= a.maxlen)) return;
+  float4 c, d;
+  int src;
+  lane_angles(a, p, lane, &c, &d, &src);
+  const float* in = a.p.in + t * a.p.ld;
+  const int64_t at = a.dense ? t * s.G * row : ((int64_t)b * s.G * a.maxlen + p) * row, stride = a.dense ? row : (int64_t)a.maxlen * row;
+  walk_heads<T>(s, in, s.dim, s.H, warp, lane, true, c, d, src, 1.f, a.eps, (T*)a.q_out + t * s.H * row, (int64_t)row);
+  walk_heads<T>(s, in + s.H * s.dim, s.dim, s.G, warp, lane, true, c, d, src, s.k_scale, a.eps, (T*)a.k_out + at, stride);
+  walk_heads<T>(s, in + (s.H + s.G) * s.dim, s.vdim, s.G, warp, lane, false, c, d, src, 1.f, a.eps, (T*)a.v_out + at, stride);
+  if (s.gate)
+    for (int h = threadIdx.x; h < s.H; h += 256) a.gate_out[t * s.H + h] = sigmoid(in[(s.H + s.G) * s.dim + s.G * s.vdim + h]);
 }
 
 template <typename T>
@@ -252,17 +280,22 @@ SB_TRACE_TU(heads)
 
 int k_head_split(strictb200_ctx* ctx, const HeadSplitArgs& a, int64_t T) {
   const HeadShape& s = a.s;
-  const int per = a.seq && a.p.splits == 1 ? 4 : 1;
   const int items = s.H + 2 * s.G + (s.gate ? 1 : 0), act_blks = act_blocks(a.act);
   const bool vec = s.dim <= 128 && s.vdim <= 128 && ((s.dim | s.vdim | (s.rot / 2) | (int)(a.p.ld & 3)) & 3) == 0;
-  const int item_blocks = (items + 8 * (vec ? per : 1) - 1) / (8 * (vec ? per : 1));
+  if (vec && a.seq && a.p.splits == 1 && !act_blks && T <= INT32_MAX) {
+    if (a.f32) SB_CUDA(sb_launch(ctx, head_rows_kernel<float>, dim3((unsigned)T), dim3(256), 0, a));
+    else SB_CUDA(sb_launch(ctx, head_rows_kernel<bf16>, dim3((unsigned)T), dim3(256), 0, a));
+    ctx->launches++;
+    return STRICTB200_OK;
+  }
+  const int item_blocks = (items + 7) / 8;
   const int64_t blocks = T * (item_blocks + act_blks);
   if (blocks > INT32_MAX || a.p.splits > 8) return sb_fail(STRICTB200_ERR_INVALID_ARG, "head split: too many rows or partial sums");
   const size_t smem = vec ? 0 : (size_t)8 * std::max(s.dim, s.vdim) * sizeof(float);
   if (smem > 48 * 1024) return sb_fail(STRICTB200_ERR_UNSUPPORTED, "heads of more than 1536 dims");
   auto go = [&](auto kernel) { return sb_launch(ctx, kernel, dim3((unsigned)blocks), dim3(256), smem, a, T, item_blocks, act_blks); };
-  if (a.f32) SB_CUDA(!vec ? go(head_split_kernel<float, false, 1>) : per > 1 ? go(head_split_kernel<float, true, 4>) : go(head_split_kernel<float, true, 1>));
-  else SB_CUDA(!vec ? go(head_split_kernel<bf16, false, 1>) : per > 1 ? go(head_split_kernel<bf16, true, 4>) : go(head_split_kernel<bf16, true, 1>));
+  if (a.f32) SB_CUDA(vec ? go(head_split_kernel<float, true>) : go(head_split_kernel<float, false>));
+  else SB_CUDA(vec ? go(head_split_kernel<bf16, true>) : go(head_split_kernel<bf16, false>));
   ctx->launches++;
   return STRICTB200_OK;
 }

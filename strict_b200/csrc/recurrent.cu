@@ -128,44 +128,45 @@ __global__ void __launch_bounds__(256) conv_hist_kernel(GatedArgs a, int64_t row
 
 // ------------------------------------------------------------------ gated recurrence
 struct Step { float a, b; };  // S <- a S + b
-// The gates' functions, for fp32 results, and for results that end in bf16: exponentials through ex2.approx (2^-22), and the
-// series of 1 - exp(x) where that would cancel (x > -1/4; the first term left out is below 2^-23 of the sum).
+// One step of the recurrence, and GELU, in fp32: with the library's functions for fp32 results, and for results that end in bf16
+// with exponentials, reciprocals and roots through the approximate instructions (relative error 2^-22 and below), and the series
+// of 1 - exp(x) where 1 - a^2 would cancel (x > -1/4; the first term left out is below 2^-23 of the sum).
 template <typename T>
-struct Gates {
-  static __device__ __forceinline__ float sig(float z) { return sigmoid(z); }
-  static __device__ __forceinline__ float ex(float z) { return expf(z); }
-  static __device__ __forceinline__ float one_minus_exp(float x) { return -expm1f(x); }
-  static __device__ __forceinline__ float root(float x) { return sqrtf(x); }
-  static __device__ __forceinline__ float gelu(float z) { return sb_gelu_tanh(z); }
-};
+__device__ __forceinline__ Step gated_step(float zr, float zi, float u, float decay);
 template <>
-struct Gates<bf16> {
-  static __device__ __forceinline__ float ex(float z) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(z * 1.4426950408889634f));
-    return y;
-  }
-  static __device__ __forceinline__ float sig(float z) { return __fdividef(1.0f, 1.0f + ex(-z)); }
-  static __device__ __forceinline__ float one_minus_exp(float x) {  // x <= 0
-    const float series = -x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 720.f, 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
-    return x > -0.25f ? series : 1.f - ex(x);
-  }
-  static __device__ __forceinline__ float root(float x) {
-    float y;
-    asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-  }
-  // 1/2 (1 + tanh(y)) = sigmoid(2 y)
-  static __device__ __forceinline__ float gelu(float z) { return z * sig(1.5957691216f * fmaf(0.044715f * z * z, z, z)); }
-};
-template <typename T>
-__device__ __forceinline__ Step gated_step(const GatedArgs& g, int64_t t, int64_t gr, int64_t gi, int64_t uo, float rb, float ib, float decay) {
-  typedef Gates<T> G;
-  const float* gates = g.gates + t * 2 * g.s.width;
-  const float r = G::sig(gates[gr] + rb), i = G::sig(gates[gi] + ib), u = to_f(((const T*)g.u)[t * g.s.ld_u() + uo]);
-  const float la = decay * r;
-  return Step{G::ex(la), G::root(G::one_minus_exp(2.f * la)) * i * u};
+__device__ __forceinline__ Step gated_step<float>(float zr, float zi, float u, float decay) {
+  const float la = decay * sigmoid(zr);
+  return Step{expf(la), sqrtf(-expm1f(2.f * la)) * sigmoid(zi) * u};
 }
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_approx(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+constexpr float LOG2E = 1.4426950408889634f;
+template <>
+__device__ __forceinline__ Step gated_step<bf16>(float zr, float zi, float u, float decay) {
+  // both sigmoids over one reciprocal; exponents are kept where the product of the denominators is finite
+  const float er = 1.f + ex2_approx(fminf(-zr * LOG2E, 60.f)), ei = 1.f + ex2_approx(fminf(-zi * LOG2E, 60.f));
+  const float inv = rcp_approx(er * ei), la = decay * (ei * inv), x = 2.f * la;
+  const float a = ex2_approx(la * LOG2E);
+  const float series = -x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 720.f, 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
+  float root;
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(root) : "f"(x > -0.25f ? series : fmaf(-a, a, 1.f)));
+  return Step{a, root * (er * inv) * u};
+}
+template <typename T>
+__device__ __forceinline__ float gelu(float z);
+template <>
+__device__ __forceinline__ float gelu<float>(float z) { return sb_gelu_tanh(z); }
+// 1/2 (1 + tanh(y)) = sigmoid(2 y)
+template <>
+__device__ __forceinline__ float gelu<bf16>(float z) { return z * rcp_approx(1.f + ex2_approx(-1.5957691216f * LOG2E * fmaf(0.044715f * z * z, z, z))); }
 constexpr int SCAN_PER = 8;  // tokens per warp and pass
 // grid (ceil(width / 32), nb), SCAN_WARPS warps: lane = channel, warp = run of tokens. Few blocks take many warps, a grid that fills
 // the GPU takes small blocks, whose loads and sums overlap each other's.
@@ -178,24 +179,36 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32, 32 / SCAN_WARPS) gated_scan_k
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, w = g.s.width;
   const int c = blockIdx.x * 32 + lane, seq = blockIdx.y;
   const bool live = c < w;
-  const int bs = g.s.bs(), blk = live ? c / bs : 0, in_blk = c - blk * bs;
-  const int64_t gr = (int64_t)blk * 2 * bs + in_blk, gi = gr + bs, uo = (int64_t)blk * g.s.bs_p() + in_blk;
+  const int bs = g.s.bs(), blk = live ? c / bs : 0, in_blk = live ? c - blk * bs : 0;
   const float rb = live ? g.r_bias[c] : 0.f, ib = live ? g.i_bias[c] : 0.f, decay = live ? g.decay[c] : 0.f, yb = live ? g.y_bias[c] : 0.f;
   pdl_wait();
   SB_TRACE_WAITED();
-  const int n = g.lens[seq] - g.past[seq];
+  const int n = live ? g.lens[seq] - g.past[seq] : 0, n_all = g.lens[seq] - g.past[seq];  // a lane without a channel has no tokens
   const int64_t row0 = g.qstart[seq];
+  const float* zr = g.gates + row0 * 2 * w + blk * 2 * bs + in_blk;
+  const T* u = (const T*)g.u + row0 * g.s.ld_u() + blk * g.s.bs_p() + in_blk;
+  const float* yp = g.p.in + row0 * g.p.ld + (live ? c : 0);  // a prompt's projection is finished
+  T* out = (T*)g.out + row0 * g.ldo + (live ? c : 0);
+  const int ld_u = (int)g.s.ld_u(), ld_y = (int)g.p.ld, ldo = (int)g.ldo;
   if (warp == 0) carry[lane] = live ? g.state[(int64_t)seq * w + c] : 0.f;
-  for (int t0 = 0; t0 < n; t0 += SCAN_WARPS * SCAN_PER) {
+  for (int t0 = 0; t0 < n_all; t0 += SCAN_WARPS * SCAN_PER) {
     const int first = t0 + warp * SCAN_PER;
-    Step st[SCAN_PER];
-    float y[SCAN_PER];
+    const float *zr0 = zr + (int64_t)first * 2 * w, *y0 = yp + (int64_t)first * ld_y;
+    const T* u0 = u + (int64_t)first * ld_u;
+    float vr[SCAN_PER], vi[SCAN_PER], vu[SCAN_PER], y[SCAN_PER];
 #pragma unroll
     for (int j = 0; j < SCAN_PER; j++) {
-      const bool on = live && first + j < n;
-      st[j] = on ? gated_step<T>(g, row0 + first + j, gr, gi, uo, rb, ib, decay) : Step{1.f, 0.f};
-      y[j] = on ? g.p.in[(row0 + first + j) * g.p.ld + c] : 0.f;  // a prompt's projection is finished
+      vr[j] = vi[j] = vu[j] = y[j] = 0.f;
+      if (first + j < n) {
+        vr[j] = __ldcs(zr0 + j * 2 * w);
+        vi[j] = __ldcs(zr0 + j * 2 * w + bs);
+        vu[j] = to_f(u0[j * ld_u]);
+        y[j] = __ldcs(y0 + j * ld_y);
+      }
     }
+    Step st[SCAN_PER];
+#pragma unroll
+    for (int j = 0; j < SCAN_PER; j++) st[j] = first + j < n ? gated_step<T>(vr[j] + rb, vi[j] + ib, vu[j], decay) : Step{1.f, 0.f};
     Step all{1.f, 0.f};
 #pragma unroll
     for (int j = 0; j < SCAN_PER; j++) { all.b = fmaf(st[j].a, all.b, st[j].b); all.a *= st[j].a; }
@@ -206,7 +219,7 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32, 32 / SCAN_WARPS) gated_scan_k
 #pragma unroll
     for (int j = 0; j < SCAN_PER; j++) {
       s = fmaf(st[j].a, s, st[j].b);
-      if (live && first + j < n) ((T*)g.out)[(row0 + first + j) * g.ldo + c] = to_t<T>(s * Gates<T>::gelu(y[j] + yb));
+      if (first + j < n) out[(int64_t)first * ldo + j * ldo] = to_t<T>(s * gelu<T>(y[j] + yb));
     }
     __syncthreads();  // everybody has read the state before this pass
     if (warp == SCAN_WARPS - 1) carry[lane] = s;
@@ -227,10 +240,12 @@ __global__ void __launch_bounds__(256) gated_step_kernel(GatedArgs g, int64_t ro
   if (c < w) {
     const int bs = g.s.bs(), blk = c / bs, in_blk = c - blk * bs;
     const int64_t gr = (int64_t)blk * 2 * bs + in_blk;
-    const Step st = gated_step<T>(g, t, gr, gr + bs, (int64_t)blk * g.s.bs_p() + in_blk, g.r_bias[c], g.i_bias[c], g.decay[c]);
+    const float* gates = g.gates + t * 2 * w + gr;
+    const float u = to_f(((const T*)g.u)[t * g.s.ld_u() + (int64_t)blk * g.s.bs_p() + in_blk]);
+    const Step st = gated_step<T>(gates[0] + g.r_bias[c], gates[bs] + g.i_bias[c], u, g.decay[c]);
     const float s = fmaf(st.a, g.state[t * w + c], st.b);
     g.state[t * w + c] = s;
-    ((T*)g.out)[t * g.ldo + c] = to_t<T>(s * Gates<T>::gelu(proj(g.p, rows, t, c) + g.y_bias[c]));
+    ((T*)g.out)[t * g.ldo + c] = to_t<T>(s * gelu<T>(proj(g.p, rows, t, c) + g.y_bias[c]));
   }
   SB_TRACE_END(SB_K_RECURRENCE, 0);
 }
