@@ -5,12 +5,14 @@
 //   log a = -8 r softplus(lam), S <- a S + sqrt(1 - a^2) i u, out = S gelu(y).
 //   * k_gated_conv: u as the operand of the gate product (rounded to bf16 there, so that the product of bf16 matrices with fp32
 //     sums is the exact product of what the recurrence uses), and the convolution's last inputs.
-//   * k_gated_scan: prompts run 64 or 256 tokens at a time in a block of 32 channels: every warp folds eight tokens into one (a, b)
+//   * k_gated_scan: prompts run 64, 128 or 256 tokens at a time in a block of 32 channels: every warp folds eight tokens into one (a, b)
 //     pair, the pairs meet in shared memory, and each warp replays its tokens from the state before them. Decode is one
 //     step per channel. sqrt(1 - a^2) is taken as sqrt(-expm1(2 log a)), which stays exact where a is close to one.
 // Retention: S <- decay S + k v^T, o = S^T q.
 //   * k_retention_decode: one block per head streams the state once, from the projection's partial sums to the gated output.
 //   * k_retention_any: any widths, token by token. Prompts of usual widths: retention_tc.cu.
+#include <algorithm>
+
 #include "mixers.cuh"
 
 using namespace mix;
@@ -74,40 +76,50 @@ __global__ void __launch_bounds__(128) gated_conv_rows_kernel(GatedArgs a, int64
   for (int j = 0; j < 4; j++)
 #pragma unroll
     for (int i = 0; i < TAPS; i++) k[j][i] = a.conv[(int64_t)(c + j) * TAPS + i];
-  auto row = [&](int64_t t) {
-    const float4 v = *(const float4*)(a.p.in + t * a.p.ld + w + c);
+  const float* in = a.p.in + t0 * a.p.ld;
+  T* u = (T*)a.u + t0 * a.s.ld_u();
+  const int ld = (int)a.p.ld, ld_u = (int)a.s.ld_u();
+  auto row = [&](int i) {  // row t0 + i
+    const float4 v = *(const float4*)(in + (int64_t)i * ld + w + c);
     return make_float4(v.x + xb.x, v.y + xb.y, v.z + xb.z, v.w + xb.w);
   };
-  float4 x[CONV_ROWS];
-#pragma unroll
-  for (int i = 0; i < CONV_ROWS; i++)
-    if (i < n) x[i] = row(t0 + i);
-  float4 win[TAPS];  // the row and the ones before it, oldest first
+  auto tap = [&](float4& o, int j, const float4& x) {
+    o.x = fmaf(k[0][j], x.x, o.x); o.y = fmaf(k[1][j], x.y, o.y); o.z = fmaf(k[2][j], x.z, o.z); o.w = fmaf(k[3][j], x.w, o.w);
+  };
   int b = a.seq[t0];
-  int64_t li = t0 - a.qstart[b];
+  int li = (int)(t0 - a.qstart[b]);  // rows of the same sequence before t0
+  if (n == CONV_ROWS && li >= TAPS - 1 && a.seq[t0 + CONV_ROWS - 1] == b) {  // all of one sequence, and so is what comes before
+    float4 x[CONV_ROWS + TAPS - 1];
 #pragma unroll
-  for (int i = 0; i < CONV_ROWS; i++) {
-    if (i >= n) break;
-    const int64_t t = t0 + i;
+    for (int i = 0; i < CONV_ROWS + TAPS - 1; i++) x[i] = row(i - (TAPS - 1));
+#pragma unroll
+    for (int i = 0; i < CONV_ROWS; i++) {
+      float4 o = cb;
+#pragma unroll
+      for (int j = 0; j < TAPS; j++) tap(o, j, x[i + j]);
+      store4<T>(u + (int64_t)i * ld_u + c, o);
+    }
+    return;
+  }
+  float4 win[TAPS];  // the row and the ones before it, oldest first
+  for (int i = 0; i < n; i++) {
     if (i > 0) {
-      const int b1 = a.seq[t];
+      const int b1 = a.seq[t0 + i];
       li = b1 == b ? li + 1 : 0;
       b = b1;
     }
     if (i == 0 || li == 0) {
 #pragma unroll
       for (int j = 0; j < TAPS - 1; j++) {
-        const int64_t back = TAPS - 1 - j;
-        win[j] = back <= li ? row(t - back) : *(const float4*)(a.hist + ((int64_t)b * (TAPS - 1) + TAPS - 1 + li - back) * w + c);
+        const int back = TAPS - 1 - j;
+        win[j] = back <= li ? row(i - back) : *(const float4*)(a.hist + ((int64_t)b * (TAPS - 1) + TAPS - 1 + li - back) * w + c);
       }
     }
-    win[TAPS - 1] = x[i];
+    win[TAPS - 1] = row(i);
     float4 o = cb;
 #pragma unroll
-    for (int j = 0; j < TAPS; j++) {
-      o.x = fmaf(k[0][j], win[j].x, o.x); o.y = fmaf(k[1][j], win[j].y, o.y); o.z = fmaf(k[2][j], win[j].z, o.z); o.w = fmaf(k[3][j], win[j].w, o.w);
-    }
-    store4<T>((T*)a.u + t * a.s.ld_u() + c, o);
+    for (int j = 0; j < TAPS; j++) tap(o, j, win[j]);
+    store4<T>(u + (int64_t)i * ld_u + c, o);
 #pragma unroll
     for (int j = 0; j < TAPS - 1; j++) win[j] = win[j + 1];
   }
@@ -185,46 +197,63 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32, 32 / SCAN_WARPS) gated_scan_k
   SB_TRACE_WAITED();
   const int n = live ? g.lens[seq] - g.past[seq] : 0, n_all = g.lens[seq] - g.past[seq];  // a lane without a channel has no tokens
   const int64_t row0 = g.qstart[seq];
-  const float* zr = g.gates + row0 * 2 * w + blk * 2 * bs + in_blk;
-  const T* u = (const T*)g.u + row0 * g.s.ld_u() + blk * g.s.bs_p() + in_blk;
-  const float* yp = g.p.in + row0 * g.p.ld + (live ? c : 0);  // a prompt's projection is finished
-  T* out = (T*)g.out + row0 * g.ldo + (live ? c : 0);
-  const int ld_u = (int)g.s.ld_u(), ld_y = (int)g.p.ld, ldo = (int)g.ldo;
+  // the same base for every lane, 32-bit offsets (the host checks that a sequence's rows fit)
+  const float* gates = g.gates + row0 * 2 * w;
+  const T* us = (const T*)g.u + row0 * g.s.ld_u();
+  const float* ys = g.p.in + row0 * g.p.ld;  // a prompt's projection is finished
+  T* out = (T*)g.out + row0 * g.ldo;
+  const uint32_t ld_g = 2 * (uint32_t)w, ld_u = (uint32_t)g.s.ld_u(), ld_y = (uint32_t)g.p.ld, ldo = (uint32_t)g.ldo;
+  const uint32_t og = blk * 2 * bs + in_blk, ou = blk * g.s.bs_p() + in_blk, oc = live ? c : 0;
   if (warp == 0) carry[lane] = live ? g.state[(int64_t)seq * w + c] : 0.f;
   for (int t0 = 0; t0 < n_all; t0 += SCAN_WARPS * SCAN_PER) {
     const int first = t0 + warp * SCAN_PER;
-    const float *zr0 = zr + (int64_t)first * 2 * w, *y0 = yp + (int64_t)first * ld_y;
-    const T* u0 = u + (int64_t)first * ld_u;
-    float vr[SCAN_PER], vi[SCAN_PER], vu[SCAN_PER], y[SCAN_PER];
+    const uint32_t f = (uint32_t)first;
+    Step st[SCAN_PER];
+    float y[SCAN_PER];
+    if (first + SCAN_PER <= n) {
+      float vr[SCAN_PER], vi[SCAN_PER], vu[SCAN_PER];
 #pragma unroll
-    for (int j = 0; j < SCAN_PER; j++) {
-      vr[j] = vi[j] = vu[j] = y[j] = 0.f;
-      if (first + j < n) {
-        vr[j] = __ldcs(zr0 + j * 2 * w);
-        vi[j] = __ldcs(zr0 + j * 2 * w + bs);
-        vu[j] = to_f(u0[j * ld_u]);
-        y[j] = __ldcs(y0 + j * ld_y);
+      for (int j = 0; j < SCAN_PER; j++) {
+        const uint32_t o = (f + j) * ld_g + og;
+        vr[j] = __ldcs(gates + o);
+        vi[j] = __ldcs(gates + o + (uint32_t)bs);
+        vu[j] = to_f(us[(f + j) * ld_u + ou]);
+        y[j] = __ldcs(ys + (f + j) * ld_y + oc);
+      }
+#pragma unroll
+      for (int j = 0; j < SCAN_PER; j++) st[j] = gated_step<T>(vr[j] + rb, vi[j] + ib, vu[j], decay);
+    } else {
+#pragma unroll
+      for (int j = 0; j < SCAN_PER; j++) {
+        st[j] = Step{1.f, 0.f};
+        y[j] = 0.f;
+        if (first + j < n) {
+          const uint32_t o = (f + j) * ld_g + og;
+          st[j] = gated_step<T>(gates[o] + rb, gates[o + (uint32_t)bs] + ib, to_f(us[(f + j) * ld_u + ou]), decay);
+          y[j] = ys[(f + j) * ld_y + oc];
+        }
       }
     }
-    Step st[SCAN_PER];
-#pragma unroll
-    for (int j = 0; j < SCAN_PER; j++) st[j] = first + j < n ? gated_step<T>(vr[j] + rb, vi[j] + ib, vu[j], decay) : Step{1.f, 0.f};
     Step all{1.f, 0.f};
 #pragma unroll
     for (int j = 0; j < SCAN_PER; j++) { all.b = fmaf(st[j].a, all.b, st[j].b); all.a *= st[j].a; }
     fold[warp][lane] = all;
     __syncthreads();
     float s = carry[lane];
-    for (int v = 0; v < warp; v++) s = fmaf(fold[v][lane].a, s, fold[v][lane].b);
+#pragma unroll 8
+    for (int v = 0; v < warp; v++) {
+      const Step x = fold[v][lane];
+      s = fmaf(x.a, s, x.b);
+    }
+    __syncthreads();  // everybody has read the state before this pass, and the runs
+    if (warp == SCAN_WARPS - 1) carry[lane] = fmaf(all.a, s, all.b);  // read after the next pass's first barrier
 #pragma unroll
     for (int j = 0; j < SCAN_PER; j++) {
       s = fmaf(st[j].a, s, st[j].b);
-      if (first + j < n) out[(int64_t)first * ldo + j * ldo] = to_t<T>(s * gelu<T>(y[j] + yb));
+      if (first + j < n) out[(f + j) * ldo + oc] = to_t<T>(s * gelu<T>(y[j] + yb));
     }
-    __syncthreads();  // everybody has read the state before this pass
-    if (warp == SCAN_WARPS - 1) carry[lane] = s;
-    __syncthreads();
   }
+  __syncthreads();
   if (warp == 0 && live) g.state[(int64_t)seq * w + c] = carry[lane];
   SB_TRACE_END(SB_K_RECURRENCE, 0);
 }
@@ -435,10 +464,13 @@ int k_gated_scan(strictb200_ctx* ctx, const GatedArgs& a, int64_t T) {
     else SB_CUDA(sb_launch(ctx, gated_step_kernel<bf16>, grid, dim3(256), 0, a, T));
   } else {
     const dim3 grid((unsigned)((a.s.width + 31) / 32), (unsigned)a.nb);
-    const bool many = (int64_t)grid.x * grid.y > 2 * ctx->sm_count;
-    auto go = [&](auto kernel) { return sb_launch(ctx, kernel, grid, dim3(many ? 256 : 1024), 0, a, T); };
-    if (a.f32) SB_CUDA(many ? go(gated_scan_kernel<float, 8>) : go(gated_scan_kernel<float, 32>));
-    else SB_CUDA(many ? go(gated_scan_kernel<bf16, 8>) : go(gated_scan_kernel<bf16, 32>));
+    if ((int64_t)a.max_new * std::max<int64_t>(std::max<int64_t>(2 * a.s.width, a.s.ld_u()), std::max(a.p.ld, a.ldo)) > UINT32_MAX)
+      return sb_fail(STRICTB200_ERR_INVALID_ARG, "gated recurrence: too many rows of a sequence in one launch");
+    const int64_t blocks = (int64_t)grid.x * grid.y;
+    const int warps = blocks > 4 * ctx->sm_count ? 8 : blocks > ctx->sm_count ? 16 : 32;
+    auto go = [&](auto kernel) { return sb_launch(ctx, kernel, grid, dim3(warps * 32), 0, a, T); };
+    if (a.f32) SB_CUDA(warps == 8 ? go(gated_scan_kernel<float, 8>) : warps == 16 ? go(gated_scan_kernel<float, 16>) : go(gated_scan_kernel<float, 32>));
+    else SB_CUDA(warps == 8 ? go(gated_scan_kernel<bf16, 8>) : warps == 16 ? go(gated_scan_kernel<bf16, 16>) : go(gated_scan_kernel<bf16, 32>));
   }
   ctx->launches++;
   return STRICTB200_OK;
