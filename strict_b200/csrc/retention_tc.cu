@@ -12,8 +12,9 @@
 // Few (sequence, head) pairs leave most SMs idle, so a prompt is then cut into segments of whole chunks, in two launches: the first
 // walks every segment but the last for its own contribution to the state alone; the second starts each segment from the state
 // that the contributions before it add up to.
-// A row thread takes its sums of a chunk out of tensor memory, prepares the operands of the next chunk (state, V'), and only
-// then norms, gates and stores, while the next chunk's products run.
+// A row thread takes its sums of a chunk out of tensor memory, prepares the next chunk's state operand, and only then is the chunk
+// finished, while the next one's products run: the sums (bf16) and their sums of squares pass through the tiles of V', which are
+// free between two chunks, so that the gates are read and the output written whole rows at a time.
 // Every mbarrier wait is bounded: on expiry the block records an error word in host-visible memory, stops, frees its tensor
 // memory and returns.
 #include <algorithm>
@@ -64,7 +65,7 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   __shared__ __align__(8) uint64_t bar_qk, bar_v, bar_s, bar_o, bar_state, s_ready, vp_ready, p_ready;
   __shared__ uint32_t tmem_base_slot;
-  __shared__ float pw[CHUNK + 1], x_sum[2][CHUNK], pw_seg;
+  __shared__ float pw[CHUNK + 1], pw_seg;
 
   const int h = blockIdx.x, b = blockIdx.y, seg = blockIdx.z;
   const int first = seg * a.seg_chunks * CHUNK, n_seq = a.lens[b] - a.past[b];
@@ -169,32 +170,41 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
     const float* S_in = (STATE || (seg == 0 && last) || a.segs == 1 ? a.state : a.seg_state + (seg ? 0 : a.segs - 1) * per_seg) + head + mine;
     float* S_out = (STATE ? a.seg_state + seg * per_seg : a.state) + head + mine;
     const bool s_vec = (a.vdim & 3) == 0;
-    const bool g_vec = ((a.vdim | (int)(a.ld_g & 3)) & 3) == 0 && ((uintptr_t)a.g & 15) == 0;
-    const bool o_vec = ((a.vdim | (int)(a.ldo & 7)) & 7) == 0 && ((uintptr_t)a.out & 15) == 0;
+    const bool vec = ((a.vdim | (int)(a.ld_g & 3) | (int)(a.ldo & 3)) & 3) == 0 && ((uintptr_t)a.g & 15) == 0 && ((uintptr_t)a.out & 7) == 0;
+    float* sums = (float*)bVl;  // [4][CHUNK] while the tile is free
 
-    // Operands of a chunk of n tokens: the state before it as two bf16 tiles, decay^n times it back to tensor memory; the values
-    // under their powers of the decay at the chunk's end.
-    auto operands = [&](int c, uint32_t* r) -> bool {
+    // A chunk of n tokens: the state before it (in tensor memory) as two bf16 tiles, and decay^n times it back to tensor memory.
+    auto state_operand = [&](int c) {
       const int n = min(CHUNK, n_all - c * CHUNK);
       const float dn = pw[n];
 #pragma unroll
-      for (int j = 0; j < 4 && !STATE; j++) {
-        uint4 hi, lo;
-        split2(__uint_as_float(r[8 * j]), __uint_as_float(r[8 * j + 1]), hi.x, lo.x);
-        split2(__uint_as_float(r[8 * j + 2]), __uint_as_float(r[8 * j + 3]), hi.y, lo.y);
-        split2(__uint_as_float(r[8 * j + 4]), __uint_as_float(r[8 * j + 5]), hi.z, lo.z);
-        split2(__uint_as_float(r[8 * j + 6]), __uint_as_float(r[8 * j + 7]), hi.w, lo.w);
-        const uint32_t off = box + box_off(row, chunk0 + j);
-        *(uint4*)(bSh + off) = hi;
-        *(uint4*)(bSl + off) = lo;
-      }
+      for (int q = 0; q < 2; q++) {
+        uint32_t r[16];
+        tc_ld16(tS + lane_base + (uint32_t)(c0 + q * 16), r);
+        tc_wait_ld();
 #pragma unroll
-      for (int j = 0; j < 32; j++) r[j] = __float_as_uint(__uint_as_float(r[j]) * dn);
-      tc_st32(tS + lane_base + (uint32_t)c0, r);
+        for (int j = 0; j < 2 && !STATE; j++) {
+          uint4 hi, lo;
+          split2(__uint_as_float(r[8 * j]), __uint_as_float(r[8 * j + 1]), hi.x, lo.x);
+          split2(__uint_as_float(r[8 * j + 2]), __uint_as_float(r[8 * j + 3]), hi.y, lo.y);
+          split2(__uint_as_float(r[8 * j + 4]), __uint_as_float(r[8 * j + 5]), hi.z, lo.z);
+          split2(__uint_as_float(r[8 * j + 6]), __uint_as_float(r[8 * j + 7]), hi.w, lo.w);
+          const uint32_t off = box + box_off(row, chunk0 + q * 2 + j);
+          *(uint4*)(bSh + off) = hi;
+          *(uint4*)(bSl + off) = lo;
+        }
+#pragma unroll
+        for (int j = 0; j < 16; j++) r[j] = __float_as_uint(__uint_as_float(r[j]) * dn);
+        tc_st16(tS + lane_base + (uint32_t)(c0 + q * 16), r);
+      }
       tc_wait_st();
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       tc_fence_before();
       arrive(&s_ready);
+    };
+    // The values under their powers of the decay at the chunk's end.
+    auto value_operand = [&](int c) -> bool {
+      const int n = min(CHUNK, n_all - c * CHUNK);
       if (!mbar_wait(smem_u32(&bar_v), (uint32_t)(c & 1))) return false;
       const float wv = row < n ? pw[n - 1 - row] : 0.f;
 #pragma unroll
@@ -262,17 +272,24 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
 #pragma unroll
       for (int j = 0; j < 32; j++) r[j] = __float_as_uint(x[j]);
       if (STATE && seg == 0) write_state(a.seg_state + (a.segs - 1) * per_seg + head + mine, r);
-      ok = operands(0, r);
+      tc_st32(tS + lane_base + (uint32_t)c0, r);
+      tc_wait_st();
+      state_operand(0);
+      ok = value_operand(0);
     }
     if constexpr (STATE) {
       for (int c = 0; c < chunks && ok; c++) {
         if (!mbar_wait(smem_u32(&bar_state), (uint32_t)(c & 1))) { ok = false; break; }
         tc_fence_after();
+        if (c + 1 < chunks) {
+          state_operand(c + 1);
+          ok = value_operand(c + 1);
+          continue;
+        }
         uint32_t r[32];
         tc_ld32(tS + lane_base + (uint32_t)c0, r);
         tc_wait_ld();
-        if (c + 1 < chunks) ok = operands(c + 1, r);
-        else write_state(S_out, r);
+        write_state(S_out, r);
       }
     } else
     for (int c = 0; c < chunks && ok; c++) {
@@ -298,78 +315,79 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
       tc_wait_st();
       tc_fence_before();
       arrive(&p_ready);
-      // ---- the gates are on their way while the products run
-      const bool live = row < n;
-      const int64_t t = row0 + c * CHUNK + row;
-      const float* g = a.g + t * a.ld_g + (int64_t)h * a.vdim + c0;
-      float gv[32];
-#pragma unroll
-      for (int j = 0; j < 8; j++) {
-        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (live && c0 + 4 * j < a.vdim) {
-          if (g_vec) x = *(const float4*)(g + 4 * j);
-          else {
-            x.x = g[4 * j];
-            if (c0 + 4 * j + 1 < a.vdim) x.y = g[4 * j + 1];
-            if (c0 + 4 * j + 2 < a.vdim) x.z = g[4 * j + 2];
-            if (c0 + 4 * j + 3 < a.vdim) x.w = g[4 * j + 3];
-          }
-        }
-        gv[4 * j] = x.x; gv[4 * j + 1] = x.y; gv[4 * j + 2] = x.z; gv[4 * j + 3] = x.w;
-      }
       // ---- sums of the chunk
       if (!mbar_wait(smem_u32(&bar_o), ph)) { ok = false; break; }
       tc_fence_after();
       const float d1 = pw[min(row + 1, CHUNK)];
-      float o[32], ss = 0.f;
-      {
-        uint32_t r[32], r2[32];
-        tc_ld32(tO + lane_base + (uint32_t)c0, r);
-        tc_ld32(tO2 + lane_base + (uint32_t)c0, r2);
+      uint32_t o[16];  // bf16 pairs
+      float ss = 0.f;
+#pragma unroll
+      for (int q = 0; q < 2; q++) {
+        uint32_t r[16], r2[16];
+        tc_ld16(tO + lane_base + (uint32_t)(c0 + q * 16), r);
+        tc_ld16(tO2 + lane_base + (uint32_t)(c0 + q * 16), r2);
         tc_wait_ld();
 #pragma unroll
-        for (int j = 0; j < 32; j++) {
-          o[j] = fmaf(d1, __uint_as_float(r2[j]), __uint_as_float(r[j]));
-          ss = fmaf(o[j], o[j], ss);  // columns beyond vdim are zero
+        for (int j = 0; j < 16; j += 2) {
+          const float u = fmaf(d1, __uint_as_float(r2[j]), __uint_as_float(r[j])), v = fmaf(d1, __uint_as_float(r2[j + 1]), __uint_as_float(r[j + 1]));
+          o[q * 8 + j / 2] = mix::pack_bf16(u, v);
+          ss = fmaf(u, u, fmaf(v, v, ss));  // columns beyond vdim are zero
         }
       }
-      if (quarter >= 2) x_sum[quarter - 2][row] = ss;
       if (!mbar_wait(smem_u32(&bar_state), ph)) { ok = false; break; }
       tc_fence_after();
-      {
+      sums[quarter * CHUNK + row] = ss;
+#pragma unroll
+      for (int j = 0; j < 4; j++) *(uint4*)(bVh + box + box_off(row, chunk0 + j)) = make_uint4(o[4 * j], o[4 * j + 1], o[4 * j + 2], o[4 * j + 3]);
+      if (c + 1 < chunks) {
+        state_operand(c + 1);
+      } else if (last) {
         uint32_t r[32];
         tc_ld32(tS + lane_base + (uint32_t)c0, r);
         tc_wait_ld();
-        if (c + 1 < chunks) {
-          ok = operands(c + 1, r);
-        } else if (last) {
-          write_state(S_out, r);
-        }
+        write_state(S_out, r);
       }
-      // ---- norm, gate, store (the sums of the four threads of a row meet in two steps)
-      rows_sync();
-      if (quarter < 2) x_sum[quarter][row] += ss;
-      rows_sync();
-      ss = x_sum[0][row] + x_sum[1][row];
-      rows_sync();
-      const float rn = rsqrtf(ss / (float)a.vdim + a.eps);
-      if (live) {
-        bf16* dst = a.out + t * a.ldo + (int64_t)h * a.vdim + c0;
+      // ---- norm, gate, store: warp w finishes rows 8 w.., four columns per lane
+      const int col = 4 * lane;
+      const int64_t t0 = row0 + c * CHUNK + 8 * warp;
+      const float* g = a.g + t0 * a.ld_g + (int64_t)h * a.vdim + col;
+      float4 z[8];
 #pragma unroll
-        for (int j = 0; j < 32; j += 8) {
-          float y[8];
-#pragma unroll
-          for (int i = 0; i < 8; i++) y[i] = o[j + i] * rn * __fdividef(gv[j + i], 1.0f + __expf(-gv[j + i]));
-          if (o_vec) {
-            if (c0 + j < a.vdim)
-              *(uint4*)(dst + j) = make_uint4(mix::pack_bf16(y[0], y[1]), mix::pack_bf16(y[2], y[3]), mix::pack_bf16(y[4], y[5]), mix::pack_bf16(y[6], y[7]));
-          } else {
-#pragma unroll
-            for (int i = 0; i < 8; i++)
-              if (c0 + j + i < a.vdim) dst[j + i] = __float2bfloat16_rn(y[i]);
+      for (int i = 0; i < 8; i++) {
+        z[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (8 * warp + i < n && col < a.vdim) {
+          const float* p = g + i * a.ld_g;
+          if (vec) z[i] = __ldcs((const float4*)p);
+          else {
+            z[i].x = p[0];
+            if (col + 1 < a.vdim) z[i].y = p[1];
+            if (col + 2 < a.vdim) z[i].z = p[2];
+            if (col + 3 < a.vdim) z[i].w = p[3];
           }
         }
       }
+      rows_sync();
+      auto silu = [](float v) { return __fdividef(v, 1.0f + __expf(-v)); };
+#pragma unroll
+      for (int i = 0; i < 8; i++) {
+        const int r = 8 * warp + i;
+        if (r >= n || col >= a.vdim) continue;
+        const float total = sums[r] + sums[CHUNK + r] + sums[2 * CHUNK + r] + sums[3 * CHUNK + r];
+        const float rn = rsqrtf(total / (float)a.vdim + a.eps);
+        const uint2 w = *(const uint2*)(bVh + (lane >> 4) * HALF_BYTES + box_off(r, (lane & 15) >> 1) + (lane & 1) * 8);
+        const float y0 = __uint_as_float(w.x << 16) * rn * silu(z[i].x), y1 = __uint_as_float(w.x & 0xFFFF0000u) * rn * silu(z[i].y);
+        const float y2 = __uint_as_float(w.y << 16) * rn * silu(z[i].z), y3 = __uint_as_float(w.y & 0xFFFF0000u) * rn * silu(z[i].w);
+        bf16* dst = a.out + (t0 + i) * a.ldo + (int64_t)h * a.vdim + col;
+        if (vec) *(uint2*)dst = make_uint2(mix::pack_bf16(y0, y1), mix::pack_bf16(y2, y3));
+        else {
+          dst[0] = __float2bfloat16_rn(y0);
+          if (col + 1 < a.vdim) dst[1] = __float2bfloat16_rn(y1);
+          if (col + 2 < a.vdim) dst[2] = __float2bfloat16_rn(y2);
+          if (col + 3 < a.vdim) dst[3] = __float2bfloat16_rn(y3);
+        }
+      }
+      rows_sync();  // the tiles are free again
+      if (c + 1 < chunks) ok = value_operand(c + 1);
     }
     if (!ok && row == 0) set_status(a.status, 18);
   }
