@@ -535,9 +535,8 @@ int k_gated_scan(strictb200_ctx*, const GatedArgs& a, int64_t T);   // the recur
 struct RetentionArgs {
   HeadShape s;
   ProjRows p;
-  const float* decay = nullptr;      // [H]
-  const float* log2_decay = nullptr; // [H]
-  float* state = nullptr;            // [B, H, dim, vdim]
+  const float* decay = nullptr;  // [H]
+  float* state = nullptr;        // [B, H, dim, vdim]
   const void *q = nullptr, *k = nullptr, *v = nullptr;  // [T, H, row] (k_head_split, dense)
   const int32_t *qstart = nullptr, *lens = nullptr, *past = nullptr;  // prompt rows of nb sequences; null: row t is the next token of sequence t
   int nb = 0, max_new = 0;

@@ -113,6 +113,14 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
       bool good = true;
       for (int c = 0; c < chunks && good; c++) {
         const uint32_t ph = (uint32_t)(c & 1);
+        if (c + 1 < chunks) {  // the next chunk's rows on their way to L2
+          const int row = (int)row0 + (c + 1) * CHUNK;
+          for (int i = 0; i < 2; i++) {
+            if (!STATE) tma_prefetch_3d(&map_q, i * 64, h, row);
+            tma_prefetch_3d(&map_k, i * 64, h, row);
+            tma_prefetch_3d(&map_v, i * 64, h, row);
+          }
+        }
         good = mbar_wait(smem_u32(&bar_qk), ph) && mbar_wait(smem_u32(&s_ready), ph);
         if (!good) break;
         tc_fence_after();
@@ -295,6 +303,11 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
     for (int c = 0; c < chunks && ok; c++) {
       const uint32_t ph = (uint32_t)(c & 1);
       const int n = min(CHUNK, n_all - c * CHUNK);
+      // ---- the chunk's gates on their way to L2: 128 bytes per thread
+      {
+        const int r = (int)threadIdx.x >> 2, col = ((int)threadIdx.x & 3) * 32;
+        if (r < n && col < a.vdim) asm volatile("prefetch.global.L2 [%0];" ::"l"(a.g + (row0 + c * CHUNK + r) * a.ld_g + (int64_t)h * a.vdim + col));
+      }
       // ---- P under the decay
       if (!mbar_wait(smem_u32(&bar_s), ph)) { ok = false; break; }
       tc_fence_after();
@@ -367,16 +380,30 @@ __global__ void __launch_bounds__(RT_THREADS) retention_prefill_kernel(const __g
         }
       }
       rows_sync();
-      auto silu = [](float v) { return __fdividef(v, 1.0f + __expf(-v)); };
+      // silu of a pair over one reciprocal; the exponents are kept where the product of the denominators is finite
+      auto silu2 = [](float u, float v, float& su, float& sv) {
+        float eu, ev, inv;
+        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(eu) : "f"(fminf(u * -1.4426950408889634f, 60.f)));
+        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(ev) : "f"(fminf(v * -1.4426950408889634f, 60.f)));
+        eu += 1.f;
+        ev += 1.f;
+        asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(inv) : "f"(eu * ev));
+        su = u * (ev * inv);
+        sv = v * (eu * inv);
+      };
+      const float per_dim = 1.0f / (float)a.vdim;
 #pragma unroll
       for (int i = 0; i < 8; i++) {
         const int r = 8 * warp + i;
         if (r >= n || col >= a.vdim) continue;
         const float total = sums[r] + sums[CHUNK + r] + sums[2 * CHUNK + r] + sums[3 * CHUNK + r];
-        const float rn = rsqrtf(total / (float)a.vdim + a.eps);
+        const float rn = rsqrtf(fmaf(total, per_dim, a.eps));
+        float s0, s1, s2, s3;
+        silu2(z[i].x, z[i].y, s0, s1);
+        silu2(z[i].z, z[i].w, s2, s3);
         const uint2 w = *(const uint2*)(bVh + (lane >> 4) * HALF_BYTES + box_off(r, (lane & 15) >> 1) + (lane & 1) * 8);
-        const float y0 = __uint_as_float(w.x << 16) * rn * silu(z[i].x), y1 = __uint_as_float(w.x & 0xFFFF0000u) * rn * silu(z[i].y);
-        const float y2 = __uint_as_float(w.y << 16) * rn * silu(z[i].z), y3 = __uint_as_float(w.y & 0xFFFF0000u) * rn * silu(z[i].w);
+        const float y0 = __uint_as_float(w.x << 16) * rn * s0, y1 = __uint_as_float(w.x & 0xFFFF0000u) * rn * s1;
+        const float y2 = __uint_as_float(w.y << 16) * rn * s2, y3 = __uint_as_float(w.y & 0xFFFF0000u) * rn * s3;
         bf16* dst = a.out + (t0 + i) * a.ldo + (int64_t)h * a.vdim + col;
         if (vec) *(uint2*)dst = make_uint2(mix::pack_bf16(y0, y1), mix::pack_bf16(y2, y3));
         else {

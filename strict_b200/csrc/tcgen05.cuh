@@ -43,6 +43,9 @@ __device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map
                "l"(map), "r"(x), "r"(y), "r"(z), "r"(bar)
                : "memory");
 }
+__device__ __forceinline__ void tma_prefetch_3d(const CUtensorMap* map, int x, int y, int z) {
+  asm volatile("cp.async.bulk.prefetch.tensor.3d.L2.global [%0, {%1, %2, %3}];" ::"l"(map), "r"(x), "r"(y), "r"(z) : "memory");
+}
 __device__ __forceinline__ void set_status(int* status, int code) {
   *(volatile int*)status = code;
   __threadfence_system();
